@@ -1,9 +1,11 @@
 """In-tree build of the native libraries.
 
-Two shared objects are produced next to this file:
+Shared objects are produced next to this file:
 
 * ``_C.so``    every sm_100a CUDA kernel plus the ``torch.ops.fllm_b200`` bindings
                (``nvcc -gencode arch=compute_100a,code=sm_100a -lineinfo``);
+* ``_C_<part>.so``  a part of it: the sources one group of models needs (``PARTS``), for a start on a machine where
+               nothing is built yet;
 * ``_cpu.so``  the CPU reference engine (quantizers, Q4_K x Q8_K dots, paged
                attention, sampler) behind a C ABI used through ``ctypes``.
 
@@ -27,6 +29,15 @@ CPU_SRC = ROOT / "csrc_cpu"
 BUILD = ROOT / "build"
 LIB_CUDA = ROOT / "_C.so"
 LIB_CPU = ROOT / "_cpu.so"
+# part name -> the sources (without suffix) its models run: dense and recurrent layers, latent attention and streams
+PARTS = {
+    "latent": ("binding", "binding_recurrent", "binding_latent", "elementwise", "sampling", "gemm_bf16", "gemm_bf16_2sm",
+               "gemm_f32", "recurrent", "attention_latent", "streams"),
+}
+
+
+def lib_part(part: str) -> Path:
+    return ROOT / f"_C_{part}.so"
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -95,19 +106,22 @@ def _compile_many(jobs, verbose):
     return True
 
 
-def build_cuda(verbose: bool = False, ptxas_info: bool = False) -> Path:
+def build_cuda(verbose: bool = False, ptxas_info: bool = False, part: str = "") -> Path:
+    """Every source into ``_C.so``, or those of one ``part`` into ``_C_<part>.so``."""
     BUILD.mkdir(exist_ok=True)
+    lib = lib_part(part) if part else LIB_CUDA
+    wanted = lambda src: not part or src.stem in PARTS[part]
     inc, torch_lib, abi = _torch_paths()
     cuda_inc = os.path.join(_cuda_home(), "include")
     headers = sorted(CSRC.glob("*.h")) + sorted(CSRC.glob("*.cuh"))
     jobs = []
     objs = []
     flags = list(NVCC_FLAGS) + (["-Xptxas", "-v"] if ptxas_info else [])
-    for src in sorted(CSRC.glob("*.cu")):
+    for src in filter(wanted, sorted(CSRC.glob("*.cu"))):
         obj = BUILD / (src.stem + ".o")
         objs.append(obj)
         jobs.append((src, obj, [_nvcc(), *flags, "-I", CSRC, "-c", src, "-o", obj], headers))
-    for src in sorted(CSRC.glob("*.cpp")):
+    for src in filter(wanted, sorted(CSRC.glob("*.cpp"))):
         obj = BUILD / (src.stem + ".cpp.o")
         objs.append(obj)
         cmd = ["g++", "-O2", "-std=c++17", "-fPIC", f"-D_GLIBCXX_USE_CXX11_ABI={abi}",
@@ -117,14 +131,14 @@ def build_cuda(verbose: bool = False, ptxas_info: bool = False) -> Path:
         cmd += ["-c", src, "-o", obj]
         jobs.append((src, obj, cmd, headers))
     changed = _compile_many(jobs, verbose)
-    if changed or not LIB_CUDA.exists():
-        tmp = LIB_CUDA.with_suffix(".so.tmp")
+    if changed or not lib.exists() or any(o.stat().st_mtime > lib.stat().st_mtime for o in objs):
+        tmp = lib.with_suffix(".so.tmp")
         cmd = [_nvcc(), "-shared", "-o", tmp, *objs, "-L", torch_lib, "-lc10", "-lc10_cuda",
                "-ltorch_cpu", "-ltorch_cuda", "-ltorch", "-lcudart",
                "-Xlinker", f"-rpath={torch_lib}"]
         _run(cmd, verbose)
-        os.replace(tmp, LIB_CUDA)
-    return LIB_CUDA
+        os.replace(tmp, lib)
+    return lib
 
 
 def build_cpu(verbose: bool = False) -> Path:

@@ -23,6 +23,8 @@ def _add_engine_flags(p: argparse.ArgumentParser) -> None:
     p.add_argument("--max-seqs", "--max-num-seqs", dest="max_seqs", type=int, default=256)
     p.add_argument("--max-batched-tokens", "--max-num-batched-tokens", dest="max_batched_tokens", type=int, default=2048)
     p.add_argument("--gpu-memory-utilization", type=float, default=0.90)
+    p.add_argument("--dtype", default="bf16", choices=["bf16", "fp32"],
+                   help="weights, activations and cache; fp32 for the families whose kernels exist in 32-bit")
     p.add_argument("--kv-cache-type", default="bf16")
     p.add_argument("--kv-blocks", type=int, default=0)
     p.add_argument("--no-prefix-cache", action="store_true")
@@ -55,7 +57,7 @@ def build_engine(args):
     device = args.device or ("cuda" if torch.cuda.is_available() else "cpu")
     ec = EngineConfig.from_env(
         max_num_seqs=args.max_seqs, max_num_batched_tokens=args.max_batched_tokens, max_model_len=args.ctx,
-        gpu_memory_utilization=args.gpu_memory_utilization, kv_cache_dtype=args.kv_cache_type,
+        gpu_memory_utilization=args.gpu_memory_utilization, dtype=args.dtype, kv_cache_dtype=args.kv_cache_type,
         num_kv_blocks=args.kv_blocks, enable_prefix_caching=not args.no_prefix_cache,
         use_cuda_graphs=not args.no_cuda_graphs, scheduling_policy=args.scheduling_policy,
         preemption=args.preemption, speculative=args.speculative, draft_tokens=args.draft_tokens, seed=args.seed,
@@ -68,7 +70,7 @@ def build_engine(args):
     args.model = hub.resolve(args.model)          # a path, a store entry, an alias that was pulled, or a preset name
     if args.model.endswith(".gguf") or os.path.isdir(args.model):
         from .formats.loader import load_model
-        cfg, weights, embedded_tok = load_model(args.model, device)
+        cfg, weights, embedded_tok = load_model(args.model, device, dtype=torch.float32 if args.dtype == "fp32" else torch.bfloat16)
         tok_path = tok_path or embedded_tok
     else:
         cfg = preset(args.model)
@@ -353,6 +355,9 @@ def main(argv: Optional[List[str]] = None) -> int:
     if argv and argv[0] == "bench-kernel":            # its own option set (a REMAINDER argument would refuse leading options)
         from .bench_kernel import main as bench_kernel_main
         return bench_kernel_main(argv[1:]) or 0
+    if argv and argv[0] == "trace-run":
+        from .runtime.replay import main as replay_main
+        return replay_main(argv[1:])
     ap = argparse.ArgumentParser(prog="fllm_b200")
     sub = ap.add_subparsers(dest="cmd", required=True)
     s = sub.add_parser("serve", help="HTTP server (OpenAI / Anthropic / Ollama dialects on one port)")
@@ -468,6 +473,7 @@ def main(argv: Optional[List[str]] = None) -> int:
     bk = sub.add_parser("bench-kernel")
     bk.add_argument("rest", nargs=argparse.REMAINDER)
     bk.set_defaults(fn=lambda a: __import__("fllm_b200.bench_kernel", fromlist=["main"]).main(a.rest) or 0)
+    sub.add_parser("trace-run", help="feed recorded token ids through a model step by step and write logits (its own option set)")
     b = sub.add_parser("bench")
     b.add_argument("rest", nargs=argparse.REMAINDER)
     b.set_defaults(fn=lambda a: subprocess.call([sys.executable, os.path.join(os.path.dirname(os.path.dirname(

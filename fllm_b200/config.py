@@ -105,6 +105,13 @@ class ModelConfig:
     # multi-head latent attention (layer kind "mla"): q_lora_rank (0 = one query projection), kv_lora_rank,
     # qk_nope_head_dim, qk_rope_head_dim, v_head_dim; head_dim is then qk_nope + qk_rope and rotary_dim qk_rope
     mla: Dict[str, Any] = field(default_factory=dict)
+    # per layer: shapes that differ from layer to layer, laid over `ssm` (recurrent kinds) or `mla` (kind "mla"; there also
+    # num_heads, scale, rope_theta, rope_style, head_gate, and kv_from = the layer whose cached rows this one attends to)
+    layer_mixers: Optional[List[Dict[str, Any]]] = None
+    # > 0: the residual is that many hyper-connected streams in fp32, mixed by learned matrices around every sublayer
+    # (models.decoder runs them); residual_mult scales what a sublayer adds
+    residual_streams: int = 0
+    residual_mult: float = 1.0
     # weight format of the big matrices
     weight_format: str = "bf16"          # bf16 | fp8_block | nvfp4 | mxfp4 | mxfp8 | mxfp4_a8 | nvfp4_a4 | int8_w8a8 | fp8_w8a8 | q4_k | ...
     name: str = "model"
@@ -137,9 +144,32 @@ class ModelConfig:
     def has_recurrent(self) -> bool:
         return bool(self.layer_kinds) and any(k not in ("attention", "mla", "none") for k in self.layer_kinds)
 
+    def ssm_of(self, layer: int) -> Dict[str, Any]:
+        """Shapes of a recurrent layer."""
+        return {**self.ssm, **self.layer_mixers[layer]} if self.layer_mixers else self.ssm
+
+    def mla_of(self, layer: int) -> Dict[str, Any]:
+        """Shapes of a latent-attention layer."""
+        return {**self.mla, **self.layer_mixers[layer]} if self.layer_mixers else self.mla
+
+    def kv_source(self, layer: int) -> int:
+        """The layer whose rows of the paged pool this one reads (itself unless it shares another's)."""
+        j = self.mla_of(layer).get("kv_from") if self.layer_kind(layer) == "mla" else None
+        return layer if j is None else int(j)
+
     def has_kv(self, layer: int) -> bool:
         """Whether the layer keeps keys and values (or latent rows) in the paged pool."""
-        return self.layer_kind(layer) in ("attention", "mla", "attention+mamba2")
+        return self.layer_kind(layer) in ("attention", "mla", "attention+mamba2") and self.kv_source(layer) == layer
+
+    @property
+    def native_f32(self) -> bool:
+        """Whether every kernel of the model's layers exists in fp32 (served with dtype fp32)."""
+        return self.residual_streams > 0 and all(k in ("gated_delta", "mla") for k in self.layer_kinds or ["attention"])
+
+    @property
+    def native_part(self) -> str:
+        """The part of the native library that holds all of the model's kernels ("" = the whole library)."""
+        return "latent" if self.native_f32 else ""
 
     @property
     def has_mla(self) -> bool:
@@ -179,7 +209,9 @@ class ModelConfig:
 
     @classmethod
     def from_hf_config(cls, hf: Dict[str, Any]) -> "ModelConfig":
-        """Map a Hugging Face ``config.json`` to the decoder description."""
+        """Map a ``config.json`` (Hugging Face keys, or those of a native design) to the decoder description."""
+        if hf.get("architecture") == "Sovanex":
+            return sovanex_from_config(cls, hf)
         mt = hf.get("model_type", "llama")
         if mt in ("glm4_moe_lite", "kimi_k2", "youtu"):    # DeepSeek-V3 under another name (Youtu: its dense form): the same tensors, router and latent attention
             hf = dict(hf, model_type="deepseek_v3")
@@ -471,6 +503,51 @@ def mla_from_hf(cls, hf: Dict[str, Any]) -> "ModelConfig":
         if mt == "deepseek_v3" and rs.get("mscale_all_dim"):        # V3 also scales the softmax by mscale squared
             cfg.attn_scale = (dn + dr) ** -0.5 * _yarn_mscale(f, rs["mscale_all_dim"]) ** 2
     return cfg
+
+
+def sovanex_from_config(cls, c: Dict[str, Any]) -> "ModelConfig":
+    """Sovanex: layers of the gated delta rule and of latent attention in any order, each with sizes of its own, squared-ReLU
+    feed-forward networks, LayerNorm with bias, hyper-connected residual streams and a tied head. Latent-attention layers
+    may share an earlier layer's cached rows."""
+    pad = lambda n: (n + 7) // 8 * 8
+    kinds, ffns, mixers, ff = [], [], [], 8
+    for i, layer in enumerate(c["layers"]):
+        m, mlp = layer["mixer"], layer.get("mlp")
+        if layer["type"] == "delta":
+            if m["heads"] % m["kv_heads"]:
+                raise ValueError(f"layer {i}: {m['heads']} value heads over {m['kv_heads']} key heads")
+            kinds.append("gated_delta")
+            mixers.append(dict(num_k_heads=m["kv_heads"], num_v_heads=m["heads"], head_k_dim=m["dim"], head_v_dim=m["vdim"],
+                               d_conv=max(m["conv"], 2), conv_taps=m["conv"]))
+        elif layer["type"] == "latent_attention":
+            rot, src = m["rot"], m.get("kv_from")
+            if rot["dims"] != m["rot_dim"]:
+                raise ValueError(f"layer {i}: a rotation of {rot['dims']} dimensions on a rotary part of {m['rot_dim']}")
+            if src is not None:
+                own = mixers[src] if 0 <= src < i and kinds[src] == "mla" else None
+                if own is None or own["kv_from"] is not None or (own["kv_lora_rank"], own["qk_rope_head_dim"], own["rope_theta"]) != \
+                        (m["kv_rank"], m["rot_dim"], float(rot["base"])):
+                    raise ValueError(f"layer {i}: layer {src} has no rows of the same layout to share")
+            kinds.append("mla")
+            mixers.append(dict(num_heads=m["heads"], q_lora_rank=0, kv_lora_rank=m["kv_rank"], qk_nope_head_dim=m["dim"],
+                               qk_rope_head_dim=m["rot_dim"], v_head_dim=m["vdim"], scale=float(m["scale"]), rope_theta=float(rot["base"]),
+                               rope_style="neox", head_gate=True, kv_from=src))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
+        if mlp is not None and mlp["kind"] != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        ffns.append("none" if mlp is None else "glu")
+        ff = max(ff, mlp["ff"] if mlp is not None else 0)
+    lat = [m for k, m in zip(kinds, mixers) if k == "mla"]
+    first = lat[0] if lat else None
+    eps = float(c["norm"]["eps"])
+    return cls(arch="sovanex", name=c.get("name") or "sovanex", vocab_size=c["vocab"], hidden_size=c["width"], num_layers=len(kinds),
+               num_heads=first["num_heads"] if first else 1, num_kv_heads=1,
+               head_dim=first["qk_nope_head_dim"] + first["qk_rope_head_dim"] if first else 64,
+               rotary_dim=first["qk_rope_head_dim"] if first else None, intermediate_size=pad(ff), rms_eps=eps,
+               tie_embeddings=True, norm_kind="layernorm", mlp_kind="plain", act="relu2", layer_kinds=kinds, ffn_kinds=ffns,
+               layer_mixers=mixers, ssm=dict(norm_eps=eps), residual_streams=int(c.get("streams") or 1),
+               residual_mult=float(c.get("residual_mult", 1.0)))
 
 
 RECURRENT_MODEL_TYPES = ("falcon_h1", "nemotron_h", "nemotron_h_moe", "mamba", "falcon_mamba", "mamba2", "bamba", "lfm2", "rwkv7", "qwen3_next", "qwen3_5_text", "qwen3_5_moe_text", "jamba", "granitemoehybrid", "granitemoe", "granitemoeshared", "glm4_moe", "ernie4_5_moe", "rwkv6")
@@ -854,6 +931,24 @@ def preset(name: str) -> ModelConfig:
                            moe_intermediate_size=128 if tiny else 1408, shared_intermediate_size=256 if tiny else 2816,
                            router_kind="deepseek_v2", router_scale=1.0, router_norm_topk=False,
                            mla=dict(q_lora_rank=0, kv_lora_rank=512, qk_nope_head_dim=128, qk_rope_head_dim=64, v_head_dim=128))
+    if n in ("sovanex-tiny", "sovanex-2b"):
+        # three gated-delta layers, then one of latent attention; every second attention layer shares the rows before it
+        tiny = n.endswith("tiny")
+        delta = dict(heads=6 if tiny else 32, kv_heads=3 if tiny else 16, dim=40 if tiny else 128, vdim=24 if tiny else 128, conv=3 if tiny else 4)
+        attn = dict(heads=2 if tiny else 16, dim=48 if tiny else 128, rot_dim=16 if tiny else 64, vdim=32 if tiny else 128,
+                    kv_rank=64 if tiny else 512, scale=(64 if tiny else 192) ** -0.5)
+        layers = []
+        for i in range(8 if tiny else 24):
+            if i % 4 < 3:
+                mixer = dict(delta)
+            else:
+                mixer = dict(attn, rot=dict(base=1e6, dims=attn["rot_dim"]))
+                if i % 8 == 7:
+                    mixer["kv_from"] = i - 4
+            layers.append(dict(type="delta" if i % 4 < 3 else "latent_attention", mixer=mixer, mlp=dict(kind="dense", ff=160 if tiny else 8192)))
+        return sovanex_from_config(ModelConfig, dict(
+            architecture="Sovanex", name=n, layers=layers, norm=dict(eps=1e-5), residual_mult=0.25, streams=2 if tiny else 4,
+            vocab=512 if tiny else 65536, width=96 if tiny else 2048))
     raise KeyError(f"unknown model preset {name!r}")
 
 
@@ -895,7 +990,9 @@ class EngineConfig:
     num_kv_blocks: int = 0               # 0 = size from gpu_memory_utilization
     gpu_memory_utilization: float = 0.90
     max_model_len: int = 8192
+    dtype: str = "bf16"                  # bf16 | fp32 (families whose kernels exist in 32-bit: weights, activations and cache)
     kv_cache_dtype: str = "bf16"         # bf16 | fp8_e4m3
+    spare_state_rows: int = 8            # recurrent models: state rows beyond one per running sequence
     enable_prefix_caching: bool = True
     scheduling_policy: str = "fcfs"      # fcfs | priority
     preemption: str = "recompute"        # recompute | swap (KV of a preempted request parked in host memory)

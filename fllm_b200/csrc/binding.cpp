@@ -240,8 +240,13 @@ void add_layernorm(Tensor x, const optional<Tensor>& delta, const Tensor& w, con
 }
 
 void act_(Tensor x, int64_t kind) {
-  check_bf16(x, "x"); check_rows(x, "x");
+  check_rows(x, "x");
   c10::cuda::CUDAGuard guard(x.device());
+  if (x.is_cuda() && x.scalar_type() == at::kFloat) {
+    fllm::act_rows_f32(x.data_ptr(), x.stride(0), (int)x.size(0), (int)x.size(1), (int)kind, cur_stream());
+    return;
+  }
+  check_bf16(x, "x");
   fllm::act_rows_bf16(x.data_ptr(), x.stride(0), (int)x.size(0), (int)x.size(1), (int)kind, cur_stream());
 }
 
@@ -250,67 +255,6 @@ void softcap_(Tensor x, double cap) {
   TORCH_CHECK(cap > 0, "softcap_: the cap must be positive");
   c10::cuda::CUDAGuard guard(x.device());
   fllm::softcap_rows_bf16(x.data_ptr(), x.stride(0), (int)x.size(0), (int)x.size(1), (float)cap, cur_stream());
-}
-
-void attention_generic(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
-                       const Tensor& block_tables, const Tensor& row_seq, const Tensor& positions,
-                       Tensor out, int64_t hq, int64_t hkv, int64_t head_dim, double scale,
-                       int64_t window, const optional<Tensor>& sinks, double softcap,
-                       const optional<Tensor>& tree_mask, const optional<Tensor>& tree_base) {
-  check_bf16(q, "q"); check_rows(q, "q"); check_bf16(out, "out"); check_rows(out, "out");
-  check_i32(block_tables, "block_tables"); check_i32(row_seq, "row_seq");
-  check_i32(positions, "positions");
-  const unsigned long long* tm = nullptr;
-  const int* tb = nullptr;
-  if (tree_mask.has_value() && tree_mask->defined()) {        // draft trees: one 64-bit ancestor mask and one context length per row
-    TORCH_CHECK(tree_base.has_value() && tree_base->defined(), "attention_generic: tree_mask needs tree_base");
-    TORCH_CHECK(tree_mask->scalar_type() == at::kLong && tree_mask->is_contiguous() && tree_mask->numel() == q.size(0), "tree_mask: int64 [rows]");
-    check_i32(*tree_base, "tree_base");
-    TORCH_CHECK(tree_base->numel() == q.size(0), "tree_base: int32 [rows]");
-    tm = reinterpret_cast<const unsigned long long*>(tree_mask->data_ptr<int64_t>());
-    tb = tree_base->data_ptr<int>();
-  }
-  const bool kv_fp8 = k_cache.element_size() == 1;            // e4m3 bytes instead of bf16
-  TORCH_CHECK(k_cache.is_cuda() && k_cache.is_contiguous() && v_cache.is_contiguous() &&
-              k_cache.element_size() == v_cache.element_size() && (kv_fp8 || k_cache.scalar_type() == at::kBFloat16),
-              "caches must be contiguous bf16 or 1-byte e4m3 tensors");
-  c10::cuda::CUDAGuard guard(q.device());
-  fllm::attention_generic_bf16(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
-                               block_tables.data_ptr<int>(), (int)block_tables.size(1),
-                               row_seq.data_ptr<int>(), positions.data_ptr<int>(), out.data_ptr(),
-                               out.stride(0), (int)q.size(0), (int)hq, (int)hkv, (int)head_dim,
-                               (int)k_cache.size(2), (float)scale, (int)window,
-                               opt_ptr<float>(sinks), (float)softcap, cur_stream(), kv_fp8 ? 1 : 0, tm, tb);
-}
-
-int64_t attention_tc(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
-                     const Tensor& block_tables, const Tensor& q_starts, const Tensor& kv_lens, Tensor out,
-                     int64_t num_seqs, int64_t max_q_len, int64_t min_q_len, int64_t max_kv_len, int64_t hq,
-                     int64_t hkv, int64_t head_dim, double scale, int64_t window,
-                     const optional<Tensor>& sinks, double softcap, const optional<Tensor>& workspace,
-                     const optional<Tensor>& status, bool bidirectional) {
-  check_bf16(q, "q"); check_rows(q, "q"); check_bf16(out, "out"); check_rows(out, "out");
-  const bool kv_fp8 = k_cache.element_size() == 1;            // e4m3 bytes: the decode kernel widens them to f16
-  TORCH_CHECK(k_cache.is_cuda() && v_cache.is_cuda() && k_cache.is_contiguous() && v_cache.is_contiguous() &&
-              k_cache.element_size() == v_cache.element_size() && (kv_fp8 || k_cache.scalar_type() == at::kBFloat16),
-              "caches must be contiguous bf16 or 1-byte e4m3 tensors");
-  check_i32(q_starts, "q_starts"); check_i32(kv_lens, "kv_lens");
-  TORCH_CHECK(block_tables.scalar_type() == at::kInt && block_tables.dim() == 2 &&
-              block_tables.stride(1) == 1 && block_tables.stride(0) == block_tables.size(1),
-              "block_tables must be a dense int32 matrix");
-  TORCH_CHECK(q_starts.numel() >= num_seqs + 1 && kv_lens.numel() >= num_seqs, "attention_tc: metadata too short");
-  c10::cuda::CUDAGuard guard(q.device());
-  void* ws = nullptr;
-  size_t ws_bytes = 0;
-  if (workspace.has_value() && workspace->defined()) { ws = workspace->data_ptr(); ws_bytes = workspace->nbytes(); }
-  return fllm::attention_tc_bf16(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
-                                 block_tables.data_ptr<int>(), (int)block_tables.size(1),
-                                 q_starts.data_ptr<int>(), kv_lens.data_ptr<int>(), out.data_ptr(),
-                                 out.stride(0), (int)q.size(0), (int)num_seqs, (int)max_q_len,
-                                 (int)min_q_len, (int)max_kv_len, (int)hq, (int)hkv, (int)head_dim,
-                                 (int)k_cache.size(2), (float)scale, (int)window, opt_ptr<float>(sinks),
-                                 (float)softcap, ws, ws_bytes, cur_stream(), (long long)k_cache.size(0),
-                                 const_cast<int*>(opt_ptr<int>(status)), kv_fp8 ? 1 : 0, bidirectional ? 1 : 0);
 }
 
 void argmax(const Tensor& logits, Tensor out_ids, const optional<Tensor>& out_vals,
@@ -447,8 +391,6 @@ TORCH_LIBRARY(fllm_b200, m) {
   m.def("softcap_(Tensor(a!) x, float cap) -> ()", &softcap_);
   m.def("add_layernorm(Tensor(a!) x, Tensor? delta, Tensor w, Tensor? b, Tensor(b!) y, float eps, float w_offset) -> ()", &add_layernorm);
   m.def("act_(Tensor(a!) x, int kind) -> ()", &act_);
-  m.def("attention_generic(Tensor q, Tensor k_cache, Tensor v_cache, Tensor block_tables, Tensor row_seq, Tensor positions, Tensor(a!) out, int hq, int hkv, int head_dim, float scale, int window, Tensor? sinks, float softcap, Tensor? tree_mask=None, Tensor? tree_base=None) -> ()", &attention_generic);
-  m.def("attention_tc(Tensor q, Tensor k_cache, Tensor v_cache, Tensor block_tables, Tensor q_starts, Tensor kv_lens, Tensor(a!) out, int num_seqs, int max_q_len, int min_q_len, int max_kv_len, int hq, int hkv, int head_dim, float scale, int window, Tensor? sinks, float softcap, Tensor? workspace, Tensor? status=None, bool bidirectional=False) -> int", &attention_tc);
   m.def("argmax(Tensor logits, Tensor(a!) out_ids, Tensor? out_vals, int id_offset) -> ()", &argmax);
   m.def("argmax_split(Tensor logits, Tensor(a!) out_ids, Tensor? out_vals, Tensor? out_pairs, int id_offset, Tensor(b!) scratch) -> ()", &argmax_split);
   m.def("argmax_pairs_select(Tensor pairs, Tensor(a!) out_ids) -> ()", &argmax_pairs_select);

@@ -729,11 +729,17 @@ void add_layernorm_bf16(void* x, long long ldx, const void* delta, long long ldd
   cuda_check(cudaGetLastError(), "add_layernorm_kernel");
 }
 
-// ---- activation of a plain MLP, in place over bf16 rows: 0 gelu (erf), 1 gelu (tanh), 2 squared relu, 3 silu, 4 relu -------------
-__global__ void act_rows_kernel(__nv_bfloat16* __restrict__ x, long long ldx, int cols, int kind) {
-  __nv_bfloat16* row = x + (size_t)blockIdx.y * ldx;
+// ---- activation of a plain MLP, in place: 0 gelu (erf), 1 gelu (tanh), 2 squared relu, 3 silu, 4 relu -------------
+__device__ __forceinline__ float2 act_load(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+__device__ __forceinline__ float2 act_load(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ void act_store(__nv_bfloat16* p, float2 v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y); }
+__device__ __forceinline__ void act_store(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
+
+template <typename T>
+__global__ void act_rows_kernel(T* __restrict__ x, long long ldx, int cols, int kind) {
+  T* row = x + (size_t)blockIdx.y * ldx;
   for (int c = (blockIdx.x * blockDim.x + threadIdx.x) * 2; c < cols; c += gridDim.x * blockDim.x * 2) {
-    float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(row + c));
+    float2 v = act_load(row + c);
     float* f = &v.x;
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
@@ -742,21 +748,28 @@ __global__ void act_rows_kernel(__nv_bfloat16* __restrict__ x, long long ldx, in
       if (kind == 0) r = 0.5f * t * (1.f + erff(t * 0.70710678118654752f));
       else if (kind == 1) r = 0.5f * t * (1.f + tanhf(0.7978845608028654f * (t + 0.044715f * t * t * t)));
       else if (kind == 2) r = t > 0.f ? t * t : 0.f;
-      else if (kind == 3) r = t / (1.f + __expf(-t));
+      else if (kind == 3) r = t / (1.f + (sizeof(T) == 4 ? expf(-t) : __expf(-t)));
       else r = fmaxf(t, 0.f);
       f[i] = r;
     }
-    *reinterpret_cast<__nv_bfloat162*>(row + c) = __floats2bfloat162_rn(v.x, v.y);
+    act_store(row + c, v);
   }
 }
 
-void act_rows_bf16(void* x, long long ldx, int rows, int cols, int kind, cudaStream_t s) {
+template <typename T>
+static void act_rows(T* x, long long ldx, int rows, int cols, int kind, cudaStream_t s) {
   if (rows <= 0 || cols <= 0) return;
-  if ((cols & 1) || (ldx & 1) || (reinterpret_cast<uintptr_t>(x) & 3) || kind < 0 || kind > 4)
-    throw std::runtime_error("act_rows_bf16: an even width and leading dimension, 4-byte aligned rows, kind 0..4");
+  if ((cols & 1) || (ldx & 1) || (reinterpret_cast<uintptr_t>(x) & (2 * sizeof(T) - 1)) || kind < 0 || kind > 4)
+    throw std::runtime_error("act_rows: an even width and leading dimension, pair-aligned rows, kind 0..4");
   const int bx = std::max(1, std::min((cols / 2 + 255) / 256, 64));
-  act_rows_kernel<<<dim3(bx, rows), 256, 0, s>>>((__nv_bfloat16*)x, ldx, cols, kind);
+  act_rows_kernel<T><<<dim3(bx, rows), 256, 0, s>>>(x, ldx, cols, kind);
   cuda_check(cudaGetLastError(), "act_rows_kernel");
+}
+void act_rows_bf16(void* x, long long ldx, int rows, int cols, int kind, cudaStream_t s) {
+  act_rows(static_cast<__nv_bfloat16*>(x), ldx, rows, cols, kind, s);
+}
+void act_rows_f32(void* x, long long ldx, int rows, int cols, int kind, cudaStream_t s) {
+  act_rows(static_cast<float*>(x), ldx, rows, cols, kind, s);
 }
 
 }  // namespace fllm

@@ -271,12 +271,13 @@ void spec_verify_sampled(const void* target_logits, long long ld_t, const void* 
 
 // ---- recurrent token mixers on ragged batches (recurrent.cu) -------------------------------------------------------
 // q_starts [B + 1] first token row per sequence, seq_state [B] row of the state pool, positions [T]: a sequence whose
-// first token of the step is at position 0 starts from zeros. Activations bf16 with leading dimensions in elements;
-// scan states fp32, convolution windows bf16 [slots][W - 1][C]. A negative return value means an argument was rejected
+// first token of the step is at position 0 starts from zeros. Activations bf16 (f32 = 1: fp32, where the launcher has the
+// argument) with leading dimensions in elements; scan states fp32, convolution windows [slots][W - 1][C] in the
+// activation type. A negative return value means an argument was rejected
 // before anything was launched.
 int causal_conv1d(const void* x, long long ldx, const float* w, const float* bias, void* state, const int* q_starts,
                   const int* seq_state, const int* positions, void* y, long long ldy, int B, int C, int W, int act,
-                  int max_q_len, cudaStream_t stream);   // max_q_len: host-side bound on a sequence's tokens in the step
+                  int max_q_len, cudaStream_t stream, int f32 = 0);   // max_q_len: host-side bound on a sequence's tokens in the step
 // Segmented scans (seg_len > 0, segs > 1): seg_state holds B * segs states (segs - 1 per sequence, then one start state per
 // sequence), seg_dt B * (segs - 1) sums of time steps per head (Mamba-2) or channel (Mamba-1).
 int mamba2_scan(const void* x, long long ldx, const void* dt, long long lddt, const void* Bm, long long ldb, const void* Cm,
@@ -296,9 +297,9 @@ int matrix_state_scan(int kind, const void* r, long long ldr, const void* k, lon
                       const void* beta, long long ldbeta, float* state, const int* q_starts, const int* seq_state,
                       const int* positions, void* y, long long ldy, int B, int H, int DK, int DV, int kv_ratio, int l2norm,
                       float q_scale, const void* gate_raw, long long ldgate, const float* gate_A, const float* gate_dt_bias,
-                      cudaStream_t stream);
+                      cudaStream_t stream, int f32 = 0);
 void gated_rmsnorm(const void* x, long long ldx, const void* z, long long ldz, const void* w, int wlen, void* y, long long ldy, int T,
-                   int D, int group_size, float eps, int norm_before_gate, cudaStream_t stream);
+                   int D, int group_size, float eps, int norm_before_gate, cudaStream_t stream, int f32 = 0);
 
 // Latent attention (attention_mla.cu). Element (t, h, e) of the absorbed query part sits at q_abs[t * qa_t + h * qa_h + e]
 // (e < 512), the rotated part in q_pe [tokens][H][64]; cache [blocks][block_size][576] = latent | rotated key part; output
@@ -327,5 +328,79 @@ void add_layernorm_bf16(void* x, long long ldx, const void* delta, long long ldd
                         int rows, int cols, float eps, float w_offset, cudaStream_t s);
 // in-place activation: 0 gelu (erf), 1 gelu (tanh), 2 squared relu, 3 silu, 4 relu
 void act_rows_bf16(void* x, long long ldx, int rows, int cols, int kind, cudaStream_t s);
+void act_rows_f32(void* x, long long ldx, int rows, int cols, int kind, cudaStream_t s);
+
+// ---- hyper-connected residual streams (streams.cu) -------------------------------------------------------------------
+// x [rows][streams][ld] fp32; element types of table, y, norm weights and h: bf16, or fp32 with f32 = 1.
+struct StreamMixParams {
+  float* x;
+  const int* ids;              // not null: the streams start as table[ids[row]] (mix, out and y are not read)
+  const void* table;
+  int vocab;
+  long long ld_table;
+  const void* y;               // output of the sublayer behind the streams, or the split-K partial sums of its projection
+  long long ld_y;
+  const float* partials;       // [splits][rows][ld], `plane` elements per split
+  int splits;
+  long long plane;
+  const float *mix, *out, *in; // [S][S] (from, to), [S], [S] of the next read
+  const int* rows;             // optional row selection of the outputs
+  const void *norm_w, *norm_b;
+  void* h;
+  long long ld_h;
+  int n_out;                   // output rows
+  int streams, width, ld;
+  float eps;
+  int rms, write, f32;
+};
+void stream_mix_norm(const StreamMixParams& p, cudaStream_t s);
+
+// ---- latent attention of any size (attention_latent.cu) ---------------------------------------------------------------
+struct LatentPrepareParams {
+  const void* ckv;             // [tokens][R + dr] rows (latent before its norm | shared key part before its rotation), or null
+  long long ld_ckv;
+  const void* q;               // head h's rotary values at q[t * ld_q + h * q_head + q_rope_offset]
+  long long ld_q;
+  int q_head, q_rope_offset;
+  const int *positions, *slots;
+  const float* inv_freq;       // [dr / 2]
+  float attn_factor;
+  const void* norm_w;
+  float eps;
+  void* cache;                 // rows of W values, addressed by slot
+  void* q_out;                 // [H][tokens][W]: columns [R, W) are written
+  long long q_out_h;
+  int tokens, H, R, dr, W, style, f32;
+};
+void latent_prepare(const LatentPrepareParams& p, cudaStream_t s);
+struct LatentAttnParams {
+  const void* q;               // [H][tokens][W], element (h, t, e) at q[h * q_h + t * W + e]
+  long long q_h;
+  const void* cache;           // [blocks][block_size][W]
+  const int* block_tables;
+  int max_blocks;
+  const int *row_seq, *positions, *q_starts;
+  void* out;                   // element (h, t, e < R) at out[h * o_h + t * o_t + e]
+  long long o_h, o_t;
+  int tokens, num_seqs, max_q_len, H, R, W, block_size;
+  float scale;
+  int f32;
+};
+bool attention_latent_tc_supported(int W, int R, int max_rows);
+int attention_latent_splits(int num_seqs, int tokens, int max_q_len, int H, int max_kv_len);
+size_t attention_latent_workspace_bytes(int tokens, int H, int R, int splits);
+int attention_latent(const LatentAttnParams& p, int splits, void* workspace, size_t workspace_bytes, bool tensor_cores, cudaStream_t s);
+// out[t][h * dv + j] = o(h, t, j) * sigmoid(gate[t][h]) (gate may be null), columns up to `cols` zero-filled
+void head_gate(const void* o, long long o_h, long long o_t, const void* gate, long long ld_gate, void* out, long long ld_out, int tokens, int H,
+               int dv, int cols, int f32, cudaStream_t s);
+
+// ---- fp32 products (gemm_f32.cu): c[b][t][n] = sum_k a[b][t][k] b[b][n][k] (+ bias[n]), strides in elements -----------------
+struct GemmF32Params {
+  const float *a, *b, *bias;
+  float* c;
+  long long a_b, a_t, a_k, b_b, b_n, b_k, c_b, c_t;
+  int batch, T, N, K;
+};
+void gemm_f32(const GemmF32Params& p, cudaStream_t s);
 
 }  // namespace fllm

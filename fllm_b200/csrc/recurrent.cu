@@ -52,6 +52,31 @@ __device__ __forceinline__ void store_f32(float* __restrict__ p, const float (&v
   for (int i = 0; i < N / 4; ++i)
     *reinterpret_cast<float4*>(p + 4 * i) = make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
 }
+// element types of the kernels that also serve in 32-bit; fp32 activations take the accurate exponential
+__device__ __forceinline__ float ld1(const bf16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ float ld1(const float* p) { return *p; }
+__device__ __forceinline__ void st1(bf16* p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ void st1(float* p, float v) { *p = v; }
+__device__ __forceinline__ float2 ld2(const bf16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+__device__ __forceinline__ float2 ld2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ void st2(bf16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
+__device__ __forceinline__ void st2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+template <typename T>
+__device__ __forceinline__ float exp_t(float x) { return sizeof(T) == 4 ? expf(x) : __expf(x); }
+template <typename T>
+__device__ __forceinline__ float silu_t(float x) { return x / (1.f + exp_t<T>(-x)); }
+template <typename T>
+__device__ __forceinline__ float softplus_t(float x) { return x > 20.f ? x : log1pf(exp_t<T>(x)); }
+template <int N>
+__device__ __forceinline__ void load_row(const bf16* p, float (&out)[N]) { load_bf16<N>(p, out); }
+template <int N>
+__device__ __forceinline__ void load_row(const float* p, float (&out)[N]) { load_f32<N>(p, out); }
+// the first n of N consecutive values, zeros behind them (any alignment)
+template <int N, typename T>
+__device__ __forceinline__ void load_part(const T* p, int n, float (&out)[N]) {
+#pragma unroll
+  for (int i = 0; i < N; ++i) out[i] = i < n ? ld1(p + i) : 0.f;
+}
 // sum over the LANES consecutive lanes that share one state row (LANES a power of two up to 32)
 template <int LANES>
 __device__ __forceinline__ float row_sum(float v) {
@@ -65,11 +90,11 @@ __device__ __forceinline__ float row_sum(float v) {
 // every thread owns two neighbouring channels. Only the CTA of a sequence's first run reads the sequence's window for
 // its channels (later runs see their whole history in x, which nothing writes), so after a barrier that CTA moves the
 // window forward in place. The last run of the grid goes on to the sequence's end.
-template <int W>
-__global__ void __launch_bounds__(256) conv1d_kernel(const bf16* __restrict__ x, long long ldx, const float* __restrict__ w,
-                                                     const float* __restrict__ bias, bf16* __restrict__ state,
+template <typename T, int W>
+__global__ void __launch_bounds__(256) conv1d_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ w,
+                                                     const float* __restrict__ bias, T* __restrict__ state,
                                                      const int* __restrict__ q_starts, const int* __restrict__ seq_state,
-                                                     const int* __restrict__ positions, bf16* __restrict__ y, long long ldy,
+                                                     const int* __restrict__ positions, T* __restrict__ y, long long ldy,
                                                      int C, int act, int seg_tokens) {
   const int s = blockIdx.y;
   const int c = (blockIdx.x * 64 + threadIdx.x) * 2;
@@ -78,7 +103,7 @@ __global__ void __launch_bounds__(256) conv1d_kernel(const bf16* __restrict__ x,
   if (n <= 0 || (p_lo >= n && blockIdx.z != 0)) return;
   const bool active = c < C;
   const bool fresh = positions[t0] == 0;
-  bf16* st = state + (long long)seq_state[s] * (W - 1) * C;
+  T* st = state + (long long)seq_state[s] * (W - 1) * C;
   float wv[2][W], hist[2][W - 1], bv[2] = {0.f, 0.f};
   if (active) {
 #pragma unroll
@@ -87,7 +112,7 @@ __global__ void __launch_bounds__(256) conv1d_kernel(const bf16* __restrict__ x,
 #pragma unroll
     for (int j = 0; j < W - 1; ++j) {
       float2 h = make_float2(0.f, 0.f);
-      if (!fresh && blockIdx.z == 0) h = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(st + (long long)j * C + c));
+      if (!fresh && blockIdx.z == 0) h = ld2(st + (long long)j * C + c);
       hist[0][j] = h.x, hist[1][j] = h.y;
     }
     // each row of threads walks a contiguous piece of the run with the last W - 1 inputs in registers: one load per token
@@ -99,22 +124,22 @@ __global__ void __launch_bounds__(256) conv1d_kernel(const bf16* __restrict__ x,
       const int i = a0 - (W - 1) + j;
       float2 v = make_float2(0.f, 0.f);
       if (a0 < a1) {
-        if (i >= 0) v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(x + (long long)(t0 + i) * ldx + c));
+        if (i >= 0) v = ld2(x + (long long)(t0 + i) * ldx + c);
         else v = make_float2(hist[0][(W - 1) + i], hist[1][(W - 1) + i]);
       }
       win[0][j] = v.x, win[1][j] = v.y;
     }
 #pragma unroll 4
     for (int p = a0; p < a1; ++p) {
-      const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(x + (long long)(t0 + p) * ldx + c));
+      const float2 v = ld2(x + (long long)(t0 + p) * ldx + c);
       float o0 = fmaf(wv[0][W - 1], v.x, bv[0]), o1 = fmaf(wv[1][W - 1], v.y, bv[1]);
 #pragma unroll
       for (int j = 0; j < W - 1; ++j) o0 = fmaf(wv[0][j], win[0][j], o0), o1 = fmaf(wv[1][j], win[1][j], o1);
 #pragma unroll
       for (int j = 0; j + 1 < W - 1; ++j) win[0][j] = win[0][j + 1], win[1][j] = win[1][j + 1];
       win[0][W - 2] = v.x, win[1][W - 2] = v.y;
-      if (act) o0 = silu_f(o0), o1 = silu_f(o1);
-      *reinterpret_cast<__nv_bfloat162*>(y + (long long)(t0 + p) * ldy + c) = __floats2bfloat162_rn(o0, o1);
+      if (act) o0 = silu_t<T>(o0), o1 = silu_t<T>(o1);
+      st2(y + (long long)(t0 + p) * ldy + c, o0, o1);
     }
   }
   if (blockIdx.z != 0) return;
@@ -123,10 +148,10 @@ __global__ void __launch_bounds__(256) conv1d_kernel(const bf16* __restrict__ x,
 #pragma unroll
     for (int j = 0; j < W - 1; ++j) {
       const int i = n - (W - 1) + j;
-      __nv_bfloat162 v;
-      if (i >= 0) v = *reinterpret_cast<const __nv_bfloat162*>(x + (long long)(t0 + i) * ldx + c);
-      else v = __floats2bfloat162_rn(hist[0][(W - 1) + i], hist[1][(W - 1) + i]);
-      *reinterpret_cast<__nv_bfloat162*>(st + (long long)j * C + c) = v;
+      float2 v;
+      if (i >= 0) v = ld2(x + (long long)(t0 + i) * ldx + c);
+      else v = make_float2(hist[0][(W - 1) + i], hist[1][(W - 1) + i]);
+      st2(st + (long long)j * C + c, v.x, v.y);
     }
   }
 }
@@ -378,28 +403,33 @@ __global__ void mamba1_combine_kernel(const Mamba1Args a) {
 //   kGatedDelta S = S d (one d per head);  m = sum_k S k;  S += k (v - m) beta;  y = sum_k S q
 //   kKda        as kGatedDelta with one d per key channel
 enum { kRwkv6 = 0, kRwkv7 = 1, kGatedDelta = 2, kKda = 3 };
+template <typename T>
 struct MatrixStateArgs {
-  const bf16 *r, *k, *v, *a, *b;     // r doubles as q; a, b only RWKV-7
+  const T *r, *k, *v, *a, *b;     // r doubles as q; a, b only RWKV-7
   const float* w;                    // log decay: [T][H*DK] (per channel) or [T][H] (kGatedDelta)
   const float* u;                    // RWKV-6 bonus [H*DK]
-  const bf16* beta;                  // [T][H] delta-rule step size (already through its sigmoid)
+  const T* beta;                  // [T][H] delta-rule step size (already through its sigmoid)
   long long ldr, ldk, ldv, lda, ldb, ldw, ldbeta, ldy;
   float* state;                      // [slots][H][DV][DK]
   const int *q_starts, *seq_state, *positions;
-  bf16* y;
+  T* y;
   int H, DV, kv_ratio;               // value heads per key head (q, k, w of head h come from head h / kv_ratio)
   int l2norm;                        // delta kinds: normalise q and k over DK inside the kernel
   float q_scale;
   // kGatedDelta with raw gates (w == nullptr): beta holds the logit of the step size, gate_raw [T][H] the logit a of the
   // decay; step size = sigmoid(beta), log decay = gate_A[h] * softplus(a + gate_dt_bias[h])
-  const bf16* gate_raw;
+  const T* gate_raw;
   long long ldgate;
   const float *gate_A, *gate_dt_bias;
+  int dk;                            // key width when it is below the kernel's (EXACT = false)
 };
 
-template <int KIND, int DK>
-__global__ void __launch_bounds__(128) matrix_state_kernel(const MatrixStateArgs a) {
-  constexpr int NPT = 16, TPK = DK / NPT, ROWS = 128 / TPK;
+// DKP key columns per row in registers. EXACT: the key width is DKP and every row is 16-byte aligned; otherwise the key
+// width is a.dk <= DKP, its missing columns are zeros in registers, and rows are read value by value.
+template <typename T, int KIND, int DKP, bool EXACT>
+__global__ void __launch_bounds__(128) matrix_state_kernel(const MatrixStateArgs<T> a) {
+  constexpr int NPT = 16, TPK = DKP / NPT, ROWS = 128 / TPK;
+  const int DK = EXACT ? DKP : a.dk;
   const int vtiles = (a.DV + ROWS - 1) / ROWS;
   const int h = blockIdx.x / vtiles, v = (blockIdx.x % vtiles) * ROWS + threadIdx.x / TPK;
   const int lk = threadIdx.x % TPK, s = blockIdx.y;
@@ -408,32 +438,39 @@ __global__ void __launch_bounds__(128) matrix_state_kernel(const MatrixStateArgs
   const bool valid = v < a.DV;
   const int vc = valid ? v : a.DV - 1;
   const int hk = h / a.kv_ratio;
+  const int nk = EXACT ? NPT : max(0, min(NPT, DK - lk * NPT));      // key columns of this lane
   float* st = a.state + (((long long)a.seq_state[s] * a.H + h) * a.DV + vc) * DK + lk * NPT;
   float S[NPT];
   if (a.positions[t0] == 0) {
 #pragma unroll
     for (int i = 0; i < NPT; ++i) S[i] = 0.f;
   } else {
-    load_f32<NPT>(st, S);
+    if (EXACT) load_f32<NPT>(st, S);
+    else load_part<NPT>(st, nk, S);
   }
   float u[NPT];
   if (KIND == kRwkv6) load_f32<NPT>(a.u + (long long)hk * DK + lk * NPT, u);
   const long long ko = (long long)hk * DK + lk * NPT;
   for (int t = t0; t < t0 + n; ++t) {
     float r[NPT], k[NPT], d[NPT];
-    load_bf16<NPT>(a.r + t * a.ldr + ko, r);
-    load_bf16<NPT>(a.k + t * a.ldk + ko, k);
-    const float vv = __bfloat162float(a.v[t * a.ldv + (long long)h * a.DV + vc]);
+    if (EXACT) {
+      load_row<NPT>(a.r + t * a.ldr + ko, r);
+      load_row<NPT>(a.k + t * a.ldk + ko, k);
+    } else {
+      load_part<NPT>(a.r + t * a.ldr + ko, nk, r);
+      load_part<NPT>(a.k + t * a.ldk + ko, nk, k);
+    }
+    const float vv = ld1(a.v + t * a.ldv + (long long)h * a.DV + vc);
     if (KIND == kGatedDelta) {
       const float dh = a.w != nullptr
-                           ? __expf(a.w[t * a.ldw + h])
-                           : __expf(a.gate_A[h] * softplus_f(__bfloat162float(a.gate_raw[t * a.ldgate + h]) + a.gate_dt_bias[h]));
+                           ? exp_t<T>(a.w[t * a.ldw + h])
+                           : exp_t<T>(a.gate_A[h] * softplus_t<T>(ld1(a.gate_raw + t * a.ldgate + h) + a.gate_dt_bias[h]));
 #pragma unroll
       for (int i = 0; i < NPT; ++i) d[i] = dh;
     } else {
       load_f32<NPT>(a.w + t * a.ldw + ko, d);
 #pragma unroll
-      for (int i = 0; i < NPT; ++i) d[i] = __expf(d[i]);
+      for (int i = 0; i < NPT; ++i) d[i] = exp_t<T>(d[i]);
     }
     float out = 0.f;
     if (KIND == kRwkv6) {
@@ -446,8 +483,8 @@ __global__ void __launch_bounds__(128) matrix_state_kernel(const MatrixStateArgs
       out = row_sum<TPK>(out);
     } else if (KIND == kRwkv7) {
       float av[NPT], bv[NPT], sa = 0.f;
-      load_bf16<NPT>(a.a + t * a.lda + ko, av);
-      load_bf16<NPT>(a.b + t * a.ldb + ko, bv);
+      load_row<NPT>(a.a + t * a.lda + ko, av);
+      load_row<NPT>(a.b + t * a.ldb + ko, bv);
 #pragma unroll
       for (int i = 0; i < NPT; ++i) sa = fmaf(S[i], av[i], sa);
       sa = row_sum<TPK>(sa);
@@ -476,8 +513,8 @@ __global__ void __launch_bounds__(128) matrix_state_kernel(const MatrixStateArgs
         m = fmaf(S[i], k[i], m);
       }
       m = row_sum<TPK>(m);
-      float step = __bfloat162float(a.beta[t * a.ldbeta + h]);
-      if (KIND == kGatedDelta && a.w == nullptr) step = 1.f / (1.f + __expf(-step));
+      float step = ld1(a.beta + t * a.ldbeta + h);
+      if (KIND == kGatedDelta && a.w == nullptr) step = 1.f / (1.f + exp_t<T>(-step));
       const float delta = (vv - m) * step;
 #pragma unroll
       for (int i = 0; i < NPT; ++i) {
@@ -486,9 +523,16 @@ __global__ void __launch_bounds__(128) matrix_state_kernel(const MatrixStateArgs
       }
       out = row_sum<TPK>(out) * qs;
     }
-    if (lk == 0 && valid) a.y[t * a.ldy + (long long)h * a.DV + vc] = __float2bfloat16(out);
+    if (lk == 0 && valid) st1(a.y + t * a.ldy + (long long)h * a.DV + vc, out);
   }
-  if (valid) store_f32<NPT>(st, S);
+  if (!valid) return;
+  if (EXACT) {
+    store_f32<NPT>(st, S);
+  } else {
+#pragma unroll
+    for (int i = 0; i < NPT; ++i)
+      if (i < nk) st[i] = S[i];
+  }
 }
 
 // ------------------------------------------------------------------------------------------ gated RMSNorm
@@ -496,31 +540,32 @@ __global__ void __launch_bounds__(128) matrix_state_kernel(const MatrixStateArgs
 //                                      mode 1  y = rmsnorm(x) * w * silu(z)   (gated delta net: norm first)
 // w has `wlen` entries (D for Mamba-2, the head width when every head shares one weight). One warp per group.
 // y may be x (every element is read and then written by the same thread).
-__global__ void __launch_bounds__(128) gated_rmsnorm_kernel(const bf16* x, long long ldx, const bf16* __restrict__ z, long long ldz,
-                                                            const bf16* __restrict__ w, int wlen, bf16* y, long long ldy, int T, int D,
+template <typename T>
+__global__ void __launch_bounds__(128) gated_rmsnorm_kernel(const T* x, long long ldx, const T* __restrict__ z, long long ldz,
+                                                            const T* __restrict__ w, int wlen, T* y, long long ldy, int n_rows, int D,
                                                             int gs, float eps, int mode) {
   const int groups = D / gs;
   const long long item = (long long)blockIdx.x * 4 + threadIdx.x / 32;
-  if (item >= (long long)T * groups) return;
+  if (item >= (long long)n_rows * groups) return;
   const int t = (int)(item / groups), g = (int)(item % groups), lane = threadIdx.x % 32;
-  const bf16* xr = x + t * ldx + (long long)g * gs;
-  const bf16* zr = z != nullptr ? z + t * ldz + (long long)g * gs : nullptr;
+  const T* xr = x + t * ldx + (long long)g * gs;
+  const T* zr = z != nullptr ? z + t * ldz + (long long)g * gs : nullptr;
   float ss = 0.f;
   for (int i = lane; i < gs; i += 32) {
-    float v = __bfloat162float(xr[i]);
-    if (mode == 0 && zr != nullptr) v *= silu_f(__bfloat162float(zr[i]));
+    float v = ld1(xr + i);
+    if (mode == 0 && zr != nullptr) v *= silu_t<T>(ld1(zr + i));
     ss = fmaf(v, v, ss);
   }
   ss = row_sum<32>(ss);
-  const float inv = rsqrtf(ss / gs + eps);
-  bf16* yr = y + t * ldy + (long long)g * gs;
+  const float inv = sizeof(T) == 4 ? 1.f / sqrtf(ss / gs + eps) : rsqrtf(ss / gs + eps);
+  T* yr = y + t * ldy + (long long)g * gs;
   for (int i = lane; i < gs; i += 32) {
-    float v = __bfloat162float(xr[i]);
-    const float gate = zr != nullptr ? silu_f(__bfloat162float(zr[i])) : 1.f;
+    float v = ld1(xr + i);
+    const float gate = zr != nullptr ? silu_t<T>(ld1(zr + i)) : 1.f;
     if (mode == 0) v *= gate;
-    v = v * inv * __bfloat162float(w[(g * gs + i) % wlen]);
+    v = v * inv * ld1(w + (g * gs + i) % wlen);
     if (mode == 1) v *= gate;
-    yr[i] = __float2bfloat16(v);
+    st1(yr + i, v);
   }
 }
 
@@ -606,19 +651,25 @@ inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 
 // Every launcher returns 0 on success or a negative code naming the argument it rejected, before any launch.
 int causal_conv1d(const void* x, long long ldx, const float* w, const float* bias, void* state, const int* q_starts,
                   const int* seq_state, const int* positions, void* y, long long ldy, int B, int C, int W, int act,
-                  int max_q_len, cudaStream_t stream) {
+                  int max_q_len, cudaStream_t stream, int f32) {
   if (B <= 0) return 0;
   if (C % 2 || (ldx % 2) || (ldy % 2) || x == y) return -1;
-  if (W < 2 || W > 4) return -2;
+  if (W < 2 || W > 8) return -2;
   constexpr int seg_tokens = 64;                       // 16 tokens per thread
   const int runs = std::min(std::max((max_q_len + seg_tokens - 1) / seg_tokens, 1), 65535);
   const dim3 grid((C / 2 + 63) / 64, B, runs), block(64, 4);
-  auto xs = static_cast<const bf16*>(x);
-  auto ys = static_cast<bf16*>(y);
-  auto ss = static_cast<bf16*>(state);
-  if (W == 2) conv1d_kernel<2><<<grid, block, 0, stream>>>(xs, ldx, w, bias, ss, q_starts, seq_state, positions, ys, ldy, C, act, seg_tokens);
-  if (W == 3) conv1d_kernel<3><<<grid, block, 0, stream>>>(xs, ldx, w, bias, ss, q_starts, seq_state, positions, ys, ldy, C, act, seg_tokens);
-  if (W == 4) conv1d_kernel<4><<<grid, block, 0, stream>>>(xs, ldx, w, bias, ss, q_starts, seq_state, positions, ys, ldy, C, act, seg_tokens);
+  auto go = [&](auto zero) {
+    using T = decltype(zero);
+    auto xs = static_cast<const T*>(x);
+    auto ys = static_cast<T*>(y);
+    auto ss = static_cast<T*>(state);
+#define FLLM_CONV(W_) \
+  case W_: conv1d_kernel<T, W_><<<grid, block, 0, stream>>>(xs, ldx, w, bias, ss, q_starts, seq_state, positions, ys, ldy, C, act, seg_tokens); break;
+    switch (W) { FLLM_CONV(2) FLLM_CONV(3) FLLM_CONV(4) FLLM_CONV(5) FLLM_CONV(6) FLLM_CONV(7) FLLM_CONV(8) }
+#undef FLLM_CONV
+  };
+  if (f32) go(float{});
+  else go(bf16{});
   return 0;
 }
 
@@ -697,46 +748,74 @@ int matrix_state_scan(int kind, const void* r, long long ldr, const void* k, lon
                       const void* beta, long long ldbeta, float* state, const int* q_starts, const int* seq_state,
                       const int* positions, void* y, long long ldy, int B, int H, int DK, int DV, int kv_ratio, int l2norm,
                       float q_scale, const void* gate_raw, long long ldgate, const float* gate_A, const float* gate_dt_bias,
-                      cudaStream_t stream) {
+                      cudaStream_t stream, int f32) {
   if (B <= 0) return 0;
-  if (!aligned16(r) || !aligned16(k) || (ldr % 8) || (ldk % 8) || kv_ratio <= 0 || H % kv_ratio) return -1;
+  if (kv_ratio <= 0 || H % kv_ratio || DK <= 0) return -1;
+  const int unit = f32 ? 4 : 8;
+  const bool exact = (DK == 16 || DK == 32 || DK == 64 || DK == 128 || DK == 256) && aligned16(r) && aligned16(k) && ldr % unit == 0 && ldk % unit == 0;
   if (w == nullptr && (kind != kGatedDelta || gate_raw == nullptr || gate_A == nullptr || gate_dt_bias == nullptr)) return -4;
+  if (kind != kGatedDelta && (!exact || DK == 16 || f32)) return exact ? -2 : -1;       // the other kinds: bf16, full key widths
   if (kind != kGatedDelta && (!aligned16(w) || (ldw % 4))) return -1;
   if (kind == kRwkv7 && (!aligned16(a_) || !aligned16(b_) || (lda % 8) || (ldb % 8))) return -1;
   if (kind == kRwkv6 && !aligned16(u)) return -1;
-  MatrixStateArgs m{static_cast<const bf16*>(r), static_cast<const bf16*>(k), static_cast<const bf16*>(v), static_cast<const bf16*>(a_),
-                    static_cast<const bf16*>(b_), w, u, static_cast<const bf16*>(beta), ldr, ldk, ldv, lda, ldb, ldw, ldbeta, ldy, state,
-                    q_starts, seq_state, positions, static_cast<bf16*>(y), H, DV, kv_ratio, l2norm, q_scale,
-                    static_cast<const bf16*>(gate_raw), ldgate, gate_A, gate_dt_bias};
-#define FLLM_MS(KIND_, DK_)                                                                        \
-  {                                                                                                \
-    constexpr int rows = 128 / (DK_ / 16);                                                         \
-    matrix_state_kernel<KIND_, DK_><<<dim3(H * ((DV + rows - 1) / rows), B), 128, 0, stream>>>(m); \
-    return 0;                                                                                      \
+  if (DK > 256) return -2;
+  auto args = [&](auto zero) {
+    using T = decltype(zero);
+    return MatrixStateArgs<T>{static_cast<const T*>(r), static_cast<const T*>(k), static_cast<const T*>(v), static_cast<const T*>(a_),
+                              static_cast<const T*>(b_), w, u, static_cast<const T*>(beta), ldr, ldk, ldv, lda, ldb, ldw, ldbeta, ldy, state,
+                              q_starts, seq_state, positions, static_cast<T*>(y), H, DV, kv_ratio, l2norm, q_scale,
+                              static_cast<const T*>(gate_raw), ldgate, gate_A, gate_dt_bias, DK};
+  };
+#define FLLM_MS(T_, KIND_, DK_, EXACT_)                                                                           \
+  {                                                                                                               \
+    constexpr int rows = 128 / (DK_ / 16);                                                                        \
+    matrix_state_kernel<T_, KIND_, DK_, EXACT_><<<dim3(H * ((DV + rows - 1) / rows), B), 128, 0, stream>>>(args(T_{})); \
+    return 0;                                                                                                     \
   }
-#define FLLM_MS_DK(KIND_)           \
-  switch (DK) {                     \
-    case 32: FLLM_MS(KIND_, 32)     \
-    case 64: FLLM_MS(KIND_, 64)     \
-    case 128: FLLM_MS(KIND_, 128)   \
-    case 256: FLLM_MS(KIND_, 256)   \
-    default: return -2;             \
+#define FLLM_MS_DK(KIND_)                       \
+  switch (DK) {                                 \
+    case 32: FLLM_MS(bf16, KIND_, 32, true)     \
+    case 64: FLLM_MS(bf16, KIND_, 64, true)     \
+    case 128: FLLM_MS(bf16, KIND_, 128, true)   \
+    case 256: FLLM_MS(bf16, KIND_, 256, true)   \
+    default: return -2;                         \
+  }
+#define FLLM_GD(T_, EXACT_)                                  \
+  {                                                          \
+    if (DK <= 16) FLLM_MS(T_, kGatedDelta, 16, EXACT_)       \
+    if (DK <= 32) FLLM_MS(T_, kGatedDelta, 32, EXACT_)       \
+    if (DK <= 64) FLLM_MS(T_, kGatedDelta, 64, EXACT_)       \
+    if (DK <= 128) FLLM_MS(T_, kGatedDelta, 128, EXACT_)     \
+    FLLM_MS(T_, kGatedDelta, 256, EXACT_)                    \
   }
   switch (kind) {
     case kRwkv6: FLLM_MS_DK(kRwkv6)
     case kRwkv7: FLLM_MS_DK(kRwkv7)
-    case kGatedDelta: FLLM_MS_DK(kGatedDelta)
     case kKda: FLLM_MS_DK(kKda)
+    case kGatedDelta:
+      if (f32) {
+        if (exact) FLLM_GD(float, true)
+        FLLM_GD(float, false)
+      }
+      if (exact) FLLM_GD(bf16, true)
+      FLLM_GD(bf16, false)
   }
+#undef FLLM_GD
 #undef FLLM_MS_DK
 #undef FLLM_MS
   return -3;
 }
 
 void gated_rmsnorm(const void* x, long long ldx, const void* z, long long ldz, const void* w, int wlen, void* y, long long ldy, int T,
-                   int D, int group_size, float eps, int norm_before_gate, cudaStream_t stream) {
+                   int D, int group_size, float eps, int norm_before_gate, cudaStream_t stream, int f32) {
   if (T <= 0) return;
   const long long items = (long long)T * (D / group_size);
+  if (f32) {
+    gated_rmsnorm_kernel<float><<<(unsigned)((items + 3) / 4), 128, 0, stream>>>(
+        static_cast<const float*>(x), ldx, static_cast<const float*>(z), ldz, static_cast<const float*>(w), wlen, static_cast<float*>(y), ldy, T, D,
+        group_size, eps, norm_before_gate);
+    return;
+  }
   const bool pairs_ok = group_size % 2 == 0 && ldx % 2 == 0 && ldy % 2 == 0 && (z == nullptr || ldz % 2 == 0) &&
                         (reinterpret_cast<uintptr_t>(x) & 3) == 0 && (reinterpret_cast<uintptr_t>(y) & 3) == 0 &&
                         (reinterpret_cast<uintptr_t>(z) & 3) == 0;
@@ -746,7 +825,7 @@ void gated_rmsnorm(const void* x, long long ldx, const void* z, long long ldz, c
                                                                    group_size, eps, norm_before_gate);
     return;
   }
-  gated_rmsnorm_kernel<<<(unsigned)((items + 3) / 4), 128, 0, stream>>>(static_cast<const bf16*>(x), ldx, static_cast<const bf16*>(z), ldz,
+  gated_rmsnorm_kernel<bf16><<<(unsigned)((items + 3) / 4), 128, 0, stream>>>(static_cast<const bf16*>(x), ldx, static_cast<const bf16*>(z), ldz,
                                                                        static_cast<const bf16*>(w), wlen, static_cast<bf16*>(y), ldy, T, D,
                                                                        group_size, eps, norm_before_gate);
 }

@@ -48,6 +48,12 @@ def load_hf_checkpoint(directory: str, device="cuda", tp: int = 1, tp_rank: int 
     def dev(t):
         return t.to(device=device, dtype=dtype if t.is_floating_point() and t.element_size() > 1 else t.dtype).contiguous()
 
+    if cfg.arch == "sovanex":
+        if tp > 1:
+            raise NotImplementedError("models with residual streams run on one rank")
+        from .sovanex_loader import sovanex_weights
+        tok = directory if os.path.exists(os.path.join(directory, "tokenizer.json")) else None
+        return cfg, sovanex_weights(cfg, get, device, dtype), tok
     if cfg.arch in CLASSIC_MODEL_TYPES:
         if tp > 1:
             raise NotImplementedError(f"{cfg.arch} runs on one rank")
@@ -399,7 +405,7 @@ def load_gguf(path: str, device="cuda", tp: int = 1, tp_rank: int = 0, dtype=tor
     return cfg, w, (path if has_tok else None)
 
 
-def load_model(path: str, device="cuda", tp: int = 1, tp_rank: int = 0):
+def load_model(path: str, device="cuda", tp: int = 1, tp_rank: int = 0, dtype=torch.bfloat16):
     if path.endswith(".gguf"):
-        return load_gguf(path, device, tp, tp_rank)
-    return load_hf_checkpoint(path, device, tp, tp_rank)
+        return load_gguf(path, device, tp, tp_rank, dtype)
+    return load_hf_checkpoint(path, device, tp, tp_rank, dtype)

@@ -63,6 +63,9 @@ class KVCache:
     def v(self, layer: int) -> torch.Tensor:
         return self.store[layer, 1]
 
+    def copy_block(self, src: int, dst: int) -> None:
+        self.store[:, :, dst].copy_(self.store[:, :, src])
+
     @staticmethod
     def bytes_per_block(num_layers, kv_heads, block_size, head_dim, elem=2) -> int:
         return num_layers * 2 * kv_heads * block_size * head_dim * elem
@@ -91,6 +94,7 @@ class Decoder:
             rot = cfg.rot_dim
             self.inv_freq_local = torch.tensor([cfg.rope_local_theta ** (-(2.0 * i) / rot) for i in range(rot // 2)],
                                                dtype=torch.float32, device=dev)
+        self._rope_tables = {}
         self.attn_factor = attn
         self.scale = cfg.attn_scale if cfg.attn_scale else cfg.head_dim ** -0.5
         self.rope_style = 0 if cfg.rope_style == "neox" else 1
@@ -126,6 +130,9 @@ class Decoder:
                        and not cfg.qk_norm_full and not cfg.clip_qkv)
         if self._defer:
             self._block_gate_up()
+        # the streams kernel also adds the split-K partial sums of the projection behind a sublayer
+        self._stream_ones = torch.ones(max(cfg.residual_streams, 1), dtype=torch.float32, device=dev)
+        self.defer_to_streams = bool(cfg.residual_streams and hasattr(ops, "k") and dev.type == "cuda")
 
     def _block_gate_up(self) -> None:
         """Re-order the rows of every dense gate|up matrix into blocks of 16 gate rows followed by the 16 up
@@ -144,6 +151,14 @@ class Decoder:
             lw.glu_layout = 16
 
     # ------------------------------------------------------------------ pieces
+    def rope_table(self, dims: int, theta: float) -> torch.Tensor:
+        """Inverse frequencies of a rotation over ``dims`` values (layers with a rotation of their own share tables)."""
+        key = (dims, theta)
+        if key not in self._rope_tables:
+            self._rope_tables[key] = torch.tensor([theta ** (-(2.0 * i) / dims) for i in range(dims // 2)], dtype=torch.float32,
+                                                  device=self.w.final_norm.device)
+        return self._rope_tables[key]
+
     def _reduce(self, x: torch.Tensor) -> torch.Tensor:
         if self._reduced:
             self._reduced = False
@@ -220,7 +235,7 @@ class Decoder:
             return y
         if cfg.mlp_kind == "plain":               # two matrices and an activation between them
             u = ops.act_(ops.linear(h, lw.w_gate_up, lw.b_up), cfg.act)
-            return ops.linear(u, lw.w_down, lw.b_down)
+            return ops.linear(u, lw.w_down, lw.b_down, defer=self.defer_to_streams)
         act = ops.linear_glu(h, lw.w_gate_up, None, self.act_kind, cfg.swiglu_alpha, cfg.swiglu_limit,
                              getattr(lw, "glu_layout", 0))
         return ops.linear(act, lw.w_down, defer=self._defer_out(lw.post_ffn_norm))
@@ -237,6 +252,8 @@ class Decoder:
         if cfg.arch == "rwkv6":
             from .rwkv import rwkv6_forward_hidden
             return rwkv6_forward_hidden(self, b)
+        if cfg.residual_streams:
+            return self._forward_streams(b)
         if self.first_stage:
             x = ops.embed(b.token_ids, self.w.embed, cfg.embed_scale)
             if cfg.learned_positions:              # the same row gather on the position table
@@ -291,6 +308,39 @@ class Decoder:
             if nvtx:
                 torch.cuda.nvtx.range_pop()
         return x, delta
+
+    def _sublayers(self):
+        """(stream coefficients, norm weight, norm bias, layer index, layer weights, is the mixer) in running order."""
+        for li, lw in zip(self.layer_range, self.w.layers):
+            yield lw.streams1, lw.attn_norm, lw.attn_norm_b, li, lw, True
+            if self.cfg.ffn_kind(li) != "none":
+                yield lw.streams2, lw.ffn_norm, lw.ffn_norm_b, li, lw, False
+
+    def _forward_streams(self, b: StepBatch):
+        """The layers of a model whose residual is several hyper-connected streams. Returns (streams, (output of the last
+        sublayer, its coefficients)): the update behind a sublayer runs together with the next one's read and norm."""
+        cfg, ops = self.cfg, self.ops
+        rms = cfg.norm_kind == "rms"
+        x = y = prev = None
+        for sm, nw, nb, li, lw, mixer in self._sublayers():
+            if self._nvtx:
+                torch.cuda.nvtx.range_push(f"layer{li}.{'mixer' if mixer else 'ffn'}")
+            if prev is None:
+                x, h = ops.streams_begin(b.token_ids, self.w.embed, cfg.residual_streams, sm.inp, nw, nb, cfg.hidden_size, cfg.rms_eps, rms)
+            else:
+                h = ops.streams_step(x, y, prev.mix, prev.out, sm.inp, nw, nb, cfg.hidden_size, cfg.rms_eps, rms)
+            if not mixer:
+                y = self._ffn_block(lw, h)
+            elif cfg.layer_kind(li) == "mla":
+                from .mla import mla_block
+                y = mla_block(self, li, lw, h, b)
+            else:
+                from .recurrent import MIXERS
+                y = MIXERS[cfg.layer_kind(li)](self, li, lw, h, b)
+            prev = sm
+            if self._nvtx:
+                torch.cuda.nvtx.range_pop()
+        return x, (y, prev)
 
     # ------------------------------------------------------------------ fused tensor parallel
     @property
@@ -369,6 +419,14 @@ class Decoder:
     def logits(self, x: torch.Tensor, delta: Optional[torch.Tensor], b: StepBatch) -> torch.Tensor:
         """Final norm + LM head on the requested rows -> [R, vocab_local]."""
         cfg, ops = self.cfg, self.ops
+        if cfg.residual_streams:                # sum of the streams, final norm, wanted rows: one kernel
+            y, sm = delta
+            rows = None if b.all_decode and b.logit_rows.numel() == x.shape[0] else b.logit_rows
+            hs = ops.streams_step(x, y, sm.mix, sm.out, self._stream_ones, self.w.final_norm, self.w.final_norm_b, cfg.hidden_size, cfg.rms_eps,
+                                  cfg.norm_kind == "rms", rows=rows, write=False)
+            if self.capture_hidden:
+                self.last_hidden = hs
+            return ops.linear(hs, self.w.lm_head, self.w.lm_head_b)
         if cfg.arch in ("rwkv7", "rwkv6"):
             from .rwkv import rwkv7_final_norm
             h = rwkv7_final_norm(self, x)

@@ -9,31 +9,48 @@ is the only one).
 """
 from __future__ import annotations
 
-from typing import Dict
+from typing import Dict, List
 
 import torch
 
 from ..config import ModelConfig
+from ..ops.latent import latent_width
 
 
 class MlaCache:
-    """Paged latent pool [layers, blocks, block_size, width]."""
+    """Paged latent pool: one [blocks, block_size, width] tensor per layer that keeps rows of its own."""
 
-    def __init__(self, num_layers: int, num_blocks: int, block_size: int, width: int, device, dtype=torch.bfloat16):
-        self.num_blocks, self.block_size, self.width = num_blocks, block_size, width
-        self.store = torch.zeros(num_layers, num_blocks, block_size, width, device=device, dtype=dtype)
+    def __init__(self, widths: List[int], num_blocks: int, block_size: int, device, dtype=torch.bfloat16):
+        self.num_blocks, self.block_size = num_blocks, block_size
+        self.rows = [torch.zeros(num_blocks, block_size, w, device=device, dtype=dtype) for w in widths]
 
     def layer(self, i: int) -> torch.Tensor:
-        return self.store[i]
+        return self.rows[i]
+
+    def copy_block(self, src: int, dst: int) -> None:
+        for t in self.rows:
+            t[dst].copy_(t[src])
 
     @staticmethod
-    def bytes_per_block(num_layers: int, block_size: int, width: int, elem: int = 2) -> int:
-        return num_layers * block_size * width * elem
+    def widths(cfg: ModelConfig, layer_range) -> List[int]:
+        out = []
+        for li in layer_range:
+            if cfg.layer_kind(li) == "mla" and cfg.has_kv(li):
+                c = cfg.mla_of(li)
+                R, dr = c["kv_lora_rank"], c["qk_rope_head_dim"]
+                out.append(latent_width(R, dr) if cfg.layer_mixers else R + dr)
+        return out
+
+    @staticmethod
+    def bytes_per_block(widths: List[int], block_size: int, elem: int = 2) -> int:
+        return sum(widths) * block_size * elem
 
 
 def mla_block(dec, li: int, lw, h: torch.Tensor, b) -> torch.Tensor:
     cfg, m, ops = dec.cfg, lw.mixer, dec.ops
-    c = cfg.mla
+    if "in_proj" in m:
+        return latent_block(dec, li, lw, h, b)
+    c = cfg.mla_of(li)
     H, dn, dr, dv, R = cfg.num_heads, c["qk_nope_head_dim"], c["qk_rope_head_dim"], c["v_head_dim"], c["kv_lora_rank"]
     T = h.shape[0]
     if "q_a" in m:
@@ -48,6 +65,44 @@ def mla_block(dec, li: int, lw, h: torch.Tensor, b) -> torch.Tensor:
     o_lat = ops.attention_mla(q_abs, q_pe, cache, b.block_tables, b.row_seq, b.positions, dec.scale, b.max_kv_len)     # [H, T, R]
     o = torch.bmm(o_lat, m["w_uv"]).transpose(0, 1).reshape(T, H * dv)
     return ops.linear(o, m["wo"], m.get("bo"))
+
+
+def latent_block(dec, li: int, lw, h: torch.Tensor, b) -> torch.Tensor:
+    """Latent attention of any size, with sizes, softmax scale and rotation of the layer's own, an optional sigmoid gate per
+    head, and optionally another layer's cached rows (``kv_from``). One projection makes [q | latent, shared key part |
+    head gates]; the absorbed query and its rotated part share one row, laid out like a cache row."""
+    m, ops, c = lw.mixer, dec.ops, dec.cfg.mla_of(li)
+    H, dn, dr, dv, R = c["num_heads"], c["qk_nope_head_dim"], c["qk_rope_head_dim"], c["v_head_dim"], c["kv_lora_rank"]
+    T, pad8 = h.shape[0], lambda n: (n + 7) // 8 * 8
+    cache = dec.kv.layer(dec.kv_index[dec.cfg.kv_source(li)])
+    proj = ops.linear(h, m["in_proj"])
+    nq, own = pad8(H * (dn + dr)), c.get("kv_from") is None
+    q = proj[:, :H * (dn + dr)]
+    ckv = proj[:, nq:nq + R + dr] if own else None
+    ql = torch.empty(H, T, cache.shape[-1], dtype=h.dtype, device=h.device)
+    q_nope = q.as_strided((H, T, dn), (dn + dr, proj.stride(0), 1))
+    ops.bmm(q_nope, m["w_uk"], out=ql[:, :, :R])
+    ops.latent_prepare(ckv, q, dn + dr, dn, b.positions, b.slots, dec.rope_table(dr, c["rope_theta"]), 1.0, m.get("kv_norm"),
+                       dec.cfg.rms_eps, cache, ql, R, 0 if c.get("rope_style") == "neox" else 1)
+    o = ops.bmm(ops.attention_latent(ql, cache, b, c["scale"], R), m["w_uv"])                     # [H, T, dv]
+    og = nq + (pad8(R + dr) if own else 0)
+    gate = proj[:, og:og + H] if c.get("head_gate") else None
+    return ops.linear(ops.head_gate(o, gate, m["wo"].shape[1]), m["wo"], defer=getattr(dec, "defer_to_streams", False))
+
+
+def pack_latent(q, dkv, kv_norm, uk, uv, gate, o_proj, c: Dict, dtype, device) -> Dict[str, torch.Tensor]:
+    """Checkpoint tensors of a layer ``latent_block`` runs: q [H * (dn + dr), in], dkv [R + dr, in] and its norm (None with
+    shared rows), uk [H * dn, R], uv [H * dv, R], gate [H, in] or None, o_proj [out, H * dv]. Row counts are padded to
+    multiples of 8."""
+    from .recurrent import pad8, pad_cols, pad_rows
+    H, dn, dv, R = c["num_heads"], c["qk_nope_head_dim"], c["v_head_dim"], c["kv_lora_rank"]
+    bf = lambda t: t.to(device=device, dtype=dtype).contiguous()
+    parts = [pad_rows(t, pad8(t.shape[0])) for t in (q, dkv, gate) if t is not None]
+    m = dict(in_proj=bf(torch.cat(parts, 0)), w_uk=bf(uk.view(H, dn, R)), w_uv=bf(uv.view(H, dv, R).transpose(1, 2)),
+             wo=bf(pad_cols(o_proj, pad8(H * dv))))
+    if dkv is not None:
+        m["kv_norm"] = bf(kv_norm)
+    return m
 
 
 def pack_mla(q_a, q_a_norm, q_b, q_proj, kv_a, kv_a_norm, kv_b, o_proj, cfg: ModelConfig, dtype, device) -> Dict[str, torch.Tensor]:

@@ -29,21 +29,21 @@ def _state_kind(kind: str) -> str:
     return "mamba2" if kind == "attention+mamba2" else kind
 
 
-def conv_channels(cfg: ModelConfig, kind: str) -> int:
-    s = cfg.ssm
+def conv_channels(cfg: ModelConfig, kind: str, layer: int = 0) -> int:
+    s = cfg.ssm_of(layer)
     if kind == "mamba1":
         return s["d_inner"]
     if kind == "mamba2":
         return s["d_inner"] + 2 * s["n_groups"] * s["d_state"]
     if kind == "gated_delta":
-        return 2 * s["num_k_heads"] * s["head_k_dim"] + s["num_v_heads"] * s["head_v_dim"]
+        return 2 * pad8(s["num_k_heads"] * s["head_k_dim"]) + pad8(s["num_v_heads"] * s["head_v_dim"])
     if kind in ("shortconv", "rwkv7", "rwkv6"):
         return cfg.hidden_size
     raise ValueError(kind)
 
 
-def scan_state_shape(cfg: ModelConfig, kind: str):
-    s = cfg.ssm
+def scan_state_shape(cfg: ModelConfig, kind: str, layer: int = 0):
+    s = cfg.ssm_of(layer)
     if kind == "mamba1":
         return (s["d_inner"], s["d_state"])
     if kind == "mamba2":
@@ -64,28 +64,28 @@ class RecurrentState:
         self.conv: Dict[int, torch.Tensor] = {}
         self.scan: Dict[int, torch.Tensor] = {}
         self.shift2: Dict[int, torch.Tensor] = {}          # RWKV: the channel mix has a token shift of its own
-        W = cfg.ssm.get("d_conv", 4)
         for li in layer_range:
             kind = _state_kind(cfg.layer_kind(li))
             if kind in ("attention", "mla", "none"):
                 continue
+            W = cfg.ssm_of(li).get("d_conv", 4)
             if kind in ("rwkv7", "rwkv6"):
                 self.shift2[li] = torch.zeros(slots, W - 1, cfg.hidden_size, dtype=act_dtype, device=device)
-            self.conv[li] = torch.zeros(slots, W - 1, conv_channels(cfg, kind), dtype=act_dtype, device=device)
-            shape = scan_state_shape(cfg, kind)
+            self.conv[li] = torch.zeros(slots, W - 1, conv_channels(cfg, kind, li), dtype=act_dtype, device=device)
+            shape = scan_state_shape(cfg, kind, li)
             if shape is not None:
                 self.scan[li] = torch.zeros(slots, *shape, dtype=torch.float32, device=device)
 
     @staticmethod
-    def bytes_per_slot(cfg: ModelConfig, layer_range: range) -> int:
+    def bytes_per_slot(cfg: ModelConfig, layer_range: range, elem: int = 2) -> int:
         n = 0
-        W = cfg.ssm.get("d_conv", 4)
         for li in layer_range:
             kind = _state_kind(cfg.layer_kind(li))
             if kind in ("attention", "mla", "none"):
                 continue
-            n += (W - 1) * conv_channels(cfg, kind) * (4 if kind in ("rwkv7", "rwkv6") else 2)
-            shape = scan_state_shape(cfg, kind)
+            W = cfg.ssm_of(li).get("d_conv", 4)
+            n += (W - 1) * conv_channels(cfg, kind, li) * (4 if kind in ("rwkv7", "rwkv6") else elem)
+            shape = scan_state_shape(cfg, kind, li)
             if shape is not None:
                 k = 4
                 for d in shape:
@@ -156,19 +156,20 @@ def gated_delta_mixer(dec, li: int, lw, h: torch.Tensor, b) -> torch.Tensor:
     """in_proj -> (q, k, v | z | beta, a); (q, k, v) = silu(conv(q, k, v)); log decay = -exp(A_log) softplus(a + dt_bias)
     and step size = sigmoid(beta), both computed inside the scan;
     delta rule with L2-normalised q, k; per-head rmsnorm(y) * w * silu(z); out_proj."""
-    s, m, ops = dec.cfg.ssm, lw.mixer, dec.ops
+    s, m, ops = dec.cfg.ssm_of(li), lw.mixer, dec.ops
     qs, ss, pos = _batch_meta(b)
     Hk, Hv, Dk, Dv = s["num_k_heads"], s["num_v_heads"], s["head_k_dim"], s["head_v_dim"]
     K, V = Hk * Dk, Hv * Dv
+    Kp, Vp = pad8(K), pad8(V)                                           # segments of the projection start on 16-byte boundaries
     proj = ops.linear(h, m["in_proj"])                                  # [q | k | v | z | beta | a] (+ padding)
-    qkv = ops.causal_conv1d(proj[:, :2 * K + V], m["conv_w"], m.get("conv_b"), dec.rstate.conv[li], qs, ss, pos, act=True, max_q_len=getattr(b, "max_q_len", 0))
-    z = proj[:, 2 * K + V:2 * K + 2 * V]
-    o = 2 * K + 2 * V                                                   # the step-size and decay logits go to the scan raw
-    y = ops.matrix_state_scan(GATED_DELTA, qkv[:, :K], qkv[:, K:2 * K], qkv[:, 2 * K:], None, None, None, None, proj[:, o:o + Hv],
+    qkv = ops.causal_conv1d(proj[:, :2 * Kp + Vp], m["conv_w"], m.get("conv_b"), dec.rstate.conv[li], qs, ss, pos, act=True, max_q_len=getattr(b, "max_q_len", 0))
+    z = proj[:, 2 * Kp + Vp:2 * Kp + Vp + V]
+    o = 2 * Kp + 2 * Vp                                                 # the step-size and decay logits go to the scan raw
+    y = ops.matrix_state_scan(GATED_DELTA, qkv[:, :K], qkv[:, Kp:Kp + K], qkv[:, 2 * Kp:2 * Kp + V], None, None, None, None, proj[:, o:o + Hv],
                               dec.rstate.scan[li], qs, ss, pos, Hv, Dk, Dv, Hv // Hk, True, Dk ** -0.5,
                               gate_raw=proj[:, o + Hv:o + 2 * Hv], gate_A=m["A"], gate_dt_bias=m["dt_bias"])
-    y = ops.gated_rmsnorm(y, z, m["norm_w"], s.get("norm_eps", dec.cfg.rms_eps), Dv, True)
-    return ops.linear(y, m["out_proj"])
+    y = ops.gated_rmsnorm(y, z, m["norm_w"], s.get("norm_eps", dec.cfg.rms_eps), Dv, True, Vp)
+    return ops.linear(y, m["out_proj"], defer=getattr(dec, "defer_to_streams", False))
 
 
 def shortconv_mixer(dec, li: int, lw, h: torch.Tensor, b) -> torch.Tensor:
@@ -237,12 +238,17 @@ def pack_mamba2(in_proj, conv_w, conv_b, dt_bias, A_log, D, norm_w, out_proj, dt
 
 
 def pack_gated_delta(q, k, v, z, b, a, conv_w, dt_bias, A_log, norm_w, out_proj, dtype, device) -> Dict[str, torch.Tensor]:
-    """Projection rows already separated by role ([Hk*Dk], [Hk*Dk], [Hv*Dv], [Hv*Dv], [Hv], [Hv]) -> one in_proj."""
+    """Projection rows already separated by role ([Hk*Dk], [Hk*Dk], [Hv*Dv], [Hv*Dv], [Hv], [Hv]) -> one in_proj whose
+    segments q, k, v and z are padded to multiples of 8 rows (``conv_w``: the rows of q, k and v, one below the other)."""
     f32 = lambda t: t.float().to(device).contiguous()
     bf = lambda t: t.to(device=device, dtype=dtype).contiguous()
-    fused = torch.cat([q, k, v, z, b, a], 0)
-    return dict(in_proj=bf(pad_rows(fused, pad8(fused.shape[0]))), conv_w=f32(conv_w.reshape(conv_w.shape[0], -1)),
-                dt_bias=f32(dt_bias), A=f32(-torch.exp(A_log.float())), norm_w=bf(norm_w), out_proj=bf(out_proj))
+    p8 = lambda t: pad_rows(t, pad8(t.shape[0]))
+    fused = torch.cat([p8(q), p8(k), p8(v), p8(z), b, a], 0)
+    K, V = q.shape[0], v.shape[0]
+    cw = conv_w.reshape(conv_w.shape[0], -1)
+    cw = torch.cat([p8(cw[:K]), p8(cw[K:2 * K]), p8(cw[2 * K:])], 0)
+    return dict(in_proj=bf(pad_rows(fused, pad8(fused.shape[0]))), conv_w=f32(cw),
+                dt_bias=f32(dt_bias), A=f32(-torch.exp(A_log.float())), norm_w=bf(norm_w), out_proj=bf(pad_cols(out_proj, pad8(V))))
 
 
 def init_random_mixer(cfg: ModelConfig, kind: str, full, li: int, dtype, device) -> Dict[str, torch.Tensor]:

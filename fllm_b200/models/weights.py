@@ -21,6 +21,15 @@ from ..config import ModelConfig
 
 
 @dataclass
+class StreamMix:
+    """How one sublayer reads and writes the residual streams (fp32): input sum_s inp[s] x_s, then
+    x_t <- sum_s mix[s, t] x_s + out[t] y; a residual multiplier is part of ``out``."""
+    inp: torch.Tensor
+    mix: torch.Tensor
+    out: torch.Tensor
+
+
+@dataclass
 class LayerWeights:
     attn_norm: torch.Tensor
     wqkv: torch.Tensor
@@ -58,6 +67,9 @@ class LayerWeights:
     b_down: Optional[torch.Tensor] = None
     # recurrent layers (Mamba, delta rule, short convolution): the mixer's tensors by name; wqkv / wo stay None
     mixer: Optional[Dict[str, torch.Tensor]] = None
+    # hyper-connected residual streams: coefficients around the mixer and around the feed-forward network
+    streams1: Optional["StreamMix"] = None
+    streams2: Optional["StreamMix"] = None
     # packed formats keep their payload here (format name -> tensors)
     packed: Dict[str, object] = field(default_factory=dict)
     # row order of w_gate_up: 0 = gate half then up half; 16 = blocks of 16 gate rows followed by the 16 up
@@ -249,6 +261,11 @@ def init_random_weights(cfg: ModelConfig, device="cpu", dtype=torch.bfloat16, se
         if tp > 1 or (layers is not None and len(layers) != cfg.num_layers):
             raise NotImplementedError("RWKV models run on one rank and one pipeline stage")
         return rwkv6_weights_from_state_dict(cfg, random_rwkv6_state_dict(cfg, seed), device, dtype)
+    if cfg.arch == "sovanex":
+        from ..formats.sovanex_loader import random_tensors, sovanex_weights
+        if tp > 1 or (layers is not None and len(layers) != cfg.num_layers):
+            raise NotImplementedError("models with residual streams run on one rank and one pipeline stage")
+        return sovanex_weights(cfg, random_tensors(cfg, seed, device), device, dtype)
     sp = make_shard_spec(cfg, tp, tp_rank, expert_parallel)
     D, H = cfg.head_dim, cfg.hidden_size
     layers = range(cfg.num_layers) if layers is None else layers

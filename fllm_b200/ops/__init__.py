@@ -8,9 +8,10 @@ import torch
 from .reference import RefOps
 
 
-def get_ops(device) -> object:
+def get_ops(device, part: str = "") -> object:
+    """``part``: the part of the native library that is enough for the caller's model (see ``_build.PARTS``)."""
     device = torch.device(device)
     if device.type == "cuda":
         from .native import NativeOps
-        return NativeOps(device)
+        return NativeOps(device, part=part)
     return RefOps()

@@ -12,6 +12,7 @@ from typing import Optional
 import torch
 
 from ._lib import load_cuda
+from .latent import LatentNative
 from .recurrent import RecurrentNative
 
 
@@ -30,11 +31,11 @@ class Deferred:
         return (self.rows, self.cols)
 
 
-class NativeOps(RecurrentNative):
+class NativeOps(RecurrentNative, LatentNative):
     name = "sm100a"
 
-    def __init__(self, device: torch.device, workspace_bytes: int = 96 << 20):
-        self.k = load_cuda()
+    def __init__(self, device: torch.device, workspace_bytes: int = 96 << 20, part: str = ""):
+        self.k = load_cuda(part=part)
         self.device = torch.device(device)
         # first 64 KiB = split-K tile counters (must start at zero; the kernels re-zero them)
         self.workspace = torch.zeros(workspace_bytes, dtype=torch.uint8, device=self.device)
@@ -60,6 +61,10 @@ class NativeOps(RecurrentNative):
             return w.apply(self, x, bias, out)
         if out is None:
             out = torch.empty(x.shape[0], w.shape[0], dtype=x.dtype, device=x.device)
+        if x.dtype == torch.float32:                 # models served in 32-bit
+            self.k.linear_f32(x, w, bias, out)
+            self.launches += 1
+            return out
         if not defer:
             self.launches += self.k.linear(x, w, bias, out, self.workspace, self.status, force_splits)
             return out
@@ -71,7 +76,7 @@ class NativeOps(RecurrentNative):
         """Tensor value of a projection result (adds a Deferred's partials with the stand-alone path)."""
         if not isinstance(y, Deferred):
             return y
-        raise RuntimeError("a deferred projection can only be consumed by rmsnorm, rope_kv_write or a gated activation")
+        raise RuntimeError("a deferred projection can only be consumed by rmsnorm, rope_kv_write, a gated activation or streams_step")
 
     def linear_glu(self, x, w, bias, act_kind=0, alpha=1.702, limit=7.0, layout=0, force_splits: int = 0):
         """act(x @ w^T + bias) for a fused gate|up weight, [T, N/2]. With a row layout the GEMM epilogue can

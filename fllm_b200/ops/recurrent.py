@@ -186,9 +186,10 @@ class RecurrentRef:
             state[slot] = S
         return y
 
-    def gated_rmsnorm(self, x, z, w, eps, group_size=0, norm_before_gate=False):
+    def gated_rmsnorm(self, x, z, w, eps, group_size=0, norm_before_gate=False, width=0):
         """Mamba-2: rmsnorm(x * silu(z)) * w over groups; gated delta net: rmsnorm(x) * w * silu(z) (norm first).
-        ``w`` may be shorter than the row (one weight vector per head): it repeats."""
+        ``w`` may be shorter than the row (one weight vector per head): it repeats. ``width``: columns of the result when
+        the next matrix is padded (zeros behind the row)."""
         T, D = x.shape
         gs = group_size or D
         xf = x.float()
@@ -201,8 +202,7 @@ class RecurrentRef:
         out = xg.reshape(T, D) * wf
         if gate is not None and norm_before_gate:
             out = out * gate
-        return out.to(x.dtype)
-
+        return F.pad(out, (0, max(width - D, 0))).to(x.dtype)
 
     def mla_prepare(self, ckv, q, rope_offset, positions, slots, inv_freq, attn_factor, norm_w, eps, cache):
         """Latent attention, per token: RMSNorm of the latent part of ``ckv`` [T, R + dr] and rotation of its last dr
@@ -317,11 +317,15 @@ class RecurrentNative:
         self.launches += 1
         return y
 
-    def gated_rmsnorm(self, x, z, w, eps, group_size=0, norm_before_gate=False):
-        y = torch.empty(x.shape, dtype=x.dtype, device=x.device)
+    def gated_rmsnorm(self, x, z, w, eps, group_size=0, norm_before_gate=False, width=0):
+        if width > x.shape[1]:
+            full = torch.zeros(x.shape[0], width, dtype=x.dtype, device=x.device)
+            y = full[:, :x.shape[1]]
+        else:
+            full = y = torch.empty(x.shape, dtype=x.dtype, device=x.device)
         self.k.gated_rmsnorm(x, z, w, y, int(group_size or x.shape[1]), float(eps), bool(norm_before_gate))
         self.launches += 1
-        return y
+        return full
 
     def mla_prepare(self, ckv, q, rope_offset, positions, slots, inv_freq, attn_factor, norm_w, eps, cache):
         if cache.shape[-1] != 576 or inv_freq.numel() != 32:      # the kernels are built for the 512 + 64 rows of the DeepSeek family

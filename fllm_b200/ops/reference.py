@@ -11,10 +11,11 @@ import numpy as np
 import torch
 import torch.nn.functional as F
 
+from .latent import LatentRef
 from .recurrent import RecurrentRef
 
 
-class RefOps(RecurrentRef):
+class RefOps(RecurrentRef, LatentRef):
     name = "reference"
 
     # ---------------------------------------------------------------- dense

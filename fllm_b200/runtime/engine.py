@@ -59,8 +59,10 @@ class LLMEngine:
         self.device = torch.device(device)
         self.is_cuda = self.device.type == "cuda"
         if self.is_cuda:
+            if self.device.index is None:
+                self.device = torch.device("cuda", torch.cuda.current_device())
             torch.cuda.set_device(self.device)
-        self.ops = ops or get_ops(self.device)
+        self.ops = ops or get_ops(self.device, model_cfg.native_part)
         self.tp_group, self.tp_rank = tp_group, tp_rank
         tp = self.par.tp
         self.spec = make_shard_spec(model_cfg, tp, tp_rank, self.par.expert_parallel)
@@ -68,8 +70,17 @@ class LLMEngine:
         self.pp_group, self.stage = pp_group, stage
         self.first_stage, self.last_stage = stage == 0, stage == self.par.pp - 1
         self.layer_range = self.par.stage_layers(model_cfg.num_layers, stage)
+        if self.cfg.dtype not in ("bf16", "fp32"):
+            raise ValueError("dtype must be bf16 or fp32")
+        if self.cfg.dtype == "fp32":
+            if hasattr(self.ops, "k") and not model_cfg.native_f32:
+                raise ValueError(f"{model_cfg.arch}: the kernels of this family run in bf16 only")
+            self.cfg = dataclasses.replace(self.cfg, kv_cache_dtype="fp32")
+        if model_cfg.residual_streams and (tp > 1 or self.par.pp > 1):
+            raise NotImplementedError("models with residual streams run on one rank and one pipeline stage")
+        act_dtype = torch.float32 if self.cfg.dtype == "fp32" else torch.bfloat16
         self.weights = weights or init_random_weights(
-            model_cfg, self.device, torch.bfloat16, seed, tp, tp_rank, self.par.expert_parallel,
+            model_cfg, self.device, act_dtype, seed, tp, tp_rank, self.par.expert_parallel,
             layers=self.layer_range, first_stage=self.first_stage, last_stage=self.last_stage)
         self.eos_token_id = eos_token_id
         if model_cfg.has_mla:
@@ -93,16 +104,15 @@ class LLMEngine:
         num_blocks = self.cfg.num_kv_blocks or self._size_kv_pool()
         if self.cfg.kv_cache_dtype not in ("bf16", "fp8", "fp8_e4m3", "fp32"):
             raise ValueError("kv_cache_dtype must be bf16 or fp8_e4m3")
-        # fp32: only with the PyTorch operators (exact comparisons against other implementations on the CPU)
+        # fp32: with the PyTorch operators (exact comparisons against other implementations), or a family with fp32 kernels
         kv_dtype = {"bf16": torch.bfloat16, "fp32": torch.float32}.get(self.cfg.kv_cache_dtype, torch.float8_e4m3fn)
-        if kv_dtype == torch.float32 and hasattr(self.ops, "k"):
-            raise ValueError("an fp32 KV pool is for the reference operators only")
+        if kv_dtype == torch.float32 and hasattr(self.ops, "k") and not (model_cfg.native_f32 and self.weights.embed.dtype == torch.float32):
+            raise ValueError("an fp32 KV pool is for the reference operators and for models served in fp32")
         if model_cfg.has_mla:
             from ..models.mla import MlaCache
             if kv_dtype not in (torch.bfloat16, torch.float32):
                 raise ValueError("the latent cache of multi-head latent attention is bf16")
-            self.kv = MlaCache(self._kv_layers(), num_blocks, self.block_size,
-                               model_cfg.mla["kv_lora_rank"] + model_cfg.mla["qk_rope_head_dim"], self.device, kv_dtype)
+            self.kv = MlaCache(MlaCache.widths(model_cfg, self.layer_range), num_blocks, self.block_size, self.device, kv_dtype)
         else:
             self.kv = KVCache(self._kv_layers(), num_blocks, self.spec.hkv_local, self.block_size,
                               model_cfg.head_dim, self.device, kv_dtype)
@@ -111,7 +121,7 @@ class LLMEngine:
             # one state row per running sequence, a few spare for sequences between two owners, and the scratch
             # row that padding sequences of a captured step write to
             from ..models.recurrent import RecurrentState
-            self.rstate = RecurrentState(model_cfg, self.layer_range, self.cfg.max_num_seqs + 9, self.device,
+            self.rstate = RecurrentState(model_cfg, self.layer_range, self._state_rows(), self.device,
                                          self.weights.embed.dtype)
         self.decoder = Decoder(model_cfg, self.weights, self.kv, self.ops, self.spec, tp_group,
                                layer_range=self.layer_range, first_stage=self.first_stage,
@@ -186,6 +196,10 @@ class LLMEngine:
                                      pin_memory=self.is_cuda)
 
     # ------------------------------------------------------------------ sizing
+    def _state_rows(self) -> int:
+        """Rows of the recurrent-state pools: one per running sequence, the spare ones, and the scratch row."""
+        return self.cfg.max_num_seqs + self.cfg.spare_state_rows + 1
+
     def _kv_layers(self) -> int:
         """Attention layers of this stage (at least one, so that the pool tensors exist)."""
         return max(1, sum(1 for li in self.layer_range if self.model_cfg.has_kv(li)))
@@ -193,18 +207,19 @@ class LLMEngine:
     def _size_kv_pool(self) -> int:
         per_block = KVCache.bytes_per_block(self._kv_layers(), self.spec.hkv_local,
                                             self.block_size, self.model_cfg.head_dim,
-                                            2 if self.cfg.kv_cache_dtype == "bf16" else 1)
+                                            {"bf16": 2, "fp32": 4}.get(self.cfg.kv_cache_dtype, 1))
         if self.model_cfg.has_mla:
             from ..models.mla import MlaCache
-            per_block = MlaCache.bytes_per_block(self._kv_layers(), self.block_size,
-                                                 self.model_cfg.mla["kv_lora_rank"] + self.model_cfg.mla["qk_rope_head_dim"])
+            per_block = max(1, MlaCache.bytes_per_block(MlaCache.widths(self.model_cfg, self.layer_range), self.block_size,
+                                                        4 if self.cfg.kv_cache_dtype == "fp32" else 2))
         if self.is_cuda:
             free, total = torch.cuda.mem_get_info(self.device)
             budget = int(total * self.cfg.gpu_memory_utilization) - (total - free)
             budget -= 4 << 30           # activations, graphs, workspaces
             if self.model_cfg.has_recurrent:
                 from ..models.recurrent import RecurrentState
-                budget -= RecurrentState.bytes_per_slot(self.model_cfg, self.layer_range) * (self.cfg.max_num_seqs + 9)
+                budget -= RecurrentState.bytes_per_slot(self.model_cfg, self.layer_range,
+                                                        4 if self.cfg.dtype == "fp32" else 2) * self._state_rows()
         else:
             budget = 256 << 20
         want = self.cfg.max_num_seqs * self.max_blocks_per_seq
@@ -243,6 +258,8 @@ class LLMEngine:
         handed to ``import_request`` of another engine of the same model and KV layout
         (rust/engine/src/disagg.rs is the reference's KV hand-over)."""
         self.drain()
+        if self.model_cfg.has_mla:
+            raise NotImplementedError("a latent cache is not handed over between engines")
         r = self.requests.get(request_id)
         if r is None or r.finished:
             raise KeyError(f"no live request {request_id!r}")
@@ -363,7 +380,9 @@ class LLMEngine:
                 sst[i] = self.blocks.state_slot(r.seq_id)
             max_q, min_q = max(max_q, n), min(min_q, n)
             if s.wants_logits:
-                if s.verify:
+                if s.rows is not None:
+                    rows.extend(t + j for j in s.rows)
+                elif s.verify:
                     rows.extend(range(t, t + n))
                 else:
                     rows.append(t + n - 1)
@@ -613,7 +632,7 @@ class LLMEngine:
         """Forward + sample + commit of one scheduled step, waiting for its result."""
         events: List[TokenEvent] = []
         for src, dst in step.cow:
-            self.kv.store[:, :, dst].copy_(self.kv.store[:, :, src])
+            self.kv.copy_block(src, dst)
         use_graph = self._graph_eligible(step)
         l0 = getattr(self.ops, "launches", 0)
         if use_graph:
@@ -870,6 +889,19 @@ class LLMEngine:
             return "length"
         return None
 
+    # ------------------------------------------------------------------ given tokens
+    @torch.inference_mode()
+    def run_forced(self, step: ScheduledStep) -> torch.Tensor:
+        """Forward of a step whose tokens are all given: fp32 logits of the rows it wants, in batch order. Pure decode steps
+        replay the captured graph of their bucket. Nothing is sampled or committed. Single pipeline stage only."""
+        self.drain()
+        if self._graph_eligible(step):
+            _, logits, _ = self._decode_with_graph(step)
+            logits = logits[[i for i, s in enumerate(step.seqs) if s.wants_logits]]
+        else:
+            logits = self.decoder.forward(self._build_batch(step))
+        return self.decoder.full_logits(logits).float()
+
     # ------------------------------------------------------------------ scoring
     @torch.inference_mode()
     def token_logits(self, tokens: Sequence[int]) -> torch.Tensor:
@@ -898,8 +930,7 @@ class LLMEngine:
             while off < n:
                 cnt = min(step_max, n - off)
                 step = ScheduledStep(seqs=[ScheduledSeq(req, off, cnt, True, verify=cnt - 1)])
-                batch = self._build_batch(step)
-                logits = self.decoder.full_logits(self.decoder.forward(batch)).float()
+                logits = self.run_forced(step)
                 out.append(logits[-1:] if cnt == 1 else logits[:cnt])
                 off += cnt
         finally:

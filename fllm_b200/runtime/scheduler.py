@@ -27,6 +27,7 @@ class ScheduledSeq:
     count: int                 # number of tokens fed this step
     wants_logits: bool         # sample after this chunk
     verify: int = 0            # number of draft tokens among `count` (rows count = 1 + verify)
+    rows: Optional[List[int]] = None   # replayed steps: the rows among `count` whose logits are wanted (None = the usual ones)
 
 
 @dataclass
