@@ -136,7 +136,7 @@ void matrix_state_scan(int64_t kind, const Tensor& r, const Tensor& k, const Ten
                                          opt_ld(beta), state.data_ptr<float>(), q_starts.data_ptr<int>(), seq_state.data_ptr<int>(),
                                          positions.data_ptr<int>(), y.data_ptr(), y.stride(0), (int)seq_state.numel(), (int)H, (int)DK, (int)DV,
                                          (int)kv_ratio, l2norm ? 1 : 0, (float)q_scale, opt_ptr(gate_raw), opt_ld(gate_raw), opt_f32(gate_A),
-                                         opt_f32(gate_dt_bias), cur_stream(), ty == at::kFloat ? 1 : 0);
+                                         opt_f32(gate_dt_bias), (int)r.size(0), cur_stream(), ty == at::kFloat ? 1 : 0);
   TORCH_CHECK(rc == 0, "matrix_state_scan: unsupported arguments (code ", rc, "): key width up to 256 (kind 2), 32 / 64 / 128 / 256 with 16-byte aligned bf16 rows (other kinds)");
 }
 

@@ -297,7 +297,7 @@ int matrix_state_scan(int kind, const void* r, long long ldr, const void* k, lon
                       const void* beta, long long ldbeta, float* state, const int* q_starts, const int* seq_state,
                       const int* positions, void* y, long long ldy, int B, int H, int DK, int DV, int kv_ratio, int l2norm,
                       float q_scale, const void* gate_raw, long long ldgate, const float* gate_A, const float* gate_dt_bias,
-                      cudaStream_t stream, int f32 = 0);
+                      int tokens, cudaStream_t stream, int f32 = 0);   // tokens: rows of the step (= B: single tokens)
 void gated_rmsnorm(const void* x, long long ldx, const void* z, long long ldz, const void* w, int wlen, void* y, long long ldy, int T,
                    int D, int group_size, float eps, int norm_before_gate, cudaStream_t stream, int f32 = 0);
 

@@ -3,7 +3,7 @@
 // follows a scan. The reference keeps one file per family (rust/engine/cuda/mamba1.cu, mamba2.cu, rwkv.cu,
 // deltanet.cu, kda.cu, shortconv.cu) and a chunk-parallel scan (scan.cu); here every family walks its tokens with the
 // state held in registers, one CTA per (sequence, head, slice of state rows): a step touches each state element
-// once, so the work per token is the state size and the per-token inputs are prefetched one token ahead. With 148 SMs
+// once, so the work per token is the state size and the per-token inputs are prefetched a token or a chunk ahead. With 148 SMs
 // the grid is sequences x heads x row tiles, which covers the machine from one 2048-token prefill chunk upwards.
 //
 // Batch layout (shared by every kernel): q_starts[B + 1] = first token row of each sequence, seq_state[B] = row of the
@@ -421,15 +421,12 @@ struct MatrixStateArgs {
   const T* gate_raw;
   long long ldgate;
   const float *gate_A, *gate_dt_bias;
-  int dk;                            // key width when it is below the kernel's (EXACT = false)
+  int dk;                            // key width (delta_scan_kernel below a full one)
 };
 
-// DKP key columns per row in registers. EXACT: the key width is DKP and every row is 16-byte aligned; otherwise the key
-// width is a.dk <= DKP, its missing columns are zeros in registers, and rows are read value by value.
-template <typename T, int KIND, int DKP, bool EXACT>
-__global__ void __launch_bounds__(128) matrix_state_kernel(const MatrixStateArgs<T> a) {
-  constexpr int NPT = 16, TPK = DKP / NPT, ROWS = 128 / TPK;
-  const int DK = EXACT ? DKP : a.dk;
+template <int KIND, int DK>
+__global__ void __launch_bounds__(128) matrix_state_kernel(const MatrixStateArgs<bf16> a) {
+  constexpr int NPT = 16, TPK = DK / NPT, ROWS = 128 / TPK;
   const int vtiles = (a.DV + ROWS - 1) / ROWS;
   const int h = blockIdx.x / vtiles, v = (blockIdx.x % vtiles) * ROWS + threadIdx.x / TPK;
   const int lk = threadIdx.x % TPK, s = blockIdx.y;
@@ -438,40 +435,25 @@ __global__ void __launch_bounds__(128) matrix_state_kernel(const MatrixStateArgs
   const bool valid = v < a.DV;
   const int vc = valid ? v : a.DV - 1;
   const int hk = h / a.kv_ratio;
-  const int nk = EXACT ? NPT : max(0, min(NPT, DK - lk * NPT));      // key columns of this lane
   float* st = a.state + (((long long)a.seq_state[s] * a.H + h) * a.DV + vc) * DK + lk * NPT;
   float S[NPT];
   if (a.positions[t0] == 0) {
 #pragma unroll
     for (int i = 0; i < NPT; ++i) S[i] = 0.f;
   } else {
-    if (EXACT) load_f32<NPT>(st, S);
-    else load_part<NPT>(st, nk, S);
+    load_f32<NPT>(st, S);
   }
   float u[NPT];
   if (KIND == kRwkv6) load_f32<NPT>(a.u + (long long)hk * DK + lk * NPT, u);
   const long long ko = (long long)hk * DK + lk * NPT;
   for (int t = t0; t < t0 + n; ++t) {
     float r[NPT], k[NPT], d[NPT];
-    if (EXACT) {
-      load_row<NPT>(a.r + t * a.ldr + ko, r);
-      load_row<NPT>(a.k + t * a.ldk + ko, k);
-    } else {
-      load_part<NPT>(a.r + t * a.ldr + ko, nk, r);
-      load_part<NPT>(a.k + t * a.ldk + ko, nk, k);
-    }
-    const float vv = ld1(a.v + t * a.ldv + (long long)h * a.DV + vc);
-    if (KIND == kGatedDelta) {
-      const float dh = a.w != nullptr
-                           ? exp_t<T>(a.w[t * a.ldw + h])
-                           : exp_t<T>(a.gate_A[h] * softplus_t<T>(ld1(a.gate_raw + t * a.ldgate + h) + a.gate_dt_bias[h]));
+    load_bf16<NPT>(a.r + t * a.ldr + ko, r);
+    load_bf16<NPT>(a.k + t * a.ldk + ko, k);
+    const float vv = __bfloat162float(a.v[t * a.ldv + (long long)h * a.DV + vc]);
+    load_f32<NPT>(a.w + t * a.ldw + ko, d);
 #pragma unroll
-      for (int i = 0; i < NPT; ++i) d[i] = dh;
-    } else {
-      load_f32<NPT>(a.w + t * a.ldw + ko, d);
-#pragma unroll
-      for (int i = 0; i < NPT; ++i) d[i] = exp_t<T>(d[i]);
-    }
+    for (int i = 0; i < NPT; ++i) d[i] = __expf(d[i]);
     float out = 0.f;
     if (KIND == kRwkv6) {
 #pragma unroll
@@ -483,8 +465,8 @@ __global__ void __launch_bounds__(128) matrix_state_kernel(const MatrixStateArgs
       out = row_sum<TPK>(out);
     } else if (KIND == kRwkv7) {
       float av[NPT], bv[NPT], sa = 0.f;
-      load_row<NPT>(a.a + t * a.lda + ko, av);
-      load_row<NPT>(a.b + t * a.ldb + ko, bv);
+      load_bf16<NPT>(a.a + t * a.lda + ko, av);
+      load_bf16<NPT>(a.b + t * a.ldb + ko, bv);
 #pragma unroll
       for (int i = 0; i < NPT; ++i) sa = fmaf(S[i], av[i], sa);
       sa = row_sum<TPK>(sa);
@@ -513,9 +495,7 @@ __global__ void __launch_bounds__(128) matrix_state_kernel(const MatrixStateArgs
         m = fmaf(S[i], k[i], m);
       }
       m = row_sum<TPK>(m);
-      float step = ld1(a.beta + t * a.ldbeta + h);
-      if (KIND == kGatedDelta && a.w == nullptr) step = 1.f / (1.f + exp_t<T>(-step));
-      const float delta = (vv - m) * step;
+      const float delta = (vv - m) * __bfloat162float(a.beta[t * a.ldbeta + h]);
 #pragma unroll
       for (int i = 0; i < NPT; ++i) {
         S[i] = fmaf(k[i], delta, S[i]);
@@ -523,16 +503,220 @@ __global__ void __launch_bounds__(128) matrix_state_kernel(const MatrixStateArgs
       }
       out = row_sum<TPK>(out) * qs;
     }
-    if (lk == 0 && valid) st1(a.y + t * a.ldy + (long long)h * a.DV + vc, out);
+    if (lk == 0 && valid) a.y[t * a.ldy + (long long)h * a.DV + vc] = __float2bfloat16(out);
   }
-  if (!valid) return;
-  if (EXACT) {
-    store_f32<NPT>(st, S);
-  } else {
+  if (valid) store_f32<NPT>(st, S);
+}
+
+// ------------------------------------------------------------------------------------------ gated delta rule
+// One CTA per (sequence, head, ROWS value rows); TPK lanes share RPT rows, lane l holding the key columns 4 (l + TPK j) + 0..3
+// of each (two rows per thread halve the shared-memory reads, which bound the walk).
+// Tokens come in chunks of kDeltaChunk: eight threads per token fetch q and k one chunk ahead into registers, normalise them
+// and leave them in shared memory as fp32 with the token's decay, step size and q . k, so the walk over a chunk touches
+// shared memory only. With m = S k and o = S q of the state before the token (one pass, two sums side by side):
+//   u = beta (v - d m);  S <- d S + u k;  y = d o + u (q . k)
+// which is the read-out behind the token's write. DKP: key columns in registers; EXACT: the key width is DKP and rows are
+// 16-byte aligned, otherwise it is a.dk <= DKP and rows are read value by value.
+constexpr int kDeltaChunk = 16, kDeltaRows = 2;
+
+// this lane's columns of a state row
+template <int TPK, bool EXACT>
+__device__ __forceinline__ void load_state(const float* st, int lk, int DK, float (&S)[16]) {
 #pragma unroll
-    for (int i = 0; i < NPT; ++i)
-      if (i < nk) st[i] = S[i];
+  for (int j = 0; j < 4; ++j) {
+    const int c = 4 * (lk + TPK * j);
+    if (EXACT) {
+      const float4 f = *reinterpret_cast<const float4*>(st + c);
+      S[4 * j] = f.x, S[4 * j + 1] = f.y, S[4 * j + 2] = f.z, S[4 * j + 3] = f.w;
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) S[4 * j + e] = c + e < DK ? st[c + e] : 0.f;
+    }
   }
+}
+template <int TPK, bool EXACT>
+__device__ __forceinline__ void store_state(float* st, int lk, int DK, const float (&S)[16]) {
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int c = 4 * (lk + TPK * j);
+    if (EXACT) {
+      *reinterpret_cast<float4*>(st + c) = make_float4(S[4 * j], S[4 * j + 1], S[4 * j + 2], S[4 * j + 3]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (c + e < DK) st[c + e] = S[4 * j + e];
+    }
+  }
+}
+
+template <typename T, int DKP, bool EXACT>
+__global__ void __launch_bounds__(128) delta_scan_kernel(const MatrixStateArgs<T> a) {
+  constexpr int NPT = 16, TPK = DKP / NPT, RPT = kDeltaRows, RG = 128 / TPK, ROWS = RPT * RG, C = kDeltaChunk, EPT = DKP / 8, VPT = ROWS * C / 128;
+  __shared__ __align__(16) float sk[C][DKP], sq[C][DKP];
+  __shared__ float sv[C][ROWS], sd[C], sb[C], skq[C];
+  const int DK = EXACT ? DKP : a.dk;
+  const int vtiles = (a.DV + ROWS - 1) / ROWS;
+  const int h = blockIdx.x / vtiles, v0 = (blockIdx.x % vtiles) * ROWS, row = threadIdx.x / TPK;      // rows v0 + row + RG r
+  const int lk = threadIdx.x % TPK, s = blockIdx.y;
+  const int t0 = a.q_starts[s], n = a.q_starts[s + 1] - t0;
+  if (n <= 0) return;
+  float* st = a.state + ((long long)a.seq_state[s] * a.H + h) * a.DV * DK;
+  float S[RPT][NPT];
+  const bool fresh = a.positions[t0] == 0;
+#pragma unroll
+  for (int r = 0; r < RPT; ++r) {
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) S[r][i] = 0.f;
+    if (!fresh) load_state<TPK, EXACT>(st + (long long)min(v0 + row + RG * r, a.DV - 1) * DK, lk, DK, S[r]);
+  }
+  // fetching: thread = (token tt of the chunk, share part of its row)
+  const int tt = threadIdx.x / 8, part = threadIdx.x % 8;
+  const long long ko = (long long)(h / a.kv_ratio) * DK + part * EPT;
+  const int np = EXACT ? EPT : max(0, min(EPT, DK - part * EPT));
+  float qr[EPT], kr[EPT], vr[VPT], gr = 0.f, br = 0.f;
+  auto fetch = [&](int base) {
+    const int left = n - base;
+    if (tt < left) {
+      const long long t = t0 + base + tt;
+      if constexpr (EXACT && EPT % 8 == 0) {
+        load_row<EPT>(a.r + t * a.ldr + ko, qr);
+        load_row<EPT>(a.k + t * a.ldk + ko, kr);
+      } else {
+        load_part<EPT>(a.r + t * a.ldr + ko, np, qr);
+        load_part<EPT>(a.k + t * a.ldk + ko, np, kr);
+      }
+      if (part == 0) {
+        gr = a.w != nullptr ? a.w[t * a.ldw + h] : ld1(a.gate_raw + t * a.ldgate + h);
+        br = ld1(a.beta + t * a.ldbeta + h);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int e = threadIdx.x + i * 128, tv = e / ROWS, rv = min(v0 + e % ROWS, a.DV - 1);
+      if (tv < left) vr[i] = ld1(a.v + (t0 + base + tv) * a.ldv + (long long)h * a.DV + rv);
+    }
+  };
+  fetch(0);
+  for (int base = 0; base < n; base += C) {
+    const int cnt = min(C, n - base);
+    __syncthreads();                                     // the chunk before is consumed
+    {
+      float qq = 0.f, kk = 0.f, qk = 0.f;
+#pragma unroll
+      for (int i = 0; i < EPT; ++i) qq = fmaf(qr[i], qr[i], qq), kk = fmaf(kr[i], kr[i], kk), qk = fmaf(qr[i], kr[i], qk);
+      qq = row_sum<8>(qq), kk = row_sum<8>(kk), qk = row_sum<8>(qk);
+      float qs = a.q_scale, ks = 1.f;
+      if (a.l2norm) qs *= 1.f / sqrtf(qq + 1e-6f), ks = 1.f / sqrtf(kk + 1e-6f);
+      if (tt < cnt) {
+#pragma unroll
+        for (int i = 0; i < EPT; ++i) sq[tt][part * EPT + i] = qr[i] * qs, sk[tt][part * EPT + i] = kr[i] * ks;
+        if (part == 0) {
+          const bool raw = a.w == nullptr;
+          sd[tt] = exp_t<T>(raw ? a.gate_A[h] * softplus_t<T>(gr + a.gate_dt_bias[h]) : gr);
+          sb[tt] = raw ? 1.f / (1.f + exp_t<T>(-br)) : br;
+          skq[tt] = qk * qs * ks;
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < VPT; ++i) {
+        const int e = threadIdx.x + i * 128;
+        if (e / ROWS < cnt) sv[e / ROWS][e % ROWS] = vr[i];
+      }
+    }
+    __syncthreads();
+    if (base + C < n) fetch(base + C);
+    T* yp = a.y + (long long)(t0 + base) * a.ldy + (long long)h * a.DV + v0 + row;
+#pragma unroll 2
+    for (int i = 0; i < cnt; ++i, yp += a.ldy) {
+      float4 k4[NPT / 4];
+      float m2[RPT][2] = {}, o2[RPT][2] = {};
+#pragma unroll
+      for (int j = 0; j < NPT / 4; ++j) {
+        k4[j] = *reinterpret_cast<const float4*>(&sk[i][4 * (lk + TPK * j)]);
+        const float4 q4 = *reinterpret_cast<const float4*>(&sq[i][4 * (lk + TPK * j)]);
+        const float *kf = &k4[j].x, *qf = &q4.x;
+#pragma unroll
+        for (int r = 0; r < RPT; ++r)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            m2[r][e & 1] = fmaf(S[r][4 * j + e], kf[e], m2[r][e & 1]);
+            o2[r][e & 1] = fmaf(S[r][4 * j + e], qf[e], o2[r][e & 1]);
+          }
+      }
+      const float d = sd[i], step = sb[i], kq = skq[i];
+#pragma unroll
+      for (int r = 0; r < RPT; ++r) {
+        const float m = row_sum<TPK>(m2[r][0] + m2[r][1]), o = row_sum<TPK>(o2[r][0] + o2[r][1]);
+        const float u = step * fmaf(-d, m, sv[i][row + RG * r]);
+#pragma unroll
+        for (int j = 0; j < NPT / 4; ++j) {
+          const float* kf = &k4[j].x;
+#pragma unroll
+          for (int e = 0; e < 4; ++e) S[r][4 * j + e] = fmaf(kf[e], u, d * S[r][4 * j + e]);
+        }
+        if (lk == 0 && v0 + row + RG * r < a.DV) st1(yp + RG * r, fmaf(d, o, u * kq));
+      }
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < RPT; ++r)
+    if (v0 + row + RG * r < a.DV) store_state<TPK, EXACT>(st + (long long)(v0 + row + RG * r) * DK, lk, DK, S[r]);
+}
+
+// The same recurrence for steps of single tokens (decode): one row per TPK lanes, inputs straight from global memory, no
+// shared memory, so that many CTAs keep state reads in flight (a decoded token reads and writes the whole state once).
+template <typename T, int DKP, bool EXACT>
+__global__ void __launch_bounds__(128) delta_decode_kernel(const MatrixStateArgs<T> a) {
+  constexpr int NPT = 16, TPK = DKP / NPT, ROWS = 128 / TPK;
+  const int DK = EXACT ? DKP : a.dk;
+  const int vtiles = (a.DV + ROWS - 1) / ROWS;
+  const int h = blockIdx.x / vtiles, v = (blockIdx.x % vtiles) * ROWS + threadIdx.x / TPK;
+  const int lk = threadIdx.x % TPK, s = blockIdx.y;
+  const int t0 = a.q_starts[s], n = a.q_starts[s + 1] - t0;
+  if (n <= 0) return;
+  const int vc = min(v, a.DV - 1);
+  float* st = a.state + (((long long)a.seq_state[s] * a.H + h) * a.DV + vc) * DK;
+  float S[NPT];
+#pragma unroll
+  for (int i = 0; i < NPT; ++i) S[i] = 0.f;
+  if (a.positions[t0] != 0) load_state<TPK, EXACT>(st, lk, DK, S);
+  const bool raw = a.w == nullptr;
+  for (long long t = t0; t < t0 + n; ++t) {
+    const T *qp = a.r + t * a.ldr + (long long)(h / a.kv_ratio) * DK, *kp = a.k + t * a.ldk + (long long)(h / a.kv_ratio) * DK;
+    float q[NPT], k[NPT];
+#pragma unroll
+    for (int j = 0; j < NPT / 4; ++j) {
+      const int c = 4 * (lk + TPK * j);
+#pragma unroll
+      for (int e = 0; e < 4; e += 2) {
+        float2 q2 = make_float2(0.f, 0.f), k2 = q2;
+        if (EXACT) {
+          q2 = ld2(qp + c + e), k2 = ld2(kp + c + e);
+        } else {
+          if (c + e < DK) q2.x = ld1(qp + c + e), k2.x = ld1(kp + c + e);
+          if (c + e + 1 < DK) q2.y = ld1(qp + c + e + 1), k2.y = ld1(kp + c + e + 1);
+        }
+        q[4 * j + e] = q2.x, q[4 * j + e + 1] = q2.y, k[4 * j + e] = k2.x, k[4 * j + e + 1] = k2.y;
+      }
+    }
+    const float g = raw ? ld1(a.gate_raw + t * a.ldgate + h) : a.w[t * a.ldw + h], b = ld1(a.beta + t * a.ldbeta + h);
+    const float vv = ld1(a.v + t * a.ldv + (long long)h * a.DV + vc);
+    float qq = 0.f, kk = 0.f, qk = 0.f, m = 0.f, o = 0.f;
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) {
+      qq = fmaf(q[i], q[i], qq), kk = fmaf(k[i], k[i], kk), qk = fmaf(q[i], k[i], qk);
+      m = fmaf(S[i], k[i], m), o = fmaf(S[i], q[i], o);
+    }
+    qk = row_sum<TPK>(qk), m = row_sum<TPK>(m), o = row_sum<TPK>(o);
+    float qs = a.q_scale, ks = 1.f;
+    if (a.l2norm) qs *= 1.f / sqrtf(row_sum<TPK>(qq) + 1e-6f), ks = 1.f / sqrtf(row_sum<TPK>(kk) + 1e-6f);
+    const float d = exp_t<T>(raw ? a.gate_A[h] * softplus_t<T>(g + a.gate_dt_bias[h]) : g), step = raw ? 1.f / (1.f + exp_t<T>(-b)) : b;
+    const float u = step * fmaf(-d, m * ks, vv);
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) S[i] = fmaf(k[i] * ks, u, d * S[i]);
+    if (lk == 0 && v < a.DV) st1(a.y + t * a.ldy + (long long)h * a.DV + v, qs * fmaf(d, o, u * qk * ks));
+  }
+  if (v < a.DV) store_state<TPK, EXACT>(st, lk, DK, S);
 }
 
 // ------------------------------------------------------------------------------------------ gated RMSNorm
@@ -748,7 +932,7 @@ int matrix_state_scan(int kind, const void* r, long long ldr, const void* k, lon
                       const void* beta, long long ldbeta, float* state, const int* q_starts, const int* seq_state,
                       const int* positions, void* y, long long ldy, int B, int H, int DK, int DV, int kv_ratio, int l2norm,
                       float q_scale, const void* gate_raw, long long ldgate, const float* gate_A, const float* gate_dt_bias,
-                      cudaStream_t stream, int f32) {
+                      int tokens, cudaStream_t stream, int f32) {
   if (B <= 0) return 0;
   if (kv_ratio <= 0 || H % kv_ratio || DK <= 0) return -1;
   const int unit = f32 ? 4 : 8;
@@ -766,27 +950,36 @@ int matrix_state_scan(int kind, const void* r, long long ldr, const void* k, lon
                               q_starts, seq_state, positions, static_cast<T*>(y), H, DV, kv_ratio, l2norm, q_scale,
                               static_cast<const T*>(gate_raw), ldgate, gate_A, gate_dt_bias, DK};
   };
-#define FLLM_MS(T_, KIND_, DK_, EXACT_)                                                                           \
-  {                                                                                                               \
-    constexpr int rows = 128 / (DK_ / 16);                                                                        \
-    matrix_state_kernel<T_, KIND_, DK_, EXACT_><<<dim3(H * ((DV + rows - 1) / rows), B), 128, 0, stream>>>(args(T_{})); \
-    return 0;                                                                                                     \
+#define FLLM_MS(KIND_, DK_)                                                                                          \
+  {                                                                                                                  \
+    constexpr int rows = 128 / (DK_ / 16);                                                                           \
+    matrix_state_kernel<KIND_, DK_><<<dim3(H * ((DV + rows - 1) / rows), B), 128, 0, stream>>>(args(bf16{}));        \
+    return 0;                                                                                                        \
   }
-#define FLLM_MS_DK(KIND_)                       \
-  switch (DK) {                                 \
-    case 32: FLLM_MS(bf16, KIND_, 32, true)     \
-    case 64: FLLM_MS(bf16, KIND_, 64, true)     \
-    case 128: FLLM_MS(bf16, KIND_, 128, true)   \
-    case 256: FLLM_MS(bf16, KIND_, 256, true)   \
-    default: return -2;                         \
+#define FLLM_MS_DK(KIND_)           \
+  switch (DK) {                     \
+    case 32: FLLM_MS(KIND_, 32)     \
+    case 64: FLLM_MS(KIND_, 64)     \
+    case 128: FLLM_MS(KIND_, 128)   \
+    case 256: FLLM_MS(KIND_, 256)   \
+    default: return -2;             \
   }
-#define FLLM_GD(T_, EXACT_)                                  \
-  {                                                          \
-    if (DK <= 16) FLLM_MS(T_, kGatedDelta, 16, EXACT_)       \
-    if (DK <= 32) FLLM_MS(T_, kGatedDelta, 32, EXACT_)       \
-    if (DK <= 64) FLLM_MS(T_, kGatedDelta, 64, EXACT_)       \
-    if (DK <= 128) FLLM_MS(T_, kGatedDelta, 128, EXACT_)     \
-    FLLM_MS(T_, kGatedDelta, 256, EXACT_)                    \
+#define FLLM_DS(T_, DK_, EXACT_)                                                                                     \
+  {                                                                                                                  \
+    constexpr int rows = 128 / (DK_ / 16);                                                                           \
+    if (tokens == B)                                                                                                 \
+      delta_decode_kernel<T_, DK_, EXACT_><<<dim3(H * ((DV + rows - 1) / rows), B), 128, 0, stream>>>(args(T_{}));   \
+    else                                                                                                             \
+      delta_scan_kernel<T_, DK_, EXACT_><<<dim3(H * ((DV + kDeltaRows * rows - 1) / (kDeltaRows * rows)), B), 128, 0, stream>>>(args(T_{})); \
+    return 0;                                                                                                        \
+  }
+#define FLLM_GD(T_, EXACT_)                  \
+  {                                          \
+    if (DK <= 16) FLLM_DS(T_, 16, EXACT_)    \
+    if (DK <= 32) FLLM_DS(T_, 32, EXACT_)    \
+    if (DK <= 64) FLLM_DS(T_, 64, EXACT_)    \
+    if (DK <= 128) FLLM_DS(T_, 128, EXACT_)  \
+    FLLM_DS(T_, 256, EXACT_)                 \
   }
   switch (kind) {
     case kRwkv6: FLLM_MS_DK(kRwkv6)
@@ -801,6 +994,7 @@ int matrix_state_scan(int kind, const void* r, long long ldr, const void* k, lon
       FLLM_GD(bf16, false)
   }
 #undef FLLM_GD
+#undef FLLM_DS
 #undef FLLM_MS_DK
 #undef FLLM_MS
   return -3;
