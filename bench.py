@@ -157,7 +157,21 @@ def main() -> None:
     ap.add_argument("--profile-step", action="store_true",
                     help="bracket ONE replay of the decode step with cudaProfilerStart/Stop (for a profiler's "
                          "launch list, run with --profile-from-start off) and exit")
+    ap.add_argument("--compare", default=None, choices=["sovanex"],
+                    help="instead of the workload above: prefill and decode throughput of this design beside the closest other "
+                         "model at equal sizes (random weights), one JSON line")
+    ap.add_argument("--sizes", default="1b,3b,7b", help="with --compare: model sizes")
+    ap.add_argument("--kernels", action="store_true", help="with --compare: also the kernels that differ, beside their like kernels")
     args = ap.parse_args()
+    if args.compare:
+        from fllm_b200.bench_compare import main as compare_main
+        args.warmup = max(args.warmup, 3)
+        sampler = ClockSampler(0)
+        sampler.start()
+        out = compare_main(args)
+        out["clocks"] = sampler.stop()
+        print(json.dumps(out))
+        return
     if args.impl == "reference":
         if int(os.environ.get("RANK", "0")) == 0:
             reference_arm(args)

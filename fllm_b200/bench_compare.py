@@ -1,0 +1,201 @@
+"""Throughput of a design beside the framework's closest other model at equal size (``bench.py --compare sovanex``).
+
+The closest other model of Sovanex is a hybrid of the layer kinds it shares with other families: the gated delta rule
+(Qwen3-Next) and 512 + 64 wide latent attention (DeepSeek), with the same layer order, heads, widths and squared-ReLU
+networks, but RMSNorm around one bf16 residual, no gate on the attention heads and no shared rows. Both run random
+weights through the engine: prompts of 1024 tokens in 2048-token steps, then captured decode steps. ``--kernels`` times
+the kernels that differ, each beside its like kernel on the same sizes.
+"""
+from __future__ import annotations
+
+import dataclasses
+import statistics
+from typing import Dict, List
+
+import torch
+
+from .config import EngineConfig, ModelConfig, sovanex_from_config
+
+# name -> width, layers, feed-forward width, value heads / key heads of the delta rule, attention heads
+SIZES = {"1b": (2048, 12, 8192, 32, 16, 16), "3b": (3072, 24, 12288, 48, 24, 24), "7b": (4096, 32, 16384, 64, 32, 32)}
+VOCAB = 65536
+
+
+def sovanex_config(size: str) -> ModelConfig:
+    W, L, ff, Hv, Hk, Ha = SIZES[size]
+    layers = []
+    for i in range(L):
+        if i % 4 < 3:
+            mixer = dict(heads=Hv, kv_heads=Hk, dim=128, vdim=128, conv=4)
+        else:
+            mixer = dict(heads=Ha, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, rot=dict(base=1e6, dims=64))
+            if i % 8 == 7:
+                mixer["kv_from"] = i - 4
+        layers.append(dict(type="delta" if i % 4 < 3 else "latent_attention", mixer=mixer, mlp=dict(kind="dense", ff=ff)))
+    return sovanex_from_config(ModelConfig, dict(architecture="Sovanex", name=f"sovanex-{size}", layers=layers, norm=dict(eps=1e-5),
+                                                 residual_mult=0.25, streams=4, vocab=VOCAB, width=W))
+
+
+def twin_config(size: str) -> ModelConfig:
+    W, L, ff, Hv, Hk, Ha = SIZES[size]
+    return ModelConfig(arch="hybrid", name=f"delta-mla-hybrid-{size}", vocab_size=VOCAB, hidden_size=W, num_layers=L, num_heads=Ha, num_kv_heads=1,
+                       head_dim=192, rotary_dim=64, rope_style="pair", intermediate_size=ff, mlp_kind="plain", act="relu2", tie_embeddings=True,
+                       layer_kinds=["gated_delta" if i % 4 < 3 else "mla" for i in range(L)],
+                       ssm=dict(num_k_heads=Hk, num_v_heads=Hv, head_k_dim=128, head_v_dim=128, d_conv=4),
+                       mla=dict(q_lora_rank=0, kv_lora_rank=512, qk_nope_head_dim=128, qk_rope_head_dim=64, v_head_dim=128))
+
+
+def throughput(cfg: ModelConfig, batch: int, prompt_len: int, steps: int, warmup: int, device, graphs: bool = True) -> Dict[str, float]:
+    """Device-timed prefill and decode of ``batch`` requests (CUDA events around whole engine steps / graph replays)."""
+    from .runtime import LLMEngine, SamplingParams
+    # sequences that prefill first decode along while the others are still prefilled
+    room = batch * prompt_len // 2048 + warmup + steps + 16
+    ec = EngineConfig(max_num_seqs=batch, max_num_batched_tokens=2048, max_model_len=prompt_len + room, enable_prefix_caching=False, use_cuda_graphs=graphs)
+    ec.num_kv_blocks = batch * (-(-ec.max_model_len // ec.block_size)) * 11 // 10 + 16
+    eng = LLMEngine(cfg, ec, device=device)
+    g = torch.Generator().manual_seed(7)
+    prompts = [torch.randint(0, cfg.vocab_size, (prompt_len,), generator=g).tolist() for _ in range(batch)]
+    sp = SamplingParams(max_tokens=room, ignore_eos=True)
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    eng.generate(prompts[:2], dataclasses.replace(sp, max_tokens=2))          # warm-up of both step kinds
+    for p in prompts:
+        eng.add_request(p, sp)
+    torch.cuda.synchronize()
+    e0.record()
+    while any(not r.output for r in eng.requests.values()):
+        eng.step()
+    e1.record()
+    torch.cuda.synchronize()
+    prefill = batch * prompt_len / (e0.elapsed_time(e1) / 1e3)
+    for _ in range(warmup):
+        eng.step()
+    eng.drain()
+    graph = eng._graphs[eng._bucket_for(batch)]
+    step = eng.scheduler.schedule()
+    eng._build_batch(step, pad_to=graph.bucket)
+    torch.cuda.synchronize()
+    e0.record()
+    for _ in range(steps):
+        graph.replay()
+    e1.record()
+    torch.cuda.synchronize()
+    ms = e0.elapsed_time(e1) / steps
+    status = eng.ops.check_status()
+    launches = graph.launches
+    eng.close()
+    del eng, graph
+    torch.cuda.empty_cache()
+    return {"prefill_tok_s": round(prefill, 1), "decode_tok_s": round(batch / (ms / 1e3), 1), "decode_ms": round(ms, 4), "launches_per_step": launches,
+            "status": status}
+
+
+# ------------------------------------------------------------------------------------------------ kernels
+def _time(fn, flush, n: int = 15) -> float:
+    """Median microseconds with a cold L2 (CUDA events on the launching stream)."""
+    for _ in range(3):
+        fn()
+    out = []
+    for _ in range(n):
+        flush.zero_()
+        torch.cuda._sleep(200000)                  # the host queues the launch while the device is busy
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        fn()
+        b.record()
+        torch.cuda.synchronize()
+        out.append(a.elapsed_time(b) * 1e3)
+    return statistics.median(out)
+
+
+def _batch(lens: List[int], ctxs: List[int], device, bs: int = 16):
+    from types import SimpleNamespace
+    B, mb = len(lens), max(-(-c // bs) for c in ctxs)
+    i32 = lambda t: t.to(device=device, dtype=torch.int32)
+    tab = torch.randperm(B * mb).view(B, mb)
+    starts = [0]
+    for n in lens:
+        starts.append(starts[-1] + n)
+    pos = torch.cat([torch.arange(c - n, c) for n, c in zip(lens, ctxs)])
+    slots = torch.cat([tab[i, torch.arange(c - n, c) // bs] * bs + torch.arange(c - n, c) % bs for i, (n, c) in enumerate(zip(lens, ctxs))])
+    return SimpleNamespace(num_seqs=B, max_q_len=max(lens), max_kv_len=max(ctxs), positions=i32(pos), slots=i32(slots), blocks=B * mb,
+                           row_seq=i32(torch.cat([torch.full((n,), i) for i, n in enumerate(lens)])), block_tables=i32(tab),
+                           q_starts=i32(torch.tensor(starts)), seq_state=i32(torch.arange(B)), tokens=starts[-1])
+
+
+def kernel_table(device, size: str = "1b") -> List[dict]:
+    """Kernels of the new layers beside their like kernels: microseconds, the floor of each (bytes at the measured copy
+    bandwidth or products at the measured GEMM rate, whichever is longer), and the ratio of the two distances."""
+    import json
+    import os
+    from .ops.native import NativeOps
+    ops, bf, g = NativeOps(device), torch.bfloat16, torch.Generator(device=device).manual_seed(1)
+    peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+    path = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "MEASURED_PEAKS.json")
+    if os.path.exists(path):
+        peaks.update({k: v for k, v in json.load(open(path)).items() if k in peaks})
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=device)
+    W, _, ff, Hv, Hk, H = SIZES[size]
+    R, dr, dn, S = 512, 64, 128, 4
+    rnd = lambda *s, dtype=bf: torch.randn(*s, device=device, generator=g).to(dtype)
+    rows = []
+
+    def floor(nbytes, flops=0.0):
+        return max(nbytes / peaks["hbm_gbs"] / 1e3, flops / peaks["bf16_tflops"] / 1e6)
+
+    def add(shape, name, us, fl, like, like_us, like_fl):
+        rows.append({"shape": shape, "kernel": name, "us": round(us, 1), "floor_us": round(fl, 2), "like": like, "like_us": round(like_us, 1),
+                     "like_floor_us": round(like_fl, 2), "times_as_far": round((us / fl) / (like_us / like_fl), 2)})
+
+    for shape, lens, ctxs in (("decode 64 x 1152", [1] * 64, [1152] * 64), ("decode 8 x 4096", [1] * 8, [4096] * 8),
+                              ("prompt 2048", [2048], [2048]), ("prompt 4 x 512 at 2048", [512] * 4, [2048] * 4)):
+        b = _batch(lens, ctxs, device)
+        T = b.tokens
+        cache, q = rnd(b.blocks, 16, R + dr), rnd(H, T, R + dr)
+        qa, qp = q[:, :, :R].contiguous(), q[:, :, R:].transpose(0, 1).contiguous()
+        keys = sum(c * n - n * (n - 1) // 2 for n, c in zip(lens, ctxs))
+        fl = floor(2 * (sum(ctxs) * (R + dr) + q.numel() + H * T * R), 2.0 * keys * H * (2 * R + dr))
+        add(shape, "attention_latent", _time(lambda: ops.attention_latent(q, cache, b, 0.07, R), flush), fl, "attention_mla",
+            _time(lambda: ops.attention_mla(qa, qp, cache, b.block_tables, b.row_seq, b.positions, 0.07, b.max_kv_len), flush), fl)
+        ckv, qh, inv, nw = rnd(T, R + dr), rnd(T, H * (dn + dr)), torch.rand(dr // 2, device=device), torch.ones(R, device=device, dtype=bf)
+        fl = floor(2 * T * (2 * (R + dr) + 2 * H * dr))
+        add(shape, "latent_prepare", _time(lambda: ops.latent_prepare(ckv, qh, dn + dr, dn, b.positions, b.slots, inv, 1.0, nw, 1e-5, cache, q, R, 0), flush), fl,
+            "mla_prepare", _time(lambda: ops.mla_prepare(ckv, qh.view(T, H, dn + dr), dn, b.positions, b.slots, inv, 1.0, nw, 1e-5, cache), flush), fl)
+    for T in (64, 2048):
+        shape = f"{T} rows"
+        x, y, res = rnd(T, S, W, dtype=torch.float32), rnd(T, W), rnd(T, W)
+        mix, vec, w = torch.eye(S, device=device), torch.ones(S, device=device), torch.ones(W, device=device, dtype=bf)
+        add(shape, "streams_step (4 fp32 streams, LayerNorm)", _time(lambda: ops.streams_step(x, y, mix, vec, vec, w, w, W, 1e-5), flush),
+            floor(T * W * (8 * S + 4)), "residual add + rmsnorm", _time(lambda: ops.rmsnorm(res, y, w, 1e-5), flush), floor(T * W * 8))
+        add(shape, "streams_step (4 fp32 streams, LayerNorm)", _time(lambda: ops.streams_step(x, y, mix, vec, vec, w, w, W, 1e-5), flush),
+            floor(T * W * (8 * S + 4)), "residual add + layernorm", _time(lambda: ops.layernorm(res, y, w, w, 1e-5), flush), floor(T * W * 8))
+        o, gate = rnd(H, T, 128), rnd(T, H)
+        add(shape, "head_gate", _time(lambda: ops.head_gate(o, gate, H * 128), flush), floor(T * H * 512), "transposing copy",
+            _time(lambda: o.transpose(0, 1).reshape(T, H * 128), flush), floor(T * H * 512))
+        D = 128
+        b = _batch([1] * T if T == 64 else [T], [1024] * T if T == 64 else [T], device)
+        qkv, gates = rnd(T, (2 * Hk + Hv) * D), rnd(T, 2 * Hv)
+        st = torch.zeros(b.num_seqs, Hv, D, D, device=device)
+        A, db = -torch.rand(Hv, device=device), torch.zeros(Hv, device=device)
+        K = Hk * D
+        us = _time(lambda: ops.matrix_state_scan(2, qkv[:, :K], qkv[:, K:2 * K], qkv[:, 2 * K:], None, None, None, None, gates[:, :Hv], st, b.q_starts,
+                                                 b.seq_state, b.positions, Hv, D, D, Hv // Hk, True, D ** -0.5, gate_raw=gates[:, Hv:], gate_A=A,
+                                                 gate_dt_bias=db), flush)
+        fl = floor(st.numel() * 8 + 2 * T * ((2 * Hk + 2 * Hv) * D))
+        add(shape, "gated delta scan", us, fl, "the same kernel", us, fl)
+    return rows
+
+
+def main(args) -> dict:
+    """``args``: design, sizes, steps, warmup, batch, prompt_len, kernels (see bench.py)."""
+    device = torch.device("cuda", 0)
+    torch.cuda.set_device(device)
+    out = {"compare": args.compare, "data": "synthetic (uniform random token ids, random weights)", "prompt_len": args.prompt_len or 1024,
+           "steps": args.steps, "warmup": args.warmup, "throughput": []}
+    for size in args.sizes.split(","):
+        for cfg in (sovanex_config(size), twin_config(size)):
+            for batch in ([args.batch] if args.batch else [8, 64]):
+                r = throughput(cfg, batch, out["prompt_len"], args.steps, args.warmup, device)
+                out["throughput"].append({"model": cfg.name, "batch": batch, **r})
+    if args.kernels:
+        out["kernels"] = kernel_table(device)
+    return out

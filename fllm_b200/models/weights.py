@@ -306,7 +306,8 @@ def init_random_weights(cfg: ModelConfig, device="cpu", dtype=torch.bfloat16, se
                     lw.shared_down = full((H, Is), li, 28)
             elif has_ffn:
                 I = cfg.intermediate_size
-                lw.w_gate_up = torch.cat([full((I, H), li, 4), full((I, H), li, 5)], 0).contiguous()
+                lw.w_gate_up = full((I, H), li, 4) if cfg.mlp_kind == "plain" else \
+                    torch.cat([full((I, H), li, 4), full((I, H), li, 5)], 0).contiguous()
                 lw.w_down = full((H, I), li, 6)
             out_layers.append(lw)
             continue
