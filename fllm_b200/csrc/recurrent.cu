@@ -553,7 +553,8 @@ template <typename T, int DKP, bool EXACT>
 __global__ void __launch_bounds__(128) delta_scan_kernel(const MatrixStateArgs<T> a) {
   constexpr int NPT = 16, TPK = DKP / NPT, RPT = kDeltaRows, RG = 128 / TPK, ROWS = RPT * RG, C = kDeltaChunk, EPT = DKP / 8, VPT = ROWS * C / 128;
   __shared__ __align__(16) float sk[C][DKP], sq[C][DKP];
-  __shared__ float sv[C][ROWS], sd[C], sb[C], skq[C];
+  __shared__ float sv[C][ROWS];
+  __shared__ float4 sg[C];                               // decay, step size, q . k
   const int DK = EXACT ? DKP : a.dk;
   const int vtiles = (a.DV + ROWS - 1) / ROWS;
   const int h = blockIdx.x / vtiles, v0 = (blockIdx.x % vtiles) * ROWS, row = threadIdx.x / TPK;      // rows v0 + row + RG r
@@ -569,31 +570,47 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const MatrixStateArgs<T
     for (int i = 0; i < NPT; ++i) S[r][i] = 0.f;
     if (!fresh) load_state<TPK, EXACT>(st + (long long)min(v0 + row + RG * r, a.DV - 1) * DK, lk, DK, S[r]);
   }
-  // fetching: thread = (token tt of the chunk, share part of its row)
+  // fetching: thread = (token tt of the chunk, share part of its row); values stay in their stored form until they are
+  // staged, so that no conversion waits for the loads while the chunk before is walked. Shares are groups of eight values
+  // (the shared-memory stores of a token's eight threads then spread over the banks).
+  constexpr bool WIDE = EXACT && EPT % 8 == 0;
+  constexpr int WORDS = WIDE ? EPT * (int)sizeof(T) / 16 : 1, LOOSE = WIDE ? 1 : EPT, PER8 = (int)sizeof(T) / 2;      // 16-byte words per group
   const int tt = threadIdx.x / 8, part = threadIdx.x % 8;
-  const long long ko = (long long)(h / a.kv_ratio) * DK + part * EPT;
-  const int np = EXACT ? EPT : max(0, min(EPT, DK - part * EPT));
-  float qr[EPT], kr[EPT], vr[VPT], gr = 0.f, br = 0.f;
+  const long long ko = (long long)(h / a.kv_ratio) * DK;
+  auto column = [&](int i) { return EPT % 8 == 0 ? 8 * (part + 8 * (i / 8)) + i % 8 : part * EPT + i; };
+  uint4 qw[WORDS], kw[WORDS];
+  float ql[LOOSE], kl[LOOSE], wr = 0.f;
+  T vr[VPT], gr{}, br{};
   auto fetch = [&](int base) {
     const int left = n - base;
     if (tt < left) {
       const long long t = t0 + base + tt;
-      if constexpr (EXACT && EPT % 8 == 0) {
-        load_row<EPT>(a.r + t * a.ldr + ko, qr);
-        load_row<EPT>(a.k + t * a.ldk + ko, kr);
+      const T *qp = a.r + t * a.ldr + ko, *kp = a.k + t * a.ldk + ko;
+      if constexpr (WIDE) {
+#pragma unroll
+        for (int i = 0; i < WORDS; ++i) {
+          const int c = 8 * (part + 8 * (i / PER8)) + (i % PER8) * (16 / (int)sizeof(T));
+          qw[i] = *reinterpret_cast<const uint4*>(qp + c);
+          kw[i] = *reinterpret_cast<const uint4*>(kp + c);
+        }
       } else {
-        load_part<EPT>(a.r + t * a.ldr + ko, np, qr);
-        load_part<EPT>(a.k + t * a.ldk + ko, np, kr);
+#pragma unroll
+        for (int i = 0; i < EPT; ++i) {
+          const int c = column(i);
+          ql[i] = c < DK ? ld1(qp + c) : 0.f;
+          kl[i] = c < DK ? ld1(kp + c) : 0.f;
+        }
       }
       if (part == 0) {
-        gr = a.w != nullptr ? a.w[t * a.ldw + h] : ld1(a.gate_raw + t * a.ldgate + h);
-        br = ld1(a.beta + t * a.ldbeta + h);
+        if (a.w != nullptr) wr = a.w[t * a.ldw + h];
+        else gr = a.gate_raw[t * a.ldgate + h];
+        br = a.beta[t * a.ldbeta + h];
       }
     }
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
       const int e = threadIdx.x + i * 128, tv = e / ROWS, rv = min(v0 + e % ROWS, a.DV - 1);
-      if (tv < left) vr[i] = ld1(a.v + (t0 + base + tv) * a.ldv + (long long)h * a.DV + rv);
+      if (tv < left) vr[i] = a.v[(t0 + base + tv) * a.ldv + (long long)h * a.DV + rv];
     }
   };
   fetch(0);
@@ -601,6 +618,15 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const MatrixStateArgs<T
     const int cnt = min(C, n - base);
     __syncthreads();                                     // the chunk before is consumed
     {
+      float qr[EPT], kr[EPT];
+      if constexpr (WIDE) {
+        const T *qt = reinterpret_cast<const T*>(qw), *kt = reinterpret_cast<const T*>(kw);
+#pragma unroll
+        for (int i = 0; i < EPT; ++i) qr[i] = ld1(qt + i), kr[i] = ld1(kt + i);
+      } else {
+#pragma unroll
+        for (int i = 0; i < EPT; ++i) qr[i] = ql[i], kr[i] = kl[i];
+      }
       float qq = 0.f, kk = 0.f, qk = 0.f;
 #pragma unroll
       for (int i = 0; i < EPT; ++i) qq = fmaf(qr[i], qr[i], qq), kk = fmaf(kr[i], kr[i], kk), qk = fmaf(qr[i], kr[i], qk);
@@ -608,33 +634,57 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const MatrixStateArgs<T
       float qs = a.q_scale, ks = 1.f;
       if (a.l2norm) qs *= 1.f / sqrtf(qq + 1e-6f), ks = 1.f / sqrtf(kk + 1e-6f);
       if (tt < cnt) {
+        if constexpr (EPT % 4 == 0) {
 #pragma unroll
-        for (int i = 0; i < EPT; ++i) sq[tt][part * EPT + i] = qr[i] * qs, sk[tt][part * EPT + i] = kr[i] * ks;
+          for (int i = 0; i < EPT; i += 4) {
+            *reinterpret_cast<float4*>(&sq[tt][column(i)]) = make_float4(qr[i] * qs, qr[i + 1] * qs, qr[i + 2] * qs, qr[i + 3] * qs);
+            *reinterpret_cast<float4*>(&sk[tt][column(i)]) = make_float4(kr[i] * ks, kr[i + 1] * ks, kr[i + 2] * ks, kr[i + 3] * ks);
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < EPT; ++i) sq[tt][column(i)] = qr[i] * qs, sk[tt][column(i)] = kr[i] * ks;
+        }
         if (part == 0) {
           const bool raw = a.w == nullptr;
-          sd[tt] = exp_t<T>(raw ? a.gate_A[h] * softplus_t<T>(gr + a.gate_dt_bias[h]) : gr);
-          sb[tt] = raw ? 1.f / (1.f + exp_t<T>(-br)) : br;
-          skq[tt] = qk * qs * ks;
+          sg[tt] = make_float4(exp_t<T>(raw ? a.gate_A[h] * softplus_t<T>(ld1(&gr) + a.gate_dt_bias[h]) : wr),
+                               raw ? 1.f / (1.f + exp_t<T>(-ld1(&br))) : ld1(&br), qk * qs * ks, 0.f);
         }
       }
 #pragma unroll
       for (int i = 0; i < VPT; ++i) {
         const int e = threadIdx.x + i * 128;
-        if (e / ROWS < cnt) sv[e / ROWS][e % ROWS] = vr[i];
+        if (e / ROWS < cnt) sv[e / ROWS][e % ROWS] = ld1(&vr[i]);
       }
     }
     __syncthreads();
     if (base + C < n) fetch(base + C);
     T* yp = a.y + (long long)(t0 + base) * a.ldy + (long long)h * a.DV + v0 + row;
-#pragma unroll 2
-    for (int i = 0; i < cnt; ++i, yp += a.ldy) {
-      float4 k4[NPT / 4];
-      float m2[RPT][2] = {}, o2[RPT][2] = {};
+    float4 kn[NPT / 4], qn[NPT / 4], gn = sg[0];           // the next token's rows travel while this one is applied
+    float vn[RPT];
+    auto rows_of = [&](int i) {
 #pragma unroll
       for (int j = 0; j < NPT / 4; ++j) {
-        k4[j] = *reinterpret_cast<const float4*>(&sk[i][4 * (lk + TPK * j)]);
-        const float4 q4 = *reinterpret_cast<const float4*>(&sq[i][4 * (lk + TPK * j)]);
-        const float *kf = &k4[j].x, *qf = &q4.x;
+        kn[j] = *reinterpret_cast<const float4*>(&sk[i][4 * (lk + TPK * j)]);
+        qn[j] = *reinterpret_cast<const float4*>(&sq[i][4 * (lk + TPK * j)]);
+      }
+      gn = sg[i];
+#pragma unroll
+      for (int r = 0; r < RPT; ++r) vn[r] = sv[i][row + RG * r];
+    };
+    rows_of(0);
+#pragma unroll 2
+    for (int i = 0; i < cnt; ++i, yp += a.ldy) {
+      float4 k4[NPT / 4], q4[NPT / 4];
+      float m2[RPT][2] = {}, o2[RPT][2] = {}, vv[RPT];
+      const float d = gn.x, step = gn.y, kq = gn.z;
+#pragma unroll
+      for (int j = 0; j < NPT / 4; ++j) k4[j] = kn[j], q4[j] = qn[j];
+#pragma unroll
+      for (int r = 0; r < RPT; ++r) vv[r] = vn[r];
+      rows_of(min(i + 1, cnt - 1));
+#pragma unroll
+      for (int j = 0; j < NPT / 4; ++j) {
+        const float *kf = &k4[j].x, *qf = &q4[j].x;
 #pragma unroll
         for (int r = 0; r < RPT; ++r)
 #pragma unroll
@@ -643,11 +693,10 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const MatrixStateArgs<T
             o2[r][e & 1] = fmaf(S[r][4 * j + e], qf[e], o2[r][e & 1]);
           }
       }
-      const float d = sd[i], step = sb[i], kq = skq[i];
 #pragma unroll
       for (int r = 0; r < RPT; ++r) {
         const float m = row_sum<TPK>(m2[r][0] + m2[r][1]), o = row_sum<TPK>(o2[r][0] + o2[r][1]);
-        const float u = step * fmaf(-d, m, sv[i][row + RG * r]);
+        const float u = step * fmaf(-d, m, vv[r]);
 #pragma unroll
         for (int j = 0; j < NPT / 4; ++j) {
           const float* kf = &k4[j].x;
