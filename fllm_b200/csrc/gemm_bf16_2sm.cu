@@ -127,9 +127,9 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tma_x, const __grid_co
   cluster_sync();                                     // the peer's barriers exist before anything arrives on them
   tc_fence_after_sync();
   const uint32_t tmem_base = *tmem_slot;
-  // No early trigger for the dependents: a kernel of single CTAs that allocates tensor memory on the SM one CTA of a pair
-  // has left, while the other still frees the pair's columns, was seen to stall. The next kernel starts when the whole
-  // grid is done.
+  // No early trigger for the dependents: with one, steps stalled at random where a one-CTA GEMM followed closely. Its
+  // CTAs could allocate tensor memory on an SM that one CTA of a pair had left while the other still freed the pair's
+  // columns. The next kernel starts when the whole grid is done.
 
   const int tiles = p.m_tiles * p.n_tiles;
   const int n_clusters = gridDim.x >> 1, cluster_id = blockIdx.x >> 1;
