@@ -30,6 +30,9 @@ class RopeScaling:
     freq_factors: Optional[List[float]] = None
 
 
+STATELESS_KINDS = ("attention", "mla", "tied", "none")       # layer kinds without a recurrent state
+
+
 @dataclass
 class ModelConfig:
     arch: str = "llama"                  # llama | qwen3 | gpt_oss
@@ -98,7 +101,7 @@ class ModelConfig:
     # layer has a gated FFN behind it ("glu") or is the mixer alone ("none"); `ssm` holds the mixer shapes
     # (d_inner, d_state, d_conv, n_groups, head_dim, n_heads, dt_rank, norm_groups, dt_min, dt_max, conv_bias,
     # num_k_heads, num_v_heads, head_k_dim, head_v_dim, bcdt_rms ...)
-    layer_kinds: Optional[List[str]] = None      # attention | mla | mamba1 | mamba2 | gated_delta | shortconv | none (FFN-only block)
+    layer_kinds: Optional[List[str]] = None      # attention | mla | tied | mamba1 | mamba2 | gated_delta | shortconv | none (FFN-only block)
                                                  # | attention+mamba2 (both read the block's input, their outputs add: Falcon-H1)
     ffn_kinds: Optional[List[str]] = None        # glu | moe | none
     ssm: Dict[str, Any] = field(default_factory=dict)
@@ -106,8 +109,17 @@ class ModelConfig:
     # qk_nope_head_dim, qk_rope_head_dim, v_head_dim; head_dim is then qk_nope + qk_rope and rotary_dim qk_rope
     mla: Dict[str, Any] = field(default_factory=dict)
     # per layer: shapes that differ from layer to layer, laid over `ssm` (recurrent kinds) or `mla` (kind "mla"; there also
-    # num_heads, scale, rope_theta, rope_style, head_gate, and kv_from = the layer whose cached rows this one attends to)
+    # num_heads, scale, rope_theta, rope_style, head_gate, and kv_from = the layer whose cached rows this one attends to); for
+    # kind "tied" all of num_heads, num_kv_heads, head_dim, scale, softcap, temp_coef, temp_every, norm_eps
     layer_mixers: Optional[List[Dict[str, Any]]] = None
+    # per layer: width and activation limit of a feed-forward network that differs from layer to layer (ff, limit)
+    layer_ffns: Optional[List[Dict[str, Any]]] = None
+    # > 0: the residual is fp32 and a block's norm follows its sum, x <- rms(alpha x + f(x)) w (models.decoder runs it)
+    postnorm_alpha: float = 0.0
+    # > 0: behind every layer a token's own embedding of that width (one table, a slice per layer) is gated by the residual,
+    # projected, normalised and added
+    token_side_dim: int = 0
+    logit_scale: float = 1.0             # factor on the logits (applied in front of the head)
     # > 0: the residual is that many hyper-connected streams in fp32, mixed by learned matrices around every sublayer
     # (models.decoder runs them); residual_mult scales what a sublayer adds
     residual_streams: int = 0
@@ -142,7 +154,7 @@ class ModelConfig:
 
     @property
     def has_recurrent(self) -> bool:
-        return bool(self.layer_kinds) and any(k not in ("attention", "mla", "none") for k in self.layer_kinds)
+        return bool(self.layer_kinds) and any(k not in STATELESS_KINDS for k in self.layer_kinds)
 
     def ssm_of(self, layer: int) -> Dict[str, Any]:
         """Shapes of a recurrent layer."""
@@ -152,28 +164,50 @@ class ModelConfig:
         """Shapes of a latent-attention layer."""
         return {**self.mla, **self.layer_mixers[layer]} if self.layer_mixers else self.mla
 
+    def attn_of(self, layer: int) -> Dict[str, Any]:
+        """Shapes of an attention layer whose values are its keys."""
+        return self.layer_mixers[layer]
+
+    def ffn_of(self, layer: int) -> Dict[str, Any]:
+        return self.layer_ffns[layer] if self.layer_ffns else dict(ff=self.intermediate_size, limit=self.swiglu_limit)
+
     def kv_source(self, layer: int) -> int:
         """The layer whose rows of the paged pool this one reads (itself unless it shares another's)."""
         j = self.mla_of(layer).get("kv_from") if self.layer_kind(layer) == "mla" else None
         return layer if j is None else int(j)
 
     def has_kv(self, layer: int) -> bool:
-        """Whether the layer keeps keys and values (or latent rows) in the paged pool."""
-        return self.layer_kind(layer) in ("attention", "mla", "attention+mamba2") and self.kv_source(layer) == layer
+        """Whether the layer keeps keys and values (or rows of another layout) in the paged pool."""
+        return self.layer_kind(layer) in ("attention", "mla", "tied", "attention+mamba2") and self.kv_source(layer) == layer
 
     @property
     def native_f32(self) -> bool:
         """Whether every kernel of the model's layers exists in fp32 (served with dtype fp32)."""
-        return self.residual_streams > 0 and all(k in ("gated_delta", "mla") for k in self.layer_kinds or ["attention"])
+        return self.native_part != ""
 
     @property
     def native_part(self) -> str:
         """The part of the native library that holds all of the model's kernels ("" = the whole library)."""
-        return "latent" if self.native_f32 else ""
+        kinds = self.layer_kinds or ["attention"]
+        if self.residual_streams > 0 and all(k in ("gated_delta", "mla") for k in kinds):
+            return "latent"
+        if self.postnorm_alpha > 0 and all(k in ("mamba2", "tied") for k in kinds):
+            return "tied"
+        return ""
+
+    @property
+    def fp32_residual(self) -> bool:
+        """Families whose residual is one or several fp32 streams with an update kernel of their own."""
+        return self.residual_streams > 0 or self.postnorm_alpha > 0
 
     @property
     def has_mla(self) -> bool:
         return bool(self.layer_kinds) and "mla" in self.layer_kinds
+
+    @property
+    def has_row_cache(self) -> bool:
+        """Whether the paged pool holds rows of a layout of their own (models.row_cache) instead of keys and values."""
+        return bool(self.layer_kinds) and any(k in ("mla", "tied") for k in self.layer_kinds)
 
     def layer_window(self, layer: int) -> int:
         if self.sliding_window <= 0:
@@ -212,6 +246,8 @@ class ModelConfig:
         """Map a ``config.json`` (Hugging Face keys, or those of a native design) to the decoder description."""
         if hf.get("architecture") == "Sovanex":
             return sovanex_from_config(cls, hf)
+        if hf.get("architecture") == "Divanex":
+            return divanex_from_config(cls, hf)
         mt = hf.get("model_type", "llama")
         if mt in ("glm4_moe_lite", "kimi_k2", "youtu"):    # DeepSeek-V3 under another name (Youtu: its dense form): the same tensors, router and latent attention
             hf = dict(hf, model_type="deepseek_v3")
@@ -548,6 +584,43 @@ def sovanex_from_config(cls, c: Dict[str, Any]) -> "ModelConfig":
                tie_embeddings=True, norm_kind="layernorm", mlp_kind="plain", act="relu2", layer_kinds=kinds, ffn_kinds=ffns,
                layer_mixers=mixers, ssm=dict(norm_eps=eps), residual_streams=int(c.get("streams") or 1),
                residual_mult=float(c.get("residual_mult", 1.0)))
+
+
+def divanex_from_config(cls, c: Dict[str, Any]) -> "ModelConfig":
+    """Divanex: layers of Mamba-2 and of attention whose values are its keys, in any order, each with sizes of its own; clamped
+    SwiGLU networks behind some of them; norms after the residual sum; a per-layer token input; a scaled, untied head."""
+    kinds, ffns, mixers, nets, ff = [], [], [], [], 8
+    for i, layer in enumerate(c["layers"]):
+        m, mlp = layer["mixer"], layer.get("mlp")
+        if layer["type"] == "mamba2":
+            inner = m["heads"] * m["vdim"]
+            if m["heads"] % m["groups"] or inner % m["norm_groups"]:
+                raise ValueError(f"layer {i}: {m['heads']} heads of {m['vdim']} over {m['groups']} groups and {m['norm_groups']} norm groups")
+            kinds.append("mamba2")
+            mixers.append(dict(d_inner=inner, d_state=m["state"], n_groups=m["groups"], n_heads=m["heads"], head_dim=m["vdim"],
+                               norm_groups=m["norm_groups"], d_conv=max(m["conv"], 2), conv_taps=m["conv"]))
+        elif layer["type"] == "attention":
+            if m["heads"] % m["kv_heads"] or m["vdim"] != m["dim"]:
+                raise ValueError(f"layer {i}: {m['heads']} query heads over {m['kv_heads']} key heads; values are the keys ({m['vdim']} != {m['dim']})")
+            temp = m.get("q_temp") or dict(coef=0.0, every=1)
+            kinds.append("tied")
+            mixers.append(dict(num_heads=m["heads"], num_kv_heads=m["kv_heads"], head_dim=m["dim"], scale=float(m["scale"]),
+                               softcap=float(m.get("softcap") or 0.0), temp_coef=float(temp["coef"]), temp_every=float(temp["every"])))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
+        if mlp is not None and mlp["kind"] != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        ffns.append("none" if mlp is None else "glu")
+        nets.append(dict(ff=mlp["ff"], limit=float(mlp["limit"])) if mlp is not None else {})
+        ff = max(ff, mlp["ff"] if mlp is not None else 0)
+    attn = [m for k, m in zip(kinds, mixers) if k == "tied"]
+    first = attn[0] if attn else dict(num_heads=1, num_kv_heads=1, head_dim=64)
+    eps = float(c["norm"]["eps"])
+    return cls(arch="divanex", name=c.get("name") or "divanex", vocab_size=c["vocab"], hidden_size=c["width"], num_layers=len(kinds),
+               num_heads=first["num_heads"], num_kv_heads=first["num_kv_heads"], head_dim=first["head_dim"], intermediate_size=(ff + 15) // 16 * 16,
+               rms_eps=eps, act="swiglu_oai", embed_scale=float((c.get("embedding") or {}).get("scale", 1.0)), use_rope=False, layer_kinds=kinds,
+               ffn_kinds=ffns, layer_mixers=mixers, layer_ffns=nets, ssm=dict(norm_eps=eps), postnorm_alpha=float(c["postln_alpha"]),
+               token_side_dim=int((c.get("token_side") or {}).get("dim", 0)), logit_scale=float(c.get("logit_scale", 1.0)))
 
 
 RECURRENT_MODEL_TYPES = ("falcon_h1", "nemotron_h", "nemotron_h_moe", "mamba", "falcon_mamba", "mamba2", "bamba", "lfm2", "rwkv7", "qwen3_next", "qwen3_5_text", "qwen3_5_moe_text", "jamba", "granitemoehybrid", "granitemoe", "granitemoeshared", "glm4_moe", "ernie4_5_moe", "rwkv6")
@@ -949,6 +1022,18 @@ def preset(name: str) -> ModelConfig:
         return sovanex_from_config(ModelConfig, dict(
             architecture="Sovanex", name=n, layers=layers, norm=dict(eps=1e-5), residual_mult=0.25, streams=2 if tiny else 4,
             vocab=512 if tiny else 65536, width=96 if tiny else 2048))
+    if n in ("divanex-tiny", "divanex-2b"):
+        # three Mamba-2 layers, then one of attention with a feed-forward network
+        tiny = n.endswith("tiny")
+        mamba = dict(heads=4 if tiny else 64, vdim=24 if tiny else 64, state=40 if tiny else 128, groups=2 if tiny else 8, norm_groups=2 if tiny else 8,
+                     conv=4)
+        dim = 48 if tiny else 128
+        attn = dict(heads=4 if tiny else 32, kv_heads=2 if tiny else 8, dim=dim, vdim=dim, scale=dim ** -0.5, softcap=30.0, q_temp=dict(coef=0.1, every=4096))
+        layers = [dict(type="attention", mixer=attn, mlp=dict(kind="dense", ff=160 if tiny else 8192, limit=7.0)) if i % 4 == 3 else
+                  dict(type="mamba2", mixer=mamba, mlp=None) for i in range(8 if tiny else 32)]
+        return divanex_from_config(ModelConfig, dict(
+            architecture="Divanex", name=n, layers=layers, norm=dict(eps=1e-5), embedding=dict(scale=4.0), postln_alpha=2.0, logit_scale=0.5,
+            token_side=dict(dim=16 if tiny else 256), vocab=512 if tiny else 65536, width=96 if tiny else 2048))
     raise KeyError(f"unknown model preset {name!r}")
 
 

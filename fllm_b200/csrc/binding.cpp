@@ -202,6 +202,14 @@ void glu_ex(const optional<Tensor>& x, Tensor out, int64_t act_kind, double alph
 }
 
 void glu(const Tensor& x, Tensor out, int64_t act_kind, double alpha, double limit) {
+  if (x.is_cuda() && x.scalar_type() == at::kFloat) {             // models served in 32-bit
+    TORCH_CHECK(out.scalar_type() == at::kFloat && x.dim() == 2 && out.dim() == 2 && x.stride(1) == 1 && out.stride(1) == 1 &&
+                    x.size(1) == 2 * out.size(1) && x.size(0) == out.size(0), "glu: fp32 rows");
+    c10::cuda::CUDAGuard guard(x.device());
+    fllm::glu_f32(x.data_ptr(), x.stride(0), out.data_ptr(), out.stride(0), (int)x.size(0), (int)out.size(1), (int)act_kind, (float)alpha,
+                  (float)limit, cur_stream());
+    return;
+  }
   check_bf16(x, "x"); check_bf16(out, "out"); check_rows(x, "x"); check_rows(out, "out");
   TORCH_CHECK(x.size(1) == 2 * out.size(1) && x.size(0) == out.size(0), "glu: shape mismatch");
   c10::cuda::CUDAGuard guard(x.device());

@@ -1,5 +1,5 @@
-// torch.ops.fllm_b200 bindings of the hyper-connected residual streams (streams.cu), latent attention of any size
-// (attention_latent.cu) and the fp32 products (gemm_f32.cu).
+// torch.ops.fllm_b200 bindings of the hyper-connected residual streams (streams.cu) and latent attention of any size
+// (attention_latent.cu).
 #include <ATen/ATen.h>
 #include <c10/cuda/CUDAGuard.h>
 #include <c10/cuda/CUDAStream.h>
@@ -161,38 +161,6 @@ void head_gate(const Tensor& o, const optional<Tensor>& gate, Tensor out) {
   fllm::head_gate(o.data_ptr(), o.stride(0), o.stride(1), g, ldg, out.data_ptr(), out.stride(0), (int)o.size(1), (int)o.size(0), (int)o.size(2),
                   (int)out.size(1), ty == at::kFloat ? 1 : 0, cur_stream());
 }
-
-// y = x @ w^T (+ bias), fp32
-void linear_f32(const Tensor& x, const Tensor& w, const optional<Tensor>& bias, Tensor y) {
-  TORCH_CHECK(x.is_cuda() && x.scalar_type() == at::kFloat && w.scalar_type() == at::kFloat && y.scalar_type() == at::kFloat && x.dim() == 2 &&
-                  w.dim() == 2 && y.dim() == 2 && y.stride(1) == 1 && x.size(1) == w.size(1) && y.size(0) == x.size(0) && y.size(1) == w.size(0),
-              "linear_f32: x [T, K], w [N, K], y [T, N] in fp32");
-  fllm::GemmF32Params p{};
-  p.a = x.data_ptr<float>(), p.a_t = x.stride(0), p.a_k = x.stride(1);
-  p.b = w.data_ptr<float>(), p.b_n = w.stride(0), p.b_k = w.stride(1);
-  if (given(bias)) {
-    TORCH_CHECK(bias->scalar_type() == at::kFloat && bias->is_contiguous() && bias->numel() == w.size(0), "linear_f32: bias");
-    p.bias = bias->data_ptr<float>();
-  }
-  p.c = y.data_ptr<float>(), p.c_t = y.stride(0);
-  p.batch = 1, p.T = (int)x.size(0), p.N = (int)w.size(0), p.K = (int)x.size(1);
-  c10::cuda::CUDAGuard guard(x.device());
-  fllm::gemm_f32(p, cur_stream());
-}
-
-// c[b] = a[b] @ m[b], fp32: a [B, T, K], m [B, K, N], c [B, T, N]
-void bmm_f32(const Tensor& a, const Tensor& m, Tensor c) {
-  TORCH_CHECK(a.is_cuda() && a.scalar_type() == at::kFloat && m.scalar_type() == at::kFloat && c.scalar_type() == at::kFloat && a.dim() == 3 &&
-                  m.dim() == 3 && c.dim() == 3 && c.stride(2) == 1 && a.size(0) == m.size(0) && a.size(2) == m.size(1) && c.size(0) == a.size(0) &&
-                  c.size(1) == a.size(1) && c.size(2) == m.size(2), "bmm_f32: a [B, T, K], m [B, K, N], c [B, T, N] in fp32");
-  fllm::GemmF32Params p{};
-  p.a = a.data_ptr<float>(), p.a_b = a.stride(0), p.a_t = a.stride(1), p.a_k = a.stride(2);
-  p.b = m.data_ptr<float>(), p.b_b = m.stride(0), p.b_n = m.stride(2), p.b_k = m.stride(1);
-  p.c = c.data_ptr<float>(), p.c_b = c.stride(0), p.c_t = c.stride(1);
-  p.batch = (int)a.size(0), p.T = (int)a.size(1), p.N = (int)m.size(2), p.K = (int)a.size(2);
-  c10::cuda::CUDAGuard guard(a.device());
-  fllm::gemm_f32(p, cur_stream());
-}
 }  // namespace
 
 TORCH_LIBRARY_FRAGMENT(fllm_b200, m) {
@@ -205,6 +173,4 @@ TORCH_LIBRARY_FRAGMENT(fllm_b200, m) {
   m.def("attention_latent(Tensor q, Tensor cache, Tensor block_tables, Tensor row_seq, Tensor positions, Tensor q_starts, Tensor(a!) out, int num_seqs, "
         "int max_q_len, float scale, int splits, Tensor? workspace, bool tensor_cores) -> int", &attention_latent);
   m.def("head_gate(Tensor o, Tensor? gate, Tensor(a!) out) -> ()", &head_gate);
-  m.def("linear_f32(Tensor x, Tensor w, Tensor? bias, Tensor(a!) y) -> ()", &linear_f32);
-  m.def("bmm_f32(Tensor a, Tensor m, Tensor(a!) c) -> ()", &bmm_f32);
 }

@@ -610,6 +610,33 @@ void glu_bf16(const void* x, long long ldx, void* out, long long ldo, int rows, 
   cuda_check(cudaGetLastError(), "glu_kernel");
 }
 
+// The same in fp32, natural layouts, accurate functions.
+__global__ void __launch_bounds__(256) glu_f32_kernel(const float* __restrict__ x, long long ldx, float* __restrict__ out, long long ldo, int inter,
+                                                      int act_kind, float alpha, float limit) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= inter) return;
+  const float* xr = x + (size_t)blockIdx.y * ldx;
+  const float g = act_kind == 2 ? xr[2 * i] : xr[i], u = act_kind == 2 ? xr[2 * i + 1] : xr[inter + i];
+  float o;
+  if (act_kind == 0) {
+    o = g / (1.f + expf(-g)) * u;
+  } else if (act_kind == 1) {
+    o = 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+  } else {
+    const float gg = fminf(g, limit);
+    o = gg / (1.f + expf(-alpha * gg)) * (fminf(fmaxf(u, -limit), limit) + 1.f);
+  }
+  out[(size_t)blockIdx.y * ldo + i] = o;
+}
+
+void glu_f32(const void* x, long long ldx, void* out, long long ldo, int rows, int inter, int act_kind, float alpha, float limit, cudaStream_t s) {
+  if (rows <= 0) return;
+  if (rows > 65535) throw std::runtime_error("glu_f32: at most 65535 rows");
+  glu_f32_kernel<<<dim3((inter + 255) / 256, rows), 256, 0, s>>>(static_cast<const float*>(x), ldx, static_cast<float*>(out), ldo, inter, act_kind, alpha,
+                                                                limit);
+  cuda_check(cudaGetLastError(), "glu_f32_kernel");
+}
+
 // ---------------------------------------------------------------------------- row gather (logit rows)
 __global__ void gather_rows_kernel(const __nv_bfloat16* __restrict__ x, long long ldx,
                                    const int* __restrict__ rows, __nv_bfloat16* __restrict__ out,

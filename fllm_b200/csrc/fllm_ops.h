@@ -285,6 +285,19 @@ int mamba2_scan(const void* x, long long ldx, const void* dt, long long lddt, co
                 const int* seq_state, const int* positions, void* y, long long ldy, int B, int H, int P, int G, int N,
                 float dt_min, float dt_max, int seg_len, int segs, float* seg_state, float* seg_dt, int skip_from,
                 cudaStream_t stream);
+// The same recurrence for any head and state width (N <= 256), bf16 or fp32 (recurrent_ssd.cu): one walk per sequence.
+struct SsdScanParams {
+  const void *x, *dt, *Bm, *Cm;
+  long long ldx, lddt, ldb, ldc, ldy;
+  const float *A, *D, *dt_bias;
+  float* state;                // [slots][H][P][N]
+  const int *q_starts, *seq_state, *positions;
+  void* y;
+  int B, tokens, H, P, G, N;   // tokens: rows of the step (= B: single tokens)
+  float dt_min, dt_max;
+  int skip_from, f32;
+};
+int ssd_scan(const SsdScanParams& p, cudaStream_t stream);
 int mamba1_scan(const void* x, long long ldx, const void* dt, long long lddt, const void* Bm, long long ldb, const void* Cm,
                 long long ldc, const void* z, long long ldz, const float* A, const float* D, const float* dt_bias, float* state,
                 const int* q_starts, const int* seq_state, const int* positions, void* y, long long ldy, int B, int Dm, int N,
@@ -329,6 +342,8 @@ void add_layernorm_bf16(void* x, long long ldx, const void* delta, long long ldd
 // in-place activation: 0 gelu (erf), 1 gelu (tanh), 2 squared relu, 3 silu, 4 relu
 void act_rows_bf16(void* x, long long ldx, int rows, int cols, int kind, cudaStream_t s);
 void act_rows_f32(void* x, long long ldx, int rows, int cols, int kind, cudaStream_t s);
+// gated activation of fp32 rows in the kind's natural layout (see glu_bf16)
+void glu_f32(const void* x, long long ldx, void* out, long long ldo, int rows, int inter, int act_kind, float alpha, float limit, cudaStream_t s);
 
 // ---- hyper-connected residual streams (streams.cu) -------------------------------------------------------------------
 // x [rows][streams][ld] fp32; element types of table, y, norm weights and h: bf16, or fp32 with f32 = 1.
@@ -393,6 +408,88 @@ int attention_latent(const LatentAttnParams& p, int splits, void* workspace, siz
 // out[t][h * dv + j] = o(h, t, j) * sigmoid(gate[t][h]) (gate may be null), columns up to `cols` zero-filled
 void head_gate(const void* o, long long o_h, long long o_t, const void* gate, long long ld_gate, void* out, long long ld_out, int tokens, int H,
                int dv, int cols, int f32, cudaStream_t s);
+
+// ---- attention whose values are the keys (attention_tied.cu) -----------------------------------------------------------
+struct TiedPrepareParams {
+  const void* x;               // [tokens] rows: query heads from column 0, key heads from column k_offset
+  long long ldx;
+  const float* partials;       // not null: the rows are the sums of split-K partials [splits][tokens][width], `plane` elements per split
+  int splits, width;
+  long long plane;
+  void* q_out;                 // with partials: [tokens] rows of H * dim
+  long long ld_qout;
+  int k_offset, H, G, dim, W, block_size, tokens;
+  const int *positions, *slots;
+  float eps;                   // of the head norms; negative: none
+  float scale, temp_coef, temp_every;
+  float* q_factor;             // [tokens][H]
+  void* cache;                 // [blocks][G][block_size][W]
+  float* key_factor;           // [blocks][G][block_size]
+  int f32;
+};
+void tied_prepare(const TiedPrepareParams& p, cudaStream_t s);
+struct TiedAttnParams {
+  const void* q;               // head h of token t at q[t * ldq + h * dim]
+  long long ldq;
+  const float* q_factor;       // [tokens][H]
+  const void* cache;           // [blocks][G][block_size][W]
+  const float* key_factor;     // [blocks][G][block_size]
+  const int* block_tables;
+  int max_blocks;
+  const int *row_seq, *positions, *q_starts;
+  void* out;                   // head h of token t at out[t * ldo + h * dim]
+  long long ldo;
+  int tokens, num_seqs, max_q_len, min_q_len, H, G, dim, W, block_size;
+  long long num_blocks;
+  float softcap;               // 0: none
+  int f32;
+};
+bool attention_tied_tc_supported(int W, int block_size, int f32);
+int attention_tied_splits(int num_seqs, int max_q_len, int H, int G, int max_kv_len);
+size_t attention_tied_workspace_bytes(int tokens, int H, int W, int splits);
+int attention_tied(const TiedAttnParams& p, int splits, void* workspace, size_t workspace_bytes, bool tensor_cores, int* status, cudaStream_t s);
+
+// ---- residual with the norm after the sum, per-layer token input (postnorm.cu) -------------------------------------------
+struct PostNormParams {
+  float* x;                    // [rows][ld] fp32, zero beyond `width`
+  const int* ids;              // not null: x = table[ids[row]] * scale
+  const void* table;
+  int vocab;
+  long long ld_table;
+  float scale;
+  const void* y;               // output of the sublayer, or the split-K partial sums [splits][rows][ld] of its projection
+  long long ld_y;
+  const float* partials;
+  int splits;
+  long long plane;
+  int add;                     // 0: x <- rms(alpha x + y) w;  1: x <- x + rms(y) w
+  float alpha;
+  const void* norm_w;
+  const void* final_w;         // not null: h = rms(x) final_w * final_scale, otherwise h = x
+  float final_scale;
+  const int* rows;             // optional row selection of the outputs
+  void* h;
+  long long ld_h;
+  int n_out, width, ld;
+  float eps;
+  int write, f32;
+};
+void postnorm(const PostNormParams& p, cudaStream_t s);
+struct SideGateParams {
+  const void* gate;            // [tokens] rows, or split-K partial sums [splits][tokens][cols]
+  long long ld_gate;
+  const float* partials;
+  int splits;
+  long long plane;
+  const int* ids;
+  const void* table;           // [vocab] rows; the layer's slice starts at column `offset`
+  int vocab, offset, dim, cols, tokens;
+  long long ld_table;
+  void* out;                   // [tokens][cols], zero beyond `dim`
+  long long ld_out;
+  int f32;
+};
+void side_gate(const SideGateParams& p, cudaStream_t s);
 
 // ---- fp32 products (gemm_f32.cu): c[b][t][n] = sum_k a[b][t][k] b[b][n][k] (+ bias[n]), strides in elements -----------------
 struct GemmF32Params {

@@ -48,11 +48,14 @@ def load_hf_checkpoint(directory: str, device="cuda", tp: int = 1, tp_rank: int 
     def dev(t):
         return t.to(device=device, dtype=dtype if t.is_floating_point() and t.element_size() > 1 else t.dtype).contiguous()
 
-    if cfg.arch == "sovanex":
+    if cfg.fp32_residual:
         if tp > 1:
-            raise NotImplementedError("models with residual streams run on one rank")
-        from .sovanex_loader import sovanex_weights
+            raise NotImplementedError("models with a residual in fp32 run on one rank")
         tok = directory if os.path.exists(os.path.join(directory, "tokenizer.json")) else None
+        if cfg.arch == "divanex":
+            from .divanex_loader import divanex_weights
+            return cfg, divanex_weights(cfg, get, device, dtype), tok
+        from .sovanex_loader import sovanex_weights
         return cfg, sovanex_weights(cfg, get, device, dtype), tok
     if cfg.arch in CLASSIC_MODEL_TYPES:
         if tp > 1:

@@ -130,9 +130,9 @@ class Decoder:
                        and not cfg.qk_norm_full and not cfg.clip_qkv)
         if self._defer:
             self._block_gate_up()
-        # the streams kernel also adds the split-K partial sums of the projection behind a sublayer
+        # the kernels of an fp32 residual also add the split-K partial sums of the projection behind a sublayer
         self._stream_ones = torch.ones(max(cfg.residual_streams, 1), dtype=torch.float32, device=dev)
-        self.defer_to_streams = bool(cfg.residual_streams and hasattr(ops, "k") and dev.type == "cuda")
+        self.defer_to_residual = bool(cfg.fp32_residual and hasattr(ops, "k") and dev.type == "cuda")
 
     def _block_gate_up(self) -> None:
         """Re-order the rows of every dense gate|up matrix into blocks of 16 gate rows followed by the 16 up
@@ -235,8 +235,8 @@ class Decoder:
             return y
         if cfg.mlp_kind == "plain":               # two matrices and an activation between them
             u = ops.act_(ops.linear(h, lw.w_gate_up, lw.b_up), cfg.act)
-            return ops.linear(u, lw.w_down, lw.b_down, defer=self.defer_to_streams)
-        act = ops.linear_glu(h, lw.w_gate_up, None, self.act_kind, cfg.swiglu_alpha, cfg.swiglu_limit,
+            return ops.linear(u, lw.w_down, lw.b_down, defer=self.defer_to_residual)
+        act = ops.linear_glu(h, lw.w_gate_up, None, self.act_kind, cfg.swiglu_alpha, cfg.swiglu_limit if lw.act_limit is None else lw.act_limit,
                              getattr(lw, "glu_layout", 0))
         return ops.linear(act, lw.w_down, defer=self._defer_out(lw.post_ffn_norm))
 
@@ -254,6 +254,8 @@ class Decoder:
             return rwkv6_forward_hidden(self, b)
         if cfg.residual_streams:
             return self._forward_streams(b)
+        if cfg.postnorm_alpha > 0:
+            return self._forward_postnorm(b)
         if self.first_stage:
             x = ops.embed(b.token_ids, self.w.embed, cfg.embed_scale)
             if cfg.learned_positions:              # the same row gather on the position table
@@ -308,6 +310,36 @@ class Decoder:
             if nvtx:
                 torch.cuda.nvtx.range_pop()
         return x, delta
+
+    def _forward_postnorm(self, b: StepBatch):
+        """The layers of a model whose norms follow the residual sum, each with its token input behind it. Returns (fp32
+        residual, (y, arguments of the last update)): that update runs together with the final norm, in ``logits``."""
+        cfg, ops, W, eps = self.cfg, self.ops, self.cfg.hidden_size, self.cfg.rms_eps
+        x, h = ops.postnorm_begin(b.token_ids, self.w.embed, cfg.embed_scale)
+        pending = None
+        for li, lw in zip(self.layer_range, self.w.layers):
+            if self._nvtx:
+                torch.cuda.nvtx.range_push(f"layer{li}")
+            if pending is not None:
+                h = ops.postnorm_step(x, *pending)
+            if cfg.layer_kind(li) == "tied":
+                from .tied import tied_attention_mixer
+                y = tied_attention_mixer(self, li, lw, h, b)
+            else:
+                from .recurrent import MIXERS
+                y = MIXERS[cfg.layer_kind(li)](self, li, lw, h, b)
+            pending = (y, lw.attn_norm, W, eps, cfg.postnorm_alpha)
+            if cfg.ffn_kind(li) != "none":
+                h = ops.postnorm_step(x, *pending)
+                pending = (self._ffn_block(lw, h), lw.ffn_norm, W, eps, cfg.postnorm_alpha)
+            if lw.side is not None:
+                h = ops.postnorm_step(x, *pending)
+                g = ops.side_gate(ops.linear(h, lw.side.gate, defer=self.defer_to_residual), b.token_ids, self.w.side_embed, li * cfg.token_side_dim,
+                                  cfg.token_side_dim)
+                pending = (ops.linear(g, lw.side.proj, defer=self.defer_to_residual), lw.side.norm, W, eps, 1.0, True)
+            if self._nvtx:
+                torch.cuda.nvtx.range_pop()
+        return x, pending
 
     def _sublayers(self):
         """(stream coefficients, norm weight, norm bias, layer index, layer weights, is the mixer) in running order."""
@@ -427,6 +459,12 @@ class Decoder:
             if self.capture_hidden:
                 self.last_hidden = hs
             return ops.linear(hs, self.w.lm_head, self.w.lm_head_b)
+        if cfg.postnorm_alpha > 0:              # last update, final norm and logit scale, wanted rows: one kernel
+            rows = None if b.all_decode and b.logit_rows.numel() == x.shape[0] else b.logit_rows
+            hs = ops.postnorm_step(x, *delta, final_w=self.w.final_norm, final_scale=cfg.logit_scale, rows=rows)
+            if self.capture_hidden:                # without the factor that belongs to the logits
+                self.last_hidden = hs / cfg.logit_scale
+            return ops.linear(hs, self.w.lm_head)
         if cfg.arch in ("rwkv7", "rwkv6"):
             from .rwkv import rwkv7_final_norm
             h = rwkv7_final_norm(self, x)

@@ -9,41 +9,11 @@ is the only one).
 """
 from __future__ import annotations
 
-from typing import Dict, List
+from typing import Dict
 
 import torch
 
 from ..config import ModelConfig
-from ..ops.latent import latent_width
-
-
-class MlaCache:
-    """Paged latent pool: one [blocks, block_size, width] tensor per layer that keeps rows of its own."""
-
-    def __init__(self, widths: List[int], num_blocks: int, block_size: int, device, dtype=torch.bfloat16):
-        self.num_blocks, self.block_size = num_blocks, block_size
-        self.rows = [torch.zeros(num_blocks, block_size, w, device=device, dtype=dtype) for w in widths]
-
-    def layer(self, i: int) -> torch.Tensor:
-        return self.rows[i]
-
-    def copy_block(self, src: int, dst: int) -> None:
-        for t in self.rows:
-            t[dst].copy_(t[src])
-
-    @staticmethod
-    def widths(cfg: ModelConfig, layer_range) -> List[int]:
-        out = []
-        for li in layer_range:
-            if cfg.layer_kind(li) == "mla" and cfg.has_kv(li):
-                c = cfg.mla_of(li)
-                R, dr = c["kv_lora_rank"], c["qk_rope_head_dim"]
-                out.append(latent_width(R, dr) if cfg.layer_mixers else R + dr)
-        return out
-
-    @staticmethod
-    def bytes_per_block(widths: List[int], block_size: int, elem: int = 2) -> int:
-        return sum(widths) * block_size * elem
 
 
 def mla_block(dec, li: int, lw, h: torch.Tensor, b) -> torch.Tensor:
@@ -87,7 +57,7 @@ def latent_block(dec, li: int, lw, h: torch.Tensor, b) -> torch.Tensor:
     o = ops.bmm(ops.attention_latent(ql, cache, b, c["scale"], R), m["w_uv"])                     # [H, T, dv]
     og = nq + (pad8(R + dr) if own else 0)
     gate = proj[:, og:og + H] if c.get("head_gate") else None
-    return ops.linear(ops.head_gate(o, gate, m["wo"].shape[1]), m["wo"], defer=getattr(dec, "defer_to_streams", False))
+    return ops.linear(ops.head_gate(o, gate, m["wo"].shape[1]), m["wo"], defer=getattr(dec, "defer_to_residual", False))
 
 
 def pack_latent(q, dkv, kv_norm, uk, uv, gate, o_proj, c: Dict, dtype, device) -> Dict[str, torch.Tensor]:

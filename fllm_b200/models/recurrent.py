@@ -15,7 +15,7 @@ from typing import Dict, Optional
 import torch
 import torch.nn.functional as F
 
-from ..config import ModelConfig
+from ..config import STATELESS_KINDS, ModelConfig
 from ..ops.recurrent import GATED_DELTA
 
 RECURRENT_KINDS = ("mamba1", "mamba2", "gated_delta", "shortconv")
@@ -34,7 +34,7 @@ def conv_channels(cfg: ModelConfig, kind: str, layer: int = 0) -> int:
     if kind == "mamba1":
         return s["d_inner"]
     if kind == "mamba2":
-        return s["d_inner"] + 2 * s["n_groups"] * s["d_state"]
+        return pad8(s["d_inner"]) + 2 * pad8(s["n_groups"] * s["d_state"])
     if kind == "gated_delta":
         return 2 * pad8(s["num_k_heads"] * s["head_k_dim"]) + pad8(s["num_v_heads"] * s["head_v_dim"])
     if kind in ("shortconv", "rwkv7", "rwkv6"):
@@ -66,7 +66,7 @@ class RecurrentState:
         self.shift2: Dict[int, torch.Tensor] = {}          # RWKV: the channel mix has a token shift of its own
         for li in layer_range:
             kind = _state_kind(cfg.layer_kind(li))
-            if kind in ("attention", "mla", "none"):
+            if kind in STATELESS_KINDS:
                 continue
             W = cfg.ssm_of(li).get("d_conv", 4)
             if kind in ("rwkv7", "rwkv6"):
@@ -81,7 +81,7 @@ class RecurrentState:
         n = 0
         for li in layer_range:
             kind = _state_kind(cfg.layer_kind(li))
-            if kind in ("attention", "mla", "none"):
+            if kind in STATELESS_KINDS:
                 continue
             W = cfg.ssm_of(li).get("d_conv", 4)
             n += (W - 1) * conv_channels(cfg, kind, li) * (4 if kind in ("rwkv7", "rwkv6") else elem)
@@ -134,13 +134,14 @@ def mamba1_mixer(dec, li: int, lw, h: torch.Tensor, b) -> torch.Tensor:
 
 def mamba2_mixer(dec, li: int, lw, h: torch.Tensor, b) -> torch.Tensor:
     """in_proj -> (z, xBC, dt); xBC = silu(conv(xBC)) -> (x, B, C); SSD scan; rmsnorm(y * silu(z)); out_proj."""
-    s, m, ops = dec.cfg.ssm, lw.mixer, dec.ops
+    s, m, ops = dec.cfg.ssm_of(li), lw.mixer, dec.ops
     qs, ss, pos = _batch_meta(b)
     Di, N, G, H, P = s["d_inner"], s["d_state"], s["n_groups"], s["n_heads"], s["head_dim"]
-    C = Di + 2 * G * N
+    Dp, bc = pad8(Di), pad8(G * N)                                      # segments of the projection start on 16-byte boundaries
+    C = Dp + 2 * bc
     zxd = ops.linear(h, m["in_proj"], m.get("in_proj_b"))
-    xbc = ops.causal_conv1d(zxd[:, Di:Di + C], m["conv_w"], m.get("conv_b"), dec.rstate.conv[li], qs, ss, pos, act=True, max_q_len=getattr(b, "max_q_len", 0))
-    y = ops.mamba2_scan(xbc[:, :Di], zxd[:, Di + C:Di + C + H], xbc[:, Di:Di + G * N], xbc[:, Di + G * N:], m["A"], m["D"],
+    xbc = ops.causal_conv1d(zxd[:, Dp:Dp + C], m["conv_w"], m.get("conv_b"), dec.rstate.conv[li], qs, ss, pos, act=True, max_q_len=getattr(b, "max_q_len", 0))
+    y = ops.mamba2_scan(xbc[:, :Di], zxd[:, Dp + C:Dp + C + H], xbc[:, Dp:Dp + G * N], xbc[:, Dp + bc:Dp + bc + G * N], m["A"], m["D"],
                         m["dt_bias"], dec.rstate.scan[li], qs, ss, pos, H, P, G, N, s.get("dt_min", 0.0),
                         s.get("dt_max", 1e30), getattr(b, "max_q_len", 0), None, getattr(b, "host_seqs", None))
     mode = s.get("gate_mode", "norm_after_gate")
@@ -148,8 +149,8 @@ def mamba2_mixer(dec, li: int, lw, h: torch.Tensor, b) -> torch.Tensor:
         y = y * F.silu(zxd[:, :Di])
     else:
         y = ops.gated_rmsnorm(y, zxd[:, :Di], m["norm_w"], s.get("norm_eps", dec.cfg.rms_eps), Di // s.get("norm_groups", 1),
-                              mode == "norm_before_gate")
-    return ops.linear(y, m["out_proj"], m.get("out_proj_b"))
+                              mode == "norm_before_gate", Dp)
+    return ops.linear(y, m["out_proj"], m.get("out_proj_b"), defer=getattr(dec, "defer_to_residual", False))
 
 
 def gated_delta_mixer(dec, li: int, lw, h: torch.Tensor, b) -> torch.Tensor:
@@ -169,7 +170,7 @@ def gated_delta_mixer(dec, li: int, lw, h: torch.Tensor, b) -> torch.Tensor:
                               dec.rstate.scan[li], qs, ss, pos, Hv, Dk, Dv, Hv // Hk, True, Dk ** -0.5,
                               gate_raw=proj[:, o + Hv:o + 2 * Hv], gate_A=m["A"], gate_dt_bias=m["dt_bias"])
     y = ops.gated_rmsnorm(y, z, m["norm_w"], s.get("norm_eps", dec.cfg.rms_eps), Dv, True, Vp)
-    return ops.linear(y, m["out_proj"], defer=getattr(dec, "defer_to_streams", False))
+    return ops.linear(y, m["out_proj"], defer=getattr(dec, "defer_to_residual", False))
 
 
 def shortconv_mixer(dec, li: int, lw, h: torch.Tensor, b) -> torch.Tensor:
@@ -223,9 +224,21 @@ def pack_mamba1(in_proj, conv_w, conv_b, x_proj, dt_proj, dt_bias, A_log, D, out
 
 
 def pack_mamba2(in_proj, conv_w, conv_b, dt_bias, A_log, D, norm_w, out_proj, dtype, device, in_proj_b=None,
-                out_proj_b=None) -> Dict[str, torch.Tensor]:
+                out_proj_b=None, shapes: Optional[dict] = None) -> Dict[str, torch.Tensor]:
+    """``shapes`` (d_inner, n_groups, d_state): needed where the segments z, x, B and C are not multiples of 8 rows; they are
+    then padded one by one."""
     f32 = lambda t: t.float().to(device).contiguous()
     bf = lambda t: t.to(device=device, dtype=dtype).contiguous()
+    if shapes is not None:
+        Di, bc = shapes["d_inner"], shapes["n_groups"] * shapes["d_state"]
+        p8 = lambda t: pad_rows(t, pad8(t.shape[0]))
+        cut = lambda t, sizes: torch.cat([p8(part) for part in torch.split(t, sizes)], 0)
+        dt = in_proj.shape[0] - 2 * Di - 2 * bc
+        in_proj = cut(in_proj, [Di, Di, bc, bc, dt])
+        in_proj_b = cut(in_proj_b, [Di, Di, bc, bc, dt]) if in_proj_b is not None else None
+        conv_w = cut(conv_w.reshape(conv_w.shape[0], -1), [Di, bc, bc])
+        conv_b = cut(conv_b, [Di, bc, bc]) if conv_b is not None else None
+        out_proj = pad_cols(out_proj, pad8(Di))
     m = dict(in_proj=bf(pad_rows(in_proj, pad8(in_proj.shape[0]))), conv_w=f32(conv_w.reshape(conv_w.shape[0], -1)),
              dt_bias=f32(dt_bias), A=f32(-torch.exp(A_log.float())), D=f32(D), norm_w=bf(norm_w), out_proj=bf(out_proj))
     if conv_b is not None:

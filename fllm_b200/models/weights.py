@@ -30,6 +30,14 @@ class StreamMix:
 
 
 @dataclass
+class SideInput:
+    """Per-layer token input: gate [dim, H], proj [H, dim], norm [H] of what is added to the residual."""
+    gate: torch.Tensor
+    proj: torch.Tensor
+    norm: torch.Tensor
+
+
+@dataclass
 class LayerWeights:
     attn_norm: torch.Tensor
     wqkv: torch.Tensor
@@ -70,6 +78,8 @@ class LayerWeights:
     # hyper-connected residual streams: coefficients around the mixer and around the feed-forward network
     streams1: Optional["StreamMix"] = None
     streams2: Optional["StreamMix"] = None
+    side: Optional["SideInput"] = None              # per-layer token input behind the layer
+    act_limit: Optional[float] = None               # clamp of this layer's gated activation (None: the model's)
     # packed formats keep their payload here (format name -> tensors)
     packed: Dict[str, object] = field(default_factory=dict)
     # row order of w_gate_up: 0 = gate half then up half; 16 = blocks of 16 gate rows followed by the 16 up
@@ -99,6 +109,7 @@ class DecoderWeights:
     final_norm_b: Optional[torch.Tensor] = None      # families whose blocks are LayerNorms (RWKV, GPT-NeoX, Phi, ...)
     lm_head_b: Optional[torch.Tensor] = None         # Phi
     pos_embed: Optional[torch.Tensor] = None         # [positions, H] learned absolute positions (GPT-2, OPT)
+    side_embed: Optional[torch.Tensor] = None        # [vocab, layers * dim]: per-layer token inputs
 
     def nbytes(self) -> int:
         n = 0
@@ -110,11 +121,13 @@ class DecoderWeights:
                 seen.add(t.data_ptr())
                 n += t.numel() * t.element_size()
 
-        add(self.embed); add(self.final_norm); add(self.lm_head)
+        add(self.embed); add(self.final_norm); add(self.lm_head); add(self.side_embed)
         for l in self.layers:
             for v in vars(l).values():
                 add(v)
             for v in (l.mixer or {}).values():
+                add(v)
+            for v in vars(l.side).values() if l.side is not None else ():
                 add(v)
         return n
 
@@ -266,6 +279,11 @@ def init_random_weights(cfg: ModelConfig, device="cpu", dtype=torch.bfloat16, se
         if tp > 1 or (layers is not None and len(layers) != cfg.num_layers):
             raise NotImplementedError("models with residual streams run on one rank and one pipeline stage")
         return sovanex_weights(cfg, random_tensors(cfg, seed, device), device, dtype)
+    if cfg.arch == "divanex":
+        from ..formats.divanex_loader import divanex_weights, random_tensors
+        if tp > 1 or (layers is not None and len(layers) != cfg.num_layers):
+            raise NotImplementedError("models with a residual in fp32 run on one rank and one pipeline stage")
+        return divanex_weights(cfg, random_tensors(cfg, seed, device), device, dtype)
     sp = make_shard_spec(cfg, tp, tp_rank, expert_parallel)
     D, H = cfg.head_dim, cfg.hidden_size
     layers = range(cfg.num_layers) if layers is None else layers

@@ -14,6 +14,7 @@ import torch
 from ._lib import load_cuda
 from .latent import LatentNative
 from .recurrent import RecurrentNative
+from .tied import TiedNative
 
 
 class Deferred:
@@ -31,7 +32,7 @@ class Deferred:
         return (self.rows, self.cols)
 
 
-class NativeOps(RecurrentNative, LatentNative):
+class NativeOps(RecurrentNative, LatentNative, TiedNative):
     name = "sm100a"
 
     def __init__(self, device: torch.device, workspace_bytes: int = 96 << 20, part: str = ""):
@@ -76,7 +77,7 @@ class NativeOps(RecurrentNative, LatentNative):
         """Tensor value of a projection result (adds a Deferred's partials with the stand-alone path)."""
         if not isinstance(y, Deferred):
             return y
-        raise RuntimeError("a deferred projection can only be consumed by rmsnorm, rope_kv_write, a gated activation or streams_step")
+        raise RuntimeError("a deferred projection can only be consumed by rmsnorm, rope_kv_write, a gated activation, or the kernels of an fp32 residual")
 
     def linear_glu(self, x, w, bias, act_kind=0, alpha=1.702, limit=7.0, layout=0, force_splits: int = 0):
         """act(x @ w^T + bias) for a fused gate|up weight, [T, N/2]. With a row layout the GEMM epilogue can
@@ -84,7 +85,7 @@ class NativeOps(RecurrentNative, LatentNative):
         when the GEMM needs split-K the activation kernel adds the partial sums instead."""
         T, N = x.shape[0], w.shape[0]
         pd = 16 if layout == 16 else (1 if act_kind == 2 else 0)
-        if not isinstance(w, torch.Tensor) or pd == 0 or N % 32:
+        if not isinstance(w, torch.Tensor) or pd == 0 or N % 32 or x.dtype == torch.float32:
             return self.glu(self.linear(x, w, bias), act_kind, alpha, limit, layout)
         out = torch.empty(T, N // 2, dtype=x.dtype, device=x.device)
         n, splits = self.k.linear_ex(x, w, bias, out, self.workspace, self.status, force_splits, act_kind + 1, pd,

@@ -12,10 +12,11 @@ import torch
 import torch.nn.functional as F
 
 from .latent import LatentRef
+from .tied import TiedRef
 from .recurrent import RecurrentRef
 
 
-class RefOps(RecurrentRef, LatentRef):
+class RefOps(RecurrentRef, LatentRef, TiedRef):
     name = "reference"
 
     # ---------------------------------------------------------------- dense

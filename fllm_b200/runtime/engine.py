@@ -76,17 +76,17 @@ class LLMEngine:
             if hasattr(self.ops, "k") and not model_cfg.native_f32:
                 raise ValueError(f"{model_cfg.arch}: the kernels of this family run in bf16 only")
             self.cfg = dataclasses.replace(self.cfg, kv_cache_dtype="fp32")
-        if model_cfg.residual_streams and (tp > 1 or self.par.pp > 1):
-            raise NotImplementedError("models with residual streams run on one rank and one pipeline stage")
+        if model_cfg.fp32_residual and (tp > 1 or self.par.pp > 1):
+            raise NotImplementedError("models with a residual in fp32 run on one rank and one pipeline stage")
         act_dtype = torch.float32 if self.cfg.dtype == "fp32" else torch.bfloat16
         self.weights = weights or init_random_weights(
             model_cfg, self.device, act_dtype, seed, tp, tp_rank, self.par.expert_parallel,
             layers=self.layer_range, first_stage=self.first_stage, last_stage=self.last_stage)
         self.eos_token_id = eos_token_id
-        if model_cfg.has_mla:
-            # the latent pool has its own layout: the host / disk tiers, swapping and block export read the K / V pool
+        if model_cfg.has_row_cache:
+            # the pool has its own layout: the host / disk tiers, swapping and block export read the K / V pool
             if tp > 1:
-                raise NotImplementedError("latent-attention layers are not cut over tensor-parallel ranks")
+                raise NotImplementedError("layers with cache rows of their own layout are not cut over tensor-parallel ranks")
             self.cfg = dataclasses.replace(self.cfg, kv_tier_host_gb=0.0, kv_tier_disk_gb=0.0, preemption="recompute")
         if model_cfg.has_recurrent:
             # A recurrent state cannot be shared, rolled back or rebuilt from cached KV blocks: prompts are always
@@ -108,11 +108,11 @@ class LLMEngine:
         kv_dtype = {"bf16": torch.bfloat16, "fp32": torch.float32}.get(self.cfg.kv_cache_dtype, torch.float8_e4m3fn)
         if kv_dtype == torch.float32 and hasattr(self.ops, "k") and not (model_cfg.native_f32 and self.weights.embed.dtype == torch.float32):
             raise ValueError("an fp32 KV pool is for the reference operators and for models served in fp32")
-        if model_cfg.has_mla:
-            from ..models.mla import MlaCache
+        if model_cfg.has_row_cache:
+            from ..models.row_cache import RowCache
             if kv_dtype not in (torch.bfloat16, torch.float32):
-                raise ValueError("the latent cache of multi-head latent attention is bf16")
-            self.kv = MlaCache(MlaCache.widths(model_cfg, self.layer_range), num_blocks, self.block_size, self.device, kv_dtype)
+                raise ValueError("a cache of latent rows or of tied keys is bf16")
+            self.kv = RowCache(RowCache.specs(model_cfg, self.layer_range), num_blocks, self.block_size, self.device, kv_dtype)
         else:
             self.kv = KVCache(self._kv_layers(), num_blocks, self.spec.hkv_local, self.block_size,
                               model_cfg.head_dim, self.device, kv_dtype)
@@ -208,9 +208,9 @@ class LLMEngine:
         per_block = KVCache.bytes_per_block(self._kv_layers(), self.spec.hkv_local,
                                             self.block_size, self.model_cfg.head_dim,
                                             {"bf16": 2, "fp32": 4}.get(self.cfg.kv_cache_dtype, 1))
-        if self.model_cfg.has_mla:
-            from ..models.mla import MlaCache
-            per_block = max(1, MlaCache.bytes_per_block(MlaCache.widths(self.model_cfg, self.layer_range), self.block_size,
+        if self.model_cfg.has_row_cache:
+            from ..models.row_cache import RowCache
+            per_block = max(1, RowCache.bytes_per_block(RowCache.specs(self.model_cfg, self.layer_range), self.block_size,
                                                         4 if self.cfg.kv_cache_dtype == "fp32" else 2))
         if self.is_cuda:
             free, total = torch.cuda.mem_get_info(self.device)
@@ -258,8 +258,8 @@ class LLMEngine:
         handed to ``import_request`` of another engine of the same model and KV layout
         (rust/engine/src/disagg.rs is the reference's KV hand-over)."""
         self.drain()
-        if self.model_cfg.has_mla:
-            raise NotImplementedError("a latent cache is not handed over between engines")
+        if self.model_cfg.has_row_cache:
+            raise NotImplementedError("a cache with rows of its own layout is not handed over between engines")
         r = self.requests.get(request_id)
         if r is None or r.finished:
             raise KeyError(f"no live request {request_id!r}")

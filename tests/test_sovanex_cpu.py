@@ -112,8 +112,8 @@ def test_checkpoint_directory_and_config(tmp_path):
     assert [mc.kv_source(i) for i in range(5)] == [0, 1, 0, 3, 0] and [mc.has_kv(i) for i in range(5)] == [True, False, False, False, False]
     assert [mc.ffn_kind(i) for i in range(5)] == ["glu", "glu", "none", "none", "glu"]
     assert ModelConfig.from_dict(mc.to_dict()) == mc
-    from fllm_b200.models.mla import MlaCache
-    assert MlaCache.widths(mc, range(5)) == [48]                                             # 37 + 6, padded; shared by three layers
+    from fllm_b200.models.row_cache import RowCache, RowSpec
+    assert RowCache.specs(mc, range(5)) == [RowSpec(48)]                                             # 37 + 6, padded; shared by three layers
     bad = dict(w)
     bad["l1.mix.k"] = bad["l1.mix.k"][:-1]
     with pytest.raises(ValueError):
