@@ -1,4 +1,4 @@
-// torch.ops.fllm_b200 bindings of the recurrent token mixers (recurrent.cu).
+// torch.ops.fllm_b200 bindings of the recurrent token mixers (recurrent.cu, recurrent_ssd.cu).
 #include <ATen/ATen.h>
 #include <c10/cuda/CUDAGuard.h>
 #include <c10/cuda/CUDAStream.h>
@@ -50,8 +50,7 @@ void causal_conv1d(const Tensor& x, const Tensor& w, const optional<Tensor>& bia
 
 void mamba2_scan(const Tensor& x, const Tensor& dt, const Tensor& Bm, const Tensor& Cm, const Tensor& A, const optional<Tensor>& D,
                  const optional<Tensor>& dt_bias, Tensor state, const Tensor& q_starts, const Tensor& seq_state, const Tensor& positions,
-                 Tensor y, int64_t H, int64_t P, int64_t G, int64_t N, double dt_min, double dt_max, int64_t seg_len, int64_t segs,
-                 const optional<Tensor>& seg_scratch, int64_t skip_from) {
+                 Tensor y, int64_t H, int64_t P, int64_t G, int64_t N, double dt_min, double dt_max, int64_t skip_from) {
   const auto ty = act_type(x);
   TORCH_CHECK(rows_of(x, ty) && rows_of(dt, ty) && rows_of(Bm, ty) && rows_of(Cm, ty) && rows_of(y, ty), "activations: rows of one type");
   TORCH_CHECK(x.size(1) == H * P && y.size(1) == H * P && dt.size(1) == H && Bm.size(1) == G * N && Cm.size(1) == G * N, "widths");
@@ -59,34 +58,15 @@ void mamba2_scan(const Tensor& x, const Tensor& dt, const Tensor& Bm, const Tens
                   state.size(3) == N, "state: fp32 [slots, H, P, N]");
   check_batch(q_starts, seq_state, positions);
   c10::cuda::CUDAGuard guard(x.device());
-  float *seg_state = nullptr, *seg_dt = nullptr;
-  const int64_t B = seq_state.numel();
-  if (seg_len <= 0 || segs <= 1) {
-    fllm::SsdScanParams p{};
-    p.x = x.data_ptr(), p.dt = dt.data_ptr(), p.Bm = Bm.data_ptr(), p.Cm = Cm.data_ptr();
-    p.ldx = x.stride(0), p.lddt = dt.stride(0), p.ldb = Bm.stride(0), p.ldc = Cm.stride(0), p.ldy = y.stride(0);
-    p.A = opt_f32(A), p.D = opt_f32(D), p.dt_bias = opt_f32(dt_bias), p.state = state.data_ptr<float>();
-    p.q_starts = q_starts.data_ptr<int>(), p.seq_state = seq_state.data_ptr<int>(), p.positions = positions.data_ptr<int>(), p.y = y.data_ptr();
-    p.B = (int)B, p.tokens = (int)x.size(0), p.H = (int)H, p.P = (int)P, p.G = (int)G, p.N = (int)N;
-    p.dt_min = (float)dt_min, p.dt_max = (float)dt_max, p.skip_from = (int)skip_from, p.f32 = ty == at::kFloat ? 1 : 0;
-    const int rc = fllm::ssd_scan(p, cur_stream());
-    TORCH_CHECK(rc == 0, "mamba2_scan: unsupported arguments (code ", rc, "): heads a multiple of the groups, state width up to 256");
-    return;
-  }
-  TORCH_CHECK(ty == at::kBFloat16, "the sequence-parallel form runs in bf16");
-  {                                              // scratch: B * segs states of [H][P][N], then [B][segs - 1][H] step sums
-    const int64_t n_state = B * segs * H * P * N, n_dt = B * (segs - 1) * H;
-    TORCH_CHECK(seg_scratch.has_value() && seg_scratch->scalar_type() == at::kFloat && seg_scratch->is_contiguous() &&
-                    seg_scratch->numel() >= n_state + n_dt, "seg_scratch: fp32, at least B * (segs * H * P * N + (segs - 1) * H) values");
-    seg_state = seg_scratch->data_ptr<float>();
-    seg_dt = seg_state + n_state;
-  }
-  const int rc = fllm::mamba2_scan(x.data_ptr(), x.stride(0), dt.data_ptr(), dt.stride(0), Bm.data_ptr(), Bm.stride(0), Cm.data_ptr(),
-                                   Cm.stride(0), opt_f32(A), opt_f32(D), opt_f32(dt_bias), state.data_ptr<float>(), q_starts.data_ptr<int>(),
-                                   seq_state.data_ptr<int>(), positions.data_ptr<int>(), y.data_ptr(), y.stride(0), (int)B,
-                                   (int)H, (int)P, (int)G, (int)N, (float)dt_min, (float)dt_max, (int)seg_len, (int)segs, seg_state, seg_dt,
-                                   (int)skip_from, cur_stream());
-  TORCH_CHECK(rc == 0, "mamba2_scan: unsupported arguments (code ", rc, "): state width 16 / 32 / 64 / 128 / 256, B and C 16-byte aligned");
+  fllm::SsdScanParams p{};
+  p.x = x.data_ptr(), p.dt = dt.data_ptr(), p.Bm = Bm.data_ptr(), p.Cm = Cm.data_ptr();
+  p.ldx = x.stride(0), p.lddt = dt.stride(0), p.ldb = Bm.stride(0), p.ldc = Cm.stride(0), p.ldy = y.stride(0);
+  p.A = opt_f32(A), p.D = opt_f32(D), p.dt_bias = opt_f32(dt_bias), p.state = state.data_ptr<float>();
+  p.q_starts = q_starts.data_ptr<int>(), p.seq_state = seq_state.data_ptr<int>(), p.positions = positions.data_ptr<int>(), p.y = y.data_ptr();
+  p.B = (int)seq_state.numel(), p.tokens = (int)x.size(0), p.H = (int)H, p.P = (int)P, p.G = (int)G, p.N = (int)N;
+  p.dt_min = (float)dt_min, p.dt_max = (float)dt_max, p.skip_from = (int)skip_from, p.f32 = ty == at::kFloat ? 1 : 0;
+  const int rc = fllm::ssd_scan(p, cur_stream());
+  TORCH_CHECK(rc == 0, "mamba2_scan: unsupported arguments (code ", rc, "): heads a multiple of the groups, state width up to 256");
 }
 
 void mamba1_scan(const Tensor& x, const Tensor& dt, const Tensor& Bm, const Tensor& Cm, const optional<Tensor>& z, const Tensor& A,
@@ -170,8 +150,7 @@ TORCH_LIBRARY_FRAGMENT(fllm_b200, m) {
   m.def("causal_conv1d(Tensor x, Tensor w, Tensor? bias, Tensor(a!) state, Tensor q_starts, Tensor seq_state, Tensor positions, Tensor(b!) y, bool act, int max_q_len) -> ()",
         &causal_conv1d);
   m.def("mamba2_scan(Tensor x, Tensor dt, Tensor Bm, Tensor Cm, Tensor A, Tensor? D, Tensor? dt_bias, Tensor(a!) state, Tensor q_starts, "
-        "Tensor seq_state, Tensor positions, Tensor(b!) y, int H, int P, int G, int N, float dt_min, float dt_max, int seg_len, int segs, "
-        "Tensor? seg_scratch, int skip_from) -> ()",
+        "Tensor seq_state, Tensor positions, Tensor(b!) y, int H, int P, int G, int N, float dt_min, float dt_max, int skip_from) -> ()",
         &mamba2_scan);
   m.def("mamba1_scan(Tensor x, Tensor dt, Tensor Bm, Tensor Cm, Tensor? z, Tensor A, Tensor? D, Tensor? dt_bias, Tensor(a!) state, "
         "Tensor q_starts, Tensor seq_state, Tensor positions, Tensor(b!) y, int seg_len, int segs, Tensor? seg_scratch) -> ()",

@@ -278,14 +278,7 @@ void spec_verify_sampled(const void* target_logits, long long ld_t, const void* 
 int causal_conv1d(const void* x, long long ldx, const float* w, const float* bias, void* state, const int* q_starts,
                   const int* seq_state, const int* positions, void* y, long long ldy, int B, int C, int W, int act,
                   int max_q_len, cudaStream_t stream, int f32 = 0);   // max_q_len: host-side bound on a sequence's tokens in the step
-// Segmented scans (seg_len > 0, segs > 1): seg_state holds B * segs states (segs - 1 per sequence, then one start state per
-// sequence), seg_dt B * (segs - 1) sums of time steps per head (Mamba-2) or channel (Mamba-1).
-int mamba2_scan(const void* x, long long ldx, const void* dt, long long lddt, const void* Bm, long long ldb, const void* Cm,
-                long long ldc, const float* A, const float* D, const float* dt_bias, float* state, const int* q_starts,
-                const int* seq_state, const int* positions, void* y, long long ldy, int B, int H, int P, int G, int N,
-                float dt_min, float dt_max, int seg_len, int segs, float* seg_state, float* seg_dt, int skip_from,
-                cudaStream_t stream);
-// The same recurrence for any head and state width (N <= 256), bf16 or fp32 (recurrent_ssd.cu): one walk per sequence.
+// The Mamba-2 recurrence for any head and state width (N <= 256), bf16 or fp32 (recurrent_ssd.cu): one walk per sequence.
 struct SsdScanParams {
   const void *x, *dt, *Bm, *Cm;
   long long ldx, lddt, ldb, ldc, ldy;
@@ -298,6 +291,8 @@ struct SsdScanParams {
   int skip_from, f32;
 };
 int ssd_scan(const SsdScanParams& p, cudaStream_t stream);
+// Segmented scan (seg_len > 0, segs > 1): seg_state holds B * segs states (segs - 1 per sequence, then one start state per
+// sequence), seg_dt B * (segs - 1) sums of time steps per channel.
 int mamba1_scan(const void* x, long long ldx, const void* dt, long long lddt, const void* Bm, long long ldb, const void* Cm,
                 long long ldc, const void* z, long long ldz, const float* A, const float* D, const float* dt_bias, float* state,
                 const int* q_starts, const int* seq_state, const int* positions, void* y, long long ldy, int B, int Dm, int N,

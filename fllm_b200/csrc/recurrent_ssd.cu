@@ -5,8 +5,9 @@
 // ssd_scan_kernel walks a sequence's tokens, one CTA per (sequence, head, slice of state rows). TPK lanes share RPT rows, lane l
 // holding the columns 4 (l + TPK j) + 0..3 of each as pairs for the packed fp32 instructions. Tokens come in chunks: eight
 // threads per token fetch B and C one chunk ahead in their stored form and leave them in shared memory as fp32 with the
-// token's decay and step size, so the walk over a chunk touches shared memory and registers only. A token's columns are
-// independent, so the walk is bound by the rate of its fp32 instructions, not by a chain.
+// token's decay and step size, so the walk over a chunk touches shared memory and registers only. Four rows per thread keep the
+// shared-memory reads below the arithmetic; the outputs of four tokens are summed over the lanes together, each exchange
+// halving the values a lane carries, so a lane ends with a sixteenth of the sums and none is computed twice.
 //
 // ssd_decode_kernel serves steps of single tokens: inputs straight from global memory, no shared memory, many CTAs that keep
 // state reads in flight (a decoded token reads and writes the whole state once).
@@ -56,15 +57,43 @@ struct SsdArgs {
   int skip_from;                      // sequences with at least this many tokens in the step are left to another path (0 = none)
 };
 
-template <typename T, int NP, bool EXACT, int RPT>
+// sums over the L lanes of a row group of V values per lane: afterwards v[i] of lane l is the sum of value (l >> rest) * left + i
+template <int L, int V>
+struct LaneSums {
+  static constexpr int left(int l, int v) { return l > 1 && v > 1 ? left(l / 2, v / 2) : v; }
+  static constexpr int rest(int l, int v) { return l > 1 && v > 1 ? rest(l / 2, v / 2) : (l > 1 ? 1 + rest(l / 2, v) : 0); }
+  static constexpr int kLeft = left(L, V), kRest = rest(L, V);
+};
+template <int L, int V, int SIZE>
+__device__ __forceinline__ void lane_sums(float (&v)[SIZE], int lane) {
+  if constexpr (L > 1 && V > 1) {
+    const bool upper = (lane & (L / 2)) != 0;
+#pragma unroll
+    for (int i = 0; i < V / 2; ++i) {
+      const float send = upper ? v[i] : v[i + V / 2], keep = upper ? v[i + V / 2] : v[i];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, send, L / 2);
+    }
+    lane_sums<L / 2, V / 2>(v, lane);
+  } else if constexpr (L > 1) {
+#pragma unroll
+    for (int o = L / 2; o > 0; o >>= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+  }
+}
+
+template <int NP>
+struct SsdTile {
+  static constexpr int NPT = NP <= 32 ? 4 : 8, TPK = NP / NPT, RG = 128 / TPK, RPT = 4, ROWS = RPT * RG, GROUP = 4;
+};
+
+template <typename T, int NP, bool EXACT>
 __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
-  constexpr int NPT = 16, TPK = NP / NPT, RG = 128 / TPK, ROWS = RPT * RG, C = kSsdChunk, EPT = NP / 8, VPT = ROWS * C / 128;
-  __shared__ __align__(16) float sb[C][NP], sc[C][NP];
-  __shared__ float sx[C][ROWS];
+  using L = SsdTile<NP>;
+  constexpr int NPT = L::NPT, TPK = L::TPK, RPT = L::RPT, ROWS = L::ROWS, GROUP = L::GROUP, C = kSsdChunk, EPT = NP / 8, VPT = ROWS * C / 128;
+  __shared__ __align__(16) float sb[C][NP], sc[C][NP], sx[C][ROWS];
   __shared__ float2 sg[C];                               // decay, step size
   const int N = EXACT ? NP : a.N;
   const int ptiles = (a.P + ROWS - 1) / ROWS;
-  const int h = blockIdx.x / ptiles, p0 = (blockIdx.x % ptiles) * ROWS, row = threadIdx.x / TPK;      // rows p0 + row + RG r
+  const int h = blockIdx.x / ptiles, p0 = (blockIdx.x % ptiles) * ROWS, row = threadIdx.x / TPK * RPT;      // rows p0 + row + r
   const int lk = threadIdx.x % TPK, s = blockIdx.y;
   const int t0 = a.q_starts[s], n = a.q_starts[s + 1] - t0;
   if (n <= 0 || (a.skip_from > 0 && n >= a.skip_from)) return;
@@ -76,7 +105,7 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
     float v[NPT];
 #pragma unroll
     for (int i = 0; i < NPT; ++i) v[i] = 0.f;
-    if (!fresh) load_state<TPK, EXACT>(st + (long long)min(p0 + row + RG * r, a.P - 1) * N, lk, N, v);
+    if (!fresh) load_state<TPK, EXACT>(st + (long long)min(p0 + row + r, a.P - 1) * N, lk, N, v);
 #pragma unroll
     for (int i = 0; i < NPT / 2; ++i) S[r][i] = pair(v[2 * i], v[2 * i + 1]);
   }
@@ -123,15 +152,17 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
   for (int base = 0; base < n; base += C) {
     const int cnt = min(C, n - base);
     __syncthreads();                                     // the chunk before is consumed
-    if (tt < cnt) {
+    {
+      // tokens past the end are steps that change nothing: decay 1, step size 0, zero inputs
+      const bool live = tt < cnt;
       float br[EPT], cr[EPT];
       if constexpr (WIDE) {
         const T *bt = reinterpret_cast<const T*>(bw), *ct = reinterpret_cast<const T*>(cw);
 #pragma unroll
-        for (int i = 0; i < EPT; ++i) br[i] = ld1(bt + i), cr[i] = ld1(ct + i);
+        for (int i = 0; i < EPT; ++i) br[i] = live ? ld1(bt + i) : 0.f, cr[i] = live ? ld1(ct + i) : 0.f;
       } else {
 #pragma unroll
-        for (int i = 0; i < EPT; ++i) br[i] = bl[i], cr[i] = cl[i];
+        for (int i = 0; i < EPT; ++i) br[i] = live ? bl[i] : 0.f, cr[i] = live ? cl[i] : 0.f;
       }
       if constexpr (EPT % 4 == 0) {
 #pragma unroll
@@ -144,76 +175,86 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
         for (int i = 0; i < EPT; ++i) sb[tt][column(i)] = br[i], sc[tt][column(i)] = cr[i];
       }
       if (part == 0) {
-        const float dt = fminf(fmaxf(softplus_t<T>(ld1(&dr) + dtb), a.dt_min), a.dt_max);
+        const float dt = live ? fminf(fmaxf(softplus_t<T>(ld1(&dr) + dtb), a.dt_min), a.dt_max) : 0.f;
         sg[tt] = make_float2(exp_t<T>(dt * A), dt);
       }
     }
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
       const int e = threadIdx.x + i * 128;
-      if (e / ROWS < cnt) sx[e / ROWS][e % ROWS] = ld1(&xr[i]);
+      sx[e / ROWS][e % ROWS] = e / ROWS < cnt ? ld1(&xr[i]) : 0.f;
     }
     __syncthreads();
     if (base + C < n) fetch(base + C);
-    T* yp = a.y + (long long)(t0 + base) * a.ldy + (long long)h * a.P + p0 + row;
-#pragma unroll 2
-    for (int i = 0; i < cnt; ++i, yp += a.ldy) {
-      uint64_t b2[NPT / 2], c2[NPT / 2];
+    for (int i0 = 0; i0 < cnt; i0 += GROUP) {
+      float o[GROUP * RPT];
 #pragma unroll
-      for (int j = 0; j < NPT / 4; ++j) {
-        const ulonglong2 bv = *reinterpret_cast<const ulonglong2*>(&sb[i][4 * (lk + TPK * j)]);
-        const ulonglong2 cv = *reinterpret_cast<const ulonglong2*>(&sc[i][4 * (lk + TPK * j)]);
-        b2[2 * j] = bv.x, b2[2 * j + 1] = bv.y, c2[2 * j] = cv.x, c2[2 * j + 1] = cv.y;
-      }
-      const float2 g = sg[i];
-      const uint64_t d2 = pair(g.x, g.x);
+      for (int k = 0; k < GROUP; ++k) {
+        const int i = i0 + k;
+        uint64_t b2[NPT / 2], c2[NPT / 2];
 #pragma unroll
-      for (int r = 0; r < RPT; ++r) {
-        const float xv = sx[i][row + RG * r], u = g.y * xv;
-        const uint64_t u2 = pair(u, u);
-        uint64_t o2[2] = {0, 0};                           // two chains of packed sums
-#pragma unroll
-        for (int j = 0; j < NPT / 2; ++j) {
-          S[r][j] = fma2(b2[j], u2, mul2(S[r][j], d2));
-          o2[j & 1] = fma2(S[r][j], c2[j], o2[j & 1]);
+        for (int j = 0; j < NPT / 4; ++j) {
+          const ulonglong2 bv = *reinterpret_cast<const ulonglong2*>(&sb[i][4 * (lk + TPK * j)]);
+          const ulonglong2 cv = *reinterpret_cast<const ulonglong2*>(&sc[i][4 * (lk + TPK * j)]);
+          b2[2 * j] = bv.x, b2[2 * j + 1] = bv.y, c2[2 * j] = cv.x, c2[2 * j + 1] = cv.y;
         }
-        const float2 e = unpair(o2[0]), f = unpair(o2[1]);
-        const float o = row_sum<TPK>((e.x + e.y) + (f.x + f.y));
-        if (lk == 0 && p0 + row + RG * r < a.P) st1(yp + RG * r, fmaf(D, xv, o));
+        const float2 g = sg[i];
+        const uint64_t d2 = pair(g.x, g.x);
+        const float4 x4 = *reinterpret_cast<const float4*>(&sx[i][row]);
+        const float xs[RPT] = {x4.x, x4.y, x4.z, x4.w};
+#pragma unroll
+        for (int r = 0; r < RPT; ++r) {
+          const float u = g.y * xs[r];
+          const uint64_t u2 = pair(u, u);
+          uint64_t o2 = 0;
+#pragma unroll
+          for (int j = 0; j < NPT / 2; ++j) {
+            S[r][j] = fma2(b2[j], u2, mul2(S[r][j], d2));
+            o2 = fma2(S[r][j], c2[j], o2);
+          }
+          const float2 e = unpair(o2);
+          o[k * RPT + r] = e.x + e.y;
+        }
+      }
+      using Sums = LaneSums<TPK, GROUP * RPT>;
+      lane_sums<TPK, GROUP * RPT>(o, lk);
+      if (Sums::kRest == 0 || (lk & ((1 << Sums::kRest) - 1)) == 0) {
+#pragma unroll
+        for (int v = 0; v < Sums::kLeft; ++v) {
+          const int at = (lk >> Sums::kRest) * Sums::kLeft + v, i = i0 + at / RPT, p = row + at % RPT;
+          if (i < cnt && p0 + p < a.P) st1(a.y + (long long)(t0 + base + i) * a.ldy + (long long)h * a.P + p0 + p, fmaf(D, sx[i][p], o[v]));
+        }
       }
     }
   }
 #pragma unroll
   for (int r = 0; r < RPT; ++r) {
-    if (p0 + row + RG * r >= a.P) continue;
+    if (p0 + row + r >= a.P) continue;
     float v[NPT];
 #pragma unroll
     for (int i = 0; i < NPT / 2; ++i) {
       const float2 f = unpair(S[r][i]);
       v[2 * i] = f.x, v[2 * i + 1] = f.y;
     }
-    store_state<TPK, EXACT>(st + (long long)(p0 + row + RG * r) * N, lk, N, v);
+    store_state<TPK, EXACT>(st + (long long)(p0 + row + r) * N, lk, N, v);
   }
 }
 
-template <typename T, int NP, bool EXACT, int RPT>
+template <typename T, int NP, bool EXACT>
 __global__ void __launch_bounds__(128) ssd_decode_kernel(const SsdArgs<T> a) {
-  constexpr int NPT = 16, TPK = NP / NPT, RG = 128 / TPK, ROWS = RPT * RG;
+  constexpr int NPT = 16, TPK = NP / NPT, ROWS = 128 / TPK;
   const int N = EXACT ? NP : a.N;
   const int ptiles = (a.P + ROWS - 1) / ROWS;
-  const int h = blockIdx.x / ptiles, p0 = (blockIdx.x % ptiles) * ROWS + threadIdx.x / TPK;      // rows p0 + RG r
+  const int h = blockIdx.x / ptiles, p = (blockIdx.x % ptiles) * ROWS + threadIdx.x / TPK;
   const int lk = threadIdx.x % TPK, s = blockIdx.y;
   const int t0 = a.q_starts[s], n = a.q_starts[s + 1] - t0;
   if (n <= 0 || (a.skip_from > 0 && n >= a.skip_from)) return;
-  float* st = a.state + ((long long)a.seq_state[s] * a.H + h) * a.P * N;
-  float S[RPT][NPT];
-  const bool fresh = a.positions[t0] == 0;
+  const int pc = min(p, a.P - 1);
+  float* st = a.state + (((long long)a.seq_state[s] * a.H + h) * a.P + pc) * N;
+  float S[NPT];
 #pragma unroll
-  for (int r = 0; r < RPT; ++r) {
-#pragma unroll
-    for (int i = 0; i < NPT; ++i) S[r][i] = 0.f;
-    if (!fresh) load_state<TPK, EXACT>(st + (long long)min(p0 + RG * r, a.P - 1) * N, lk, N, S[r]);
-  }
+  for (int i = 0; i < NPT; ++i) S[i] = 0.f;
+  if (a.positions[t0] != 0) load_state<TPK, EXACT>(st, lk, N, S);
   const float A = a.A[h], D = a.D != nullptr ? a.D[h] : 0.f, dtb = a.dt_bias != nullptr ? a.dt_bias[h] : 0.f;
   const long long go = (long long)(h / (a.H / a.G)) * N;
   for (long long t = t0; t < t0 + n; ++t) {
@@ -235,24 +276,17 @@ __global__ void __launch_bounds__(128) ssd_decode_kernel(const SsdArgs<T> a) {
       }
     }
     const float dt = fminf(fmaxf(softplus_t<T>(ld1(a.dt + t * a.lddt + h) + dtb), a.dt_min), a.dt_max);
-    const float d = exp_t<T>(dt * A);
+    const float d = exp_t<T>(dt * A), xv = ld1(a.x + t * a.ldx + (long long)h * a.P + pc), u = dt * xv;
+    float o[2] = {0.f, 0.f};
 #pragma unroll
-    for (int r = 0; r < RPT; ++r) {
-      const int p = p0 + RG * r;
-      const float xv = ld1(a.x + t * a.ldx + (long long)h * a.P + min(p, a.P - 1)), u = dt * xv;
-      float o[2] = {0.f, 0.f};
-#pragma unroll
-      for (int i = 0; i < NPT; ++i) {
-        S[r][i] = fmaf(B[i], u, d * S[r][i]);
-        o[i & 1] = fmaf(S[r][i], C[i], o[i & 1]);
-      }
-      const float tot = row_sum<TPK>(o[0] + o[1]);
-      if (lk == 0 && p < a.P) st1(a.y + t * a.ldy + (long long)h * a.P + p, fmaf(D, xv, tot));
+    for (int i = 0; i < NPT; ++i) {
+      S[i] = fmaf(B[i], u, d * S[i]);
+      o[i & 1] = fmaf(S[i], C[i], o[i & 1]);
     }
+    const float tot = row_sum<TPK>(o[0] + o[1]);
+    if (lk == 0 && p < a.P) st1(a.y + t * a.ldy + (long long)h * a.P + p, fmaf(D, xv, tot));
   }
-#pragma unroll
-  for (int r = 0; r < RPT; ++r)
-    if (p0 + RG * r < a.P) store_state<TPK, EXACT>(st + (long long)(p0 + RG * r) * N, lk, N, S[r]);
+  if (p < a.P) store_state<TPK, EXACT>(st, lk, N, S);
 }
 }  // namespace
 
@@ -270,11 +304,11 @@ int ssd_scan(const SsdScanParams& p, cudaStream_t stream) {
   };
 #define FLLM_SSD(T_, NP_, EXACT_)                                                                                     \
   {                                                                                                                   \
-    constexpr int rows = 128 / (NP_ / 16);                                                                            \
+    constexpr int drows = 128 / (NP_ / 16), rows = SsdTile<NP_>::ROWS;                                                \
     if (p.tokens == p.B)                                                                                              \
-      ssd_decode_kernel<T_, NP_, EXACT_, 1><<<dim3(p.H * ((p.P + rows - 1) / rows), p.B), 128, 0, stream>>>(args(T_{}));             \
+      ssd_decode_kernel<T_, NP_, EXACT_><<<dim3(p.H * ((p.P + drows - 1) / drows), p.B), 128, 0, stream>>>(args(T_{}));     \
     else                                                                                                              \
-      ssd_scan_kernel<T_, NP_, EXACT_, 2><<<dim3(p.H * ((p.P + 2 * rows - 1) / (2 * rows)), p.B), 128, 0, stream>>>(args(T_{}));     \
+      ssd_scan_kernel<T_, NP_, EXACT_><<<dim3(p.H * ((p.P + rows - 1) / rows), p.B), 128, 0, stream>>>(args(T_{}));   \
     return 0;                                                                                                         \
   }
 #define FLLM_SSD_N(T_, EXACT_)                    \

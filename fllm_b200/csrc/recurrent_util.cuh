@@ -74,11 +74,11 @@ __device__ __forceinline__ float row_sum(float v) {
   return v;
 }
 
-// this lane's columns of a state row
-template <int TPK, bool EXACT>
-__device__ __forceinline__ void load_state(const float* st, int lk, int DK, float (&S)[16]) {
+// this lane's columns 4 (lk + TPK j) + 0..3 of a state row
+template <int TPK, bool EXACT, int NPT>
+__device__ __forceinline__ void load_state(const float* st, int lk, int DK, float (&S)[NPT]) {
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
+  for (int j = 0; j < NPT / 4; ++j) {
     const int c = 4 * (lk + TPK * j);
     if (EXACT) {
       const float4 f = *reinterpret_cast<const float4*>(st + c);
@@ -89,10 +89,10 @@ __device__ __forceinline__ void load_state(const float* st, int lk, int DK, floa
     }
   }
 }
-template <int TPK, bool EXACT>
-__device__ __forceinline__ void store_state(float* st, int lk, int DK, const float (&S)[16]) {
+template <int TPK, bool EXACT, int NPT>
+__device__ __forceinline__ void store_state(float* st, int lk, int DK, const float (&S)[NPT]) {
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
+  for (int j = 0; j < NPT / 4; ++j) {
     const int c = 4 * (lk + TPK * j);
     if (EXACT) {
       *reinterpret_cast<float4*>(st + c) = make_float4(S[4 * j], S[4 * j + 1], S[4 * j + 2], S[4 * j + 3]);

@@ -143,7 +143,7 @@ def mamba2_mixer(dec, li: int, lw, h: torch.Tensor, b) -> torch.Tensor:
     xbc = ops.causal_conv1d(zxd[:, Dp:Dp + C], m["conv_w"], m.get("conv_b"), dec.rstate.conv[li], qs, ss, pos, act=True, max_q_len=getattr(b, "max_q_len", 0))
     y = ops.mamba2_scan(xbc[:, :Di], zxd[:, Dp + C:Dp + C + H], xbc[:, Dp:Dp + G * N], xbc[:, Dp + bc:Dp + bc + G * N], m["A"], m["D"],
                         m["dt_bias"], dec.rstate.scan[li], qs, ss, pos, H, P, G, N, s.get("dt_min", 0.0),
-                        s.get("dt_max", 1e30), getattr(b, "max_q_len", 0), None, getattr(b, "host_seqs", None))
+                        s.get("dt_max", 1e30), getattr(b, "max_q_len", 0), getattr(b, "host_seqs", None))
     mode = s.get("gate_mode", "norm_after_gate")
     if mode == "gate_only":                       # Falcon-H1 without the mixer norm: y * silu(z)
         y = y * F.silu(zxd[:, :Di])

@@ -21,10 +21,10 @@ import torch.nn.functional as F
 RWKV6, RWKV7, GATED_DELTA, KDA = 0, 1, 2, 3
 # Mamba-2 prompt chunks from this many tokens on take the matrix form (``ssd_chunked``) instead of the token walk; 0 = never.
 # Off by default: as a chain of PyTorch operators (about 40 launches per layer and sequence over [chunks, heads, 128, 128]
-# tensors) it measured slower than the sequence-parallel scan kernel on a B200 (Mamba-2 2.7B prefill 15.3 k against
-# 16.6 k tok/s); it is kept as the tested statement of the algorithm a fused kernel would implement.
+# tensors) it measured slower than the scan kernel on a B200; it is kept as the tested statement of the algorithm a fused
+# kernel would implement.
 SSD_MIN_TOKENS = int(__import__("os").environ.get("FLLM_SSD_MIN_TOKENS", "0"))
-# Tokens per segment of the sequence-parallel Mamba scans (0: always one walk per sequence).
+# Tokens per segment of the sequence-parallel Mamba-1 scan (0: always one walk per sequence).
 SCAN_SEG_LEN = int(__import__("os").environ.get("FLLM_SCAN_SEG_LEN", "128"))
 
 
@@ -105,7 +105,7 @@ class RecurrentRef:
         return y
 
     def mamba2_scan(self, x, dt, Bm, Cm, A, D, dt_bias, state, q_starts, seq_state, positions, H, P, G, N,
-                    dt_min=0.0, dt_max=float("inf"), max_q_len=0, seg_len=None, host_seqs=None):
+                    dt_min=0.0, dt_max=float("inf"), max_q_len=0, host_seqs=None):
         """h = exp(dt A) h + dt x (x) B;  y = h C + D x per head; dt = clamp(softplus(dt + dt_bias))."""
         y = torch.empty_like(x)
         rep = H // G
@@ -254,14 +254,11 @@ class RecurrentNative:
         return y
 
     def mamba2_scan(self, x, dt, Bm, Cm, A, D, dt_bias, state, q_starts, seq_state, positions, H, P, G, N,
-                    dt_min=0.0, dt_max=float("inf"), max_q_len=0, seg_len=None, host_seqs=None):
-        """``max_q_len`` (host-side bound on the tokens of a sequence in this step) lets long prompts of few sequences run
-        sequence-parallel: segments of ``seg_len`` tokens side by side, a short combine pass, then the outputs.
-        ``host_seqs`` (the step's sequences as (first row, rows, state row, fresh) known on the host) sends prompt chunks
+                    dt_min=0.0, dt_max=float("inf"), max_q_len=0, host_seqs=None):
+        """``host_seqs`` (the step's sequences as (first row, rows, state row, fresh) known on the host) sends prompt chunks
         of ``SSD_MIN_TOKENS`` tokens or more through the matrix form (``ssd_chunked``: batched matrix products on tensor
         cores); the scan kernel then leaves those sequences alone."""
         y = torch.empty(x.shape, dtype=x.dtype, device=x.device)
-        B = seq_state.numel()
         skip = 0
         if host_seqs:
             long = [q for q in host_seqs if SSD_MIN_TOKENS and q[1] >= SSD_MIN_TOKENS]
@@ -273,21 +270,10 @@ class RecurrentNative:
             if long:
                 if len(long) == len(host_seqs):
                     return y
-                skip, max_q_len = SSD_MIN_TOKENS, SSD_MIN_TOKENS - 1
-        if seg_len is None:
-            # CTAs that walk long sequences (a mixed step's decode rows finish at once and do not fill the GPU)
-            ctas = max(1, min(B, x.shape[0] // 256)) * H * max(1, P * max(N // 16, 1) // 128)
-            seg_len = SCAN_SEG_LEN if (max_q_len >= 512 and ctas < 4 * 148) else 0
-        segs = -(-int(max_q_len) // seg_len) if seg_len else 1
-        scratch = None
-        if segs > 1:
-            need = B * (segs * H * P * N + (segs - 1) * H)
-            scratch = getattr(self, "_scan_scratch", None)
-            if scratch is None or scratch.numel() < need:
-                scratch = self._scan_scratch = torch.empty(need, dtype=torch.float32, device=x.device)
+                skip = SSD_MIN_TOKENS
         self.k.mamba2_scan(x, dt, Bm, Cm, A, D, dt_bias, state, q_starts, seq_state, positions, y, H, P, G, N,
-                           float(dt_min), float(min(dt_max, 3.0e38)), int(seg_len if segs > 1 else 0), int(segs), scratch, int(skip))
-        self.launches += 3 if segs > 1 else 1
+                           float(dt_min), float(min(dt_max, 3.0e38)), int(skip))
+        self.launches += 1
         return y
 
     def mamba1_scan(self, x, dt, Bm, Cm, z, A, D, dt_bias, state, q_starts, seq_state, positions, max_q_len=0, seg_len=None):
