@@ -1,10 +1,12 @@
-"""Throughput of a design beside the framework's closest other model at equal size (``bench.py --compare sovanex``).
+"""Throughput of a design beside the framework's closest other model at equal size (``bench.py --compare sovanex|divanex``).
 
 The closest other model of Sovanex is a hybrid of the layer kinds it shares with other families: the gated delta rule
 (Qwen3-Next) and 512 + 64 wide latent attention (DeepSeek), with the same layer order, heads, widths and squared-ReLU
-networks, but RMSNorm around one bf16 residual, no gate on the attention heads and no shared rows. Both run random
-weights through the engine: prompts of 1024 tokens in 2048-token steps, then captured decode steps. ``--kernels`` times
-the kernels that differ, each beside its like kernel on the same sizes.
+networks, but RMSNorm around one bf16 residual, no gate on the attention heads and no shared rows. That of Divanex is a
+hybrid of Mamba-2 and grouped-query attention with normalised queries and keys and capped scores (Bamba, Gemma-2), the same
+layer order, sizes and clamped SwiGLU networks (gpt-oss), but separate values, norms in front of the blocks around one bf16
+residual, and no token input. Both models run random weights through the engine: prompts of 1024 tokens in 2048-token
+steps, then captured decode steps. ``--kernels`` times the kernels that differ, each beside its like kernel on the same sizes.
 """
 from __future__ import annotations
 
@@ -14,7 +16,7 @@ from typing import Dict, List
 
 import torch
 
-from .config import EngineConfig, ModelConfig, sovanex_from_config
+from .config import EngineConfig, ModelConfig, divanex_from_config, sovanex_from_config
 
 # name -> width, layers, feed-forward width, value heads / key heads of the delta rule, attention heads
 SIZES = {"1b": (2048, 12, 8192, 32, 16, 16), "3b": (3072, 24, 12288, 48, 24, 24), "7b": (4096, 32, 16384, 64, 32, 32)}
@@ -43,6 +45,29 @@ def twin_config(size: str) -> ModelConfig:
                        layer_kinds=["gated_delta" if i % 4 < 3 else "mla" for i in range(L)],
                        ssm=dict(num_k_heads=Hk, num_v_heads=Hv, head_k_dim=128, head_v_dim=128, d_conv=4),
                        mla=dict(q_lora_rank=0, kv_lora_rank=512, qk_nope_head_dim=128, qk_rope_head_dim=64, v_head_dim=128))
+
+
+# name -> width, layers, feed-forward width, Mamba-2 heads (of 64, state 128, 8 groups), query / key heads (of 128), token input
+DIVANEX_SIZES = {"1b": (2048, 24, 8192, 64, 16, 4, 256), "3b": (3072, 32, 12288, 96, 24, 6, 256), "7b": (4096, 40, 16384, 128, 32, 8, 256)}
+
+
+def divanex_config(size: str) -> ModelConfig:
+    W, L, ff, Hm, H, G, side = DIVANEX_SIZES[size]
+    mamba = dict(heads=Hm, vdim=64, state=128, groups=8, norm_groups=8, conv=4)
+    attn = dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, q_temp=dict(coef=0.1, every=8192))
+    layers = [dict(type="attention", mixer=attn, mlp=dict(kind="dense", ff=ff, limit=7.0)) if i % 4 == 3 else dict(type="mamba2", mixer=mamba, mlp=None)
+              for i in range(L)]
+    return divanex_from_config(ModelConfig, dict(architecture="Divanex", name=f"divanex-{size}", layers=layers, norm=dict(eps=1e-5), embedding=dict(scale=4.0),
+                                                 postln_alpha=2.0, logit_scale=0.5, token_side=dict(dim=side), vocab=VOCAB, width=W))
+
+
+def divanex_twin_config(size: str) -> ModelConfig:
+    W, L, ff, Hm, H, G, _ = DIVANEX_SIZES[size]
+    return ModelConfig(arch="hybrid", name=f"mamba2-gqa-hybrid-{size}", vocab_size=VOCAB, hidden_size=W, num_layers=L, num_heads=H, num_kv_heads=G, head_dim=128,
+                       use_rope=False, qk_norm=True, attn_softcap=30.0, intermediate_size=ff, act="swiglu_oai", tie_embeddings=False,
+                       layer_kinds=["attention" if i % 4 == 3 else "mamba2" for i in range(L)], ffn_kinds=["glu" if i % 4 == 3 else "none" for i in range(L)],
+                       ssm=dict(d_inner=Hm * 64, d_state=128, d_conv=4, n_groups=8, head_dim=64, n_heads=Hm, norm_groups=8, conv_bias=True, dt_min=0.0,
+                                dt_max=1e30))
 
 
 def throughput(cfg: ModelConfig, batch: int, prompt_len: int, steps: int, warmup: int, device, graphs: bool = True) -> Dict[str, float]:
@@ -122,30 +147,42 @@ def _batch(lens: List[int], ctxs: List[int], device, bs: int = 16):
                            q_starts=i32(torch.tensor(starts)), seq_state=i32(torch.arange(B)), tokens=starts[-1])
 
 
-def kernel_table(device, size: str = "1b") -> List[dict]:
-    """Kernels of the new layers beside their like kernels: microseconds, the floor of each (bytes at the measured copy
-    bandwidth or products at the measured GEMM rate, whichever is longer), and the ratio of the two distances."""
-    import json
-    import os
-    from .ops.native import NativeOps
-    ops, bf, g = NativeOps(device), torch.bfloat16, torch.Generator(device=device).manual_seed(1)
-    peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
-    path = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "MEASURED_PEAKS.json")
-    if os.path.exists(path):
-        peaks.update({k: v for k, v in json.load(open(path)).items() if k in peaks})
-    flush = torch.empty(256 << 20, dtype=torch.uint8, device=device)
+class _Table:
+    """Rows of kernels beside their like kernels: microseconds, the floor of each (bytes at the measured copy bandwidth or
+    products at the measured GEMM rate, whichever is longer), and the ratio of the two distances."""
+
+    def __init__(self, device):
+        import json
+        import os
+        from .ops.native import NativeOps
+        self.ops, self.device, self.rows = NativeOps(device), device, []
+        self.gen = torch.Generator(device=device).manual_seed(1)
+        self.peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+        path = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "MEASURED_PEAKS.json")
+        if os.path.exists(path):
+            self.peaks.update({k: v for k, v in json.load(open(path)).items() if k in self.peaks})
+        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device=device)
+
+    def rnd(self, *shape, dtype=torch.bfloat16):
+        return torch.randn(*shape, device=self.device, generator=self.gen).to(dtype)
+
+    def time(self, fn) -> float:
+        return _time(fn, self.flush)
+
+    def floor(self, nbytes, flops=0.0) -> float:
+        return max(nbytes / self.peaks["hbm_gbs"] / 1e3, flops / self.peaks["bf16_tflops"] / 1e6)
+
+    def add(self, shape, name, us, fl, like, like_us, like_fl) -> None:
+        self.rows.append({"shape": shape, "kernel": name, "us": round(us, 1), "floor_us": round(fl, 2), "like": like, "like_us": round(like_us, 1),
+                          "like_floor_us": round(like_fl, 2), "times_as_far": round((us / fl) / (like_us / like_fl), 2)})
+
+
+def sovanex_kernels(device, size: str = "1b") -> List[dict]:
+    tab = _Table(device)
+    ops, rnd, floor, add = tab.ops, tab.rnd, tab.floor, tab.add
+    bf = torch.bfloat16
     W, _, ff, Hv, Hk, H = SIZES[size]
     R, dr, dn, S = 512, 64, 128, 4
-    rnd = lambda *s, dtype=bf: torch.randn(*s, device=device, generator=g).to(dtype)
-    rows = []
-
-    def floor(nbytes, flops=0.0):
-        return max(nbytes / peaks["hbm_gbs"] / 1e3, flops / peaks["bf16_tflops"] / 1e6)
-
-    def add(shape, name, us, fl, like, like_us, like_fl):
-        rows.append({"shape": shape, "kernel": name, "us": round(us, 1), "floor_us": round(fl, 2), "like": like, "like_us": round(like_us, 1),
-                     "like_floor_us": round(like_fl, 2), "times_as_far": round((us / fl) / (like_us / like_fl), 2)})
-
     for shape, lens, ctxs in (("decode 64 x 1152", [1] * 64, [1152] * 64), ("decode 8 x 4096", [1] * 8, [4096] * 8),
                               ("prompt 2048", [2048], [2048]), ("prompt 4 x 512 at 2048", [512] * 4, [2048] * 4)):
         b = _batch(lens, ctxs, device)
@@ -154,35 +191,84 @@ def kernel_table(device, size: str = "1b") -> List[dict]:
         qa, qp = q[:, :, :R].contiguous(), q[:, :, R:].transpose(0, 1).contiguous()
         keys = sum(c * n - n * (n - 1) // 2 for n, c in zip(lens, ctxs))
         fl = floor(2 * (sum(ctxs) * (R + dr) + q.numel() + H * T * R), 2.0 * keys * H * (2 * R + dr))
-        add(shape, "attention_latent", _time(lambda: ops.attention_latent(q, cache, b, 0.07, R), flush), fl, "attention_mla",
-            _time(lambda: ops.attention_mla(qa, qp, cache, b.block_tables, b.row_seq, b.positions, 0.07, b.max_kv_len), flush), fl)
+        add(shape, "attention_latent", tab.time(lambda: ops.attention_latent(q, cache, b, 0.07, R)), fl, "attention_mla",
+            tab.time(lambda: ops.attention_mla(qa, qp, cache, b.block_tables, b.row_seq, b.positions, 0.07, b.max_kv_len)), fl)
         ckv, qh, inv, nw = rnd(T, R + dr), rnd(T, H * (dn + dr)), torch.rand(dr // 2, device=device), torch.ones(R, device=device, dtype=bf)
         fl = floor(2 * T * (2 * (R + dr) + 2 * H * dr))
-        add(shape, "latent_prepare", _time(lambda: ops.latent_prepare(ckv, qh, dn + dr, dn, b.positions, b.slots, inv, 1.0, nw, 1e-5, cache, q, R, 0), flush), fl,
-            "mla_prepare", _time(lambda: ops.mla_prepare(ckv, qh.view(T, H, dn + dr), dn, b.positions, b.slots, inv, 1.0, nw, 1e-5, cache), flush), fl)
+        add(shape, "latent_prepare", tab.time(lambda: ops.latent_prepare(ckv, qh, dn + dr, dn, b.positions, b.slots, inv, 1.0, nw, 1e-5, cache, q, R, 0)), fl,
+            "mla_prepare", tab.time(lambda: ops.mla_prepare(ckv, qh.view(T, H, dn + dr), dn, b.positions, b.slots, inv, 1.0, nw, 1e-5, cache)), fl)
     for T in (64, 2048):
         shape = f"{T} rows"
         x, y, res = rnd(T, S, W, dtype=torch.float32), rnd(T, W), rnd(T, W)
         mix, vec, w = torch.eye(S, device=device), torch.ones(S, device=device), torch.ones(W, device=device, dtype=bf)
-        add(shape, "streams_step (4 fp32 streams, LayerNorm)", _time(lambda: ops.streams_step(x, y, mix, vec, vec, w, w, W, 1e-5), flush),
-            floor(T * W * (8 * S + 4)), "residual add + rmsnorm", _time(lambda: ops.rmsnorm(res, y, w, 1e-5), flush), floor(T * W * 8))
-        add(shape, "streams_step (4 fp32 streams, LayerNorm)", _time(lambda: ops.streams_step(x, y, mix, vec, vec, w, w, W, 1e-5), flush),
-            floor(T * W * (8 * S + 4)), "residual add + layernorm", _time(lambda: ops.layernorm(res, y, w, w, 1e-5), flush), floor(T * W * 8))
+        add(shape, "streams_step (4 fp32 streams, LayerNorm)", tab.time(lambda: ops.streams_step(x, y, mix, vec, vec, w, w, W, 1e-5)),
+            floor(T * W * (8 * S + 4)), "residual add + rmsnorm", tab.time(lambda: ops.rmsnorm(res, y, w, 1e-5)), floor(T * W * 8))
+        add(shape, "streams_step (4 fp32 streams, LayerNorm)", tab.time(lambda: ops.streams_step(x, y, mix, vec, vec, w, w, W, 1e-5)),
+            floor(T * W * (8 * S + 4)), "residual add + layernorm", tab.time(lambda: ops.layernorm(res, y, w, w, 1e-5)), floor(T * W * 8))
         o, gate = rnd(H, T, 128), rnd(T, H)
-        add(shape, "head_gate", _time(lambda: ops.head_gate(o, gate, H * 128), flush), floor(T * H * 512), "transposing copy",
-            _time(lambda: o.transpose(0, 1).reshape(T, H * 128), flush), floor(T * H * 512))
+        add(shape, "head_gate", tab.time(lambda: ops.head_gate(o, gate, H * 128)), floor(T * H * 512), "transposing copy",
+            tab.time(lambda: o.transpose(0, 1).reshape(T, H * 128)), floor(T * H * 512))
         D = 128
         b = _batch([1] * T if T == 64 else [T], [1024] * T if T == 64 else [T], device)
         qkv, gates = rnd(T, (2 * Hk + Hv) * D), rnd(T, 2 * Hv)
         st = torch.zeros(b.num_seqs, Hv, D, D, device=device)
         A, db = -torch.rand(Hv, device=device), torch.zeros(Hv, device=device)
         K = Hk * D
-        us = _time(lambda: ops.matrix_state_scan(2, qkv[:, :K], qkv[:, K:2 * K], qkv[:, 2 * K:], None, None, None, None, gates[:, :Hv], st, b.q_starts,
+        us = tab.time(lambda: ops.matrix_state_scan(2, qkv[:, :K], qkv[:, K:2 * K], qkv[:, 2 * K:], None, None, None, None, gates[:, :Hv], st, b.q_starts,
                                                  b.seq_state, b.positions, Hv, D, D, Hv // Hk, True, D ** -0.5, gate_raw=gates[:, Hv:], gate_A=A,
-                                                 gate_dt_bias=db), flush)
+                                                 gate_dt_bias=db))
         fl = floor(st.numel() * 8 + 2 * T * ((2 * Hk + 2 * Hv) * D))
         add(shape, "gated delta scan", us, fl, "the same kernel", us, fl)
-    return rows
+    return tab.rows
+
+
+def divanex_kernels(device, size: str = "1b") -> List[dict]:
+    tab = _Table(device)
+    ops, rnd, floor, bf = tab.ops, tab.rnd, tab.floor, torch.bfloat16
+    W, _, ff, Hm, H, G, side = DIVANEX_SIZES[size]
+    D = 128
+    for shape, lens, ctxs in (("decode 64 x 1152", [1] * 64, [1152] * 64), ("decode 8 x 4096", [1] * 8, [4096] * 8), ("prompt 2048", [2048], [2048]),
+                              ("prompt 8192", [8192], [8192]), ("prompt 4 x 512 at 2048", [512] * 4, [2048] * 4)):
+        b = _batch(lens, ctxs, device)
+        T = b.tokens
+        b.min_q_len, b.seq_lens = min(lens), torch.tensor(ctxs, dtype=torch.int32, device=device)
+        cache, factor = rnd(b.blocks, G, 16, D), torch.rand(b.blocks, G, 16, device=device) + 0.5
+        kc, vc = rnd(b.blocks, G, 16, D), rnd(b.blocks, G, 16, D)
+        q, qf = rnd(T, H * D), torch.full((T, H), D ** -0.5, device=device)
+        flops = 4.0 * sum(c * n - n * (n - 1) // 2 for n, c in zip(lens, ctxs)) * H * D
+        tied, split = floor(sum(ctxs) * G * (2 * D + 4) + 4 * T * H * D, flops), floor(sum(ctxs) * G * 4 * D + 4 * T * H * D, flops)
+        us = tab.time(lambda: ops.attention_tied(q, qf, cache, factor, D, b, 30.0))
+        for cap in (30.0, 0.0):
+            like = tab.time(lambda: ops.attention(q, kc, vc, b.block_tables, b.row_seq, b.positions, H, G, D, D ** -0.5, 0, None, cap, meta=b))
+            tab.add(shape, "attention_tied", us, tied, "attention" + (", capped" if cap else ""), like, split)
+        if len(lens) == 4:
+            continue
+        x, w, inv = rnd(T, (H + 2 * G) * D), torch.ones(D, device=device, dtype=bf), torch.zeros(D // 2, device=device)
+        tab.add(shape, "tied_prepare", tab.time(lambda: ops.tied_prepare(x, H * D, H, D, b.positions, b.slots, 1e-5, 0.1, 0.1, 8192.0, cache, factor)),
+                floor(2 * T * (H + 2 * G) * D), "rope_kv_write",
+                tab.time(lambda: ops.rope_kv_write(x, b.positions, b.slots, inv, w, w, kc, vc, H, G, D, D, 0, 1e-5)), floor(2 * T * (2 * H + 4 * G) * D))
+    for T in (64, 2048):
+        shape = f"{T} rows"
+        x, y, res, w = rnd(T, W, dtype=torch.float32), rnd(T, W), rnd(T, W), torch.ones(W, device=device, dtype=bf)
+        norm, norm_fl = tab.time(lambda: ops.rmsnorm(res, y, w, 1e-5)), floor(T * W * 8)
+        tab.add(shape, "postnorm, norm of the sum", tab.time(lambda: ops.postnorm_step(x, y, w, W, 1e-5, 2.0)), floor(T * W * 12), "residual add + rmsnorm", norm, norm_fl)
+        tab.add(shape, "postnorm, norm of what is added", tab.time(lambda: ops.postnorm_step(x, y, w, W, 1e-5, 1.0, True)), floor(T * W * 12),
+                "residual add + rmsnorm", norm, norm_fl)
+        gate, gu, table = rnd(T, side), rnd(T, 2 * side), rnd(4096, 4 * side)
+        ids = torch.randint(0, 4096, (T,), device=device, generator=tab.gen).int()
+        tab.add(shape, "side_gate", tab.time(lambda: ops.side_gate(gate, ids, table, side, side)), floor(6 * T * side), "geglu", tab.time(lambda: ops.glu(gu, 1)),
+                floor(6 * T * side))
+        b = _batch([1] * T if T == 64 else [T], [1024] * T if T == 64 else [T], device)
+        P, N, Gm = 64, 128, 8
+        xs, bc, dt = rnd(T, Hm * P), rnd(T, 2 * Gm * N), rnd(T, Hm)
+        st, A, Dv = torch.zeros(b.num_seqs, Hm, P, N, device=device), -torch.rand(Hm, device=device), torch.ones(Hm, device=device)
+        us = tab.time(lambda: ops.mamba2_scan(xs, dt, bc[:, :Gm * N], bc[:, Gm * N:], A, Dv, Dv, st, b.q_starts, b.seq_state, b.positions, Hm, P, Gm, N))
+        fl = floor(st.numel() * 8 + 2 * T * (2 * Hm * P + 2 * Gm * N))
+        tab.add(shape, "Mamba-2 scan", us, fl, "the same kernel", us, fl)
+    return tab.rows
+
+
+DESIGNS = {"sovanex": (sovanex_config, twin_config, sovanex_kernels), "divanex": (divanex_config, divanex_twin_config, divanex_kernels)}
 
 
 def main(args) -> dict:
@@ -191,11 +277,12 @@ def main(args) -> dict:
     torch.cuda.set_device(device)
     out = {"compare": args.compare, "data": "synthetic (uniform random token ids, random weights)", "prompt_len": args.prompt_len or 1024,
            "steps": args.steps, "warmup": args.warmup, "throughput": []}
-    for size in args.sizes.split(","):
-        for cfg in (sovanex_config(size), twin_config(size)):
+    design, twin, kernels = DESIGNS[args.compare]
+    for size in args.sizes.split(",") if args.sizes else ():
+        for cfg in (design(size), twin(size)):
             for batch in ([args.batch] if args.batch else [8, 64]):
                 r = throughput(cfg, batch, out["prompt_len"], args.steps, args.warmup, device)
                 out["throughput"].append({"model": cfg.name, "batch": batch, **r})
     if args.kernels:
-        out["kernels"] = kernel_table(device)
+        out["kernels"] = kernels(device)
     return out

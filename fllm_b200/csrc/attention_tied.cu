@@ -59,6 +59,10 @@ __device__ __forceinline__ float rcp(float x) {
 // the row goes to the cache with f = 1 / rms(k). rms(x) = sqrt(mean x^2 + eps); eps < 0: no norm (factor 1). temperature =
 // 1 + coef ln(floor((position + 1) / every) + 1). With split-K partial sums as the source, queries are also written to q_out.
 template <typename T>
+struct Four { using type = uint2; };
+template <>
+struct Four<float> { using type = float4; };
+template <typename T>
 __global__ void __launch_bounds__(128) tied_prepare_kernel(const TiedPrepareParams p) {
   pdl_launch_dependents();
   pdl_wait();
@@ -76,17 +80,38 @@ __global__ void __launch_bounds__(128) tied_prepare_kernel(const TiedPreparePara
   if (!is_q) dst = static_cast<T*>(p.cache) + (((long long)(slot / p.block_size) * p.G + (h - p.H)) * p.block_size + slot % p.block_size) * p.W;
   else if (part) dst = static_cast<T*>(p.q_out) + (long long)t * p.ld_qout + h * p.dim;
   float ss = 0.f;
-  for (int c = lane; c < p.dim; c += 32) {
-    T v;
-    if (part) {
-      float acc = 0.f;
-      for (int s = 0; s < p.splits; ++s) acc += __ldcg(part + s * p.plane + c);
-      v = from_f32<T>(acc);
-    } else {
-      v = src[c];
+  if (p.vec) {                                             // four values per lane
+    using V4 = typename Four<T>::type;
+    for (int c = 4 * lane; c < p.dim; c += 128) {
+      V4 raw;
+      T* v = reinterpret_cast<T*>(&raw);
+      if (part) {
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int s = 0; s < p.splits; ++s) {
+          const float4 q = __ldcg(reinterpret_cast<const float4*>(part + s * p.plane + c));
+          acc.x += q.x, acc.y += q.y, acc.z += q.z, acc.w += q.w;
+        }
+        v[0] = from_f32<T>(acc.x), v[1] = from_f32<T>(acc.y), v[2] = from_f32<T>(acc.z), v[3] = from_f32<T>(acc.w);
+      } else {
+        raw = *reinterpret_cast<const V4*>(src + c);
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) ss = fmaf(to_f32(v[e]), to_f32(v[e]), ss);
+      if (dst) *reinterpret_cast<V4*>(dst + c) = raw;
     }
-    ss = fmaf(to_f32(v), to_f32(v), ss);
-    if (dst) dst[c] = v;
+  } else {
+    for (int c = lane; c < p.dim; c += 32) {
+      T v;
+      if (part) {
+        float acc = 0.f;
+        for (int s = 0; s < p.splits; ++s) acc += __ldcg(part + s * p.plane + c);
+        v = from_f32<T>(acc);
+      } else {
+        v = src[c];
+      }
+      ss = fmaf(to_f32(v), to_f32(v), ss);
+      if (dst) dst[c] = v;
+    }
   }
   if (!is_q)
     for (int c = p.dim + lane; c < p.W; c += 32) dst[c] = from_f32<T>(0.f);
@@ -828,8 +853,12 @@ int attention_tied(const TiedAttnParams& p, int splits, void* workspace, size_t 
 #undef FLLM_TIED
 }
 
-void tied_prepare(const TiedPrepareParams& p, cudaStream_t s) {
-  if (p.tokens <= 0) return;
+void tied_prepare(const TiedPrepareParams& params, cudaStream_t s) {
+  if (params.tokens <= 0) return;
+  TiedPrepareParams p = params;
+  const uintptr_t any = reinterpret_cast<uintptr_t>(p.x) | reinterpret_cast<uintptr_t>(p.cache) | reinterpret_cast<uintptr_t>(p.q_out);
+  p.vec = p.dim % 4 == 0 && p.k_offset % 4 == 0 && p.W % 4 == 0 && any % 16 == 0 &&
+          (p.partials ? p.width % 4 == 0 && p.plane % 4 == 0 && p.ld_qout % 4 == 0 && reinterpret_cast<uintptr_t>(p.partials) % 16 == 0 : p.ldx % 4 == 0);
   const unsigned blocks = (unsigned)(((long long)p.tokens * (p.H + p.G) + 3) / 4);
   if (p.f32) launch_pdl(tied_prepare_kernel<float>, dim3(blocks), dim3(128), 0, s, p);
   else launch_pdl(tied_prepare_kernel<bf16>, dim3(blocks), dim3(128), 0, s, p);

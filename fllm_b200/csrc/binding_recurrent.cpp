@@ -43,7 +43,7 @@ void causal_conv1d(const Tensor& x, const Tensor& w, const optional<Tensor>& bia
   c10::cuda::CUDAGuard guard(x.device());
   const int rc = fllm::causal_conv1d(x.data_ptr(), x.stride(0), w.data_ptr<float>(), opt_f32(bias), state.data_ptr(), q_starts.data_ptr<int>(),
                                      seq_state.data_ptr<int>(), positions.data_ptr<int>(), y.data_ptr(), y.stride(0), (int)seq_state.numel(),
-                                     (int)C, (int)W, act ? 1 : 0, (int)(max_q_len > 0 ? max_q_len : x.size(0)), cur_stream(),
+                                     (int)C, (int)W, act ? 1 : 0, (int)x.size(0), (int)(max_q_len > 0 ? max_q_len : x.size(0)), cur_stream(),
                                      ty == at::kFloat ? 1 : 0);
   TORCH_CHECK(rc == 0, "causal_conv1d: unsupported arguments (code ", rc, "): even C and strides, 2 <= W <= 8, y distinct from x");
 }

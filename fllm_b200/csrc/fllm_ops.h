@@ -277,7 +277,8 @@ void spec_verify_sampled(const void* target_logits, long long ld_t, const void* 
 // before anything was launched.
 int causal_conv1d(const void* x, long long ldx, const float* w, const float* bias, void* state, const int* q_starts,
                   const int* seq_state, const int* positions, void* y, long long ldy, int B, int C, int W, int act,
-                  int max_q_len, cudaStream_t stream, int f32 = 0);   // max_q_len: host-side bound on a sequence's tokens in the step
+                  int tokens, int max_q_len, cudaStream_t stream, int f32 = 0);   // tokens: rows of the step (= B: single tokens);
+                                                                                  // max_q_len: host-side bound on a sequence's tokens in it
 // The Mamba-2 recurrence for any head and state width (N <= 256), bf16 or fp32 (recurrent_ssd.cu): one walk per sequence.
 struct SsdScanParams {
   const void *x, *dt, *Bm, *Cm;
@@ -421,6 +422,7 @@ struct TiedPrepareParams {
   void* cache;                 // [blocks][G][block_size][W]
   float* key_factor;           // [blocks][G][block_size]
   int f32;
+  int vec;                     // set by tied_prepare: rows move four values at a time
 };
 void tied_prepare(const TiedPrepareParams& p, cudaStream_t s);
 struct TiedAttnParams {

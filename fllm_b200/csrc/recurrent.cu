@@ -14,7 +14,9 @@
 #include <cuda_runtime.h>
 
 #include "fllm_ops.h"
+#include "ptx.cuh"
 #include "recurrent_util.cuh"
+#include "tma_host.h"
 
 namespace fllm {
 namespace {
@@ -29,6 +31,7 @@ __global__ void __launch_bounds__(256) conv1d_kernel(const T* __restrict__ x, lo
                                                      const int* __restrict__ q_starts, const int* __restrict__ seq_state,
                                                      const int* __restrict__ positions, T* __restrict__ y, long long ldy,
                                                      int C, int act, int seg_tokens) {
+  pdl_wait();
   const int s = blockIdx.y;
   const int c = (blockIdx.x * 64 + threadIdx.x) * 2;
   const int t0 = q_starts[s], n = q_starts[s + 1] - t0;
@@ -87,6 +90,43 @@ __global__ void __launch_bounds__(256) conv1d_kernel(const T* __restrict__ x, lo
       st2(st + (long long)j * C + c, v.x, v.y);
     }
   }
+}
+
+// Steps of single tokens (decode): one thread per two channels and sequence, every load in flight at once.
+template <typename T, int W>
+__global__ void __launch_bounds__(128) conv1d_decode_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ w,
+                                                            const float* __restrict__ bias, T* __restrict__ state,
+                                                            const int* __restrict__ q_starts, const int* __restrict__ seq_state,
+                                                            const int* __restrict__ positions, T* __restrict__ y, long long ldy, int C, int act) {
+  pdl_launch_dependents();
+  const int s = blockIdx.y, c = (blockIdx.x * 128 + threadIdx.x) * 2;
+  float wv[2][W], bv[2] = {0.f, 0.f};
+  if (c < C) {                                               // weights do not wait for the kernel before
+#pragma unroll
+    for (int j = 0; j < W; ++j) wv[0][j] = w[(long long)c * W + j], wv[1][j] = w[(long long)(c + 1) * W + j];
+    if (bias != nullptr) bv[0] = bias[c], bv[1] = bias[c + 1];
+  }
+  pdl_wait();
+  const int t0 = q_starts[s], n = q_starts[s + 1] - t0;
+  if (n <= 0 || c >= C) return;
+  const bool fresh = positions[t0] == 0;
+  T* st = state + (long long)seq_state[s] * (W - 1) * C + c;
+  float2 win[W - 1];
+#pragma unroll
+  for (int j = 0; j < W - 1; ++j) win[j] = fresh ? make_float2(0.f, 0.f) : ld2(st + (long long)j * C);
+  for (int p = 0; p < n; ++p) {
+    const float2 v = ld2(x + (long long)(t0 + p) * ldx + c);
+    float o0 = fmaf(wv[0][W - 1], v.x, bv[0]), o1 = fmaf(wv[1][W - 1], v.y, bv[1]);
+#pragma unroll
+    for (int j = 0; j < W - 1; ++j) o0 = fmaf(wv[0][j], win[j].x, o0), o1 = fmaf(wv[1][j], win[j].y, o1);
+#pragma unroll
+    for (int j = 0; j + 1 < W - 1; ++j) win[j] = win[j + 1];
+    win[W - 2] = v;
+    if (act) o0 = silu_t<T>(o0), o1 = silu_t<T>(o1);
+    st2(y + (long long)(t0 + p) * ldy + c, o0, o1);
+  }
+#pragma unroll
+  for (int j = 0; j < W - 1; ++j) st2(st + (long long)j * C, win[j].x, win[j].y);
 }
 
 // ------------------------------------------------------------------------------------------ Mamba-1
@@ -550,6 +590,8 @@ template <typename T>
 __global__ void __launch_bounds__(128) gated_rmsnorm_kernel(const T* x, long long ldx, const T* __restrict__ z, long long ldz,
                                                             const T* __restrict__ w, int wlen, T* y, long long ldy, int n_rows, int D,
                                                             int gs, float eps, int mode) {
+  pdl_launch_dependents();
+  pdl_wait();
   const int groups = D / gs;
   const long long item = (long long)blockIdx.x * 4 + threadIdx.x / 32;
   if (item >= (long long)n_rows * groups) return;
@@ -575,12 +617,14 @@ __global__ void __launch_bounds__(128) gated_rmsnorm_kernel(const T* x, long lon
   }
 }
 
-// The same for wide groups (Mamba-2 normalises the whole inner width at once): one CTA of 256 threads per (token, group),
-// two channels per thread and step, the (gated) row kept in registers between the two passes when it fits (up to 8192 channels).
-__global__ void __launch_bounds__(256) gated_rmsnorm_wide_kernel(const bf16* x, long long ldx, const bf16* __restrict__ z, long long ldz,
-                                                                 const bf16* __restrict__ w, int wlen, bf16* y, long long ldy, int D, int gs,
-                                                                 float eps, int mode) {
-  constexpr int KEEP = 16;                                 // pairs kept per thread: 256 * 16 * 2 = 8192 channels
+// The same for wide groups (Mamba-2 normalises up to the whole inner width at once): one CTA per (token, group), two channels
+// per thread and step, the (gated) row kept in registers between the two passes when it fits (2 * THREADS * KEEP channels).
+template <int THREADS, int KEEP>
+__global__ void __launch_bounds__(THREADS) gated_rmsnorm_wide_kernel(const bf16* x, long long ldx, const bf16* __restrict__ z, long long ldz,
+                                                                     const bf16* __restrict__ w, int wlen, bf16* y, long long ldy, int D, int gs,
+                                                                     float eps, int mode) {
+  pdl_launch_dependents();
+  pdl_wait();
   const int groups = D / gs;
   const int t = blockIdx.x / groups, g = blockIdx.x % groups;
   const __nv_bfloat162* xr = reinterpret_cast<const __nv_bfloat162*>(x + t * ldx + (long long)g * gs);
@@ -590,7 +634,7 @@ __global__ void __launch_bounds__(256) gated_rmsnorm_wide_kernel(const bf16* x, 
   float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
-    const int p = threadIdx.x + i * 256;
+    const int p = threadIdx.x + i * THREADS;
     keep[i] = make_float2(0.f, 0.f);
     if (p < pairs) {
       keep[i] = __bfloat1622float2(xr[p]);
@@ -601,7 +645,7 @@ __global__ void __launch_bounds__(256) gated_rmsnorm_wide_kernel(const bf16* x, 
       ss = fmaf(keep[i].x, keep[i].x, fmaf(keep[i].y, keep[i].y, ss));
     }
   }
-  for (int p = threadIdx.x + KEEP * 256; p < pairs; p += 256) {     // beyond the kept part: read again in the second pass
+  for (int p = threadIdx.x + KEEP * THREADS; p < pairs; p += THREADS) {     // beyond the kept part: read again in the second pass
     float2 v = __bfloat1622float2(xr[p]);
     if (mode == 0 && zr != nullptr) {
       const float2 zz = __bfloat1622float2(zr[p]);
@@ -609,13 +653,13 @@ __global__ void __launch_bounds__(256) gated_rmsnorm_wide_kernel(const bf16* x, 
     }
     ss = fmaf(v.x, v.x, fmaf(v.y, v.y, ss));
   }
-  __shared__ float part[8];
+  __shared__ float part[THREADS / 32];
   ss = row_sum<32>(ss);
   if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = ss;
   __syncthreads();
   float tot = 0.f;
 #pragma unroll
-  for (int i = 0; i < 8; ++i) tot += part[i];
+  for (int i = 0; i < THREADS / 32; ++i) tot += part[i];
   const float inv = rsqrtf(tot / gs + eps);
   __nv_bfloat162* yr = reinterpret_cast<__nv_bfloat162*>(y + t * ldy + (long long)g * gs);
   auto weight = [&](int p) {
@@ -624,7 +668,7 @@ __global__ void __launch_bounds__(256) gated_rmsnorm_wide_kernel(const bf16* x, 
   };
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
-    const int p = threadIdx.x + i * 256;
+    const int p = threadIdx.x + i * THREADS;
     if (p < pairs) {
       const float2 ww = weight(p);
       float2 v = make_float2(keep[i].x * inv * ww.x, keep[i].y * inv * ww.y);
@@ -635,7 +679,7 @@ __global__ void __launch_bounds__(256) gated_rmsnorm_wide_kernel(const bf16* x, 
       yr[p] = __floats2bfloat162_rn(v.x, v.y);
     }
   }
-  for (int p = threadIdx.x + KEEP * 256; p < pairs; p += 256) {
+  for (int p = threadIdx.x + KEEP * THREADS; p < pairs; p += THREADS) {
     float2 v = __bfloat1622float2(xr[p]);
     float2 gt = make_float2(1.f, 1.f);
     if (zr != nullptr) {
@@ -656,7 +700,7 @@ __global__ void __launch_bounds__(256) gated_rmsnorm_wide_kernel(const bf16* x, 
 // Every launcher returns 0 on success or a negative code naming the argument it rejected, before any launch.
 int causal_conv1d(const void* x, long long ldx, const float* w, const float* bias, void* state, const int* q_starts,
                   const int* seq_state, const int* positions, void* y, long long ldy, int B, int C, int W, int act,
-                  int max_q_len, cudaStream_t stream, int f32) {
+                  int tokens, int max_q_len, cudaStream_t stream, int f32) {
   if (B <= 0) return 0;
   if (C % 2 || (ldx % 2) || (ldy % 2) || x == y) return -1;
   if (W < 2 || W > 8) return -2;
@@ -668,8 +712,14 @@ int causal_conv1d(const void* x, long long ldx, const float* w, const float* bia
     auto xs = static_cast<const T*>(x);
     auto ys = static_cast<T*>(y);
     auto ss = static_cast<T*>(state);
-#define FLLM_CONV(W_) \
-  case W_: conv1d_kernel<T, W_><<<grid, block, 0, stream>>>(xs, ldx, w, bias, ss, q_starts, seq_state, positions, ys, ldy, C, act, seg_tokens); break;
+#define FLLM_CONV(W_)                                                                                                                               \
+  case W_:                                                                                                                                          \
+    if (tokens == B)                                                                                                                                \
+      launch_pdl(conv1d_decode_kernel<T, W_>, dim3((C / 2 + 127) / 128, B), dim3(128), 0, stream, xs, ldx, w, bias, ss, q_starts, seq_state, positions, ys, \
+                 ldy, C, act);                                                                                                                      \
+    else                                                                                                                                            \
+      launch_pdl(conv1d_kernel<T, W_>, grid, block, 0, stream, xs, ldx, w, bias, ss, q_starts, seq_state, positions, ys, ldy, C, act, (int)seg_tokens);   \
+    break;
     switch (W) { FLLM_CONV(2) FLLM_CONV(3) FLLM_CONV(4) FLLM_CONV(5) FLLM_CONV(6) FLLM_CONV(7) FLLM_CONV(8) }
 #undef FLLM_CONV
   };
@@ -796,15 +846,15 @@ void gated_rmsnorm(const void* x, long long ldx, const void* z, long long ldz, c
   const bool pairs_ok = group_size % 2 == 0 && ldx % 2 == 0 && ldy % 2 == 0 && (z == nullptr || ldz % 2 == 0) &&
                         (reinterpret_cast<uintptr_t>(x) & 3) == 0 && (reinterpret_cast<uintptr_t>(y) & 3) == 0 &&
                         (reinterpret_cast<uintptr_t>(z) & 3) == 0;
-  if (group_size >= 1024 && pairs_ok) {
-    gated_rmsnorm_wide_kernel<<<(unsigned)items, 256, 0, stream>>>(static_cast<const bf16*>(x), ldx, static_cast<const bf16*>(z), ldz,
-                                                                   static_cast<const bf16*>(w), wlen, static_cast<bf16*>(y), ldy, D,
-                                                                   group_size, eps, norm_before_gate);
-    return;
-  }
-  gated_rmsnorm_kernel<bf16><<<(unsigned)((items + 3) / 4), 128, 0, stream>>>(static_cast<const bf16*>(x), ldx, static_cast<const bf16*>(z), ldz,
-                                                                       static_cast<const bf16*>(w), wlen, static_cast<bf16*>(y), ldy, T, D,
-                                                                       group_size, eps, norm_before_gate);
+  auto go = [&](auto kernel, unsigned grid, unsigned threads) {
+    launch_pdl(kernel, dim3(grid), dim3(threads), 0, stream, static_cast<const bf16*>(x), ldx, static_cast<const bf16*>(z), ldz, static_cast<const bf16*>(w), wlen,
+               static_cast<bf16*>(y), ldy, D, group_size, eps, norm_before_gate);
+  };
+  if (group_size > 1024 && pairs_ok) go(gated_rmsnorm_wide_kernel<256, 16>, (unsigned)items, 256);
+  else if (group_size > 256 && pairs_ok) go(gated_rmsnorm_wide_kernel<128, 4>, (unsigned)items, 128);
+  else
+    launch_pdl(gated_rmsnorm_kernel<bf16>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, static_cast<const bf16*>(x), ldx, static_cast<const bf16*>(z), ldz,
+               static_cast<const bf16*>(w), wlen, static_cast<bf16*>(y), ldy, T, D, group_size, eps, norm_before_gate);
 }
 
 }  // namespace fllm

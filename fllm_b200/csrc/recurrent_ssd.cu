@@ -15,7 +15,9 @@
 // NP: state columns in registers; EXACT: the state width is NP and rows are 16-byte aligned, otherwise it is N <= NP and rows
 // are read value by value.
 #include "fllm_ops.h"
+#include "ptx.cuh"
 #include "recurrent_util.cuh"
+#include "tma_host.h"
 
 namespace fllm {
 namespace {
@@ -87,6 +89,7 @@ struct SsdTile {
 
 template <typename T, int NP, bool EXACT>
 __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
+  pdl_wait();
   using L = SsdTile<NP>;
   constexpr int NPT = L::NPT, TPK = L::TPK, RPT = L::RPT, ROWS = L::ROWS, GROUP = L::GROUP, C = kSsdChunk, EPT = NP / 8, VPT = ROWS * C / 128;
   __shared__ __align__(16) float sb[C][NP], sc[C][NP], sx[C][ROWS];
@@ -242,6 +245,8 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
 
 template <typename T, int NP, bool EXACT>
 __global__ void __launch_bounds__(128) ssd_decode_kernel(const SsdArgs<T> a) {
+  pdl_launch_dependents();
+  pdl_wait();
   constexpr int NPT = 16, TPK = NP / NPT, ROWS = 128 / TPK;
   const int N = EXACT ? NP : a.N;
   const int ptiles = (a.P + ROWS - 1) / ROWS;
@@ -306,9 +311,9 @@ int ssd_scan(const SsdScanParams& p, cudaStream_t stream) {
   {                                                                                                                   \
     constexpr int drows = 128 / (NP_ / 16), rows = SsdTile<NP_>::ROWS;                                                \
     if (p.tokens == p.B)                                                                                              \
-      ssd_decode_kernel<T_, NP_, EXACT_><<<dim3(p.H * ((p.P + drows - 1) / drows), p.B), 128, 0, stream>>>(args(T_{}));     \
+      launch_pdl(ssd_decode_kernel<T_, NP_, EXACT_>, dim3(p.H * ((p.P + drows - 1) / drows), p.B), dim3(128), 0, stream, args(T_{}));     \
     else                                                                                                              \
-      ssd_scan_kernel<T_, NP_, EXACT_><<<dim3(p.H * ((p.P + rows - 1) / rows), p.B), 128, 0, stream>>>(args(T_{}));   \
+      launch_pdl(ssd_scan_kernel<T_, NP_, EXACT_>, dim3(p.H * ((p.P + rows - 1) / rows), p.B), dim3(128), 0, stream, args(T_{}));   \
     return 0;                                                                                                         \
   }
 #define FLLM_SSD_N(T_, EXACT_)                    \
