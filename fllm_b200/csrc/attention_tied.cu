@@ -266,7 +266,7 @@ __device__ __forceinline__ bf16* tile_ptr(bf16* base, int row, int chunk) {
 
 template <int D>
 struct DecodeTile {
-  static constexpr int kStages = 5;
+  static constexpr int kStages = 4;
   static constexpr int kRowBytes = kPage * D * 2, kStage = kRowBytes + kPage * 4;      // key rows, then their factors
   static constexpr int kQ = 16 * D * 2, kRing = 4 * kStages * kStage;
   static constexpr int kMerge = 4 * 16 * D * 4 + 4 * 16 * 2 * 4;
@@ -275,7 +275,7 @@ struct DecodeTile {
 
 // FIXED: the cap bounds the scores, reference 0; otherwise a running maximum
 template <int D, bool CAP, bool FIXED>
-__global__ void __launch_bounds__(128) tied_decode_kernel(const Tied p, int row_tiles, int max_rows) {
+__global__ void __launch_bounds__(128, 3) tied_decode_kernel(const Tied p, int row_tiles, int max_rows) {
   using L = DecodeTile<D>;
   extern __shared__ __align__(128) uint8_t smem[];
   bf16* qtile = reinterpret_cast<bf16*>(smem);

@@ -6,14 +6,19 @@
 // holding the columns 4 (l + TPK j) + 0..3 of each as pairs for the packed fp32 instructions. Tokens come in chunks: eight
 // threads per token fetch B and C one chunk ahead in their stored form and leave them in shared memory as fp32 with the
 // token's decay and step size, so the walk over a chunk touches shared memory and registers only. Four rows per thread keep the
-// shared-memory reads below the arithmetic; the outputs of four tokens are summed over the lanes together, each exchange
-// halving the values a lane carries, so a lane ends with a sixteenth of the sums and none is computed twice.
+// shared-memory reads below the arithmetic (two where four would leave half the SMs idle). The outputs of four tokens are
+// summed over the lanes together, each exchange halving the values a lane carries, so that no sum is computed twice. Inside
+// such a group the state is kept over the product of the decays so far (S = P_t S', S' += (dt / P_t) x B, y = P_t S' C): one
+// multiplication by the group's whole decay replaces four. Groups that decay too far for that (P below kMinDecay) multiply
+// token by token.
 //
 // ssd_decode_kernel serves steps of single tokens: inputs straight from global memory, no shared memory, many CTAs that keep
 // state reads in flight (a decoded token reads and writes the whole state once).
 //
 // NP: state columns in registers; EXACT: the state width is NP and rows are 16-byte aligned, otherwise it is N <= NP and rows
 // are read value by value.
+#include <type_traits>
+
 #include "fllm_ops.h"
 #include "ptx.cuh"
 #include "recurrent_util.cuh"
@@ -23,6 +28,7 @@ namespace fllm {
 namespace {
 
 constexpr int kSsdChunk = 16;
+constexpr float kMinDecay = 2e-9f;           // e^-20: the rounding of the exponents stays at 2e-6
 
 // pairs of fp32 values in one 64-bit register
 __device__ __forceinline__ uint64_t pair(float a, float b) {
@@ -82,18 +88,18 @@ __device__ __forceinline__ void lane_sums(float (&v)[SIZE], int lane) {
   }
 }
 
-template <int NP>
+template <int NP, int RPT>
 struct SsdTile {
-  static constexpr int NPT = NP <= 32 ? 4 : 8, TPK = NP / NPT, RG = 128 / TPK, RPT = 4, ROWS = RPT * RG, GROUP = 4;
+  static constexpr int NPT = NP <= 32 ? 4 : 8, TPK = NP / NPT, RG = 128 / TPK, ROWS = RPT * RG, GROUP = 4;
 };
 
-template <typename T, int NP, bool EXACT>
+template <typename T, int NP, bool EXACT, int RPT>
 __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
   pdl_wait();
-  using L = SsdTile<NP>;
-  constexpr int NPT = L::NPT, TPK = L::TPK, RPT = L::RPT, ROWS = L::ROWS, GROUP = L::GROUP, C = kSsdChunk, EPT = NP / 8, VPT = ROWS * C / 128;
+  using L = SsdTile<NP, RPT>;
+  constexpr int NPT = L::NPT, TPK = L::TPK, ROWS = L::ROWS, GROUP = L::GROUP, C = kSsdChunk, EPT = NP / 8, VPT = ROWS * C / 128;
   __shared__ __align__(16) float sb[C][NP], sc[C][NP], sx[C][ROWS];
-  __shared__ float2 sg[C];                               // decay, step size
+  __shared__ float4 sg[C];                               // P, dt / P, decay, dt
   const int N = EXACT ? NP : a.N;
   const int ptiles = (a.P + ROWS - 1) / ROWS;
   const int h = blockIdx.x / ptiles, p0 = (blockIdx.x % ptiles) * ROWS, row = threadIdx.x / TPK * RPT;      // rows p0 + row + r
@@ -143,7 +149,7 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
           cl[i] = c < N ? ld1(cp + c) : 0.f;
         }
       }
-      if (part == 0) dr = a.dt[t * a.lddt + h];
+      dr = a.dt[t * a.lddt + h];
     }
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
@@ -177,10 +183,15 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
 #pragma unroll
         for (int i = 0; i < EPT; ++i) sb[tt][column(i)] = br[i], sc[tt][column(i)] = cr[i];
       }
-      if (part == 0) {
-        const float dt = live ? fminf(fmaxf(softplus_t<T>(ld1(&dr) + dtb), a.dt_min), a.dt_max) : 0.f;
-        sg[tt] = make_float2(exp_t<T>(dt * A), dt);
-      }
+      // a warp holds the four tokens of a group: running sum of the exponents over them
+      static_assert(GROUP == 4, "eight threads per token");
+      const float dt = live ? fminf(fmaxf(softplus_t<T>(ld1(&dr) + dtb), a.dt_min), a.dt_max) : 0.f, e = dt * A;
+      float c = e;
+      const float c1 = __shfl_up_sync(0xffffffffu, c, 8);
+      if (tt % 4 >= 1) c += c1;
+      const float c2 = __shfl_up_sync(0xffffffffu, c, 16);
+      if (tt % 4 >= 2) c += c2;
+      if (part == 0) sg[tt] = make_float4(exp_t<T>(c), dt * exp_t<T>(-c), exp_t<T>(e), dt);
     }
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
@@ -191,33 +202,53 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
     if (base + C < n) fetch(base + C);
     for (int i0 = 0; i0 < cnt; i0 += GROUP) {
       float o[GROUP * RPT];
+      auto walk = [&](auto scaled) {
+        constexpr bool SCALED = decltype(scaled)::value;
 #pragma unroll
-      for (int k = 0; k < GROUP; ++k) {
-        const int i = i0 + k;
-        uint64_t b2[NPT / 2], c2[NPT / 2];
+        for (int k = 0; k < GROUP; ++k) {
+          const int i = i0 + k;
+          uint64_t b2[NPT / 2], c2[NPT / 2];
 #pragma unroll
-        for (int j = 0; j < NPT / 4; ++j) {
-          const ulonglong2 bv = *reinterpret_cast<const ulonglong2*>(&sb[i][4 * (lk + TPK * j)]);
-          const ulonglong2 cv = *reinterpret_cast<const ulonglong2*>(&sc[i][4 * (lk + TPK * j)]);
-          b2[2 * j] = bv.x, b2[2 * j + 1] = bv.y, c2[2 * j] = cv.x, c2[2 * j + 1] = cv.y;
-        }
-        const float2 g = sg[i];
-        const uint64_t d2 = pair(g.x, g.x);
-        const float4 x4 = *reinterpret_cast<const float4*>(&sx[i][row]);
-        const float xs[RPT] = {x4.x, x4.y, x4.z, x4.w};
-#pragma unroll
-        for (int r = 0; r < RPT; ++r) {
-          const float u = g.y * xs[r];
-          const uint64_t u2 = pair(u, u);
-          uint64_t o2 = 0;
-#pragma unroll
-          for (int j = 0; j < NPT / 2; ++j) {
-            S[r][j] = fma2(b2[j], u2, mul2(S[r][j], d2));
-            o2 = fma2(S[r][j], c2[j], o2);
+          for (int j = 0; j < NPT / 4; ++j) {
+            const ulonglong2 bv = *reinterpret_cast<const ulonglong2*>(&sb[i][4 * (lk + TPK * j)]);
+            const ulonglong2 cv = *reinterpret_cast<const ulonglong2*>(&sc[i][4 * (lk + TPK * j)]);
+            b2[2 * j] = bv.x, b2[2 * j + 1] = bv.y, c2[2 * j] = cv.x, c2[2 * j + 1] = cv.y;
           }
-          const float2 e = unpair(o2);
-          o[k * RPT + r] = e.x + e.y;
+          const float4 g = sg[i];
+          float xs[RPT];
+          if constexpr (RPT == 4) {
+            const float4 v = *reinterpret_cast<const float4*>(&sx[i][row]);
+            xs[0] = v.x, xs[1] = v.y, xs[2] = v.z, xs[3] = v.w;
+          } else {
+            const float2 v = *reinterpret_cast<const float2*>(&sx[i][row]);
+            xs[0] = v.x, xs[1] = v.y;
+          }
+          const uint64_t d2 = pair(g.z, g.z);
+#pragma unroll
+          for (int r = 0; r < RPT; ++r) {
+            const float u = (SCALED ? g.y : g.w) * xs[r];
+            const uint64_t u2 = pair(u, u);
+            uint64_t o2 = 0;
+#pragma unroll
+            for (int j = 0; j < NPT / 2; ++j) {
+              S[r][j] = fma2(b2[j], u2, SCALED ? S[r][j] : mul2(S[r][j], d2));
+              o2 = fma2(S[r][j], c2[j], o2);
+            }
+            const float2 e = unpair(o2);
+            o[k * RPT + r] = SCALED ? g.x * (e.x + e.y) : e.x + e.y;
+          }
         }
+      };
+      const float whole = sg[i0 + GROUP - 1].x;
+      if (whole > kMinDecay) {
+        walk(std::true_type{});
+        const uint64_t w2 = pair(whole, whole);
+#pragma unroll
+        for (int r = 0; r < RPT; ++r)
+#pragma unroll
+          for (int j = 0; j < NPT / 2; ++j) S[r][j] = mul2(S[r][j], w2);
+      } else {
+        walk(std::false_type{});
       }
       using Sums = LaneSums<TPK, GROUP * RPT>;
       lane_sums<TPK, GROUP * RPT>(o, lk);
@@ -307,13 +338,17 @@ int ssd_scan(const SsdScanParams& p, cudaStream_t stream) {
                       p.ldx, p.lddt, p.ldb, p.ldc, p.ldy, p.A, p.D, p.dt_bias, p.state, p.q_starts, p.seq_state, p.positions,
                       static_cast<T*>(p.y), p.H, p.P, p.G, p.N, p.dt_min, p.dt_max, p.skip_from};
   };
+  // few sequences and heads: two rows per thread instead of four, so that twice as many SMs work
 #define FLLM_SSD(T_, NP_, EXACT_)                                                                                     \
   {                                                                                                                   \
-    constexpr int drows = 128 / (NP_ / 16), rows = SsdTile<NP_>::ROWS;                                                \
+    constexpr int drows = 128 / (NP_ / 16), rows4 = SsdTile<NP_, 4>::ROWS, rows2 = SsdTile<NP_, 2>::ROWS;             \
+    const int tiles4 = p.H * ((p.P + rows4 - 1) / rows4), tiles2 = p.H * ((p.P + rows2 - 1) / rows2);                 \
     if (p.tokens == p.B)                                                                                              \
-      launch_pdl(ssd_decode_kernel<T_, NP_, EXACT_>, dim3(p.H * ((p.P + drows - 1) / drows), p.B), dim3(128), 0, stream, args(T_{}));     \
+      launch_pdl(ssd_decode_kernel<T_, NP_, EXACT_>, dim3(p.H * ((p.P + drows - 1) / drows), p.B), dim3(128), 0, stream, args(T_{}));  \
+    else if (2LL * tiles4 * p.B <= sm_count() && tiles2 > tiles4)                                                     \
+      launch_pdl(ssd_scan_kernel<T_, NP_, EXACT_, 2>, dim3(tiles2, p.B), dim3(128), 0, stream, args(T_{}));           \
     else                                                                                                              \
-      launch_pdl(ssd_scan_kernel<T_, NP_, EXACT_>, dim3(p.H * ((p.P + rows - 1) / rows), p.B), dim3(128), 0, stream, args(T_{}));   \
+      launch_pdl(ssd_scan_kernel<T_, NP_, EXACT_, 4>, dim3(tiles4, p.B), dim3(128), 0, stream, args(T_{}));           \
     return 0;                                                                                                         \
   }
 #define FLLM_SSD_N(T_, EXACT_)                    \

@@ -238,6 +238,7 @@ def test_ssd_scan(ops, H, P, N, G, dtype):
     oB, oC, oD = p8(H * P), p8(H * P) + p8(G * N), p8(H * P) + 2 * p8(G * N)
     rows = [torch.randn(n, p8(oD + H), device=DEV, generator=g).to(dtype) for n in lens]
     A = -torch.exp(torch.randn(H, device=DEV, generator=g))
+    A[-1] *= 30                                                        # a head that forgets within a token or two
     D, bias = torch.randn(H, device=DEV, generator=g), torch.randn(H, device=DEV, generator=g) - 2
     state = torch.full((6, H, P, N), 9.0, device=DEV)                  # stale rows of earlier requests
     got, at = [[] for _ in lens], [0, 0, 0]
