@@ -141,7 +141,7 @@ def dense(q, qf, cache, kf, tab, starts, lens, ctxs, H, G, dim, cap, bs=16):
     return out
 
 
-SHAPES = [(8, 2, 64), (12, 1, 128), (3, 3, 24), (40, 2, 128), (5, 1, 80), (6, 2, 20), (4, 4, 136), (1, 1, 8)]
+SHAPES = [(8, 2, 64), (80, 1, 64), (12, 1, 128), (3, 3, 24), (40, 2, 128), (5, 1, 80), (6, 2, 20), (4, 4, 136), (1, 1, 8)]
 BATCHES = [([1, 1, 1], [1, 40, 129]), ([5, 1, 23], [5, 17, 60]), ([70], [133]), ([1], [700]), ([150, 1, 130], [150, 300, 400])]
 
 
