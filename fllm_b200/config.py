@@ -30,7 +30,23 @@ class RopeScaling:
     freq_factors: Optional[List[float]] = None
 
 
-STATELESS_KINDS = ("attention", "mla", "tied", "none")       # layer kinds without a recurrent state
+STATELESS_KINDS = ("attention", "mla", "tied", "maps", "none")       # layer kinds without a recurrent state
+ROW_CACHE_KINDS = ("mla", "tied", "maps", "maps+lightning")          # layer kinds whose cache rows have a layout of their own
+
+
+@dataclass(frozen=True)
+class MoeSpec:
+    """Routed experts of one layer. ``weigh_input``: an expert's routing weight multiplies its input instead of its output."""
+    experts: int
+    top: int
+    router: str = "softmax_topk"         # softmax_topk | softmax_all | deepseek_v2 (softmax scores) | deepseek_v3 (sigmoid scores)
+    norm_topk: bool = False
+    scale: float = 1.0
+    groups: int = 1
+    topk_groups: int = 1
+    act: str = "swiglu"
+    weigh_input: bool = False
+    fp32_router: bool = False            # the router's logits stay fp32 (otherwise they take the activation type)
 
 
 @dataclass
@@ -101,8 +117,9 @@ class ModelConfig:
     # layer has a gated FFN behind it ("glu") or is the mixer alone ("none"); `ssm` holds the mixer shapes
     # (d_inner, d_state, d_conv, n_groups, head_dim, n_heads, dt_rank, norm_groups, dt_min, dt_max, conv_bias,
     # num_k_heads, num_v_heads, head_k_dim, head_v_dim, bcdt_rms ...)
-    layer_kinds: Optional[List[str]] = None      # attention | mla | tied | mamba1 | mamba2 | gated_delta | shortconv | none (FFN-only block)
+    layer_kinds: Optional[List[str]] = None      # attention | mla | tied | maps | mamba1 | mamba2 | gated_delta | shortconv | none (FFN-only block)
                                                  # | attention+mamba2 (both read the block's input, their outputs add: Falcon-H1)
+                                                 # | maps+lightning (the same, each output normalised, their mean: models.maps)
     ffn_kinds: Optional[List[str]] = None        # glu | moe | none
     ssm: Dict[str, Any] = field(default_factory=dict)
     # multi-head latent attention (layer kind "mla"): q_lora_rank (0 = one query projection), kv_lora_rank,
@@ -110,12 +127,17 @@ class ModelConfig:
     mla: Dict[str, Any] = field(default_factory=dict)
     # per layer: shapes that differ from layer to layer, laid over `ssm` (recurrent kinds) or `mla` (kind "mla"; there also
     # num_heads, scale, rope_theta, rope_style, head_gate, and kv_from = the layer whose cached rows this one attends to); for
-    # kind "tied" all of num_heads, num_kv_heads, head_dim, scale, softcap, temp_coef, temp_every, norm_eps
+    # kind "tied" all of num_heads, num_kv_heads, head_dim, scale, softcap, temp_coef, temp_every, norm_eps; for kind "maps"
+    # num_heads, num_kv_heads, head_dim, v_dim, maps, window, scale, rope (dims, theta, scaling), qk_norm ("head" | "full"), and
+    # with two maps diff; for "maps+lightning" those and lin_heads, lin_k_dim, lin_v_dim, lin_decay
     layer_mixers: Optional[List[Dict[str, Any]]] = None
-    # per layer: width and activation limit of a feed-forward network that differs from layer to layer (ff, limit)
+    # per layer: width and activation limit of a feed-forward network that differs from layer to layer (ff, limit), or its
+    # routed experts (experts, top, ff, shared_ff, router ...: the fields of MoeSpec)
     layer_ffns: Optional[List[Dict[str, Any]]] = None
     # > 0: the residual is fp32 and a block's norm follows its sum, x <- rms(alpha x + f(x)) w (models.decoder runs it)
     postnorm_alpha: float = 0.0
+    # the residual is fp32 and a sublayer reads it as it is; its output is normalised before it is added, x <- x + rms(f(x)) w
+    outnorm: bool = False
     # > 0: behind every layer a token's own embedding of that width (one table, a slice per layer) is gated by the residual,
     # projected, normalised and added
     token_side_dim: int = 0
@@ -165,11 +187,22 @@ class ModelConfig:
         return {**self.mla, **self.layer_mixers[layer]} if self.layer_mixers else self.mla
 
     def attn_of(self, layer: int) -> Dict[str, Any]:
-        """Shapes of an attention layer whose values are its keys."""
+        """Shapes of an attention layer of kind "tied" or "maps"."""
         return self.layer_mixers[layer]
 
     def ffn_of(self, layer: int) -> Dict[str, Any]:
         return self.layer_ffns[layer] if self.layer_ffns else dict(ff=self.intermediate_size, limit=self.swiglu_limit)
+
+    def moe_of(self, layer: int) -> MoeSpec:
+        """The routed experts of a layer whose network differs from layer to layer."""
+        f, names = self.layer_ffns[layer], {x.name for x in dataclasses.fields(MoeSpec)}
+        return MoeSpec(**{k: v for k, v in f.items() if k in names})
+
+    @property
+    def moe(self) -> MoeSpec:
+        """The routed experts of a model that has the same in every routed layer."""
+        return MoeSpec(self.num_experts, self.experts_per_token, self.router_kind, self.router_norm_topk, self.router_scale, self.router_groups,
+                       self.router_topk_groups, self.act)
 
     def kv_source(self, layer: int) -> int:
         """The layer whose rows of the paged pool this one reads (itself unless it shares another's)."""
@@ -178,7 +211,7 @@ class ModelConfig:
 
     def has_kv(self, layer: int) -> bool:
         """Whether the layer keeps keys and values (or rows of another layout) in the paged pool."""
-        return self.layer_kind(layer) in ("attention", "mla", "tied", "attention+mamba2") and self.kv_source(layer) == layer
+        return self.layer_kind(layer) in ("attention", "attention+mamba2") + ROW_CACHE_KINDS and self.kv_source(layer) == layer
 
     @property
     def native_f32(self) -> bool:
@@ -193,12 +226,14 @@ class ModelConfig:
             return "latent"
         if self.postnorm_alpha > 0 and all(k in ("mamba2", "tied") for k in kinds):
             return "tied"
+        if self.outnorm and all(k in ("maps", "maps+lightning") for k in kinds):
+            return "maps"
         return ""
 
     @property
     def fp32_residual(self) -> bool:
         """Families whose residual is one or several fp32 streams with an update kernel of their own."""
-        return self.residual_streams > 0 or self.postnorm_alpha > 0
+        return self.residual_streams > 0 or self.postnorm_alpha > 0 or self.outnorm
 
     @property
     def has_mla(self) -> bool:
@@ -207,7 +242,7 @@ class ModelConfig:
     @property
     def has_row_cache(self) -> bool:
         """Whether the paged pool holds rows of a layout of their own (models.row_cache) instead of keys and values."""
-        return bool(self.layer_kinds) and any(k in ("mla", "tied") for k in self.layer_kinds)
+        return bool(self.layer_kinds) and any(k in ROW_CACHE_KINDS for k in self.layer_kinds)
 
     def layer_window(self, layer: int) -> int:
         if self.sliding_window <= 0:
@@ -248,6 +283,8 @@ class ModelConfig:
             return sovanex_from_config(cls, hf)
         if hf.get("architecture") == "Divanex":
             return divanex_from_config(cls, hf)
+        if hf.get("architecture") == "Dorevik":
+            return dorevik_from_config(cls, hf)
         mt = hf.get("model_type", "llama")
         if mt in ("glm4_moe_lite", "kimi_k2", "youtu"):    # DeepSeek-V3 under another name (Youtu: its dense form): the same tensors, router and latent attention
             hf = dict(hf, model_type="deepseek_v3")
@@ -623,6 +660,67 @@ def divanex_from_config(cls, c: Dict[str, Any]) -> "ModelConfig":
                token_side_dim=int((c.get("token_side") or {}).get("dim", 0)), logit_scale=float(c.get("logit_scale", 1.0)))
 
 
+def _attention_maps(i: int, m: Dict[str, Any], maps: int) -> Dict[str, Any]:
+    """One Dorevik attention as the fields of a layer of kind "maps"."""
+    rot = m["rot"]
+    if m["heads"] % m["kv_heads"]:
+        raise ValueError(f"layer {i}: {m['heads']} query heads over {m['kv_heads']} key heads")
+    if not 0 < rot["dims"] <= m["dim"] or rot["dims"] % 2:
+        raise ValueError(f"layer {i}: a rotation of {rot['dims']} dimensions on heads of {m['dim']}")
+    if int(m["mask"]["size"]) < 1:
+        raise ValueError(f"layer {i}: a window of {m['mask']['size']} tokens")
+    rope, s = dict(dims=rot["dims"], theta=float(rot["base"])), rot.get("scaling")
+    if s is not None:
+        rope["scaling"] = dict(kind="yarn", factor=float(s["factor"]), original_max_position=s["original"], beta_fast=float(s["fast"]),
+                               beta_slow=float(s["slow"]))
+    return dict(num_heads=m["heads"], num_kv_heads=m["kv_heads"], head_dim=m["dim"], v_dim=m["vdim"], maps=maps, window=int(m["mask"]["size"]),
+                scale=float(m["scale"]), rope=rope)
+
+
+def dorevik_from_config(cls, c: Dict[str, Any]) -> "ModelConfig":
+    """Dorevik: layers of differential attention and of windowed attention beside lightning attention, in any order, each with
+    sizes of its own; GeGLU networks or routed SwiGLU experts behind some of them; sublayers that read an fp32 residual as it is
+    and whose outputs are normalised; a capped, untied head."""
+    kinds, ffns, mixers, nets, ff = [], [], [], [], 8
+    for i, layer in enumerate(c["layers"]):
+        m, mlp = layer["mixer"], layer.get("mlp")
+        if layer["type"] == "attention":
+            kinds.append("maps")
+            mixers.append(dict(_attention_maps(i, m, 2), qk_norm="head", diff=float(m["diff"])))
+        elif layer["type"] == "parallel":
+            lin = m["right"]
+            if len(lin["decay"]) != lin["heads"]:
+                raise ValueError(f"layer {i}: {len(lin['decay'])} decays for {lin['heads']} heads")
+            kinds.append("maps+lightning")
+            mixers.append(dict(_attention_maps(i, m["left"], 1), qk_norm="full", lin_heads=lin["heads"], lin_k_dim=lin["dim"], lin_v_dim=lin["vdim"],
+                               lin_decay=[float(d) for d in lin["decay"]]))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
+        if mlp is None:
+            ffns.append("none")
+            nets.append({})
+        elif mlp["kind"] == "dense":
+            ffns.append("glu")
+            nets.append(dict(ff=mlp["ff"]))
+            ff = max(ff, mlp["ff"])
+        elif mlp["kind"] == "moe":
+            r = mlp["router"]
+            if not 0 < r["top"] <= r["experts"]:
+                raise ValueError(f"layer {i}: the best {r['top']} of {r['experts']} experts")
+            ffns.append("moe")
+            nets.append(dict(experts=r["experts"], top=r["top"], ff=mlp["expert"]["ff"], shared_ff=(mlp.get("shared") or {}).get("ff", 0),
+                             router="deepseek_v3", act="swiglu", weigh_input=True, fp32_router=True))
+        else:
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+    first = mixers[0]
+    eps = float(c["norm"]["eps"])
+    return cls(arch="dorevik", name=c.get("name") or "dorevik", vocab_size=c["vocab"], hidden_size=c["width"], num_layers=len(kinds),
+               num_heads=first["num_heads"], num_kv_heads=first["num_kv_heads"], head_dim=first["head_dim"], intermediate_size=(ff + 15) // 16 * 16,
+               rms_eps=eps, act="geglu", use_rope=False, layer_kinds=kinds, ffn_kinds=ffns, layer_mixers=mixers, layer_ffns=nets,
+               ssm=dict(norm_eps=eps), sliding_window=max(m["window"] for m in mixers), outnorm=True,
+               logit_softcap=float(c.get("logit_softcap") or 0.0))
+
+
 RECURRENT_MODEL_TYPES = ("falcon_h1", "nemotron_h", "nemotron_h_moe", "mamba", "falcon_mamba", "mamba2", "bamba", "lfm2", "rwkv7", "qwen3_next", "qwen3_5_text", "qwen3_5_moe_text", "jamba", "granitemoehybrid", "granitemoe", "granitemoeshared", "glm4_moe", "ernie4_5_moe", "rwkv6")
 
 
@@ -866,9 +964,12 @@ def rope_inv_freq(cfg: ModelConfig) -> "tuple[List[float], float]":
     """Per-pair inverse frequencies (length rot_dim/2) and the attention factor that
     multiplies cos/sin. Covers plain, linear, Llama-3 and YaRN scaling
     (rust/engine/src/rope.rs:1 builds the same families of tables)."""
-    rot = cfg.rot_dim
-    base = [cfg.rope_theta ** (-(2.0 * i) / rot) for i in range(rot // 2)]
-    rs = cfg.rope_scaling
+    return scaled_inv_freq(cfg.rot_dim, cfg.rope_theta, cfg.rope_scaling)
+
+
+def scaled_inv_freq(rot: int, theta: float, rs: RopeScaling) -> "tuple[List[float], float]":
+    """The same for a rotation over ``rot`` values with base ``theta`` (layers with a rotation of their own)."""
+    base = [theta ** (-(2.0 * i) / rot) for i in range(rot // 2)]
     attn = 1.0
     if rs.kind == "linear":
         base = [f / rs.factor for f in base]
@@ -894,7 +995,7 @@ def rope_inv_freq(cfg: ModelConfig) -> "tuple[List[float], float]":
     elif rs.kind == "yarn":
         def corr_dim(n_rot: float) -> float:
             return (rot * math.log(rs.original_max_position / (n_rot * 2 * math.pi))) / (
-                2 * math.log(cfg.rope_theta))
+                2 * math.log(theta))
         lo, hi = corr_dim(rs.beta_fast), corr_dim(rs.beta_slow)
         if rs.truncate:
             lo, hi = math.floor(lo), math.ceil(hi)
@@ -1034,6 +1135,23 @@ def preset(name: str) -> ModelConfig:
         return divanex_from_config(ModelConfig, dict(
             architecture="Divanex", name=n, layers=layers, norm=dict(eps=1e-5), embedding=dict(scale=4.0), postln_alpha=2.0, logit_scale=0.5,
             token_side=dict(dim=16 if tiny else 256), vocab=512 if tiny else 65536, width=96 if tiny else 2048))
+    if n in ("dorevik-tiny", "dorevik-2b"):
+        # three layers of differential attention, then one of windowed beside lightning attention; experts in every second layer
+        tiny = n.endswith("tiny")
+        dim, vdim = (40, 56) if tiny else (64, 128)
+        diff = dict(heads=4 if tiny else 16, kv_heads=2 if tiny else 4, dim=dim, vdim=vdim, scale=dim ** -0.5, diff=0.7, mask=dict(size=24 if tiny else 2048),
+                    rot=dict(base=1e4, dims=16 if tiny else 64, scaling=dict(factor=4.0, original=64 if tiny else 4096, fast=32.0, slow=1.0)))
+        left = dict(heads=4 if tiny else 16, kv_heads=2 if tiny else 4, dim=32 if tiny else 128, vdim=24 if tiny else 128, scale=(32 if tiny else 128) ** -0.5,
+                    mask=dict(size=10 if tiny else 512), rot=dict(base=1e6, dims=32 if tiny else 128))
+        heads = 2 if tiny else 16
+        right = dict(heads=heads, dim=24 if tiny else 128, vdim=40 if tiny else 128, decay=[math.exp(-0.5 ** (1 + 8 * i / heads)) for i in range(heads)])
+        dense = dict(kind="dense", ff=160 if tiny else 6144)
+        moe = dict(kind="moe", expert=dict(ff=48 if tiny else 768), router=dict(experts=10 if tiny else 32, top=2 if tiny else 4),
+                   shared=dict(ff=64 if tiny else 1536))
+        layers = [dict(type="parallel" if i % 4 == 3 else "attention", mixer=dict(left=left, right=right) if i % 4 == 3 else diff,
+                       mlp=moe if i % 2 else dense) for i in range(8 if tiny else 24)]
+        return dorevik_from_config(ModelConfig, dict(
+            architecture="Dorevik", name=n, layers=layers, norm=dict(eps=1e-6), logit_softcap=30.0, vocab=512 if tiny else 65536, width=96 if tiny else 2048))
     raise KeyError(f"unknown model preset {name!r}")
 
 

@@ -17,10 +17,9 @@ from typing import List, Optional
 
 import torch
 
-from ..config import ModelConfig, rope_inv_freq
+from ..config import ModelConfig, RopeScaling, rope_inv_freq, scaled_inv_freq
+from .moe import ACT_KIND
 from .weights import DecoderWeights, ShardSpec, make_shard_spec
-
-ACT_KIND = {"swiglu": 0, "geglu": 1, "swiglu_oai": 2}
 
 
 @dataclass
@@ -141,14 +140,15 @@ class Decoder:
         if self.cfg.is_moe or self.cfg.act not in ("swiglu", "geglu"):
             return
         for lw in self.w.layers:
-            w = lw.w_gate_up
-            if not isinstance(w, torch.Tensor) or getattr(lw, "glu_layout", 0) or (w.shape[0] // 2) % 16:
-                continue
-            I, K = w.shape[0] // 2, w.shape[1]
-            blocked = torch.stack([w[:I].view(I // 16, 16, K), w[I:].view(I // 16, 16, K)], 1).reshape(2 * I, K)
-            w.copy_(blocked)
-            del blocked
-            lw.glu_layout = 16
+            for name, layout in (("w_gate_up", "glu_layout"), ("shared_gate_up", "shared_layout")):
+                w = getattr(lw, name)
+                if not isinstance(w, torch.Tensor) or w.dtype == torch.float32 or getattr(lw, layout, 0) or (w.shape[0] // 2) % 16:
+                    continue
+                I, K = w.shape[0] // 2, w.shape[1]
+                blocked = torch.stack([w[:I].view(I // 16, 16, K), w[I:].view(I // 16, 16, K)], 1).reshape(2 * I, K)
+                w.copy_(blocked)
+                del blocked
+                setattr(lw, layout, 16)
 
     # ------------------------------------------------------------------ pieces
     def rope_table(self, dims: int, theta: float) -> torch.Tensor:
@@ -157,6 +157,15 @@ class Decoder:
         if key not in self._rope_tables:
             self._rope_tables[key] = torch.tensor([theta ** (-(2.0 * i) / dims) for i in range(dims // 2)], dtype=torch.float32,
                                                   device=self.w.final_norm.device)
+        return self._rope_tables[key]
+
+    def layer_rope(self, rope: dict) -> "tuple[torch.Tensor, float]":
+        """Inverse frequencies and the factor of cosine and sine of a layer's own rotation (dims, theta, optionally scaling)."""
+        scaling = rope.get("scaling") or {}
+        key = (rope["dims"], rope["theta"], tuple(sorted(scaling.items())))
+        if key not in self._rope_tables:
+            inv, factor = scaled_inv_freq(rope["dims"], rope["theta"], RopeScaling(**scaling))
+            self._rope_tables[key] = (torch.tensor(inv, dtype=torch.float32, device=self.w.final_norm.device), factor)
         return self._rope_tables[key]
 
     def _reduce(self, x: torch.Tensor) -> torch.Tensor:
@@ -215,24 +224,24 @@ class Decoder:
     def _ffn_block(self, lw, h: torch.Tensor) -> torch.Tensor:
         cfg, ops = self.cfg, self.ops
         if lw.router_w is not None:
-            from .moe import moe_ffn, moe_ffn_alltoall
+            from .moe import moe_ffn, moe_ffn_alltoall, spec_of
             if self.ep_a2a is not None:
                 self._reduced = True                 # rows come back complete: nothing left to reduce
                 return moe_ffn_alltoall(self, lw, h)
-            if lw.moe_latent_in is not None:         # the router reads the hidden state, the experts a projection of it
-                y = ops.linear(moe_ffn(self, lw, h, ops.linear(h, lw.moe_latent_in)), lw.moe_latent_out)
-            else:
-                y = moe_ffn(self, lw, h)
+            ys = None
             if lw.shared_gate_up is not None:        # always-on shared experts: one dense MLP beside the routed ones
                 if cfg.mlp_kind == "plain":
                     act = ops.act_(ops.linear(h, lw.shared_gate_up), cfg.act)
                 else:
-                    act = ops.linear_glu(h, lw.shared_gate_up, None, self.act_kind, cfg.swiglu_alpha, cfg.swiglu_limit, 0)
+                    act = ops.linear_glu(h, lw.shared_gate_up, None, ACT_KIND.get(spec_of(cfg, lw).act, 0), cfg.swiglu_alpha, cfg.swiglu_limit,
+                                         lw.shared_layout)
                 ys = ops.linear(act, lw.shared_down)
                 if lw.shared_gate_w is not None:
                     ys = (ys.float() * torch.sigmoid(ops.linear(h, lw.shared_gate_w)[:, :1].float())).to(ys.dtype)
-                y = y + ys
-            return y
+            if lw.moe_latent_in is not None:         # the router reads the hidden state, the experts a projection of it
+                y = ops.linear(moe_ffn(self, lw, h, ops.linear(h, lw.moe_latent_in)), lw.moe_latent_out)
+                return y if ys is None else y + ys
+            return moe_ffn(self, lw, h, add=ys)
         if cfg.mlp_kind == "plain":               # two matrices and an activation between them
             u = ops.act_(ops.linear(h, lw.w_gate_up, lw.b_up), cfg.act)
             return ops.linear(u, lw.w_down, lw.b_down, defer=self.defer_to_residual)
@@ -254,7 +263,7 @@ class Decoder:
             return rwkv6_forward_hidden(self, b)
         if cfg.residual_streams:
             return self._forward_streams(b)
-        if cfg.postnorm_alpha > 0:
+        if cfg.postnorm_alpha > 0 or cfg.outnorm:
             return self._forward_postnorm(b)
         if self.first_stage:
             x = ops.embed(b.token_ids, self.w.embed, cfg.embed_scale)
@@ -312,9 +321,11 @@ class Decoder:
         return x, delta
 
     def _forward_postnorm(self, b: StepBatch):
-        """The layers of a model whose norms follow the residual sum, each with its token input behind it. Returns (fp32
-        residual, (y, arguments of the last update)): that update runs together with the final norm, in ``logits``."""
+        """The layers of a model whose sublayers read an fp32 residual as it is, with norms behind the residual sum or on what is
+        added (``outnorm``), each with its token input, if any, behind it. Returns (residual, (y, arguments of the last
+        update)): that update runs together with the final norm, in ``logits``."""
         cfg, ops, W, eps = self.cfg, self.ops, self.cfg.hidden_size, self.cfg.rms_eps
+        how = (W, eps, 1.0, True) if cfg.outnorm else (W, eps, cfg.postnorm_alpha)
         x, h = ops.postnorm_begin(b.token_ids, self.w.embed, cfg.embed_scale)
         pending = None
         for li, lw in zip(self.layer_range, self.w.layers):
@@ -325,13 +336,16 @@ class Decoder:
             if cfg.layer_kind(li) == "tied":
                 from .tied import tied_attention_mixer
                 y = tied_attention_mixer(self, li, lw, h, b)
+            elif cfg.layer_kind(li) in ("maps", "maps+lightning"):
+                from .maps import MAPS_MIXERS
+                y = MAPS_MIXERS[cfg.layer_kind(li)](self, li, lw, h, b)
             else:
                 from .recurrent import MIXERS
                 y = MIXERS[cfg.layer_kind(li)](self, li, lw, h, b)
-            pending = (y, lw.attn_norm, W, eps, cfg.postnorm_alpha)
+            pending = (y, lw.attn_norm, *how)
             if cfg.ffn_kind(li) != "none":
                 h = ops.postnorm_step(x, *pending)
-                pending = (self._ffn_block(lw, h), lw.ffn_norm, W, eps, cfg.postnorm_alpha)
+                pending = (self._ffn_block(lw, h), lw.ffn_norm, *how)
             if lw.side is not None:
                 h = ops.postnorm_step(x, *pending)
                 g = ops.side_gate(ops.linear(h, lw.side.gate, defer=self.defer_to_residual), b.token_ids, self.w.side_embed, li * cfg.token_side_dim,
@@ -459,12 +473,13 @@ class Decoder:
             if self.capture_hidden:
                 self.last_hidden = hs
             return ops.linear(hs, self.w.lm_head, self.w.lm_head_b)
-        if cfg.postnorm_alpha > 0:              # last update, final norm and logit scale, wanted rows: one kernel
+        if cfg.postnorm_alpha > 0 or cfg.outnorm:    # last update, final norm and logit scale, wanted rows: one kernel
             rows = None if b.all_decode and b.logit_rows.numel() == x.shape[0] else b.logit_rows
             hs = ops.postnorm_step(x, *delta, final_w=self.w.final_norm, final_scale=cfg.logit_scale, rows=rows)
             if self.capture_hidden:                # without the factor that belongs to the logits
                 self.last_hidden = hs / cfg.logit_scale
-            return ops.linear(hs, self.w.lm_head)
+            lg = ops.linear(hs, self.w.lm_head)
+            return ops.softcap_(lg, cfg.logit_softcap) if cfg.logit_softcap > 0 else lg
         if cfg.arch in ("rwkv7", "rwkv6"):
             from .rwkv import rwkv7_final_norm
             h = rwkv7_final_norm(self, x)

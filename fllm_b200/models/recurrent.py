@@ -26,7 +26,7 @@ def pad8(n: int) -> int:
 
 
 def _state_kind(kind: str) -> str:
-    return "mamba2" if kind == "attention+mamba2" else kind
+    return {"attention+mamba2": "mamba2", "maps+lightning": "lightning"}.get(kind, kind)
 
 
 def conv_channels(cfg: ModelConfig, kind: str, layer: int = 0) -> int:
@@ -50,14 +50,16 @@ def scan_state_shape(cfg: ModelConfig, kind: str, layer: int = 0):
         return (s["n_heads"], s["head_dim"], s["d_state"])
     if kind == "gated_delta":
         return (s["num_v_heads"], s["head_v_dim"], s["head_k_dim"])
+    if kind == "lightning":
+        return (s["lin_heads"], s["lin_v_dim"], s["lin_k_dim"])
     if kind in ("rwkv7", "rwkv6"):
         return (cfg.hidden_size // s["head_dim"], s["head_dim"], s["head_dim"])
     return None
 
 
 class RecurrentState:
-    """State pools of this stage's recurrent layers: per layer a convolution window [slots, W - 1, C] in the activation type (bf16 on a GPU) and (except
-    for the short convolution) an fp32 scan state [slots, ...]. The last row is the scratch row of padding sequences."""
+    """State pools of this stage's recurrent layers: per layer a convolution window [slots, W - 1, C] in the activation type (bf16 on a GPU; none for
+    lightning attention) and (except for the short convolution) an fp32 scan state [slots, ...]. The last row is the scratch row of padding sequences."""
 
     def __init__(self, cfg: ModelConfig, layer_range: range, slots: int, device, act_dtype=torch.bfloat16):
         self.slots = slots
@@ -71,7 +73,8 @@ class RecurrentState:
             W = cfg.ssm_of(li).get("d_conv", 4)
             if kind in ("rwkv7", "rwkv6"):
                 self.shift2[li] = torch.zeros(slots, W - 1, cfg.hidden_size, dtype=act_dtype, device=device)
-            self.conv[li] = torch.zeros(slots, W - 1, conv_channels(cfg, kind, li), dtype=act_dtype, device=device)
+            if kind != "lightning":
+                self.conv[li] = torch.zeros(slots, W - 1, conv_channels(cfg, kind, li), dtype=act_dtype, device=device)
             shape = scan_state_shape(cfg, kind, li)
             if shape is not None:
                 self.scan[li] = torch.zeros(slots, *shape, dtype=torch.float32, device=device)
@@ -84,7 +87,8 @@ class RecurrentState:
             if kind in STATELESS_KINDS:
                 continue
             W = cfg.ssm_of(li).get("d_conv", 4)
-            n += (W - 1) * conv_channels(cfg, kind, li) * (4 if kind in ("rwkv7", "rwkv6") else elem)
+            if kind != "lightning":
+                n += (W - 1) * conv_channels(cfg, kind, li) * (4 if kind in ("rwkv7", "rwkv6") else elem)
             shape = scan_state_shape(cfg, kind, li)
             if shape is not None:
                 k = 4

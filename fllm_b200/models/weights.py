@@ -17,7 +17,7 @@ from typing import Dict, List, Optional
 
 import torch
 
-from ..config import ModelConfig
+from ..config import ModelConfig, MoeSpec
 
 
 @dataclass
@@ -80,11 +80,13 @@ class LayerWeights:
     streams2: Optional["StreamMix"] = None
     side: Optional["SideInput"] = None              # per-layer token input behind the layer
     act_limit: Optional[float] = None               # clamp of this layer's gated activation (None: the model's)
+    moe: Optional[MoeSpec] = None                   # routed experts that differ from layer to layer (None: the model's)
     # packed formats keep their payload here (format name -> tensors)
     packed: Dict[str, object] = field(default_factory=dict)
     # row order of w_gate_up: 0 = gate half then up half; 16 = blocks of 16 gate rows followed by the 16 up
     # rows of the same features (set by the decoder on a GPU, where the GEMM epilogue applies the activation)
     glu_layout: int = 0
+    shared_layout: int = 0                          # the same of shared_gate_up
 
 
 def gate_up_natural(lw: "LayerWeights") -> torch.Tensor:
@@ -284,6 +286,11 @@ def init_random_weights(cfg: ModelConfig, device="cpu", dtype=torch.bfloat16, se
         if tp > 1 or (layers is not None and len(layers) != cfg.num_layers):
             raise NotImplementedError("models with a residual in fp32 run on one rank and one pipeline stage")
         return divanex_weights(cfg, random_tensors(cfg, seed, device), device, dtype)
+    if cfg.arch == "dorevik":
+        from ..formats.dorevik_loader import dorevik_weights, random_tensors
+        if tp > 1 or (layers is not None and len(layers) != cfg.num_layers):
+            raise NotImplementedError("models with a residual in fp32 run on one rank and one pipeline stage")
+        return dorevik_weights(cfg, random_tensors(cfg, seed, device), device, dtype)
     sp = make_shard_spec(cfg, tp, tp_rank, expert_parallel)
     D, H = cfg.head_dim, cfg.hidden_size
     layers = range(cfg.num_layers) if layers is None else layers

@@ -1,0 +1,146 @@
+"""Attention of one or two maps over shared values, and the recurrence of lightning attention: the fp32 PyTorch statement of each
+op (``MapsRef``, mixed into the reference ops) and the wrappers of the sm_100a kernels (``MapsNative``).
+
+A map is a softmax attention with queries and keys of its own. Every query head has ``maps`` of them over the values of its
+key/value head; two maps are combined as ``rms(a1 - lam a2) * out_scale`` over the head's values. Map m of query head h is row
+``h * maps + m`` of the query heads and reads key row ``g * maps + m``. Cache rows are padded with zeros to ``maps_width``; key
+and value rows have widths of their own. A query at position i sees the keys j with 0 <= i - j < window (0: all up to i).
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+import torch.nn.functional as F
+
+from .latent import _rotate
+from .tied import tied_width
+
+
+def maps_width(dim: int) -> int:
+    """Padded length of a key, value or query row."""
+    return tied_width(dim)
+
+
+@dataclass
+class Combine:
+    """How the two maps of a head become its output."""
+    lam: float
+    out_scale: float
+    eps: float
+
+
+@dataclass
+class NormedPair:
+    """A sublayer output that is half the sum of two projections, each over its root mean square times a weight. ``b`` may be a
+    deferred projection; ``postnorm_step`` takes the pair in place of a tensor."""
+    a: torch.Tensor
+    b: object
+    wa: torch.Tensor
+    wb: torch.Tensor
+
+
+def _rms(x, eps):
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+
+
+class MapsRef:
+    def maps_prepare(self, x, offsets, heads, dim, v_dim, positions, slots, inv_freq, rope_factor, q_norm, k_norm, full, eps, k_cache, v_cache):
+        """``x`` [T, ...]: query maps at column offsets[0], key maps at offsets[1], values at offsets[2]. Norms (over a map, or with
+        ``full`` over all maps at once), rotates the first 2 len(inv_freq) values of every map, writes the tokens' cache rows
+        (slot < 0: none) and returns the queries [T, heads, W], padded like the key rows."""
+        T, W, bs = x.shape[0], k_cache.shape[3], k_cache.shape[2]
+        rot = 2 * inv_freq.numel()
+
+        def part(off, n, w):
+            t = x[:, off:off + n * dim].float()
+            t = _rms(t, eps) * w.float() if full else _rms(t.reshape(T, n, dim), eps) * w.float()
+            t = t.reshape(T, n, dim)
+            return F.pad(torch.cat([_rotate(t[..., :rot], positions, inv_freq, rope_factor, 0), t[..., rot:]], -1), (0, W - dim)).to(k_cache.dtype)
+        q, k = part(offsets[0], heads, q_norm), part(offsets[1], k_cache.shape[1], k_norm)
+        G = v_cache.shape[1]
+        v = F.pad(x[:, offsets[2]:offsets[2] + G * v_dim].reshape(T, G, v_dim), (0, v_cache.shape[3] - v_dim)).to(v_cache.dtype)
+        keep = slots[:T] >= 0
+        s = slots[:T][keep].long()
+        k_cache[s // bs, :, s % bs] = k[keep]
+        v_cache[s // bs, :, s % bs] = v[keep]
+        return q
+
+    def attention_maps(self, q, k_cache, v_cache, dim, v_dim, b, scale, window=0, combine: Optional[Combine] = None, out_cols=0, tensor_cores=True, splits=None):
+        """q [T, heads * maps, W] against the rows every token may see -> [T, out_cols or heads * v_dim]. ``b``: the step batch."""
+        T, HM = q.shape[:2]
+        G, bs = v_cache.shape[1], v_cache.shape[2]
+        M = k_cache.shape[1] // G
+        H = HM // M
+        out = torch.zeros(T, max(out_cols, H * v_dim), dtype=q.dtype, device=q.device)
+        for t in range(T):
+            n = int(b.positions[t]) + 1
+            lo = max(0, n - window) if window > 0 else 0
+            blocks = b.block_tables[int(b.row_seq[t]), lo // bs:(n + bs - 1) // bs].long()
+            cut = slice(lo - lo // bs * bs, n - lo // bs * bs)
+            k = k_cache[blocks].transpose(1, 2).reshape(-1, G, M, k_cache.shape[3])[cut].float()
+            v = v_cache[blocks].transpose(1, 2).reshape(-1, G, v_cache.shape[3])[cut, :, :v_dim].float()
+            s = torch.einsum("ghmd,ngmd->ghmn", q[t].float().view(G, H // G, M, -1), k) * scale
+            a = torch.einsum("ghmn,ngd->ghmd", torch.softmax(s, -1), v)
+            y = _rms(a[:, :, 0] - combine.lam * a[:, :, 1], combine.eps) * combine.out_scale if M == 2 else a[:, :, 0]
+            out[t, :H * v_dim] = y.reshape(-1).to(out.dtype)
+        return out
+
+    def decay_scan(self, q, k, v, decay, state, q_starts, seq_state, positions, H, K, V, width=0):
+        """Per head S <- decay S + silu(v) silu(k)^T, o = S silu(q), with S [V, K] in fp32: [T, width or H * V]."""
+        from .recurrent import _seqs
+        T = q.shape[0]
+        out = torch.zeros(T, max(width, H * V), dtype=v.dtype, device=v.device)
+        d = decay.float()[:, None, None]
+        act = lambda x, n: F.silu(x.float()).reshape(-1, H, n)
+        for t0, t1, slot, fresh in _seqs(q_starts, seq_state, positions):
+            S = torch.zeros(H, V, K, dtype=torch.float32, device=v.device) if fresh else state[slot].clone()
+            qf, kf, vf = act(q[t0:t1], K), act(k[t0:t1], K), act(v[t0:t1], V)
+            for i in range(t1 - t0):
+                S = d * S + vf[i][:, :, None] * kf[i][:, None, :]
+                out[t0 + i, :H * V] = (S * qf[i][:, None, :]).sum(-1).reshape(-1).to(out.dtype)
+            state[slot] = S
+        return out
+
+
+class MapsNative:
+    """Kernel wrappers; ``self.k`` is the loaded extension and ``self.launches`` the launch counter of the ops object. The
+    projection ``maps_prepare`` reads may be deferred: its split-K partial sums are added by the kernel."""
+
+    def maps_prepare(self, x, offsets, heads, dim, v_dim, positions, slots, inv_freq, rope_factor, q_norm, k_norm, full, eps, k_cache, v_cache):
+        T, splits = x.shape[0], getattr(x, "splits", 0)
+        q = torch.empty(T, heads, k_cache.shape[3], dtype=k_cache.dtype, device=k_cache.device)
+        self.k.maps_prepare(None if splits else x, self.workspace if splits else None, int(splits), int(x.shape[1]), x.bias if splits else None,
+                            int(offsets[0]), int(offsets[1]), int(offsets[2]), int(dim), int(v_dim), positions, slots, inv_freq, float(rope_factor), q_norm,
+                            k_norm, bool(full), float(eps), q, k_cache, v_cache)
+        self.launches += 1
+        return q
+
+    def attention_maps(self, q, k_cache, v_cache, dim, v_dim, b, scale, window=0, combine: Optional[Combine] = None, out_cols=0, tensor_cores=True, splits=None):
+        T, HM = q.shape[:2]
+        M = k_cache.shape[1] // v_cache.shape[1]
+        H = HM // M
+        make = torch.zeros if out_cols > H * v_dim else torch.empty
+        out = make(T, max(out_cols, H * v_dim), dtype=q.dtype, device=q.device)
+        if splits is None:
+            splits = int(self.k.attention_maps_splits(b.num_seqs, b.max_q_len, H, v_cache.shape[1], M, b.max_kv_len, int(window))) if q.dtype == torch.bfloat16 else 1
+        ws = None
+        if splits > 1:
+            need = int(self.k.attention_maps_workspace_bytes(T, HM, v_cache.shape[3], splits))
+            held = self.__dict__.setdefault("_maps_ws", [])        # grow-only; captured graphs may still use the smaller ones
+            if not held or held[-1].numel() < need:
+                held.append(torch.empty(need, dtype=torch.uint8, device=q.device))
+            ws = held[-1]
+        c = combine or Combine(0.0, 1.0, 0.0)
+        self.launches += self.k.attention_maps(q, k_cache, v_cache, int(dim), int(v_dim), b.block_tables, b.row_seq, b.positions, b.q_starts, out, b.num_seqs,
+                                               b.max_q_len, b.min_q_len, float(scale), int(window), float(c.lam), float(c.out_scale), float(c.eps),
+                                               int(splits), ws, bool(tensor_cores), self.status)
+        return out
+
+    def decay_scan(self, q, k, v, decay, state, q_starts, seq_state, positions, H, K, V, width=0):
+        make = torch.zeros if width > H * V else torch.empty
+        out = make(q.shape[0], max(width, H * V), dtype=v.dtype, device=v.device)
+        self.k.decay_scan(q, k, v, decay, state, q_starts, seq_state, positions, out, int(H), int(K), int(V))
+        self.launches += 1
+        return out

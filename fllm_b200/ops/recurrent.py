@@ -186,14 +186,15 @@ class RecurrentRef:
             state[slot] = S
         return y
 
-    def gated_rmsnorm(self, x, z, w, eps, group_size=0, norm_before_gate=False, width=0):
-        """Mamba-2: rmsnorm(x * silu(z)) * w over groups; gated delta net: rmsnorm(x) * w * silu(z) (norm first).
+    def gated_rmsnorm(self, x, z, w, eps, group_size=0, norm_before_gate=False, width=0, gate="silu"):
+        """Mamba-2: rmsnorm(x * silu(z)) * w over groups; gated delta net: rmsnorm(x) * w * silu(z) (norm first); ``gate``
+        "sigmoid" (lightning attention): sigmoid(z) in place of silu(z).
         ``w`` may be shorter than the row (one weight vector per head): it repeats. ``width``: columns of the result when
         the next matrix is padded (zeros behind the row)."""
         T, D = x.shape
         gs = group_size or D
         xf = x.float()
-        gate = F.silu(z.float()) if z is not None else None
+        gate = {"silu": F.silu, "sigmoid": torch.sigmoid}[gate](z.float()) if z is not None else None
         if gate is not None and not norm_before_gate:
             xf = xf * gate
         xg = xf.view(T, D // gs, gs)
@@ -303,13 +304,13 @@ class RecurrentNative:
         self.launches += 1
         return y
 
-    def gated_rmsnorm(self, x, z, w, eps, group_size=0, norm_before_gate=False, width=0):
+    def gated_rmsnorm(self, x, z, w, eps, group_size=0, norm_before_gate=False, width=0, gate="silu"):
         if width > x.shape[1]:
             full = torch.zeros(x.shape[0], width, dtype=x.dtype, device=x.device)
             y = full[:, :x.shape[1]]
         else:
             full = y = torch.empty(x.shape, dtype=x.dtype, device=x.device)
-        self.k.gated_rmsnorm(x, z, w, y, int(group_size or x.shape[1]), float(eps), bool(norm_before_gate))
+        self.k.gated_rmsnorm(x, z, w, y, int(group_size or x.shape[1]), float(eps), bool(norm_before_gate), gate == "sigmoid")
         self.launches += 1
         return full
 

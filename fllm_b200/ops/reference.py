@@ -12,11 +12,12 @@ import torch
 import torch.nn.functional as F
 
 from .latent import LatentRef
+from .maps import MapsRef
 from .tied import TiedRef
 from .recurrent import RecurrentRef
 
 
-class RefOps(RecurrentRef, LatentRef, TiedRef):
+class RefOps(RecurrentRef, LatentRef, TiedRef, MapsRef):
     name = "reference"
 
     # ---------------------------------------------------------------- dense

@@ -7,7 +7,8 @@ every query head has an fp32 factor of its own (norm, temperature by position, s
 therefore exist only inside the fp32 scores.
 
 The residual is fp32 [rows, width]. ``postnorm_step`` with ``add`` off is ``x <- rms(alpha x + y) w``, with ``add`` on
-``x <- x + rms(y) w``; it returns the row in the activation type, or its final norm.
+``x <- x + rms(y) w``; it returns the row in the activation type, or its final norm. Its ``y`` may be a pair of projections
+with norms of their own (``ops.maps.NormedPair``).
 """
 from __future__ import annotations
 
@@ -70,7 +71,10 @@ class TiedRef:
         return x, x.to(table.dtype)
 
     def postnorm_step(self, x, y, norm_w, width, eps, alpha=1.0, add=False, final_w=None, final_scale=1.0, rows=None):
-        """``rows`` (with ``final_w``): only these rows, the residual is left as it is."""
+        """``rows`` (with ``final_w``): only these rows, the residual is left as it is. ``y``: a tensor or a NormedPair."""
+        if hasattr(y, "wa"):
+            norm = lambda t, w: F.pad(_rms(t.float()[:, :width], eps), (0, x.shape[1] - width)) * w.float()
+            y = 0.5 * (norm(y.a, y.wa) + norm(y.b, y.wb))
         y = y.float()
         v = y if add else alpha * x + y
         v = F.pad(_rms(v[:, :width], eps), (0, x.shape[1] - width)) * norm_w.float()
@@ -119,15 +123,17 @@ class TiedNative:
         T, ld = ids.numel(), table.shape[1]
         x = torch.empty(T, ld, dtype=torch.float32, device=table.device)
         h = torch.empty(T, ld, dtype=table.dtype, device=table.device)
-        self.k.postnorm(x, ids, table, float(scale), None, None, 0, False, 0.0, None, None, 1.0, None, h, ld, 0.0, True)
+        self.k.postnorm(x, ids, table, float(scale), None, None, 0, False, 0.0, None, None, 1.0, None, h, ld, 0.0, True, None, None, None)
         self.launches += 1
         return x, h
 
     def postnorm_step(self, x, y, norm_w, width, eps, alpha=1.0, add=False, final_w=None, final_scale=1.0, rows=None):
         h = torch.empty(x.shape[0] if rows is None else rows.numel(), x.shape[1], dtype=norm_w.dtype, device=x.device)
+        first, wa, wb = (y.a, y.wa, y.wb) if hasattr(y, "wa") else (None, None, None)
+        y = y.b if first is not None else y
         splits = getattr(y, "splits", 0)
         self.k.postnorm(x, None, None, 1.0, None if splits else y, self.workspace if splits else None, int(splits), bool(add), float(alpha), norm_w, final_w,
-                        float(final_scale), rows, h, int(width), float(eps), rows is None)
+                        float(final_scale), rows, h, int(width), float(eps), rows is None, first, wa, wb)
         self.launches += 1
         return h
 
