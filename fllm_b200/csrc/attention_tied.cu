@@ -22,32 +22,16 @@
 #include <stdexcept>
 #include <unordered_map>
 
+#include "attention_util.cuh"
 #include "fllm_ops.h"
 #include "ptx.cuh"
 #include "tma_host.h"
 
 namespace fllm {
 namespace {
-using bf16 = __nv_bfloat16;
-constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kFixedCap = 64.f;
-constexpr int kPage = 16;                 // tokens fetched as one piece (blocks are multiples of it)
 constexpr int kDecodeRows = 64;           // sequences with at most this many query rows per kv head run in the decode kernel
 
-__device__ __forceinline__ float to_f32(float v) { return v; }
-__device__ __forceinline__ float to_f32(bf16 v) { return __bfloat162float(v); }
-template <typename T>
-__device__ __forceinline__ T from_f32(float v);
-template <>
-__device__ __forceinline__ float from_f32<float>(float v) { return v; }
-template <>
-__device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16(v); }
-
-__device__ __forceinline__ float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 __device__ __forceinline__ float rcp(float x) {
   float y;
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -58,10 +42,6 @@ __device__ __forceinline__ float rcp(float x) {
 // One warp per (token, head), query heads first. Query head: q_factor[t][h] = scale * temperature(position) / rms(q). Key head:
 // the row goes to the cache with f = 1 / rms(k). rms(x) = sqrt(mean x^2 + eps); eps < 0: no norm (factor 1). temperature =
 // 1 + coef ln(floor((position + 1) / every) + 1). With split-K partial sums as the source, queries are also written to q_out.
-template <typename T>
-struct Four { using type = uint2; };
-template <>
-struct Four<float> { using type = float4; };
 template <typename T>
 __global__ void __launch_bounds__(128) tied_prepare_kernel(const TiedPrepareParams p) {
   pdl_launch_dependents();
@@ -234,36 +214,6 @@ __device__ __forceinline__ int page_row(const Tied& p, const int* table, int tok
 }
 
 // ------------------------------------------------------------------------------------------ decode
-__device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(smem)), "l"(gmem) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() {
-  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
-}
-__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void ldsm_x4_t(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// 16-byte piece c of row r of a row-major tile lies at piece c ^ (r & 7): ldmatrix row fetches hit distinct banks
-template <int D>
-__device__ __forceinline__ bf16* tile_ptr(bf16* base, int row, int chunk) {
-  return base + row * D + ((chunk ^ (row & 7)) << 3);
-}
-
 template <int D>
 struct DecodeTile {
   static constexpr int kStages = 4;
@@ -486,10 +436,7 @@ __global__ void __launch_bounds__(128) tied_merge_kernel(const Tied p, int T) {
 // issues the MMAs, warps 2 - 5 are the softmax, one thread per query row. The weights of 32 tokens overwrite the 32 columns
 // their scores came from: 16 columns of leading bf16 terms, 16 of remainders. Tensor memory: S / P 128 columns, O 128; two
 // CTAs share an SM, so one's softmax runs under the other's MMAs. Every wait is bounded.
-constexpr int kRows = 128, kTile = 128, kThreads = 192, kHalf = 128 * 128;      // kHalf: bytes of a 64-column half of a tile
-constexpr float kLazyRescale = 8.f;
-template <int D>
-constexpr int tile_bytes() { return (D / 64) * kHalf; }
+constexpr int kThreads = 192;
 template <int D>
 constexpr int prefill_smem() { return 3 * tile_bytes<D>() + 2 * kTile * 4 + 256 + 1024; }
 
@@ -498,12 +445,6 @@ __device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t b
   asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst)), "l"(src), "r"(bytes),
                "r"(smem_u32(bar))
                : "memory");
-}
-
-// MN-major operand: 128-byte swizzled rows, 1024 bytes between groups of eight rows, kHalf between the 64-column halves
-template <int D>
-__device__ __forceinline__ uint64_t desc_mn_major(uint32_t saddr) {
-  return (uint64_t)((saddr & 0x3FFFFu) >> 4) | (uint64_t)((D > 64 ? kHalf : 1024) >> 4) << 16 | (uint64_t)(1024 >> 4) << 32 | (uint64_t)1 << 46 | (uint64_t)2 << 61;
 }
 
 template <int D, bool FULL, bool CAP, bool FIXED>

@@ -259,10 +259,12 @@ void act_(Tensor x, int64_t kind) {
 }
 
 void softcap_(Tensor x, double cap) {
-  check_bf16(x, "x"); check_rows(x, "x");
+  const bool f32 = x.is_cuda() && x.scalar_type() == at::kFloat;
+  if (!f32) check_bf16(x, "x");
+  check_rows(x, "x");
   TORCH_CHECK(cap > 0, "softcap_: the cap must be positive");
   c10::cuda::CUDAGuard guard(x.device());
-  fllm::softcap_rows_bf16(x.data_ptr(), x.stride(0), (int)x.size(0), (int)x.size(1), (float)cap, cur_stream());
+  fllm::softcap_rows(x.data_ptr(), x.stride(0), (int)x.size(0), (int)x.size(1), (float)cap, f32 ? 1 : 0, cur_stream());
 }
 
 void argmax(const Tensor& logits, Tensor out_ids, const optional<Tensor>& out_vals,

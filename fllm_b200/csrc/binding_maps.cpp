@@ -1,0 +1,120 @@
+// torch.ops.fllm_b200 bindings of attention of one or two maps over shared values (attention_maps.cu).
+#include <ATen/ATen.h>
+#include <c10/cuda/CUDAGuard.h>
+#include <c10/cuda/CUDAStream.h>
+#include <torch/library.h>
+
+#include <algorithm>
+
+#include "fllm_ops.h"
+
+namespace {
+using at::Tensor;
+using c10::optional;
+inline cudaStream_t cur_stream() { return c10::cuda::getCurrentCUDAStream().stream(); }
+inline bool given(const optional<Tensor>& t) { return t.has_value() && t->defined(); }
+inline bool i32(const Tensor& t) { return t.is_cuda() && t.scalar_type() == at::kInt && t.is_contiguous(); }
+inline bool rows_of(const Tensor& t, at::ScalarType ty) { return t.is_cuda() && t.scalar_type() == ty && t.dim() == 2 && t.stride(1) == 1; }
+inline at::ScalarType act_type(const Tensor& t) {
+  TORCH_CHECK(t.is_cuda() && (t.scalar_type() == at::kBFloat16 || t.scalar_type() == at::kFloat), "activations are bf16 or fp32 on a GPU");
+  return t.scalar_type();
+}
+// key and value pools of one layer: [blocks, G * maps, block_size, wk] and [blocks, G, block_size, wv], maps 1 or 2
+inline void check_pools(const Tensor& k, const Tensor& v, at::ScalarType ty, int64_t dim, int64_t v_dim) {
+  TORCH_CHECK(k.dim() == 4 && v.dim() == 4 && k.is_contiguous() && v.is_contiguous() && k.is_cuda() && v.is_cuda() && k.scalar_type() == ty &&
+                  v.scalar_type() == ty && k.size(0) == v.size(0) && k.size(2) == v.size(2) && k.size(3) >= dim && v.size(3) >= v_dim && dim > 0 && v_dim > 0 &&
+                  (k.size(1) == v.size(1) || k.size(1) == 2 * v.size(1)),
+              "pools: [blocks, heads (or twice as many), block_size, width] of one type");
+}
+
+// x [T, >= all segments], or its split-K partial sums [splits][T][width] (bias added here)
+void maps_prepare(const optional<Tensor>& x, const optional<Tensor>& workspace, int64_t splits, int64_t width, const optional<Tensor>& bias,
+                  int64_t q_offset, int64_t k_offset, int64_t v_offset, int64_t dim, int64_t v_dim, const Tensor& positions, const Tensor& slots,
+                  const Tensor& inv_freq, double rope_factor, const Tensor& q_norm, const Tensor& k_norm, bool full, double eps, Tensor q_out,
+                  Tensor k_cache, Tensor v_cache) {
+  const auto ty = act_type(k_cache);
+  check_pools(k_cache, v_cache, ty, dim, v_dim);
+  TORCH_CHECK(q_out.is_cuda() && q_out.scalar_type() == ty && q_out.is_contiguous() && q_out.dim() == 3 && q_out.size(2) == k_cache.size(3),
+              "q_out: [T, query maps, width of the key rows]");
+  fllm::MapsPrepareParams p{};
+  const int64_t T = q_out.size(0), HQ = q_out.size(1), HK = k_cache.size(1), G = v_cache.size(1);
+  const int64_t end = std::max({q_offset + HQ * dim, k_offset + HK * dim, v_offset + G * v_dim});
+  TORCH_CHECK(i32(positions) && i32(slots) && positions.numel() >= T && slots.numel() >= T && q_offset >= 0 && k_offset >= 0 && v_offset >= 0, "positions, slots int32 [T]");
+  TORCH_CHECK(inv_freq.is_cuda() && inv_freq.scalar_type() == at::kFloat && inv_freq.is_contiguous() && 2 * inv_freq.numel() <= dim, "inv_freq: fp32, half the rotated values");
+  TORCH_CHECK(q_norm.is_cuda() && q_norm.scalar_type() == ty && q_norm.is_contiguous() && k_norm.is_cuda() && k_norm.scalar_type() == ty && k_norm.is_contiguous() &&
+                  q_norm.numel() == (full ? HQ * dim : dim) && k_norm.numel() == (full ? HK * dim : dim), "norm weights: one map wide, or all maps (full)");
+  if (splits > 0) {
+    TORCH_CHECK(width >= end && given(workspace) && workspace->is_contiguous() && workspace->nbytes() >= fllm::kLinearPartialsOffset + (size_t)splits * T * width * 4,
+                "workspace too small for the split-K partials");
+    p.partials = reinterpret_cast<const float*>(reinterpret_cast<const uint8_t*>(workspace->data_ptr()) + fllm::kLinearPartialsOffset);
+    p.splits = (int)splits, p.width = (int)width, p.plane = T * width;
+    if (given(bias)) {
+      TORCH_CHECK(bias->is_cuda() && bias->scalar_type() == ty && bias->is_contiguous() && bias->numel() >= end, "bias: [width]");
+      p.bias = bias->data_ptr();
+    }
+  } else {
+    TORCH_CHECK(given(x) && rows_of(*x, ty) && x->size(0) == T && x->size(1) >= end, "x: [T, >= all segments]");
+    p.x = x->data_ptr(), p.ldx = x->stride(0);
+  }
+  p.q_offset = (int)q_offset, p.k_offset = (int)k_offset, p.v_offset = (int)v_offset, p.q_heads = (int)HQ, p.k_heads = (int)HK, p.v_heads = (int)G;
+  p.dim = (int)dim, p.v_dim = (int)v_dim, p.wk = (int)k_cache.size(3), p.wv = (int)v_cache.size(3), p.block_size = (int)k_cache.size(2), p.tokens = (int)T;
+  p.positions = positions.data_ptr<int>(), p.slots = slots.data_ptr<int>(), p.inv_freq = inv_freq.data_ptr<float>();
+  p.rot = 2 * (int)inv_freq.numel(), p.rope_factor = (float)rope_factor;
+  p.q_norm = q_norm.data_ptr(), p.k_norm = k_norm.data_ptr(), p.full = full ? 1 : 0, p.eps = (float)eps;
+  p.q_out = q_out.data_ptr(), p.k_cache = k_cache.data_ptr(), p.v_cache = v_cache.data_ptr(), p.f32 = ty == at::kFloat ? 1 : 0;
+  c10::cuda::CUDAGuard guard(k_cache.device());
+  fllm::maps_prepare(p, cur_stream());
+}
+
+int64_t attention_maps_splits(int64_t num_seqs, int64_t max_q_len, int64_t H, int64_t G, int64_t maps, int64_t max_kv_len, int64_t window) {
+  return fllm::attention_maps_splits((int)num_seqs, (int)max_q_len, (int)H, (int)G, (int)maps, (int)max_kv_len, (int)window);
+}
+int64_t attention_maps_workspace_bytes(int64_t tokens, int64_t q_heads, int64_t wv, int64_t splits) {
+  return (int64_t)fllm::attention_maps_workspace_bytes((int)tokens, (int)q_heads, (int)wv, (int)splits);
+}
+
+// q [T, H * maps, wk], out [T, >= H * v_dim]; returns the number of kernels launched
+int64_t attention_maps(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, int64_t dim, int64_t v_dim, const Tensor& block_tables,
+                       const Tensor& row_seq, const Tensor& positions, const Tensor& q_starts, Tensor out, int64_t num_seqs, int64_t max_q_len,
+                       int64_t min_q_len, double scale, int64_t window, double lam, double out_scale, double eps, int64_t splits,
+                       const optional<Tensor>& workspace, bool tensor_cores, const optional<Tensor>& status) {
+  const auto ty = act_type(q);
+  check_pools(k_cache, v_cache, ty, dim, v_dim);
+  const int64_t T = q.size(0), G = v_cache.size(1), M = k_cache.size(1) / G;
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && q.size(2) == k_cache.size(3) && q.size(1) % (G * M) == 0, "q: contiguous [T, H * maps, width of the key rows]");
+  const int64_t H = q.size(1) / M;
+  TORCH_CHECK(rows_of(out, ty) && out.size(0) == T && out.size(1) >= H * v_dim && window >= 0, "out: [T, >= H * v_dim] like q");
+  TORCH_CHECK(block_tables.is_cuda() && block_tables.scalar_type() == at::kInt && block_tables.dim() == 2 && block_tables.stride(1) == 1 && i32(row_seq) &&
+                  i32(positions) && i32(q_starts) && row_seq.numel() >= T && positions.numel() >= T && q_starts.numel() >= num_seqs + 1,
+              "block_tables [B, max_blocks], row_seq [T], positions [T], q_starts [B + 1]: int32");
+  void* ws = nullptr;
+  size_t ws_bytes = 0;
+  if (given(workspace)) {
+    TORCH_CHECK(workspace->is_cuda() && workspace->is_contiguous(), "workspace: contiguous CUDA tensor");
+    ws = workspace->data_ptr();
+    ws_bytes = workspace->nbytes();
+  }
+  fllm::MapsAttnParams p{};
+  p.q = q.data_ptr(), p.k_cache = k_cache.data_ptr(), p.v_cache = v_cache.data_ptr();
+  p.block_tables = block_tables.data_ptr<int>(), p.max_blocks = (int)block_tables.stride(0);
+  p.row_seq = row_seq.data_ptr<int>(), p.positions = positions.data_ptr<int>(), p.q_starts = q_starts.data_ptr<int>();
+  p.out = out.data_ptr(), p.ldo = out.stride(0);
+  p.tokens = (int)T, p.num_seqs = (int)num_seqs, p.max_q_len = (int)max_q_len, p.min_q_len = (int)min_q_len;
+  p.H = (int)H, p.G = (int)G, p.maps = (int)M, p.dim = (int)dim, p.v_dim = (int)v_dim, p.wk = (int)k_cache.size(3), p.wv = (int)v_cache.size(3);
+  p.block_size = (int)k_cache.size(2), p.num_blocks = k_cache.size(0);
+  p.scale = (float)scale, p.window = (int)window, p.lam = (float)lam, p.out_scale = (float)out_scale, p.eps = (float)eps, p.f32 = ty == at::kFloat ? 1 : 0;
+  c10::cuda::CUDAGuard guard(q.device());
+  return fllm::attention_maps(p, (int)splits, ws, ws_bytes, tensor_cores, given(status) ? status->data_ptr<int>() : nullptr, cur_stream());
+}
+}  // namespace
+
+TORCH_LIBRARY_FRAGMENT(fllm_b200, m) {
+  m.def("maps_prepare(Tensor? x, Tensor? workspace, int splits, int width, Tensor? bias, int q_offset, int k_offset, int v_offset, int dim, int v_dim, "
+        "Tensor positions, Tensor slots, Tensor inv_freq, float rope_factor, Tensor q_norm, Tensor k_norm, bool full, float eps, Tensor(a!) q_out, "
+        "Tensor(b!) k_cache, Tensor(c!) v_cache) -> ()", &maps_prepare);
+  m.def("attention_maps_splits(int num_seqs, int max_q_len, int H, int G, int maps, int max_kv_len, int window) -> int", &attention_maps_splits);
+  m.def("attention_maps_workspace_bytes(int tokens, int q_heads, int wv, int splits) -> int", &attention_maps_workspace_bytes);
+  m.def("attention_maps(Tensor q, Tensor k_cache, Tensor v_cache, int dim, int v_dim, Tensor block_tables, Tensor row_seq, Tensor positions, Tensor q_starts, "
+        "Tensor(a!) out, int num_seqs, int max_q_len, int min_q_len, float scale, int window, float lam, float out_scale, float eps, int splits, "
+        "Tensor? workspace, bool tensor_cores, Tensor? status) -> int", &attention_maps);
+}

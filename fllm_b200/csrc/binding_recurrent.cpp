@@ -69,6 +69,27 @@ void mamba2_scan(const Tensor& x, const Tensor& dt, const Tensor& Bm, const Tens
   TORCH_CHECK(rc == 0, "mamba2_scan: unsupported arguments (code ", rc, "): heads a multiple of the groups, state width up to 256");
 }
 
+// q, k [T, H * K], v, out [T, >= H * V], decay fp32 [H], state fp32 [slots, H, V, K]: S <- decay S + silu(v) silu(k)^T, out = S silu(q)
+void decay_scan(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& decay, Tensor state, const Tensor& q_starts,
+                const Tensor& seq_state, const Tensor& positions, Tensor out, int64_t H, int64_t K, int64_t V) {
+  const auto ty = act_type(v);
+  TORCH_CHECK(rows_of(q, ty) && rows_of(k, ty) && rows_of(v, ty) && rows_of(out, ty), "activations: rows of one type");
+  TORCH_CHECK(q.size(1) == H * K && k.size(1) == H * K && v.size(1) == H * V && out.size(1) >= H * V && out.size(0) == v.size(0) && decay.numel() == H, "widths");
+  TORCH_CHECK(state.scalar_type() == at::kFloat && state.is_contiguous() && state.dim() == 4 && state.size(1) == H && state.size(2) == V &&
+                  state.size(3) == K, "state: fp32 [slots, H, V, K]");
+  check_batch(q_starts, seq_state, positions);
+  c10::cuda::CUDAGuard guard(v.device());
+  fllm::SsdScanParams p{};
+  p.x = v.data_ptr(), p.Bm = k.data_ptr(), p.Cm = q.data_ptr();
+  p.ldx = v.stride(0), p.ldb = k.stride(0), p.ldc = q.stride(0), p.ldy = out.stride(0);
+  p.A = opt_f32(decay), p.state = state.data_ptr<float>();
+  p.q_starts = q_starts.data_ptr<int>(), p.seq_state = seq_state.data_ptr<int>(), p.positions = positions.data_ptr<int>(), p.y = out.data_ptr();
+  p.B = (int)seq_state.numel(), p.tokens = (int)v.size(0), p.H = (int)H, p.P = (int)V, p.G = (int)H, p.N = (int)K;
+  p.f32 = ty == at::kFloat ? 1 : 0;
+  const int rc = fllm::ssd_scan(p, cur_stream());
+  TORCH_CHECK(rc == 0, "decay_scan: unsupported arguments (code ", rc, "): key width up to 256");
+}
+
 void mamba1_scan(const Tensor& x, const Tensor& dt, const Tensor& Bm, const Tensor& Cm, const optional<Tensor>& z, const Tensor& A,
                  const optional<Tensor>& D, const optional<Tensor>& dt_bias, Tensor state, const Tensor& q_starts, const Tensor& seq_state,
                  const Tensor& positions, Tensor y, int64_t seg_len, int64_t segs, const optional<Tensor>& seg_scratch) {
@@ -134,14 +155,15 @@ void matrix_state_scan(int64_t kind, const Tensor& r, const Tensor& k, const Ten
   TORCH_CHECK(rc == 0, "matrix_state_scan: unsupported arguments (code ", rc, "): key width up to 256 (kind 2), 32 / 64 / 128 / 256 with 16-byte aligned bf16 rows (other kinds)");
 }
 
-void gated_rmsnorm(const Tensor& x, const optional<Tensor>& z, const Tensor& w, Tensor y, int64_t group_size, double eps, bool norm_before_gate) {
+void gated_rmsnorm(const Tensor& x, const optional<Tensor>& z, const Tensor& w, Tensor y, int64_t group_size, double eps, bool norm_before_gate,
+                   bool sigmoid_gate) {
   const auto ty = act_type(x);
   TORCH_CHECK(rows_of(x, ty) && rows_of(y, ty) && x.sizes() == y.sizes(), "x, y: rows of one shape and type");
   TORCH_CHECK(w.scalar_type() == ty && w.is_contiguous() && x.size(1) % group_size == 0, "w: like x; D a multiple of the group");
   TORCH_CHECK(!z.has_value() || !z->defined() || (rows_of(*z, ty) && z->sizes() == x.sizes()), "z: rows like x");
   c10::cuda::CUDAGuard guard(x.device());
   fllm::gated_rmsnorm(x.data_ptr(), x.stride(0), opt_ptr(z), opt_ld(z), w.data_ptr(), (int)w.numel(), y.data_ptr(), y.stride(0), (int)x.size(0),
-                      (int)x.size(1), (int)group_size, (float)eps, norm_before_gate ? 1 : 0, cur_stream(), ty == at::kFloat ? 1 : 0);
+                      (int)x.size(1), (int)group_size, (float)eps, norm_before_gate ? 1 : 0, cur_stream(), ty == at::kFloat ? 1 : 0, sigmoid_gate ? 1 : 0);
 }
 
 }  // namespace
@@ -152,6 +174,8 @@ TORCH_LIBRARY_FRAGMENT(fllm_b200, m) {
   m.def("mamba2_scan(Tensor x, Tensor dt, Tensor Bm, Tensor Cm, Tensor A, Tensor? D, Tensor? dt_bias, Tensor(a!) state, Tensor q_starts, "
         "Tensor seq_state, Tensor positions, Tensor(b!) y, int H, int P, int G, int N, float dt_min, float dt_max, int skip_from) -> ()",
         &mamba2_scan);
+  m.def("decay_scan(Tensor q, Tensor k, Tensor v, Tensor decay, Tensor(a!) state, Tensor q_starts, Tensor seq_state, Tensor positions, Tensor(b!) out, "
+        "int H, int K, int V) -> ()", &decay_scan);
   m.def("mamba1_scan(Tensor x, Tensor dt, Tensor Bm, Tensor Cm, Tensor? z, Tensor A, Tensor? D, Tensor? dt_bias, Tensor(a!) state, "
         "Tensor q_starts, Tensor seq_state, Tensor positions, Tensor(b!) y, int seg_len, int segs, Tensor? seg_scratch) -> ()",
         &mamba1_scan);
@@ -159,5 +183,5 @@ TORCH_LIBRARY_FRAGMENT(fllm_b200, m) {
         "Tensor q_starts, Tensor seq_state, Tensor positions, Tensor(b!) y, int H, int DK, int DV, int kv_ratio, bool l2norm, float q_scale, "
         "Tensor? gate_raw, Tensor? gate_A, Tensor? gate_dt_bias) -> ()",
         &matrix_state_scan);
-  m.def("gated_rmsnorm(Tensor x, Tensor? z, Tensor w, Tensor(a!) y, int group_size, float eps, bool norm_before_gate) -> ()", &gated_rmsnorm);
+  m.def("gated_rmsnorm(Tensor x, Tensor? z, Tensor w, Tensor(a!) y, int group_size, float eps, bool norm_before_gate, bool sigmoid_gate=False) -> ()", &gated_rmsnorm);
 }

@@ -1,5 +1,4 @@
-// torch.ops.fllm_b200 bindings of attention whose values are the keys (attention_tied.cu) and of the residual with the norm
-// after the sum (postnorm.cu).
+// torch.ops.fllm_b200 bindings of attention whose values are the keys (attention_tied.cu).
 #include <ATen/ATen.h>
 #include <c10/cuda/CUDAGuard.h>
 #include <c10/cuda/CUDAStream.h>
@@ -96,70 +95,6 @@ int64_t attention_tied(const Tensor& q, const Tensor& q_factor, const Tensor& ca
   c10::cuda::CUDAGuard guard(q.device());
   return fllm::attention_tied(p, (int)splits, ws, ws_bytes, tensor_cores, given(status) ? status->data_ptr<int>() : nullptr, cur_stream());
 }
-
-// x fp32 [rows, ld]. Start: ids + table. Otherwise y [rows, ld] or, with splits > 0, its split-K partial sums in `workspace`.
-void postnorm(Tensor x, const optional<Tensor>& ids, const optional<Tensor>& table, double scale, const optional<Tensor>& y,
-              const optional<Tensor>& workspace, int64_t splits, bool add, double alpha, const optional<Tensor>& norm_w, const optional<Tensor>& final_w,
-              double final_scale, const optional<Tensor>& rows, Tensor h, int64_t width, double eps, bool write) {
-  const auto ty = act_type(h);
-  TORCH_CHECK(f32(x) && x.dim() == 2, "x: contiguous fp32 [rows, ld]");
-  const int64_t n = x.size(0), ld = x.size(1);
-  TORCH_CHECK(rows_of(h, ty) && h.size(1) == ld, "h: rows of the residual's padded width");
-  auto vec = [&](const optional<Tensor>& t) -> const void* {
-    TORCH_CHECK(t->scalar_type() == ty && t->is_cuda() && t->is_contiguous() && t->numel() == ld, "norm weights: the padded width, like h");
-    return t->data_ptr();
-  };
-  fllm::PostNormParams p{};
-  p.x = x.data_ptr<float>();
-  if (given(ids)) {
-    TORCH_CHECK(i32(*ids) && ids->numel() == n && given(table) && rows_of(*table, ty) && table->size(1) == ld, "ids int32 [rows], table [vocab, ld]");
-    p.ids = ids->data_ptr<int>(), p.table = table->data_ptr(), p.vocab = (int)table->size(0), p.ld_table = table->stride(0), p.scale = (float)scale;
-  } else {
-    TORCH_CHECK(given(norm_w), "an update needs a norm weight");
-    p.norm_w = vec(norm_w);
-    if (splits > 0) {
-      p.partials = partial_sums(workspace, splits, n, ld);
-      p.splits = (int)splits, p.plane = n * ld;
-    } else {
-      TORCH_CHECK(given(y) && rows_of(*y, ty) && y->size(0) == n && y->size(1) == ld, "y: [rows, ld] like h");
-      p.y = y->data_ptr(), p.ld_y = y->stride(0);
-    }
-  }
-  p.n_out = (int)n;
-  if (given(rows)) {
-    TORCH_CHECK(i32(*rows) && !write, "rows: int32; a selection of rows does not update the residual");
-    p.rows = rows->data_ptr<int>(), p.n_out = (int)rows->numel();
-  }
-  TORCH_CHECK(h.size(0) == p.n_out, "h: one row per output");
-  if (given(final_w)) p.final_w = vec(final_w);
-  p.add = add ? 1 : 0, p.alpha = (float)alpha, p.final_scale = (float)final_scale;
-  p.h = h.data_ptr(), p.ld_h = h.stride(0), p.width = (int)width, p.ld = (int)ld, p.eps = (float)eps;
-  p.write = write ? 1 : 0, p.f32 = ty == at::kFloat ? 1 : 0;
-  c10::cuda::CUDAGuard guard(h.device());
-  fllm::postnorm(p, cur_stream());
-}
-
-// out [T, cols] = gelu_tanh(gate) * table[ids, offset : offset + dim], zeros behind; gate [T, cols] or its split-K partial sums
-void side_gate(const optional<Tensor>& gate, const optional<Tensor>& workspace, int64_t splits, const Tensor& ids, const Tensor& table, int64_t offset,
-               int64_t dim, Tensor out) {
-  const auto ty = act_type(out);
-  TORCH_CHECK(rows_of(out, ty) && rows_of(table, ty) && i32(ids) && ids.numel() >= out.size(0) && offset >= 0 && dim <= out.size(1) &&
-                  offset + dim <= table.size(1), "out [T, cols >= dim], table [vocab, >= offset + dim], ids int32 [T]");
-  fllm::SideGateParams p{};
-  const int64_t T = out.size(0), cols = out.size(1);
-  if (splits > 0) {
-    p.partials = partial_sums(workspace, splits, T, cols);
-    p.splits = (int)splits, p.plane = T * cols;
-  } else {
-    TORCH_CHECK(given(gate) && rows_of(*gate, ty) && gate->size(0) == T && gate->size(1) == cols, "gate: [T, cols]");
-    p.gate = gate->data_ptr(), p.ld_gate = gate->stride(0);
-  }
-  p.ids = ids.data_ptr<int>(), p.table = table.data_ptr(), p.vocab = (int)table.size(0), p.ld_table = table.stride(0);
-  p.offset = (int)offset, p.dim = (int)dim, p.cols = (int)cols, p.tokens = (int)T;
-  p.out = out.data_ptr(), p.ld_out = out.stride(0), p.f32 = ty == at::kFloat ? 1 : 0;
-  c10::cuda::CUDAGuard guard(out.device());
-  fllm::side_gate(p, cur_stream());
-}
 }  // namespace
 
 TORCH_LIBRARY_FRAGMENT(fllm_b200, m) {
@@ -170,7 +105,4 @@ TORCH_LIBRARY_FRAGMENT(fllm_b200, m) {
   m.def("attention_tied(Tensor q, Tensor q_factor, Tensor cache, Tensor key_factor, int dim, Tensor block_tables, Tensor row_seq, Tensor positions, "
         "Tensor q_starts, Tensor(a!) out, int num_seqs, int max_q_len, int min_q_len, float softcap, int splits, Tensor? workspace, bool tensor_cores, "
         "Tensor? status) -> int", &attention_tied);
-  m.def("postnorm(Tensor(a!) x, Tensor? ids, Tensor? table, float scale, Tensor? y, Tensor? workspace, int splits, bool add, float alpha, Tensor? norm_w, "
-        "Tensor? final_w, float final_scale, Tensor? rows, Tensor(b!) h, int width, float eps, bool write) -> ()", &postnorm);
-  m.def("side_gate(Tensor? gate, Tensor? workspace, int splits, Tensor ids, Tensor table, int offset, int dim, Tensor(a!) out) -> ()", &side_gate);
 }

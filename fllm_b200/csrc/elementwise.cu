@@ -657,23 +657,29 @@ void gather_rows_bf16(const void* x, long long ldx, const int* rows, void* out, 
 
 // ---- logit soft-cap: x = cap * tanh(x / cap), in place over bf16 rows (Gemma-2 final logits; the reference keeps it with
 // its small architecture ops in rust/engine/cuda/arch_ops.cu) -------------------------------------------------------
-__global__ void softcap_rows_kernel(__nv_bfloat16* __restrict__ x, long long ldx, int cols, float cap, float inv_cap) {
-  __nv_bfloat16* row = x + (size_t)blockIdx.y * ldx;
+template <typename T>
+__global__ void softcap_rows_kernel(T* __restrict__ x, long long ldx, int cols, float cap, float inv_cap) {
+  T* row = x + (size_t)blockIdx.y * ldx;
+  auto capped = [&](float v) { return cap * tanhf(v * inv_cap); };
   for (int c = (blockIdx.x * blockDim.x + threadIdx.x) * 2; c < cols; c += gridDim.x * blockDim.x * 2) {
-    if (c + 1 < cols) {
+    if constexpr (sizeof(T) == 4) {
+      row[c] = capped(row[c]);
+      if (c + 1 < cols) row[c + 1] = capped(row[c + 1]);
+    } else if (c + 1 < cols) {
       const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(row + c));
-      *reinterpret_cast<__nv_bfloat162*>(row + c) = __floats2bfloat162_rn(cap * tanhf(v.x * inv_cap), cap * tanhf(v.y * inv_cap));
+      *reinterpret_cast<__nv_bfloat162*>(row + c) = __floats2bfloat162_rn(capped(v.x), capped(v.y));
     } else {
-      row[c] = __float2bfloat16(cap * tanhf(__bfloat162float(row[c]) * inv_cap));
+      row[c] = __float2bfloat16(capped(__bfloat162float(row[c])));
     }
   }
 }
 
-void softcap_rows_bf16(void* x, long long ldx, int rows, int cols, float cap, cudaStream_t s) {
+void softcap_rows(void* x, long long ldx, int rows, int cols, float cap, int f32, cudaStream_t s) {
   if (rows <= 0 || cols <= 0) return;
-  if ((ldx & 1) || (reinterpret_cast<uintptr_t>(x) & 3)) throw std::runtime_error("softcap_rows_bf16: even leading dimension, 4-byte aligned rows");
-  const int bx = std::min((cols / 2 + 255) / 256, 64);
-  softcap_rows_kernel<<<dim3(std::max(bx, 1), rows), 256, 0, s>>>((__nv_bfloat16*)x, ldx, cols, cap, 1.f / cap);
+  if (!f32 && ((ldx & 1) || (reinterpret_cast<uintptr_t>(x) & 3))) throw std::runtime_error("softcap_rows: even leading dimension, 4-byte aligned rows");
+  const dim3 grid(std::max(std::min((cols / 2 + 255) / 256, 64), 1), rows);
+  if (f32) softcap_rows_kernel<float><<<grid, 256, 0, s>>>((float*)x, ldx, cols, cap, 1.f / cap);
+  else softcap_rows_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>((__nv_bfloat16*)x, ldx, cols, cap, 1.f / cap);
   cuda_check(cudaGetLastError(), "softcap_rows_kernel");
 }
 

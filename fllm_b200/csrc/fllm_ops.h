@@ -170,14 +170,19 @@ int moe_grouped_linear_bf16(const void* xp, long long ldx, const void* w_stack, 
 // score-weighted routers (score_kind 1 softmax over all experts, 2 sigmoid; selection on score + select_bias; optional renormalisation; scale)
 void moe_route_scored(const void* logits, long long ld, const float* select_bias, int tokens, int experts, int k, int score_kind,
                       int renorm, float scale, int* ids, float* weights, cudaStream_t s);
+// the same rule (without a selection bias) on fp32 logits: the sum of `splits` planes of [tokens][ld], `plane` elements each
+void moe_route_fp32(const float* logits, int splits, long long plane, long long ld, int tokens, int experts, int k, int score_kind, int renorm,
+                    float scale, int* ids, float* weights, cudaStream_t s);
 void moe_route(const void* logits, long long ld, const void* bias, int tokens, int experts, int k, int softmax_all,
                int* ids, float* weights, cudaStream_t s);
 void moe_align(const int* ids, int tokens, int k, int experts, int expert_lo, int expert_hi, int bn, int* row_of,
                int* token_of, int rows_cap, int* tile_expert, int* tile_row0, int* num_tiles, int max_tiles,
-               cudaStream_t s);
-void moe_gather(const void* x, long long ldx, const int* token_of, void* xp, int rows_cap, int hidden, cudaStream_t s);
+               cudaStream_t s, const float* weights = nullptr, float* row_weight = nullptr);   // row_weight [rows_cap]: weights [tokens * k] by row
+void moe_gather(const void* x, long long ldx, const int* token_of, void* xp, int rows_cap, int hidden, cudaStream_t s,
+                const float* row_weight = nullptr, int f32 = 0);
+// weights null: the rows are summed as they are; add (optional): [tokens] rows added to the result
 void moe_combine(const void* y, long long ldy, const int* row_of, const float* weights, int tokens, int k, void* out,
-                 long long ldo, int hidden, cudaStream_t s);
+                 long long ldo, int hidden, cudaStream_t s, const void* add = nullptr, long long ld_add = 0, int f32 = 0);
 
 // ---- elementwise --------------------------------------------------------------------
 void embed_bf16(const int* ids, const void* table, void* out, int tokens, int hidden, int vocab,
@@ -280,6 +285,7 @@ int causal_conv1d(const void* x, long long ldx, const float* w, const float* bia
                   int tokens, int max_q_len, cudaStream_t stream, int f32 = 0);   // tokens: rows of the step (= B: single tokens);
                                                                                   // max_q_len: host-side bound on a sequence's tokens in it
 // The Mamba-2 recurrence for any head and state width (N <= 256), bf16 or fp32 (recurrent_ssd.cu): one walk per sequence.
+// dt = null: lightning attention, a constant decay A[h] per head, step size 1 and silu on x, Bm and Cm (D, dt_bias unused).
 struct SsdScanParams {
   const void *x, *dt, *Bm, *Cm;
   long long ldx, lddt, ldb, ldc, ldy;
@@ -308,7 +314,7 @@ int matrix_state_scan(int kind, const void* r, long long ldr, const void* k, lon
                       float q_scale, const void* gate_raw, long long ldgate, const float* gate_A, const float* gate_dt_bias,
                       int tokens, cudaStream_t stream, int f32 = 0);   // tokens: rows of the step (= B: single tokens)
 void gated_rmsnorm(const void* x, long long ldx, const void* z, long long ldz, const void* w, int wlen, void* y, long long ldy, int T,
-                   int D, int group_size, float eps, int norm_before_gate, cudaStream_t stream, int f32 = 0);
+                   int D, int group_size, float eps, int norm_before_gate, cudaStream_t stream, int f32 = 0, int sigmoid_gate = 0);   // gate: silu(z) or sigmoid(z)
 
 // Latent attention (attention_mla.cu). Element (t, h, e) of the absorbed query part sits at q_abs[t * qa_t + h * qa_h + e]
 // (e < 512), the rotated part in q_pe [tokens][H][64]; cache [blocks][block_size][576] = latent | rotated key part; output
@@ -329,8 +335,8 @@ void mla_prepare_bf16(const void* ckv, long long ldc, const void* q, long long l
                       const int* positions, const int* slots, const float* inv_freq, float attn_factor, const void* norm_w, float eps,
                       void* cache, void* q_pe, int tokens, int H, cudaStream_t s);
 
-// x = cap * tanh(x / cap) in place over bf16 rows
-void softcap_rows_bf16(void* x, long long ldx, int rows, int cols, float cap, cudaStream_t s);
+// x = cap * tanh(x / cap) in place over rows of bf16, or fp32 with f32 = 1
+void softcap_rows(void* x, long long ldx, int rows, int cols, float cap, int f32, cudaStream_t s);
 
 // x += delta (in place, delta may be null), y = LayerNorm(x) * (w + w_offset) + b (b may be null)
 void add_layernorm_bf16(void* x, long long ldx, const void* delta, long long ldd, const void* w, const void* b, void* y, long long ldy,
@@ -446,6 +452,48 @@ int attention_tied_splits(int num_seqs, int max_q_len, int H, int G, int max_kv_
 size_t attention_tied_workspace_bytes(int tokens, int H, int W, int splits);
 int attention_tied(const TiedAttnParams& p, int splits, void* workspace, size_t workspace_bytes, bool tensor_cores, int* status, cudaStream_t s);
 
+// ---- attention of one or two maps over shared values (attention_maps.cu) -----------------------------------------------
+struct MapsPrepareParams {
+  const void* x;               // [tokens] rows: query maps from column q_offset, key maps from k_offset, values from v_offset
+  long long ldx;
+  const float* partials;       // not null: the rows are the sums of split-K partials [splits][tokens][width] (plus bias), `plane` elements per split
+  int splits, width;
+  long long plane;
+  const void* bias;            // [width], with partials only
+  int q_offset, k_offset, v_offset, q_heads, k_heads, v_heads, dim, v_dim, wk, wv, block_size, tokens;
+  const int *positions, *slots;
+  const float* inv_freq;       // [rot / 2]: pairs (i, i + rot / 2) of a map's first rot values turn
+  int rot;
+  float rope_factor;           // on cosine and sine
+  const void *q_norm, *k_norm; // [dim], or with full [heads * dim]
+  int full;                    // 1: one root mean square over all maps, 0: one per map
+  float eps;
+  void* q_out;                 // [tokens][q_heads][wk]
+  void *k_cache, *v_cache;     // [blocks][k_heads][block_size][wk], [blocks][v_heads][block_size][wv]
+  int f32;
+  int vec;                     // set by maps_prepare: rows move four values at a time
+};
+void maps_prepare(const MapsPrepareParams& p, cudaStream_t s);
+struct MapsAttnParams {
+  const void* q;               // [tokens][H * maps][wk]
+  const void *k_cache, *v_cache;   // [blocks][G * maps][block_size][wk], [blocks][G][block_size][wv]
+  const int* block_tables;
+  int max_blocks;
+  const int *row_seq, *positions, *q_starts;
+  void* out;                   // head h of token t at out[t * ldo + h * v_dim]
+  long long ldo;
+  int tokens, num_seqs, max_q_len, min_q_len, H, G, maps, dim, v_dim, wk, wv, block_size;
+  long long num_blocks;
+  float scale;
+  int window;                  // keys a query sees, itself included (0: all)
+  float lam, out_scale, eps;   // two maps: out = rms(a1 - lam a2) * out_scale
+  int f32;
+};
+bool attention_maps_tc_supported(int wk, int wv, int block_size, int f32);
+int attention_maps_splits(int num_seqs, int max_q_len, int H, int G, int maps, int max_kv_len, int window);
+size_t attention_maps_workspace_bytes(int tokens, int q_heads, int wv, int splits);
+int attention_maps(const MapsAttnParams& p, int splits, void* workspace, size_t workspace_bytes, bool tensor_cores, int* status, cudaStream_t s);
+
 // ---- residual with the norm after the sum, per-layer token input (postnorm.cu) -------------------------------------------
 struct PostNormParams {
   float* x;                    // [rows][ld] fp32, zero beyond `width`
@@ -459,6 +507,9 @@ struct PostNormParams {
   const float* partials;
   int splits;
   long long plane;
+  const void* pair_a;          // not null: what is added is (rms(pair_a) pair_wa + rms(y) pair_wb) / 2 in place of y
+  long long ld_pair;
+  const void *pair_wa, *pair_wb;
   int add;                     // 0: x <- rms(alpha x + y) w;  1: x <- x + rms(y) w
   float alpha;
   const void* norm_w;
@@ -496,5 +547,8 @@ struct GemmF32Params {
   int batch, T, N, K;
 };
 void gemm_f32(const GemmF32Params& p, cudaStream_t s);
+// Mixture of experts over a device-built tile list of 64-row tiles: b is the stack of matrices [experts][N][K] (b_b between them),
+// tile i multiplies rows tile_row0[i] ... of a with matrix tile_expert[i]
+void moe_grouped_f32(const GemmF32Params& p, const int* tile_expert, const int* tile_row0, const int* num_tiles, int max_tiles, cudaStream_t s);
 
 }  // namespace fllm

@@ -1,6 +1,7 @@
 // True fp32 matrix products on the CUDA cores (no reduced-precision tensor mode), for models served in 32-bit:
 // C[b][t][n] = sum_k A[b][t][k] B[b][n][k] (+ bias[n]) with arbitrary strides, so the same kernel is the linear layer
 // (B = weight rows) and the batched per-head products. 64 x 64 tiles, 4 x 4 results per thread, K in steps of 16.
+// Grouped form (mixture of experts): the row tiles come from a list built on the device, each with a matrix of its own.
 #include <cuda_runtime.h>
 
 #include <stdexcept>
@@ -12,11 +13,17 @@ namespace fllm {
 namespace {
 constexpr int TM = 64, TN = 64, TK = 16;
 
-__global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Params p) {
+struct TileList {
+  const int *expert, *row0, *count;
+};
+
+template <bool GROUPED>
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Params p, const TileList g) {
   __shared__ float As[TK][TM + 4], Bs[TK][TN + 4];
-  const int t0 = blockIdx.y * TM, n0 = blockIdx.x * TN, tid = threadIdx.x;
+  if (GROUPED && (int)blockIdx.y >= *g.count) return;
+  const int t0 = GROUPED ? g.row0[blockIdx.y] : blockIdx.y * TM, n0 = blockIdx.x * TN, tid = threadIdx.x;
   const float* A = p.a + (long long)blockIdx.z * p.a_b;
-  const float* B = p.b + (long long)blockIdx.z * p.b_b;
+  const float* B = p.b + (long long)(GROUPED ? g.expert[blockIdx.y] : blockIdx.z) * p.b_b;
   const int tx = tid % 16, ty = tid / 16;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < p.K; k0 += TK) {
@@ -59,8 +66,15 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Params p) {
 void gemm_f32(const GemmF32Params& p, cudaStream_t s) {
   if (p.T <= 0 || p.N <= 0 || p.batch <= 0) return;
   if ((p.T + TM - 1) / TM > 65535 || p.batch > 65535) throw std::runtime_error("gemm_f32: too many rows for one launch");
-  gemm_f32_kernel<<<dim3((p.N + TN - 1) / TN, (p.T + TM - 1) / TM, p.batch), 256, 0, s>>>(p);
+  gemm_f32_kernel<false><<<dim3((p.N + TN - 1) / TN, (p.T + TM - 1) / TM, p.batch), 256, 0, s>>>(p, TileList{});
   cuda_check(cudaGetLastError(), "gemm_f32_kernel");
+}
+
+void moe_grouped_f32(const GemmF32Params& p, const int* tile_expert, const int* tile_row0, const int* num_tiles, int max_tiles, cudaStream_t s) {
+  if (p.T <= 0 || p.N <= 0 || max_tiles <= 0) return;
+  if (max_tiles > 65535) throw std::runtime_error("moe_grouped_f32: too many row tiles for one launch");
+  gemm_f32_kernel<true><<<dim3((p.N + TN - 1) / TN, max_tiles, 1), 256, 0, s>>>(p, TileList{tile_expert, tile_row0, num_tiles});
+  cuda_check(cudaGetLastError(), "moe_grouped_f32");
 }
 
 }  // namespace fllm

@@ -6,7 +6,8 @@
 //   moe_align_kernel    one CTA: count rows per expert, lay the experts' row segments out back to
 //                       back, each padded to the token-tile width, and emit the tile list
 //                       (expert, first row) that the grouped GEMM walks; sizes stay on the device
-//                       so the whole layer can live in a CUDA graph;
+//                       so the whole layer can live in a CUDA graph; optionally each row's routing
+//                       weight;
 //   moe_gather_kernel   permuted activations xp[row] = x[token(row)] (zero rows for padding);
 //   moe_combine_kernel  out[token] = sum_j weight[token, j] * y[row(token, j)] in slot order, so
 //                       the result does not depend on scheduling.
@@ -80,19 +81,38 @@ __global__ void moe_route_kernel(const __nv_bfloat16* __restrict__ logits, long 
 // Routers that weigh experts by their score: score = softmax over all experts (score_kind 1) or sigmoid (2) of the logit; the
 // k experts with the largest score + select_bias are taken (the bias only steers the choice: DeepSeek-V3, GLM-4.5, ERNIE 4.5);
 // weights = the scores of the chosen experts, renormalised on request, times `scale`. One warp per token, up to 256 experts.
-__global__ void moe_route_scored_kernel(const __nv_bfloat16* __restrict__ logits, long long ld, const float* __restrict__ select_bias,
-                                        int tokens, int experts, int k, int score_kind, int renorm, float scale, int* __restrict__ ids,
-                                        float* __restrict__ weights) {
+// Logits: bf16, or (Sum) fp32 as the sum of planes, then with the accurate exponential.
+struct Bf16Logits {
+  const __nv_bfloat16* p;
+  long long ld;
+  static constexpr bool kAccurate = false;
+  __device__ __forceinline__ float operator()(int t, int e) const { return __bfloat162float(p[(size_t)t * ld + e]); }
+};
+struct SumLogits {
+  const float* p;
+  long long ld, plane;
+  int splits;
+  static constexpr bool kAccurate = true;
+  __device__ __forceinline__ float operator()(int t, int e) const {
+    float v = 0.f;
+    for (int s = 0; s < splits; ++s) v += __ldcg(p + s * plane + (size_t)t * ld + e);
+    return v;
+  }
+};
+template <typename Logits>
+__global__ void moe_route_scored_kernel(const Logits logits, const float* __restrict__ select_bias, int tokens, int experts, int k,
+                                        int score_kind, int renorm, float scale, int* __restrict__ ids, float* __restrict__ weights) {
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (t >= tokens) return;
   constexpr int MAXPL = 8;
+  auto ex = [](float x) { return Logits::kAccurate ? expf(x) : __expf(x); };
   float sc[MAXPL], ch[MAXPL];
   float vmax = -INFINITY;
 #pragma unroll
   for (int i = 0; i < MAXPL; ++i) {
     const int e = lane + 32 * i;
-    sc[i] = e < experts ? __bfloat162float(logits[(size_t)t * ld + e]) : -INFINITY;
+    sc[i] = e < experts ? logits(t, e) : -INFINITY;
     vmax = fmaxf(vmax, sc[i]);
   }
   if (score_kind == 1) {
@@ -100,7 +120,7 @@ __global__ void moe_route_scored_kernel(const __nv_bfloat16* __restrict__ logits
     float den = 0.f;
 #pragma unroll
     for (int i = 0; i < MAXPL; ++i) {
-      sc[i] = sc[i] == -INFINITY ? 0.f : __expf(sc[i] - vmax);
+      sc[i] = sc[i] == -INFINITY ? 0.f : ex(sc[i] - vmax);
       den += sc[i];
     }
     den = warp_sum(den);
@@ -108,7 +128,7 @@ __global__ void moe_route_scored_kernel(const __nv_bfloat16* __restrict__ logits
     for (int i = 0; i < MAXPL; ++i) sc[i] /= den;
   } else {
 #pragma unroll
-    for (int i = 0; i < MAXPL; ++i) sc[i] = sc[i] == -INFINITY ? 0.f : 1.f / (1.f + __expf(-sc[i]));
+    for (int i = 0; i < MAXPL; ++i) sc[i] = sc[i] == -INFINITY ? 0.f : 1.f / (1.f + ex(-sc[i]));
   }
 #pragma unroll
   for (int i = 0; i < MAXPL; ++i) {
@@ -150,9 +170,18 @@ void moe_route_scored(const void* logits, long long ld, const float* select_bias
                       int renorm, float scale, int* ids, float* weights, cudaStream_t s) {
   if (tokens <= 0) return;
   if (experts > 256 || k > 8 || (score_kind != 1 && score_kind != 2)) throw std::runtime_error("moe_route_scored: at most 256 experts, top-8, score kind 1 or 2");
-  moe_route_scored_kernel<<<(tokens + 3) / 4, 128, 0, s>>>((const __nv_bfloat16*)logits, ld, select_bias, tokens, experts, k, score_kind,
-                                                           renorm, scale, ids, weights);
+  moe_route_scored_kernel<<<(tokens + 3) / 4, 128, 0, s>>>(Bf16Logits{(const __nv_bfloat16*)logits, ld}, select_bias, tokens, experts, k,
+                                                           score_kind, renorm, scale, ids, weights);
   cuda_check(cudaGetLastError(), "moe_route_scored_kernel");
+}
+
+void moe_route_fp32(const float* logits, int splits, long long plane, long long ld, int tokens, int experts, int k, int score_kind, int renorm,
+                    float scale, int* ids, float* weights, cudaStream_t s) {
+  if (tokens <= 0) return;
+  if (experts > 256 || k > 8 || (score_kind != 1 && score_kind != 2)) throw std::runtime_error("moe_route_fp32: at most 256 experts, top-8, score kind 1 or 2");
+  moe_route_scored_kernel<<<(tokens + 3) / 4, 128, 0, s>>>(SumLogits{logits, ld, plane, splits}, (const float*)nullptr, tokens, experts, k, score_kind,
+                                                           renorm, scale, ids, weights);
+  cuda_check(cudaGetLastError(), "moe_route_fp32");
 }
 
 void moe_route(const void* logits, long long ld, const void* bias, int tokens, int experts, int k, int softmax_all,
@@ -172,7 +201,8 @@ __global__ void __launch_bounds__(1024) moe_align_kernel(const int* __restrict__
                                                          int* __restrict__ row_of, int* __restrict__ token_of,
                                                          int rows_cap, int* __restrict__ tile_expert,
                                                          int* __restrict__ tile_row0, int* __restrict__ num_tiles,
-                                                         int max_tiles, int staged) {
+                                                         int max_tiles, int staged, const float* __restrict__ weights,
+                                                         float* __restrict__ row_weight) {
   __shared__ int cnt[512], off[513], fill[512];
   extern __shared__ int ids_s[];              // the first `staged` ids: the per-expert scans below read them from here
   for (int e = threadIdx.x; e < 512; e += blockDim.x) { cnt[e] = 0; fill[e] = 0; }
@@ -218,7 +248,10 @@ __global__ void __launch_bounds__(1024) moe_align_kernel(const int* __restrict__
         if (valid) {
           const int pos = off[e] + fill[e] + __popc(same & ((1u << lane) - 1u));
           row_of[i] = pos;
-          if (pos < rows_cap) token_of[pos] = i / k;
+          if (pos < rows_cap) {
+            token_of[pos] = i / k;
+            if (row_weight) row_weight[pos] = weights[i];
+          }
         }
         __syncwarp();
         if (valid && lane == __ffs(same) - 1) fill[e] += __popc(same);
@@ -231,66 +264,87 @@ __global__ void __launch_bounds__(1024) moe_align_kernel(const int* __restrict__
 
 void moe_align(const int* ids, int tokens, int k, int experts, int expert_lo, int expert_hi, int bn, int* row_of,
                int* token_of, int rows_cap, int* tile_expert, int* tile_row0, int* num_tiles, int max_tiles,
-               cudaStream_t s) {
+               cudaStream_t s, const float* weights, float* row_weight) {
   if (expert_hi - expert_lo > 512) throw std::runtime_error("moe_align: at most 512 local experts");
   const int staged = std::min(tokens * k, 10240);              // 40 KiB of dynamic shared memory at most
   moe_align_kernel<<<1, 1024, (size_t)staged * sizeof(int), s>>>(ids, tokens * k, experts, expert_lo, expert_hi, bn, k, row_of, token_of,
-                                                                 rows_cap, tile_expert, tile_row0, num_tiles, max_tiles, staged);
+                                                                 rows_cap, tile_expert, tile_row0, num_tiles, max_tiles, staged, weights, row_weight);
   cuda_check(cudaGetLastError(), "moe_align_kernel");
 }
 
-__global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const int* __restrict__ token_of,
-                                  __nv_bfloat16* __restrict__ xp, int hidden) {
+// four values of a row as fp32
+__device__ __forceinline__ float4 row4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 row4(const __nv_bfloat16* p) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void put4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put4(__nv_bfloat16* p, const float4& v) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+}
+
+// row_weight (optional): routers that weigh an expert's input
+template <typename T>
+__global__ void moe_gather_kernel(const T* __restrict__ x, long long ldx, const int* __restrict__ token_of, const float* __restrict__ row_weight,
+                                  T* __restrict__ xp, int hidden) {
+  constexpr int V = 16 / sizeof(T);
   const int row = blockIdx.x;
   const int t = token_of[row];
   uint4* dst = reinterpret_cast<uint4*>(xp + (size_t)row * hidden);
   if (t < 0) {
-    for (int i = threadIdx.x; i < hidden / 8; i += blockDim.x) dst[i] = make_uint4(0, 0, 0, 0);
+    for (int i = threadIdx.x; i < hidden / V; i += blockDim.x) dst[i] = make_uint4(0, 0, 0, 0);
     return;
   }
-  const uint4* src = reinterpret_cast<const uint4*>(x + (size_t)t * ldx);
-  for (int i = threadIdx.x; i < hidden / 8; i += blockDim.x) dst[i] = src[i];
+  const T* src = x + (size_t)t * ldx;
+  if (row_weight != nullptr) {
+    const float w = row_weight[row];
+    for (int i = threadIdx.x; i < hidden / 4; i += blockDim.x) {
+      const float4 v = row4(src + 4 * i);
+      put4(xp + (size_t)row * hidden + 4 * i, make_float4(v.x * w, v.y * w, v.z * w, v.w * w));
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < hidden / V; i += blockDim.x) dst[i] = reinterpret_cast<const uint4*>(src)[i];
 }
 
-void moe_gather(const void* x, long long ldx, const int* token_of, void* xp, int rows_cap, int hidden, cudaStream_t s) {
+void moe_gather(const void* x, long long ldx, const int* token_of, void* xp, int rows_cap, int hidden, cudaStream_t s, const float* row_weight, int f32) {
   if (rows_cap <= 0) return;
-  moe_gather_kernel<<<rows_cap, 128, 0, s>>>((const __nv_bfloat16*)x, ldx, token_of, (__nv_bfloat16*)xp, hidden);
+  if (f32) moe_gather_kernel<float><<<rows_cap, 128, 0, s>>>((const float*)x, ldx, token_of, row_weight, (float*)xp, hidden);
+  else moe_gather_kernel<__nv_bfloat16><<<rows_cap, 128, 0, s>>>((const __nv_bfloat16*)x, ldx, token_of, row_weight, (__nv_bfloat16*)xp, hidden);
   cuda_check(cudaGetLastError(), "moe_gather_kernel");
 }
 
-__global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, long long ldy, const int* __restrict__ row_of,
-                                   const float* __restrict__ weights, int k, __nv_bfloat16* __restrict__ out,
-                                   long long ldo, int hidden) {
+// weights (optional; none: the rows are summed as they are), add (optional): rows added to the result
+template <typename T>
+__global__ void moe_combine_kernel(const T* __restrict__ y, long long ldy, const int* __restrict__ row_of, const float* __restrict__ weights, int k,
+                                   const T* __restrict__ add, long long ld_add, T* __restrict__ out, long long ldo, int hidden) {
   const int t = blockIdx.x;
-  for (int i = threadIdx.x; i < hidden / 8; i += blockDim.x) {
-    float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  for (int i = threadIdx.x; i < hidden / 4; i += blockDim.x) {
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int j = 0; j < k; ++j) {
       const int row = row_of[(size_t)t * k + j];
       if (row < 0) continue;                                  // expert lives on another rank
-      const float w = weights[(size_t)t * k + j];
-      const uint4 v = reinterpret_cast<const uint4*>(y + (size_t)row * ldy)[i];
-      const uint32_t* vw = reinterpret_cast<const uint32_t*>(&v);
-#pragma unroll
-      for (int q = 0; q < 4; ++q) {
-        const float2 f = unpack_bf16x2(vw[q]);
-        acc[2 * q] += w * f.x;
-        acc[2 * q + 1] += w * f.y;
-      }
+      const float w = weights != nullptr ? weights[(size_t)t * k + j] : 1.f;
+      const float4 v = row4(y + (size_t)row * ldy + 4 * i);
+      acc.x += w * v.x, acc.y += w * v.y, acc.z += w * v.z, acc.w += w * v.w;
     }
-    uint4 o;
-    o.x = pack_bf16x2(acc[0], acc[1]);
-    o.y = pack_bf16x2(acc[2], acc[3]);
-    o.z = pack_bf16x2(acc[4], acc[5]);
-    o.w = pack_bf16x2(acc[6], acc[7]);
-    reinterpret_cast<uint4*>(out + (size_t)t * ldo)[i] = o;
+    if (add != nullptr) {
+      const float4 v = row4(add + (size_t)t * ld_add + 4 * i);
+      acc.x += v.x, acc.y += v.y, acc.z += v.z, acc.w += v.w;
+    }
+    put4(out + (size_t)t * ldo + 4 * i, acc);
   }
 }
 
 void moe_combine(const void* y, long long ldy, const int* row_of, const float* weights, int tokens, int k, void* out,
-                 long long ldo, int hidden, cudaStream_t s) {
+                 long long ldo, int hidden, cudaStream_t s, const void* add, long long ld_add, int f32) {
   if (tokens <= 0) return;
-  moe_combine_kernel<<<tokens, 128, 0, s>>>((const __nv_bfloat16*)y, ldy, row_of, weights, k, (__nv_bfloat16*)out, ldo,
-                                            hidden);
+  if (f32)
+    moe_combine_kernel<float><<<tokens, 128, 0, s>>>((const float*)y, ldy, row_of, weights, k, (const float*)add, ld_add, (float*)out, ldo, hidden);
+  else
+    moe_combine_kernel<__nv_bfloat16><<<tokens, 128, 0, s>>>((const __nv_bfloat16*)y, ldy, row_of, weights, k, (const __nv_bfloat16*)add, ld_add,
+                                                              (__nv_bfloat16*)out, ldo, hidden);
   cuda_check(cudaGetLastError(), "moe_combine_kernel");
 }
 

@@ -3,7 +3,8 @@
 //   start      x = table[id] * scale
 //   norm sum   x <- rms(alpha x + y) w                 a block whose norm follows the residual sum
 //   add norm   x <- x + rms(y) w                       an output that is normalised before it is added
-// where rms(v) = v / sqrt(mean v^2 + eps). Behind it the row goes on to the next projection, rounded to the activation type, or
+// where rms(v) = v / sqrt(mean v^2 + eps). y may itself be half the sum of two projections, each normalised with a weight of its
+// own (PAIR): y = (rms(a) wa + rms(b) wb) / 2. Behind it the row goes on to the next projection, rounded to the activation type, or
 // through a second RMS norm (times a factor) in front of the head, then only for the rows whose logits are wanted.
 //
 // side_gate: g = gelu_tanh(gate) * e with e a slice of the token's row in a table of per-layer embeddings.
@@ -46,7 +47,16 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return t;
 }
 
-template <typename T, int ITERS>
+__device__ __forceinline__ float2 block_sum2(float a, float b, float2* red) {
+  a = warp_sum(a), b = warp_sum(b);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(a, b);
+  __syncthreads();
+  float2 t = make_float2(0.f, 0.f);
+  for (int i = 0; i < (int)(blockDim.x >> 5); ++i) t.x += red[i].x, t.y += red[i].y;
+  return t;
+}
+
+template <typename T, int ITERS, bool PAIR>
 __global__ void __launch_bounds__(512) postnorm_kernel(const PostNormParams p) {
   __shared__ float red[16];
   pdl_launch_dependents();
@@ -67,8 +77,8 @@ __global__ void __launch_bounds__(512) postnorm_kernel(const PostNormParams p) {
       v[it] = make_float4(e.x * p.scale, e.y * p.scale, e.z * p.scale, e.w * p.scale);
     }
   } else {
-    float4 x[ITERS];
-    float sq = 0.f;
+    float4 x[ITERS], a[PAIR ? ITERS : 1];
+    float sq = 0.f, sqa = 0.f;
 #pragma unroll
     for (int it = 0; it < ITERS; ++it) {
       const int i = threadIdx.x + it * blockDim.x;
@@ -86,9 +96,32 @@ __global__ void __launch_bounds__(512) postnorm_kernel(const PostNormParams p) {
       } else {
         y = load4(static_cast<const T*>(p.y) + (size_t)row * p.ld_y + 4 * i);
       }
+      if constexpr (PAIR) {
+        v[it] = y;
+        a[it] = load4(static_cast<const T*>(p.pair_a) + (size_t)row * p.ld_pair + 4 * i);
+        sqa += dot4(a[it]), sq += dot4(y);
+        continue;
+      }
       if (!p.add) y = make_float4(fmaf(p.alpha, x[it].x, y.x), fmaf(p.alpha, x[it].y, y.y), fmaf(p.alpha, x[it].z, y.z), fmaf(p.alpha, x[it].w, y.w));
       v[it] = y;
       sq += dot4(y);                                       // the padding is zero
+    }
+    if constexpr (PAIR) {
+      __shared__ float2 red2[16];
+      const float2 s2 = block_sum2(sqa, sq, red2);
+      const float ra = 0.5f / sqrtf(s2.x / (float)p.width + p.eps), rb = 0.5f / sqrtf(s2.y / (float)p.width + p.eps);
+      sq = 0.f;
+#pragma unroll
+      for (int it = 0; it < ITERS; ++it) {
+        const int i = threadIdx.x + it * blockDim.x;
+        if (i >= nvec) continue;
+        const float4 wa = load4(static_cast<const T*>(p.pair_wa) + 4 * i), wb = load4(static_cast<const T*>(p.pair_wb) + 4 * i);
+        float4 y = make_float4(fmaf(a[it].x * ra, wa.x, v[it].x * rb * wb.x), fmaf(a[it].y * ra, wa.y, v[it].y * rb * wb.y),
+                               fmaf(a[it].z * ra, wa.z, v[it].z * rb * wb.z), fmaf(a[it].w * ra, wa.w, v[it].w * rb * wb.w));
+        if (!p.add) y = make_float4(fmaf(p.alpha, x[it].x, y.x), fmaf(p.alpha, x[it].y, y.y), fmaf(p.alpha, x[it].z, y.z), fmaf(p.alpha, x[it].w, y.w));
+        v[it] = y;
+        sq += dot4(y);
+      }
     }
     const float r = 1.f / sqrtf(block_sum(sq, red) / (float)p.width + p.eps);
 #pragma unroll
@@ -130,14 +163,14 @@ __global__ void __launch_bounds__(512) postnorm_kernel(const PostNormParams p) {
   }
 }
 
-template <typename T>
+template <typename T, bool PAIR>
 void run_postnorm(const PostNormParams& p, cudaStream_t s) {
   const int nvec = p.ld / 4, threads = std::min(512, (nvec + 31) / 32 * 32), iters = (nvec + threads - 1) / threads;
   const dim3 grid(p.n_out), block(threads);
-  if (iters <= 1) launch_pdl(postnorm_kernel<T, 1>, grid, block, 0, s, p);
-  else if (iters <= 2) launch_pdl(postnorm_kernel<T, 2>, grid, block, 0, s, p);
-  else if (iters <= 4) launch_pdl(postnorm_kernel<T, 4>, grid, block, 0, s, p);
-  else if (iters <= 8) launch_pdl(postnorm_kernel<T, 8>, grid, block, 0, s, p);
+  if (iters <= 1) launch_pdl(postnorm_kernel<T, 1, PAIR>, grid, block, 0, s, p);
+  else if (iters <= 2) launch_pdl(postnorm_kernel<T, 2, PAIR>, grid, block, 0, s, p);
+  else if (iters <= 4) launch_pdl(postnorm_kernel<T, 4, PAIR>, grid, block, 0, s, p);
+  else if (iters <= 8) launch_pdl(postnorm_kernel<T, 8, PAIR>, grid, block, 0, s, p);
   else throw std::runtime_error("postnorm: rows of at most 16384 values");
   cuda_check(cudaGetLastError(), "postnorm_kernel");
 }
@@ -172,8 +205,14 @@ void postnorm(const PostNormParams& p, cudaStream_t s) {
   if (p.n_out <= 0) return;
   if ((p.ld & 3) || (p.ld_h & 3) || (p.ld_y & 3) || (p.ld_table & 3) || p.width > p.ld || p.width <= 0)
     throw std::runtime_error("postnorm: padded row lengths in multiples of 4");
-  if (p.f32) run_postnorm<float>(p, s);
-  else run_postnorm<bf16>(p, s);
+  if (p.pair_a != nullptr) {
+    if (p.ld_pair & 3) throw std::runtime_error("postnorm: padded row lengths in multiples of 4");
+    if (p.f32) run_postnorm<float, true>(p, s);
+    else run_postnorm<bf16, true>(p, s);
+    return;
+  }
+  if (p.f32) run_postnorm<float, false>(p, s);
+  else run_postnorm<bf16, false>(p, s);
 }
 
 void side_gate(const SideGateParams& p, cudaStream_t s) {

@@ -586,6 +586,11 @@ __global__ void __launch_bounds__(128) delta_decode_kernel(const MatrixStateArgs
 //                                      mode 1  y = rmsnorm(x) * w * silu(z)   (gated delta net: norm first)
 // w has `wlen` entries (D for Mamba-2, the head width when every head shares one weight). One warp per group.
 // y may be x (every element is read and then written by the same thread).
+// mode: bit 0 = the norm comes before the gate, bit 1 = the gate is sigmoid(z) instead of silu(z)
+template <typename T>
+__device__ __forceinline__ float gate_t(float z, int mode) {
+  return ((mode & 2) ? 1.f : z) / (1.f + exp_t<T>(-z));
+}
 template <typename T>
 __global__ void __launch_bounds__(128) gated_rmsnorm_kernel(const T* x, long long ldx, const T* __restrict__ z, long long ldz,
                                                             const T* __restrict__ w, int wlen, T* y, long long ldy, int n_rows, int D,
@@ -601,7 +606,7 @@ __global__ void __launch_bounds__(128) gated_rmsnorm_kernel(const T* x, long lon
   float ss = 0.f;
   for (int i = lane; i < gs; i += 32) {
     float v = ld1(xr + i);
-    if (mode == 0 && zr != nullptr) v *= silu_t<T>(ld1(zr + i));
+    if ((mode & 1) == 0 && zr != nullptr) v *= gate_t<T>(ld1(zr + i), mode);
     ss = fmaf(v, v, ss);
   }
   ss = row_sum<32>(ss);
@@ -609,10 +614,10 @@ __global__ void __launch_bounds__(128) gated_rmsnorm_kernel(const T* x, long lon
   T* yr = y + t * ldy + (long long)g * gs;
   for (int i = lane; i < gs; i += 32) {
     float v = ld1(xr + i);
-    const float gate = zr != nullptr ? silu_t<T>(ld1(zr + i)) : 1.f;
-    if (mode == 0) v *= gate;
+    const float gate = zr != nullptr ? gate_t<T>(ld1(zr + i), mode) : 1.f;
+    if ((mode & 1) == 0) v *= gate;
     v = v * inv * ld1(w + (g * gs + i) % wlen);
-    if (mode == 1) v *= gate;
+    if ((mode & 1)) v *= gate;
     st1(yr + i, v);
   }
 }
@@ -638,18 +643,18 @@ __global__ void __launch_bounds__(THREADS) gated_rmsnorm_wide_kernel(const bf16*
     keep[i] = make_float2(0.f, 0.f);
     if (p < pairs) {
       keep[i] = __bfloat1622float2(xr[p]);
-      if (mode == 0 && zr != nullptr) {
+      if ((mode & 1) == 0 && zr != nullptr) {
         const float2 zz = __bfloat1622float2(zr[p]);
-        keep[i].x *= silu_f(zz.x), keep[i].y *= silu_f(zz.y);
+        keep[i].x *= gate_t<bf16>(zz.x, mode), keep[i].y *= gate_t<bf16>(zz.y, mode);
       }
       ss = fmaf(keep[i].x, keep[i].x, fmaf(keep[i].y, keep[i].y, ss));
     }
   }
   for (int p = threadIdx.x + KEEP * THREADS; p < pairs; p += THREADS) {     // beyond the kept part: read again in the second pass
     float2 v = __bfloat1622float2(xr[p]);
-    if (mode == 0 && zr != nullptr) {
+    if ((mode & 1) == 0 && zr != nullptr) {
       const float2 zz = __bfloat1622float2(zr[p]);
-      v.x *= silu_f(zz.x), v.y *= silu_f(zz.y);
+      v.x *= gate_t<bf16>(zz.x, mode), v.y *= gate_t<bf16>(zz.y, mode);
     }
     ss = fmaf(v.x, v.x, fmaf(v.y, v.y, ss));
   }
@@ -672,9 +677,9 @@ __global__ void __launch_bounds__(THREADS) gated_rmsnorm_wide_kernel(const bf16*
     if (p < pairs) {
       const float2 ww = weight(p);
       float2 v = make_float2(keep[i].x * inv * ww.x, keep[i].y * inv * ww.y);
-      if (mode == 1 && zr != nullptr) {
+      if ((mode & 1) && zr != nullptr) {
         const float2 zz = __bfloat1622float2(zr[p]);
-        v.x *= silu_f(zz.x), v.y *= silu_f(zz.y);
+        v.x *= gate_t<bf16>(zz.x, mode), v.y *= gate_t<bf16>(zz.y, mode);
       }
       yr[p] = __floats2bfloat162_rn(v.x, v.y);
     }
@@ -684,12 +689,12 @@ __global__ void __launch_bounds__(THREADS) gated_rmsnorm_wide_kernel(const bf16*
     float2 gt = make_float2(1.f, 1.f);
     if (zr != nullptr) {
       const float2 zz = __bfloat1622float2(zr[p]);
-      gt = make_float2(silu_f(zz.x), silu_f(zz.y));
+      gt = make_float2(gate_t<bf16>(zz.x, mode), gate_t<bf16>(zz.y, mode));
     }
-    if (mode == 0) v.x *= gt.x, v.y *= gt.y;
+    if ((mode & 1) == 0) v.x *= gt.x, v.y *= gt.y;
     const float2 ww = weight(p);
     v = make_float2(v.x * inv * ww.x, v.y * inv * ww.y);
-    if (mode == 1) v.x *= gt.x, v.y *= gt.y;
+    if ((mode & 1)) v.x *= gt.x, v.y *= gt.y;
     yr[p] = __floats2bfloat162_rn(v.x, v.y);
   }
 }
@@ -834,13 +839,14 @@ int matrix_state_scan(int kind, const void* r, long long ldr, const void* k, lon
 }
 
 void gated_rmsnorm(const void* x, long long ldx, const void* z, long long ldz, const void* w, int wlen, void* y, long long ldy, int T,
-                   int D, int group_size, float eps, int norm_before_gate, cudaStream_t stream, int f32) {
+                   int D, int group_size, float eps, int norm_before_gate, cudaStream_t stream, int f32, int sigmoid_gate) {
   if (T <= 0) return;
+  const int mode = norm_before_gate | (sigmoid_gate << 1);
   const long long items = (long long)T * (D / group_size);
   if (f32) {
     gated_rmsnorm_kernel<float><<<(unsigned)((items + 3) / 4), 128, 0, stream>>>(
         static_cast<const float*>(x), ldx, static_cast<const float*>(z), ldz, static_cast<const float*>(w), wlen, static_cast<float*>(y), ldy, T, D,
-        group_size, eps, norm_before_gate);
+        group_size, eps, mode);
     return;
   }
   const bool pairs_ok = group_size % 2 == 0 && ldx % 2 == 0 && ldy % 2 == 0 && (z == nullptr || ldz % 2 == 0) &&
@@ -848,13 +854,13 @@ void gated_rmsnorm(const void* x, long long ldx, const void* z, long long ldz, c
                         (reinterpret_cast<uintptr_t>(z) & 3) == 0;
   auto go = [&](auto kernel, unsigned grid, unsigned threads) {
     launch_pdl(kernel, dim3(grid), dim3(threads), 0, stream, static_cast<const bf16*>(x), ldx, static_cast<const bf16*>(z), ldz, static_cast<const bf16*>(w), wlen,
-               static_cast<bf16*>(y), ldy, D, group_size, eps, norm_before_gate);
+               static_cast<bf16*>(y), ldy, D, group_size, eps, mode);
   };
   if (group_size > 1024 && pairs_ok) go(gated_rmsnorm_wide_kernel<256, 16>, (unsigned)items, 256);
   else if (group_size > 256 && pairs_ok) go(gated_rmsnorm_wide_kernel<128, 4>, (unsigned)items, 128);
   else
     launch_pdl(gated_rmsnorm_kernel<bf16>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, static_cast<const bf16*>(x), ldx, static_cast<const bf16*>(z), ldz,
-               static_cast<const bf16*>(w), wlen, static_cast<bf16*>(y), ldy, T, D, group_size, eps, norm_before_gate);
+               static_cast<const bf16*>(w), wlen, static_cast<bf16*>(y), ldy, T, D, group_size, eps, mode);
 }
 
 }  // namespace fllm

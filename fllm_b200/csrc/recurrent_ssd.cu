@@ -15,6 +15,9 @@
 // ssd_decode_kernel serves steps of single tokens: inputs straight from global memory, no shared memory, many CTAs that keep
 // state reads in flight (a decoded token reads and writes the whole state once).
 //
+// LIN: lightning attention, the same recurrence with a constant decay per head (A holds it), step size 1 and silu on all three
+// inputs: S[p][n] <- d S[p][n] + silu(x[p]) silu(B[n]), y[p] = sum_n S[p][n] silu(C[n]).
+//
 // NP: state columns in registers; EXACT: the state width is NP and rows are 16-byte aligned, otherwise it is N <= NP and rows
 // are read value by value.
 #include <type_traits>
@@ -93,7 +96,7 @@ struct SsdTile {
   static constexpr int NPT = NP <= 32 ? 4 : 8, TPK = NP / NPT, RG = 128 / TPK, ROWS = RPT * RG, GROUP = 4;
 };
 
-template <typename T, int NP, bool EXACT, int RPT>
+template <typename T, int NP, bool EXACT, int RPT, bool LIN>
 __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
   pdl_wait();
   using L = SsdTile<NP, RPT>;
@@ -149,7 +152,7 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
           cl[i] = c < N ? ld1(cp + c) : 0.f;
         }
       }
-      dr = a.dt[t * a.lddt + h];
+      if constexpr (!LIN) dr = a.dt[t * a.lddt + h];
     }
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
@@ -173,6 +176,10 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
 #pragma unroll
         for (int i = 0; i < EPT; ++i) br[i] = live ? bl[i] : 0.f, cr[i] = live ? cl[i] : 0.f;
       }
+      if constexpr (LIN) {
+#pragma unroll
+        for (int i = 0; i < EPT; ++i) br[i] = silu_t<T>(br[i]), cr[i] = silu_t<T>(cr[i]);
+      }
       if constexpr (EPT % 4 == 0) {
 #pragma unroll
         for (int i = 0; i < EPT; i += 4) {
@@ -185,6 +192,11 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
       }
       // a warp holds the four tokens of a group: running sum of the exponents over them
       static_assert(GROUP == 4, "eight threads per token");
+      if constexpr (LIN) {
+        const int n_live = min(tt % 4 + 1, cnt - tt / 4 * 4);      // of the group's tokens up to this one (0 or less: none)
+        const float p2 = A * A, P = n_live >= 4 ? p2 * p2 : n_live == 3 ? p2 * A : n_live == 2 ? p2 : n_live == 1 ? A : 1.f;
+        if (part == 0) sg[tt] = make_float4(P, live ? 1.f / P : 0.f, live ? A : 1.f, live ? 1.f : 0.f);
+      } else {
       const float dt = live ? fminf(fmaxf(softplus_t<T>(ld1(&dr) + dtb), a.dt_min), a.dt_max) : 0.f, e = dt * A;
       float c = e;
       const float c1 = __shfl_up_sync(0xffffffffu, c, 8);
@@ -192,11 +204,13 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
       const float c2 = __shfl_up_sync(0xffffffffu, c, 16);
       if (tt % 4 >= 2) c += c2;
       if (part == 0) sg[tt] = make_float4(exp_t<T>(c), dt * exp_t<T>(-c), exp_t<T>(e), dt);
+      }
     }
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
       const int e = threadIdx.x + i * 128;
-      sx[e / ROWS][e % ROWS] = e / ROWS < cnt ? ld1(&xr[i]) : 0.f;
+      const float v = e / ROWS < cnt ? ld1(&xr[i]) : 0.f;
+      sx[e / ROWS][e % ROWS] = LIN ? silu_t<T>(v) : v;
     }
     __syncthreads();
     if (base + C < n) fetch(base + C);
@@ -274,7 +288,7 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
   }
 }
 
-template <typename T, int NP, bool EXACT>
+template <typename T, int NP, bool EXACT, bool LIN>
 __global__ void __launch_bounds__(128) ssd_decode_kernel(const SsdArgs<T> a) {
   pdl_launch_dependents();
   pdl_wait();
@@ -311,8 +325,16 @@ __global__ void __launch_bounds__(128) ssd_decode_kernel(const SsdArgs<T> a) {
         B[4 * j + e] = b2.x, B[4 * j + e + 1] = b2.y, C[4 * j + e] = c2.x, C[4 * j + e + 1] = c2.y;
       }
     }
-    const float dt = fminf(fmaxf(softplus_t<T>(ld1(a.dt + t * a.lddt + h) + dtb), a.dt_min), a.dt_max);
-    const float d = exp_t<T>(dt * A), xv = ld1(a.x + t * a.ldx + (long long)h * a.P + pc), u = dt * xv;
+    float d = A, u = ld1(a.x + t * a.ldx + (long long)h * a.P + pc);
+    const float xv = u;
+    if constexpr (LIN) {
+      u = silu_t<T>(u);
+#pragma unroll
+      for (int i = 0; i < NPT; ++i) B[i] = silu_t<T>(B[i]), C[i] = silu_t<T>(C[i]);
+    } else {
+      const float dt = fminf(fmaxf(softplus_t<T>(ld1(a.dt + t * a.lddt + h) + dtb), a.dt_min), a.dt_max);
+      d = exp_t<T>(dt * A), u = dt * xv;
+    }
     float o[2] = {0.f, 0.f};
 #pragma unroll
     for (int i = 0; i < NPT; ++i) {
@@ -339,32 +361,40 @@ int ssd_scan(const SsdScanParams& p, cudaStream_t stream) {
                       static_cast<T*>(p.y), p.H, p.P, p.G, p.N, p.dt_min, p.dt_max, p.skip_from};
   };
   // few sequences and heads: two rows per thread instead of four, so that twice as many SMs work
-#define FLLM_SSD(T_, NP_, EXACT_)                                                                                     \
+#define FLLM_SSD(T_, NP_, EXACT_, LIN_)                                                                                     \
   {                                                                                                                   \
     constexpr int drows = 128 / (NP_ / 16), rows4 = SsdTile<NP_, 4>::ROWS, rows2 = SsdTile<NP_, 2>::ROWS;             \
     const int tiles4 = p.H * ((p.P + rows4 - 1) / rows4), tiles2 = p.H * ((p.P + rows2 - 1) / rows2);                 \
     if (p.tokens == p.B)                                                                                              \
-      launch_pdl(ssd_decode_kernel<T_, NP_, EXACT_>, dim3(p.H * ((p.P + drows - 1) / drows), p.B), dim3(128), 0, stream, args(T_{}));  \
+      launch_pdl(ssd_decode_kernel<T_, NP_, EXACT_, LIN_>, dim3(p.H * ((p.P + drows - 1) / drows), p.B), dim3(128), 0, stream, args(T_{}));  \
     else if (2LL * tiles4 * p.B <= sm_count() && tiles2 > tiles4)                                                     \
-      launch_pdl(ssd_scan_kernel<T_, NP_, EXACT_, 2>, dim3(tiles2, p.B), dim3(128), 0, stream, args(T_{}));           \
+      launch_pdl(ssd_scan_kernel<T_, NP_, EXACT_, 2, LIN_>, dim3(tiles2, p.B), dim3(128), 0, stream, args(T_{}));           \
     else                                                                                                              \
-      launch_pdl(ssd_scan_kernel<T_, NP_, EXACT_, 4>, dim3(tiles4, p.B), dim3(128), 0, stream, args(T_{}));           \
+      launch_pdl(ssd_scan_kernel<T_, NP_, EXACT_, 4, LIN_>, dim3(tiles4, p.B), dim3(128), 0, stream, args(T_{}));           \
     return 0;                                                                                                         \
   }
-#define FLLM_SSD_N(T_, EXACT_)                    \
-  {                                               \
-    if (p.N <= 16) FLLM_SSD(T_, 16, EXACT_)       \
-    if (p.N <= 32) FLLM_SSD(T_, 32, EXACT_)       \
-    if (p.N <= 64) FLLM_SSD(T_, 64, EXACT_)       \
-    if (p.N <= 128) FLLM_SSD(T_, 128, EXACT_)     \
-    FLLM_SSD(T_, 256, EXACT_)                     \
+#define FLLM_SSD_N(T_, EXACT_, LIN_)                    \
+  {                                                     \
+    if (p.N <= 16) FLLM_SSD(T_, 16, EXACT_, LIN_)       \
+    if (p.N <= 32) FLLM_SSD(T_, 32, EXACT_, LIN_)       \
+    if (p.N <= 64) FLLM_SSD(T_, 64, EXACT_, LIN_)       \
+    if (p.N <= 128) FLLM_SSD(T_, 128, EXACT_, LIN_)     \
+    FLLM_SSD(T_, 256, EXACT_, LIN_)                     \
+  }
+  if (p.dt == nullptr) {               // constant decay
+    if (p.f32) {
+      if (exact) FLLM_SSD_N(float, true, true)
+      FLLM_SSD_N(float, false, true)
+    }
+    if (exact) FLLM_SSD_N(bf16, true, true)
+    FLLM_SSD_N(bf16, false, true)
   }
   if (p.f32) {
-    if (exact) FLLM_SSD_N(float, true)
-    FLLM_SSD_N(float, false)
+    if (exact) FLLM_SSD_N(float, true, false)
+    FLLM_SSD_N(float, false, false)
   }
-  if (exact) FLLM_SSD_N(bf16, true)
-  FLLM_SSD_N(bf16, false)
+  if (exact) FLLM_SSD_N(bf16, true, false)
+  FLLM_SSD_N(bf16, false, false)
 #undef FLLM_SSD_N
 #undef FLLM_SSD
 }

@@ -38,13 +38,11 @@ def frequencies(rot):
 def rotate(x, rot, start=0):
     """x [T, d] of one head; row t stands at position start + t. Value i of the first dims / 2 turns with value i + dims / 2."""
     f, factor = frequencies(rot)
+    pos = torch.arange(start, start + x.shape[0], dtype=x.dtype)
     y, half = x.clone(), rot["dims"] // 2
-    for t in range(x.shape[0]):
-        for i in range(half):
-            a = (start + t) * f[i]
-            c, s = factor * math.cos(a), factor * math.sin(a)
-            u, v = x[t, i], x[t, i + half]
-            y[t, i], y[t, i + half] = u * c - v * s, v * c + u * s
+    for i in range(half):
+        c, s = factor * torch.cos(pos * f[i]), factor * torch.sin(pos * f[i])
+        y[:, i], y[:, i + half] = x[:, i] * c - x[:, i + half] * s, x[:, i + half] * c + x[:, i] * s
     return y
 
 
