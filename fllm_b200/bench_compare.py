@@ -1,11 +1,14 @@
-"""Throughput of a design beside the framework's closest other model at equal size (``bench.py --compare sovanex|divanex``).
+"""Throughput of a design beside the framework's closest other model at equal size (``bench.py --compare sovanex|divanex|dorevik``).
 
 The closest other model of Sovanex is a hybrid of the layer kinds it shares with other families: the gated delta rule
 (Qwen3-Next) and 512 + 64 wide latent attention (DeepSeek), with the same layer order, heads, widths and squared-ReLU
 networks, but RMSNorm around one bf16 residual, no gate on the attention heads and no shared rows. That of Divanex is a
 hybrid of Mamba-2 and grouped-query attention with normalised queries and keys and capped scores (Bamba, Gemma-2), the same
 layer order, sizes and clamped SwiGLU networks (gpt-oss), but separate values, norms in front of the blocks around one bf16
-residual, and no token input. Both models run random weights through the engine: prompts of 1024 tokens in 2048-token
+residual, and no token input. That of Dorevik is a hybrid of windowed grouped-query attention with normalised queries and keys,
+of that attention beside Mamba-2 (Falcon-H1) and of routed experts beside a shared one (DeepSeek-V3's router), with the same
+layer order and as many weights and products, but one softmax per head, weights on the experts' outputs, and norms in front of
+the blocks around one bf16 residual. Both models run random weights through the engine: prompts of 1024 tokens in 2048-token
 steps, then captured decode steps. ``--kernels`` times the kernels that differ, each beside its like kernel on the same sizes.
 """
 from __future__ import annotations
@@ -16,7 +19,7 @@ from typing import Dict, List
 
 import torch
 
-from .config import EngineConfig, ModelConfig, divanex_from_config, sovanex_from_config
+from .config import EngineConfig, ModelConfig, divanex_from_config, dorevik_from_config, sovanex_from_config
 
 # name -> width, layers, feed-forward width, value heads / key heads of the delta rule, attention heads
 SIZES = {"1b": (2048, 12, 8192, 32, 16, 16), "3b": (3072, 24, 12288, 48, 24, 24), "7b": (4096, 32, 16384, 64, 32, 32)}
@@ -68,6 +71,36 @@ def divanex_twin_config(size: str) -> ModelConfig:
                        layer_kinds=["attention" if i % 4 == 3 else "mamba2" for i in range(L)], ffn_kinds=["glu" if i % 4 == 3 else "none" for i in range(L)],
                        ssm=dict(d_inner=Hm * 64, d_state=128, d_conv=4, n_groups=8, head_dim=64, n_heads=Hm, norm_groups=8, conv_bias=True, dt_min=0.0,
                                 dt_max=1e30))
+
+
+# name -> width, layers, feed-forward width, query / key heads (values of 128; differential: two maps of 64), experts, their width, shared
+# width, tokens of every window
+DOREVIK_SIZES = {"1b": (2048, 16, 6144, 16, 4, 32, 768, 1536, 1024), "3b": (3072, 20, 9216, 24, 6, 32, 1024, 2048, 1024),
+                 "7b": (4096, 24, 12288, 32, 8, 32, 1536, 3072, 1024)}
+DOREVIK_TOP = 4
+
+
+def dorevik_config(size: str) -> ModelConfig:
+    W, L, ff, H, G, E, fe, fs, window = DOREVIK_SIZES[size]
+    rot = lambda n: dict(base=1e6, dims=n)
+    diff = dict(heads=H, kv_heads=G, dim=64, vdim=128, scale=64 ** -0.5, diff=0.7, mask=dict(size=window), rot=rot(64))
+    left = dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=window), rot=rot(128))
+    right = dict(heads=H, dim=128, vdim=128, decay=[1 - 2.0 ** (-3 - 6 * i / H) for i in range(H)])
+    moe = dict(kind="moe", expert=dict(ff=fe), router=dict(experts=E, top=DOREVIK_TOP), shared=dict(ff=fs))
+    layers = [dict(type="parallel" if i % 4 == 3 else "attention", mixer=dict(left=left, right=right) if i % 4 == 3 else diff,
+                   mlp=moe if i % 2 else dict(kind="dense", ff=ff)) for i in range(L)]
+    return dorevik_from_config(ModelConfig, dict(architecture="Dorevik", name=f"dorevik-{size}", layers=layers, norm=dict(eps=1e-6), logit_softcap=30.0,
+                                                 vocab=VOCAB, width=W))
+
+
+def dorevik_twin_config(size: str) -> ModelConfig:
+    W, L, ff, H, G, E, fe, fs, window = DOREVIK_SIZES[size]
+    return ModelConfig(arch="hybrid", name=f"gqa-mamba2-moe-hybrid-{size}", vocab_size=VOCAB, hidden_size=W, num_layers=L, num_heads=H, num_kv_heads=G,
+                       head_dim=128, rope_theta=1e6, qk_norm=True, sliding_window=window, intermediate_size=ff, act="swiglu", tie_embeddings=False,
+                       logit_softcap=30.0, num_experts=E, experts_per_token=DOREVIK_TOP, moe_intermediate_size=fe, shared_intermediate_size=fs,
+                       router_kind="deepseek_v3", layer_kinds=["attention+mamba2" if i % 4 == 3 else "attention" for i in range(L)],
+                       ffn_kinds=["moe" if i % 2 else "glu" for i in range(L)],
+                       ssm=dict(d_inner=H * 128, d_state=128, d_conv=4, n_groups=H, head_dim=64, n_heads=2 * H, norm_groups=1, conv_bias=True, dt_min=0.0, dt_max=1e30))
 
 
 def throughput(cfg: ModelConfig, batch: int, prompt_len: int, steps: int, warmup: int, device, graphs: bool = True) -> Dict[str, float]:
@@ -268,7 +301,82 @@ def divanex_kernels(device, size: str = "1b") -> List[dict]:
     return tab.rows
 
 
-DESIGNS = {"sovanex": (sovanex_config, twin_config, sovanex_kernels), "divanex": (divanex_config, divanex_twin_config, divanex_kernels)}
+def dorevik_kernels(device, size: str = "1b") -> List[dict]:
+    from .ops.maps import Combine, NormedPair
+    tab = _Table(device)
+    ops, rnd, floor, bf = tab.ops, tab.rnd, tab.floor, torch.bfloat16
+    W, _, ff, H, G, E, fe, fs, _ = DOREVIK_SIZES[size]
+    D, K = 128, 64
+    for shape, lens, ctxs, windows in (("decode 64 x 1152", [1] * 64, [1152] * 64, (0, 512)), ("decode 8 x 4096", [1] * 8, [4096] * 8, (0, 512)),
+                                       ("prompt 2048", [2048], [2048], (0, 512)), ("prompt 8192", [8192], [8192], (0, 1024)),
+                                       ("prompt 4 x 512 at 2048", [512] * 4, [2048] * 4, (0, 512))):
+        b = _batch(lens, ctxs, device)
+        T = b.tokens
+        b.min_q_len, b.seq_lens = min(lens), torch.tensor(ctxs, dtype=torch.int32, device=device)
+        kc, vc, k2 = rnd(b.blocks, G, 16, D), rnd(b.blocks, G, 16, D), rnd(b.blocks, 2 * G, 16, K)
+        q, q1, q2 = rnd(T, H * D), rnd(T, H, D), rnd(T, 2 * H, K)
+        for window in windows:
+            see = lambda i: min(i + 1, window or i + 1)
+            keys = sum(see(i) for n, c in zip(lens, ctxs) for i in range(c - n, c))
+            rows = sum(min(c, n + (window or c) - 1) for n, c in zip(lens, ctxs))
+            fl = floor(rows * G * 4 * D + 4 * T * H * D, 4.0 * keys * H * D)
+            fl2 = floor(rows * G * 4 * D + 4 * T * H * D, 2.0 * keys * H * (2 * K + 2 * D))       # two maps: each weighs all values
+            like = tab.time(lambda: ops.attention(q, kc, vc, b.block_tables, b.row_seq, b.positions, H, G, D, D ** -0.5, window, None, 0.0, meta=b))
+            at = f"{shape}, window {window}" if window else shape
+            tab.add(at, "attention_maps, two maps of 64", tab.time(lambda: ops.attention_maps(q2, k2, vc, K, D, b, K ** -0.5, window, Combine(0.5, 0.3, 1e-6))), fl2,
+                    "attention", like, fl)
+            tab.add(at, "attention_maps, one map of 128", tab.time(lambda: ops.attention_maps(q1, kc, vc, D, D, b, D ** -0.5, window)), fl, "attention", like, fl)
+        if len(lens) == 4:
+            continue
+        x, w, inv = rnd(T, (H + 2 * G) * D), torch.ones(H * D, device=device, dtype=bf), torch.rand(D // 2, device=device)
+        fl = floor(2 * T * (2 * H + 4 * G) * D)
+        like = tab.time(lambda: ops.rope_kv_write(x, b.positions, b.slots, inv, w[:D], w[:D], kc, vc, H, G, D, D, 0, 1e-5))
+        tab.add(shape, "maps_prepare, norm per map", tab.time(lambda: ops.maps_prepare(x, (0, H * D, (H + G) * D), 2 * H, K, D, b.positions, b.slots, inv[:K // 2], 1.0,
+                                                                                   w[:K], w[:K], False, 1e-5, k2, vc)), fl, "rope_kv_write", like, fl)
+        tab.add(shape, "maps_prepare, norm over all heads", tab.time(lambda: ops.maps_prepare(x, (0, H * D, (H + G) * D), H, D, D, b.positions, b.slots, inv, 1.0,
+                                                                                          w, w[:G * D], True, 1e-5, kc, vc)), fl, "rope_kv_write", like, fl)
+    for T in (64, 2048):
+        shape = f"{T} rows"
+        x, y, y2, res, w = rnd(T, W, dtype=torch.float32), rnd(T, W), rnd(T, W), rnd(T, W), torch.ones(W, device=device, dtype=bf)
+        norm, norm_fl = tab.time(lambda: ops.rmsnorm(res, y, w, 1e-5)), floor(T * W * 8)
+        tab.add(shape, "postnorm, norm of what is added", tab.time(lambda: ops.postnorm_step(x, y, w, W, 1e-5, 1.0, True)), floor(T * W * 12),
+                "residual add + rmsnorm", norm, norm_fl)
+        tab.add(shape, "postnorm of a normed pair", tab.time(lambda: ops.postnorm_step(x, NormedPair(y2, y, w, w), w, W, 1e-5, 1.0, True)), floor(T * W * 14),
+                "residual add + rmsnorm", norm, norm_fl)
+        o, z, wn = rnd(T, H * D), rnd(T, H * D), torch.ones(H * D, device=device, dtype=bf)
+        fl = floor(6 * T * H * D)
+        tab.add(shape, "norm before a sigmoid gate", tab.time(lambda: ops.gated_rmsnorm(o, z, wn, 1e-5, H * D, True, 0, "sigmoid")), fl, "norm behind a silu gate",
+                tab.time(lambda: ops.gated_rmsnorm(o, z, wn, 1e-5, H * D)), fl)
+        rw, bias = rnd(E, W), torch.zeros(E, device=device)
+        ids, wts = torch.empty(T, DOREVIK_TOP, dtype=torch.int32, device=device), torch.empty(T, DOREVIK_TOP, device=device)
+
+        def routed(fp32):
+            z = ops.linear(y, rw, force_splits=2 if fp32 else 0, defer=fp32)
+            if fp32:
+                ops.k.moe_route_fp32(None, ops.workspace, z.splits, E, E, DOREVIK_TOP, 2, False, 1.0, ids, wts)
+            else:
+                ops.k.moe_route_scored(z, bias, DOREVIK_TOP, 2, False, 1.0, ids, wts)
+        fl = floor(2 * (T * W + E * W))
+        tab.add(shape, "router, fp32 logits", tab.time(lambda: routed(True)), fl, "router, bf16 logits", tab.time(lambda: routed(False)), fl)
+        n = T * DOREVIK_TOP
+        token_of, row_w, xp, row_of = torch.arange(n, device=device).int() // DOREVIK_TOP, torch.rand(n, device=device), rnd(n, W), torch.arange(n, device=device).int().view(T, -1)
+        fl = floor(2 * (T + n) * W)
+        tab.add(shape, "gather of weighed rows", tab.time(lambda: ops.k.moe_gather(y, token_of, xp, row_w)), fl, "gather", tab.time(lambda: ops.k.moe_gather(y, token_of, xp)), fl)
+        tab.add(shape, "combine with the shared expert", tab.time(lambda: ops.k.moe_combine(xp, row_of, None, y2, res)), floor(2 * (2 * T + n) * W), "combine",
+                tab.time(lambda: ops.k.moe_combine(xp, row_of, wts, y2)), fl)
+        b = _batch([1] * T if T == 64 else [T], [1024] * T if T == 64 else [T], device)
+        qkv, dt = rnd(T, 3 * H * D), rnd(T, 2 * H)
+        st, A, dec = torch.zeros(b.num_seqs, H, D, D, device=device), -torch.rand(2 * H, device=device), torch.full((H,), 0.99, device=device)
+        us = tab.time(lambda: ops.decay_scan(qkv[:, :H * D], qkv[:, H * D:2 * H * D], qkv[:, 2 * H * D:], dec, st, b.q_starts, b.seq_state, b.positions, H, D, D))
+        st2 = st.view(b.num_seqs, 2 * H, 64, D)
+        like = tab.time(lambda: ops.mamba2_scan(qkv[:, 2 * H * D:], dt, qkv[:, H * D:2 * H * D], qkv[:, :H * D], A, A, A, st2, b.q_starts, b.seq_state, b.positions,
+                                                2 * H, 64, H, D))
+        fl = floor(st.numel() * 8 + 2 * T * 4 * H * D)
+        tab.add(shape, "constant-decay scan", us, fl, "Mamba-2 scan", like, fl)
+    return tab.rows
+
+
+DESIGNS = {"dorevik": (dorevik_config, dorevik_twin_config, dorevik_kernels), "sovanex": (sovanex_config, twin_config, sovanex_kernels), "divanex": (divanex_config, divanex_twin_config, divanex_kernels)}
 
 
 def main(args) -> dict:

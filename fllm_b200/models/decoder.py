@@ -176,7 +176,7 @@ class Decoder:
             return self.tp.all_reduce(x)
         return x
 
-    def _attention_block(self, li: int, lw, h: torch.Tensor, b: StepBatch) -> torch.Tensor:
+    def _attention_block(self, li: int, lw, h: torch.Tensor, b: StepBatch, defer_out: bool = True) -> torch.Tensor:
         cfg, sp, ops = self.cfg, self.spec, self.ops
         gated = lw.w_attn_gate is not None
         qkv = ops.linear(h, lw.wqkv, lw.bqkv, defer=self._defer and not gated)
@@ -202,7 +202,7 @@ class Decoder:
                           meta=b)
         if gated:                                # the attention output passes through a sigmoid gate of its own projection
             a = (a.float() * torch.sigmoid(ops.linear(h, lw.w_attn_gate).float())).to(a.dtype)
-        return ops.linear(a, lw.wo, lw.bo, defer=self._defer_out(lw.post_attn_norm))
+        return ops.linear(a, lw.wo, lw.bo, defer=defer_out and self._defer_out(lw.post_attn_norm))
 
     def _defer_out(self, post_norm) -> bool:
         """May a row-parallel projection hand its split-K partials to the next norm? Only when nothing
@@ -295,7 +295,7 @@ class Decoder:
                 o = self._reduce(self._attention_block(li, lw, h, b))
             elif kind == "attention+mamba2":          # two mixers on one normed input
                 from .recurrent import mamba2_mixer
-                o = ops.materialize(self._reduce(self._attention_block(li, lw, h, b))) + mamba2_mixer(self, li, lw, h, b)
+                o = self._reduce(self._attention_block(li, lw, h, b, defer_out=False)) + mamba2_mixer(self, li, lw, h, b)
             elif kind == "mla":
                 from .mla import mla_block
                 o = mla_block(self, li, lw, h, b)

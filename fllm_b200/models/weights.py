@@ -307,7 +307,8 @@ def init_random_weights(cfg: ModelConfig, device="cpu", dtype=torch.bfloat16, se
     ones = lambda n: torch.ones(n, device=device, dtype=dtype)
     out_layers = []
     for li in layers:
-        if cfg.layer_kind(li) != "attention":
+        kind = cfg.layer_kind(li)
+        if kind not in ("attention", "attention+mamba2"):
             from .recurrent import init_random_mixer
             if tp > 1:
                 raise NotImplementedError("recurrent and latent-attention layers are not cut over tensor-parallel ranks")
@@ -345,6 +346,11 @@ def init_random_weights(cfg: ModelConfig, device="cpu", dtype=torch.bfloat16, se
         wo = full((H, cfg.q_size), li, 3)[:, qs].contiguous()
         lw = LayerWeights(attn_norm=ones(H), wqkv=wqkv, wo=wo, ffn_norm=ones(H))
         del wq, wk, wv
+        if kind == "attention+mamba2":
+            from .recurrent import init_random_mixer
+            if tp > 1:
+                raise NotImplementedError("recurrent layers are not cut over tensor-parallel ranks")
+            lw.mixer = init_random_mixer(cfg, "mamba2", full, li, dtype, device)
         if cfg.attn_bias:
             bq = full((cfg.q_size,), li, 10)
             bk = full((cfg.kv_size,), li, 11)
@@ -360,8 +366,12 @@ def init_random_weights(cfg: ModelConfig, device="cpu", dtype=torch.bfloat16, se
         if cfg.attn_sinks:
             s = torch.randn(cfg.num_heads, generator=gen_for(li, 14), device=device) * 0.5
             lw.sinks = s[sp.q_head_start: sp.q_head_start + sp.hq_local].float().contiguous()
-        if cfg.is_moe:
+        if cfg.is_moe and (cfg.ffn_kinds is None or cfg.ffn_kind(li) == "moe"):
             E, I = cfg.num_experts, cfg.moe_intermediate_size
+            if cfg.ffn_kinds is not None and cfg.shared_intermediate_size:
+                Is = cfg.shared_intermediate_size
+                lw.shared_gate_up = torch.cat([full((Is, H), li, 26), full((Is, H), li, 27)], 0).contiguous()
+                lw.shared_down = full((H, Is), li, 28)
             lw.router_w = full((E, H), li, 20)
             lw.router_b = full((E,), li, 21) if cfg.expert_bias else None
             gu = full((E, 2 * I, H), li, 22)

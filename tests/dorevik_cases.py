@@ -50,8 +50,8 @@ CONFIGS = {
     "wide": config([diff(heads(2, 1, 136, 72, 30, 100), 0.5, dense(40)), parallel(heads(3, 3, 72, 200, 18, 72), [0.99], 200, 72, dense(24)),
                     diff(heads(2, 2, 16, 140, 45, 8), 0.8, moe(3, 2, 24, 16))], 160, 64, cap=20.0, eps=1e-6),
     # sizes, windows and counts of one
-    "ones": config([diff(heads(1, 1, 8, 8, 1, 2), 0.1, moe(1, 1, 8)), parallel(heads(1, 1, 8, 8, 1, 8), [0.5], 8, 8, dense(8)),
-                    diff(heads(1, 1, 2, 3, 2, 2), 0.9), parallel(heads(2, 1, 8, 3, 3, 4), [1.0, 0.5, 0.9], 1, 1)], 48, 24, cap=1.0, eps=1e-3),
+    "ones": config([diff(heads(1, 1, 8, 24, 1, 2), 0.1, moe(1, 1, 16)), parallel(heads(1, 1, 8, 24, 1, 8), [0.5], 8, 24, dense(16)),
+                    diff(heads(1, 1, 2, 16, 2, 2), 0.5), parallel(heads(2, 1, 8, 24, 3, 4), [0.5] * 12 + [1.0] * 12, 1, 1)], 48, 24, cap=1.0, eps=1e-3),
 }
 
 
