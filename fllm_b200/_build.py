@@ -31,7 +31,7 @@ LIB_CUDA = ROOT / "_C.so"
 LIB_CPU = ROOT / "_cpu.so"
 # part name -> the sources (without suffix) its models run: dense and recurrent layers, 32-bit products and a kind of attention
 _COMMON = ("binding", "binding_recurrent", "binding_f32", "elementwise", "sampling", "gemm_bf16", "gemm_bf16_2sm", "gemm_f32", "recurrent",
-           "recurrent_ssd")
+           "recurrent_ssd", "recurrent_chunk")
 PARTS = {
     "latent": _COMMON + ("binding_latent", "attention_latent", "streams"),
     "tied": _COMMON + ("binding_tied", "binding_postnorm", "attention_tied", "postnorm"),

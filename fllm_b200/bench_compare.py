@@ -367,7 +367,8 @@ def dorevik_kernels(device, size: str = "1b") -> List[dict]:
         b = _batch([1] * T if T == 64 else [T], [1024] * T if T == 64 else [T], device)
         qkv, dt = rnd(T, 3 * H * D), rnd(T, 2 * H)
         st, A, dec = torch.zeros(b.num_seqs, H, D, D, device=device), -torch.rand(2 * H, device=device), torch.full((H,), 0.99, device=device)
-        us = tab.time(lambda: ops.decay_scan(qkv[:, :H * D], qkv[:, H * D:2 * H * D], qkv[:, 2 * H * D:], dec, st, b.q_starts, b.seq_state, b.positions, H, D, D))
+        us = tab.time(lambda: ops.decay_scan(qkv[:, :H * D], qkv[:, H * D:2 * H * D], qkv[:, 2 * H * D:], dec, st, b.q_starts, b.seq_state, b.positions, H, D, D, 0,
+                                             b.max_q_len, b.max_q_len))
         st2 = st.view(b.num_seqs, 2 * H, 64, D)
         like = tab.time(lambda: ops.mamba2_scan(qkv[:, 2 * H * D:], dt, qkv[:, H * D:2 * H * D], qkv[:, :H * D], A, A, A, st2, b.q_starts, b.seq_state, b.positions,
                                                 2 * H, 64, H, D))

@@ -102,10 +102,41 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
     all.x = 1.f / sqrtf(all.x / (float)(p.q_heads * p.dim) + p.eps), all.y = 1.f / sqrtf(all.y / (float)(p.k_heads * p.dim) + p.eps);
   }
   __syncthreads();
+  if (p.lanes > 0) {
+    // maps of 64 or 128 values: 16 or 32 lanes with four values each, so that a warp has one or two maps at a time and a
+    // rotation partner is a shuffle away
+    const int maps = p.q_heads + (slot >= 0 ? p.k_heads : 0), per = 32 / p.lanes, sub = lane / p.lanes, li = lane % p.lanes, c = 4 * li;
+    const bool low = c < half, turns = c < p.rot;
+    const int mate = turns ? lane + (low ? half / 4 : -half / 4) : lane;
+    float2 cs[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) cs[e] = turns ? turn[(low ? c : c - half) + e] : make_float2(1.f, 0.f);
+    for (int i0 = (blockIdx.y * 4 + warp) * per; i0 < maps; i0 += 4 * per * gridDim.y) {
+      const int item = min(i0 + sub, maps - 1);                   // (lanes past the end repeat the last map)
+      const bool is_q = item < p.q_heads;
+      const int h = is_q ? item : item - p.q_heads;
+      const float4 f = load4((is_q ? p.q_offset : p.k_offset) + h * p.dim, c, p.dim);
+      float ss = sq(f);
+      for (int o = p.lanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      const float inv = p.full ? (is_q ? all.x : all.y) : 1.f / sqrtf(ss / (float)p.dim + p.eps);
+      const T* w = static_cast<const T*>(is_q ? p.q_norm : p.k_norm) + (p.full ? h * p.dim : 0) + c;
+      const typename Four<T>::type raw = *reinterpret_cast<const typename Four<T>::type*>(w);
+      const T* wv = reinterpret_cast<const T*>(&raw);
+      float v[4] = {f.x * inv * to_f32(wv[0]), f.y * inv * to_f32(wv[1]), f.z * inv * to_f32(wv[2]), f.w * inv * to_f32(wv[3])};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float m = __shfl_sync(0xffffffffu, v[e], mate);
+        v[e] = low ? v[e] * cs[e].x - m * cs[e].y : v[e] * cs[e].x + m * cs[e].y;
+      }
+      T* dst = is_q ? static_cast<T*>(p.q_out) + ((long long)t * p.q_heads + h) * p.wk
+                    : static_cast<T*>(p.k_cache) + (((long long)(slot / p.block_size) * p.k_heads + h) * p.block_size + slot % p.block_size) * p.wk;
+      if (i0 + sub < maps) store4(dst + c, v);
+    }
+  }
   const int items = p.q_heads + (slot >= 0 ? p.k_heads + p.v_heads : 0);
   const long long block = slot >= 0 ? slot / p.block_size : 0;
   const int at = slot >= 0 ? slot % p.block_size : 0;
-  for (int item = blockIdx.y * 4 + warp; item < items; item += 4 * gridDim.y) {
+  for (int item = (p.lanes > 0 ? p.q_heads + p.k_heads : 0) + blockIdx.y * 4 + warp; item < items; item += 4 * gridDim.y) {
     float v[4];
     if (item >= p.q_heads + p.k_heads) {                          // values go to the pool as they are
       const int g = item - p.q_heads - p.k_heads;
@@ -973,6 +1004,8 @@ void maps_prepare(const MapsPrepareParams& params, cudaStream_t s) {
   const uintptr_t any = reinterpret_cast<uintptr_t>(p.x) | reinterpret_cast<uintptr_t>(p.bias) | reinterpret_cast<uintptr_t>(p.partials);
   p.vec = p.dim % 4 == 0 && p.v_dim % 4 == 0 && p.q_offset % 4 == 0 && p.k_offset % 4 == 0 && p.v_offset % 4 == 0 && any % 16 == 0 &&
           (p.partials ? p.width % 4 == 0 && p.plane % 4 == 0 : p.ldx % 4 == 0);
+  const uintptr_t norms = reinterpret_cast<uintptr_t>(p.q_norm) | reinterpret_cast<uintptr_t>(p.k_norm);
+  p.lanes = p.vec && (p.dim == 64 || p.dim == 128) && p.wk == p.dim && p.rot % 8 == 0 && norms % 16 == 0 ? p.dim / 4 : 0;
   const int heads = p.q_heads + p.k_heads + p.v_heads;
   const int shares = std::max(1, std::min((heads + 3) / 4, 4 * sm_count() / std::max(p.tokens, 1)));
   const size_t smem = (size_t)(p.rot + 4 * p.dim) * sizeof(float);

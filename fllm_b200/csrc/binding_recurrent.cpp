@@ -1,4 +1,4 @@
-// torch.ops.fllm_b200 bindings of the recurrent token mixers (recurrent.cu, recurrent_ssd.cu).
+// torch.ops.fllm_b200 bindings of the recurrent token mixers (recurrent.cu, recurrent_ssd.cu, recurrent_chunk.cu).
 #include <ATen/ATen.h>
 #include <c10/cuda/CUDAGuard.h>
 #include <c10/cuda/CUDAStream.h>
@@ -69,9 +69,11 @@ void mamba2_scan(const Tensor& x, const Tensor& dt, const Tensor& Bm, const Tens
   TORCH_CHECK(rc == 0, "mamba2_scan: unsupported arguments (code ", rc, "): heads a multiple of the groups, state width up to 256");
 }
 
-// q, k [T, H * K], v, out [T, >= H * V], decay fp32 [H], state fp32 [slots, H, V, K]: S <- decay S + silu(v) silu(k)^T, out = S silu(q)
+// q, k [T, H * K], v, out [T, >= H * V], decay fp32 [H], state fp32 [slots, H, V, K]: S <- decay S + v' k'^T, out = S q'.
+// chunked: q' = q (activations applied), the sequences with at least min_tokens tokens, over chunks on the tensor cores. Otherwise
+// q' = silu(q), the sequences below skip_from (0: all), token by token.
 void decay_scan(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& decay, Tensor state, const Tensor& q_starts,
-                const Tensor& seq_state, const Tensor& positions, Tensor out, int64_t H, int64_t K, int64_t V) {
+                const Tensor& seq_state, const Tensor& positions, Tensor out, int64_t H, int64_t K, int64_t V, bool chunked, int64_t from) {
   const auto ty = act_type(v);
   TORCH_CHECK(rows_of(q, ty) && rows_of(k, ty) && rows_of(v, ty) && rows_of(out, ty), "activations: rows of one type");
   TORCH_CHECK(q.size(1) == H * K && k.size(1) == H * K && v.size(1) == H * V && out.size(1) >= H * V && out.size(0) == v.size(0) && decay.numel() == H, "widths");
@@ -86,8 +88,9 @@ void decay_scan(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor&
   p.q_starts = q_starts.data_ptr<int>(), p.seq_state = seq_state.data_ptr<int>(), p.positions = positions.data_ptr<int>(), p.y = out.data_ptr();
   p.B = (int)seq_state.numel(), p.tokens = (int)v.size(0), p.H = (int)H, p.P = (int)V, p.G = (int)H, p.N = (int)K;
   p.f32 = ty == at::kFloat ? 1 : 0;
-  const int rc = fllm::ssd_scan(p, cur_stream());
-  TORCH_CHECK(rc == 0, "decay_scan: unsupported arguments (code ", rc, "): key width up to 256");
+  p.skip_from = chunked ? 0 : (int)from;
+  const int rc = chunked ? fllm::decay_chunk(p, (int)from, cur_stream()) : fllm::ssd_scan(p, cur_stream());
+  TORCH_CHECK(rc == 0, "decay_scan: unsupported arguments (code ", rc, "): key width up to 256; chunked: bf16, widths in multiples of 8, keys up to 128, aligned rows");
 }
 
 void mamba1_scan(const Tensor& x, const Tensor& dt, const Tensor& Bm, const Tensor& Cm, const optional<Tensor>& z, const Tensor& A,
@@ -175,7 +178,7 @@ TORCH_LIBRARY_FRAGMENT(fllm_b200, m) {
         "Tensor seq_state, Tensor positions, Tensor(b!) y, int H, int P, int G, int N, float dt_min, float dt_max, int skip_from) -> ()",
         &mamba2_scan);
   m.def("decay_scan(Tensor q, Tensor k, Tensor v, Tensor decay, Tensor(a!) state, Tensor q_starts, Tensor seq_state, Tensor positions, Tensor(b!) out, "
-        "int H, int K, int V) -> ()", &decay_scan);
+        "int H, int K, int V, bool chunked, int from_tokens) -> ()", &decay_scan);
   m.def("mamba1_scan(Tensor x, Tensor dt, Tensor Bm, Tensor Cm, Tensor? z, Tensor A, Tensor? D, Tensor? dt_bias, Tensor(a!) state, "
         "Tensor q_starts, Tensor seq_state, Tensor positions, Tensor(b!) y, int seg_len, int segs, Tensor? seg_scratch) -> ()",
         &mamba1_scan);

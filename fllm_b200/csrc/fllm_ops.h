@@ -298,6 +298,11 @@ struct SsdScanParams {
   int skip_from, f32;
 };
 int ssd_scan(const SsdScanParams& p, cudaStream_t stream);
+// Lightning attention over chunks on the tensor cores (recurrent_chunk.cu), bf16: the sequences with at least min_tokens tokens in
+// the step, from x, Bm and Cm with their activations already applied. Returns a negative code, before any launch, for what it does
+// not cover: widths that are no multiples of 8, keys above 128, rows that are not 16-byte aligned.
+bool decay_chunk_supported(int K, int V);
+int decay_chunk(const SsdScanParams& p, int min_tokens, cudaStream_t s);
 // Segmented scan (seg_len > 0, segs > 1): seg_state holds B * segs states (segs - 1 per sequence, then one start state per
 // sequence), seg_dt B * (segs - 1) sums of time steps per channel.
 int mamba1_scan(const void* x, long long ldx, const void* dt, long long lddt, const void* Bm, long long ldb, const void* Cm,
@@ -471,7 +476,7 @@ struct MapsPrepareParams {
   void* q_out;                 // [tokens][q_heads][wk]
   void *k_cache, *v_cache;     // [blocks][k_heads][block_size][wk], [blocks][v_heads][block_size][wv]
   int f32;
-  int vec;                     // set by maps_prepare: rows move four values at a time
+  int vec, lanes;              // set by maps_prepare: rows move four values at a time; lanes of a map held in registers (0: through shared memory)
 };
 void maps_prepare(const MapsPrepareParams& p, cudaStream_t s);
 struct MapsAttnParams {

@@ -310,6 +310,18 @@ __global__ void __launch_bounds__(128) ssd_decode_kernel(const SsdArgs<T> a) {
   for (long long t = t0; t < t0 + n; ++t) {
     const T *bp = a.Bm + t * a.ldb + go, *cp = a.Cm + t * a.ldc + go;
     float B[NPT], C[NPT];
+    if constexpr (LIN) {                                   // the activations once per CTA
+      __shared__ __align__(16) float sb[NP], sc[NP];
+      __syncthreads();
+      for (int i = threadIdx.x; i < NP; i += 128) sb[i] = i < N ? silu_t<T>(ld1(bp + i)) : 0.f, sc[i] = i < N ? silu_t<T>(ld1(cp + i)) : 0.f;
+      __syncthreads();
+#pragma unroll
+      for (int j = 0; j < NPT / 4; ++j) {
+        const float4 b4 = *reinterpret_cast<const float4*>(&sb[4 * (lk + TPK * j)]), c4 = *reinterpret_cast<const float4*>(&sc[4 * (lk + TPK * j)]);
+        B[4 * j] = b4.x, B[4 * j + 1] = b4.y, B[4 * j + 2] = b4.z, B[4 * j + 3] = b4.w;
+        C[4 * j] = c4.x, C[4 * j + 1] = c4.y, C[4 * j + 2] = c4.z, C[4 * j + 3] = c4.w;
+      }
+    } else {
 #pragma unroll
     for (int j = 0; j < NPT / 4; ++j) {
       const int c = 4 * (lk + TPK * j);
@@ -325,12 +337,11 @@ __global__ void __launch_bounds__(128) ssd_decode_kernel(const SsdArgs<T> a) {
         B[4 * j + e] = b2.x, B[4 * j + e + 1] = b2.y, C[4 * j + e] = c2.x, C[4 * j + e + 1] = c2.y;
       }
     }
+    }
     float d = A, u = ld1(a.x + t * a.ldx + (long long)h * a.P + pc);
     const float xv = u;
     if constexpr (LIN) {
       u = silu_t<T>(u);
-#pragma unroll
-      for (int i = 0; i < NPT; ++i) B[i] = silu_t<T>(B[i]), C[i] = silu_t<T>(C[i]);
     } else {
       const float dt = fminf(fmaxf(softplus_t<T>(ld1(a.dt + t * a.lddt + h) + dtb), a.dt_min), a.dt_max);
       d = exp_t<T>(dt * A), u = dt * xv;

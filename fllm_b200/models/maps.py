@@ -43,7 +43,7 @@ def maps_lightning_mixer(dec, li: int, lw, h: torch.Tensor, b) -> NormedPair:
     at, nk = m["lin_offset"], pad8(H * K)
     q, k, v = proj[:, at:at + H * K], proj[:, at + nk:at + nk + H * K], proj[:, at + 2 * nk:at + 2 * nk + H * V]
     gate = proj[:, at + 2 * nk + pad8(H * V):at + 2 * nk + pad8(H * V) + H * V]
-    o = ops.decay_scan(q, k, v, m["lin_decay"], dec.rstate.scan[li], qs, ss, pos, H, K, V)
+    o = ops.decay_scan(q, k, v, m["lin_decay"], dec.rstate.scan[li], qs, ss, pos, H, K, V, 0, b.max_q_len, b.min_q_len)
     o = ops.gated_rmsnorm(o, gate, m["lin_norm"], s.get("norm_eps", dec.cfg.rms_eps), H * V, True, m["lin_wo"].shape[1], "sigmoid")
     return NormedPair(ya, ops.linear(o, m["lin_wo"], defer=dec.defer_to_residual), m["out_a"], m["out_b"])
 

@@ -18,6 +18,9 @@ from .latent import _rotate
 from .tied import tied_width
 
 
+DECAY_CHUNK_TOKENS = 32          # sequences with at least this many tokens in a step run lightning attention in matrix form
+
+
 def maps_width(dim: int) -> int:
     """Padded length of a key, value or query row."""
     return tied_width(dim)
@@ -87,7 +90,7 @@ class MapsRef:
             out[t, :H * v_dim] = y.reshape(-1).to(out.dtype)
         return out
 
-    def decay_scan(self, q, k, v, decay, state, q_starts, seq_state, positions, H, K, V, width=0):
+    def decay_scan(self, q, k, v, decay, state, q_starts, seq_state, positions, H, K, V, width=0, max_q_len=0, min_q_len=0, chunk_from=0):
         """Per head S <- decay S + silu(v) silu(k)^T, o = S silu(q), with S [V, K] in fp32: [T, width or H * V]."""
         from .recurrent import _seqs
         T = q.shape[0]
@@ -138,9 +141,25 @@ class MapsNative:
                                                int(splits), ws, bool(tensor_cores), self.status)
         return out
 
-    def decay_scan(self, q, k, v, decay, state, q_starts, seq_state, positions, H, K, V, width=0):
+    def decay_scan(self, q, k, v, decay, state, q_starts, seq_state, positions, H, K, V, width=0, max_q_len=0, min_q_len=0, chunk_from=DECAY_CHUNK_TOKENS):
+        """``max_q_len`` / ``min_q_len``: host-side bounds on a sequence's tokens in the step (0: unknown). Sequences with at least
+        ``chunk_from`` tokens run in matrix form on the tensor cores where it covers the sizes; q, k and v then hold their
+        activations afterwards."""
         make = torch.zeros if width > H * V else torch.empty
         out = make(q.shape[0], max(width, H * V), dtype=v.dtype, device=v.device)
-        self.k.decay_scan(q, k, v, decay, state, q_starts, seq_state, positions, out, int(H), int(K), int(V))
-        self.launches += 1
+        args = (decay, state, q_starts, seq_state, positions, out, int(H), int(K), int(V))
+        aligned = all(t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in (q, k, v)) and out.stride(0) % 2 == 0
+        chunks = chunk_from > 0 and max_q_len >= chunk_from and v.dtype == torch.bfloat16 and aligned and K % 8 == 0 and V % 8 == 0 and K <= 128
+        if not chunks or min_q_len < chunk_from:
+            self.k.decay_scan(q, k, v, *args, False, int(chunk_from) if chunks else 0)
+            self.launches += 1
+        if chunks:
+            ld, at = q.stride(0), q.data_ptr()
+            if k.stride(0) == ld == v.stride(0) and k.data_ptr() == at + 2 * H * K and v.data_ptr() == at + 4 * H * K:     # one segment behind the other
+                self.act_(q.as_strided((q.shape[0], 2 * H * K + H * V), (ld, 1)), "silu")
+            else:
+                for t in (q, k, v):
+                    self.act_(t, "silu")
+            self.k.decay_scan(q, k, v, *args, True, int(chunk_from))
+            self.launches += 1
         return out

@@ -226,9 +226,13 @@ def test_single_keys_at_every_border(ops, lens, ctx, M, dtype):
 
 # ------------------------------------------------------------------------------------------------ lightning attention
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,V,K", [(4, 13, 20), (1, 8, 8), (3, 40, 16), (4, 24, 64), (2, 64, 128), (2, 20, 256), (3, 300, 100), (16, 128, 128), (2, 7, 32), (1, 1, 1), (2, 64, 32)])
-def test_decay_scan(ops, H, V, K, dtype):
-    """Ragged steps that continue each other: prompts, portions of 2 .. 130 tokens and single tokens, rows of the pool in any order."""
+@pytest.mark.parametrize("H,V,K", [(4, 13, 20), (1, 8, 8), (3, 40, 16), (4, 24, 64), (2, 64, 128), (2, 20, 256), (3, 300, 100), (16, 128, 128), (2, 7, 32), (1, 1, 1), (2, 64, 32), (60, 40, 72)])
+@pytest.mark.parametrize("chunks", [0, 32, 2])
+def test_decay_scan(ops, H, V, K, dtype, chunks):
+    """Ragged steps that continue each other: prompts, portions of 2 .. 130 tokens and single tokens, rows of the pool in any order;
+    token by token, in matrix form from 32 tokens on, and in matrix form down to portions of two tokens."""
+    if chunks and (dtype == torch.float32 or K % 8 or V % 8 or K > 128):
+        pytest.skip("sizes and types of the token-by-token form")
     g = gen(K)
     lens, slots = [245, 170, 3], [2, 0, 4]
     p8 = lambda n: (n + 7) // 8 * 8
@@ -242,7 +246,9 @@ def test_decay_scan(ops, H, V, K, dtype):
         x = torch.cat([rows[i][at[i]:at[i] + n] for i, n in part])
         qs = ints([sum(n for _, n in part[:j]) for j in range(len(part) + 1)])
         pos = ints([p for i, n in part for p in range(at[i], at[i] + n)])
-        y = ops.decay_scan(x[:, :H * K], x[:, ok:ok + H * K], x[:, ov:ov + H * V], decay, state, qs, ints([slots[i] for i, _ in part]), pos, H, K, V, H * V + 3)
+        many = [n for _, n in part] if chunks else [0]
+        y = ops.decay_scan(x[:, :H * K], x[:, ok:ok + H * K], x[:, ov:ov + H * V], decay, state, qs, ints([slots[i] for i, _ in part]), pos, H, K, V, H * V + 4,
+                           max(many), min(many), chunks)
         assert not y[:, H * V:].any()
         for j, (i, n) in enumerate(part):
             got[i].append(y[int(qs[j]):int(qs[j + 1]), :H * V])
@@ -252,8 +258,27 @@ def test_decay_scan(ops, H, V, K, dtype):
         cut = lambda o, w, h: x[:, o + h * w:o + (h + 1) * w]
         want = [O.decayed_sum(cut(0, K, h), cut(ok, K, h), cut(ov, V, h), d64(decay)[h]) for h in range(H)]
         assert rel(torch.cat(got[i]), torch.cat([y for y, _ in want], 1)) < (2e-6 if dtype == torch.float32 else 4e-3)
-        assert rel(state[slots[i]], torch.stack([s.t() for _, s in want])) < 2e-6                # fp32 in both modes
+        # fp32 in both modes (in matrix form the activations are bf16 operands)
+        assert rel(state[slots[i]], torch.stack([s.t() for _, s in want])) < (4e-3 if chunks else 2e-6)
     assert bool((state[[1, 3, 5]] == 9).all())
+
+
+def test_chunks_keep_the_precision_of_the_state(ops):
+    """1000 tokens in matrix form against the recurrence on the same bf16 activations: the state has fp32 precision, the outputs
+    that of their own rounding; decays from hardly to at once."""
+    H, V, K, n, g = 5, 40, 72, 1000, gen(9)
+    x = torch.randn(n, 2 * H * K + H * V, device=DEV, generator=g).bfloat16()
+    decay, state = torch.tensor([0.9999, 0.99, 0.7, 0.01, 1.0], device=DEV), torch.zeros(2, H, V, K, device=DEV)
+    q, k, v = x[:, :H * K], x[:, H * K:2 * H * K], x[:, 2 * H * K:]
+    for t0, t1 in ((0, 500), (500, 502), (502, 1000)):
+        y = ops.decay_scan(q[t0:t1], k[t0:t1], v[t0:t1], decay, state, ints([0, t1 - t0]), ints([1]), ints(list(range(t0, t1))), H, K, V, 0, t1 - t0, t1 - t0, 2)
+        x[t0:t1, :H * V] = y                                            # (the activations replaced q, k and v; the outputs go over q)
+    f = d64(torch.cat([k, v], 1))                                       # bf16 activations
+    for h in range(H):
+        kh, vh = f[:, h * K:(h + 1) * K], f[:, H * K + h * V:H * K + (h + 1) * V]
+        _, S = O.decayed_sum(torch.zeros_like(kh), kh, vh, d64(decay)[h])
+        assert rel(state[1, h], S.t()) < 3e-6, h
+    assert not state[0].any()
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
