@@ -115,7 +115,7 @@ def throughput(cfg: ModelConfig, batch: int, prompt_len: int, steps: int, warmup
     prompts = [torch.randint(0, cfg.vocab_size, (prompt_len,), generator=g).tolist() for _ in range(batch)]
     sp = SamplingParams(max_tokens=room, ignore_eos=True)
     e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-    eng.generate(prompts[:2], dataclasses.replace(sp, max_tokens=2))          # warm-up of both step kinds
+    eng.generate(prompts[:8], dataclasses.replace(sp, max_tokens=2))          # warm-up of both step kinds, and of the allocator
     for p in prompts:
         eng.add_request(p, sp)
     torch.cuda.synchronize()

@@ -61,13 +61,13 @@ void moe_align(const Tensor& ids, int64_t experts, int64_t expert_lo, int64_t ex
                Tensor token_of, Tensor tile_expert, Tensor tile_row0, Tensor num_tiles, const optional<Tensor>& weights,
                const optional<Tensor>& row_weight) {
   TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == at::kInt && ids.dim() == 2 && ids.is_contiguous(), "ids: [tokens, k] int32");
-  TORCH_CHECK(num_tiles.numel() >= 2, "num_tiles needs two ints");
+  TORCH_CHECK(num_tiles.numel() >= 2 && expert_lo >= 0 && expert_lo <= expert_hi && expert_hi <= experts, "num_tiles needs two ints; a range of the experts");
   const bool weighed = row_weight.has_value() && row_weight->defined();
   TORCH_CHECK(!weighed || (weights.has_value() && weights->scalar_type() == at::kFloat && weights->is_contiguous() && weights->numel() == ids.numel() &&
                            row_weight->scalar_type() == at::kFloat && row_weight->is_contiguous() && row_weight->numel() >= token_of.numel()),
               "weights fp32 like ids, row_weight fp32 like token_of");
   c10::cuda::CUDAGuard guard(ids.device());
-  fllm::moe_align(ids.data_ptr<int>(), (int)ids.size(0), (int)ids.size(1), (int)experts, (int)expert_lo, (int)expert_hi,
+  fllm::moe_align(ids.data_ptr<int>(), (int)ids.size(0), (int)ids.size(1), (int)expert_lo, (int)expert_hi,
                   (int)bn, row_of.data_ptr<int>(), token_of.data_ptr<int>(), (int)token_of.numel(),
                   tile_expert.data_ptr<int>(), tile_row0.data_ptr<int>(), num_tiles.data_ptr<int>(),
                   (int)tile_expert.numel(), cur_stream(), weighed ? weights->data_ptr<float>() : nullptr,

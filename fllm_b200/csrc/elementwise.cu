@@ -768,24 +768,28 @@ __device__ __forceinline__ float2 act_load(const float* p) { return *reinterpret
 __device__ __forceinline__ void act_store(__nv_bfloat16* p, float2 v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y); }
 __device__ __forceinline__ void act_store(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
 
-template <typename T>
+__device__ __forceinline__ float act_value(float t, int kind, bool accurate) {
+  if (kind == 0) return 0.5f * t * (1.f + erff(t * 0.70710678118654752f));
+  if (kind == 1) return 0.5f * t * (1.f + tanhf(0.7978845608028654f * (t + 0.044715f * t * t * t)));
+  if (kind == 2) return t > 0.f ? t * t : 0.f;
+  if (kind == 3) return t / (1.f + (accurate ? expf(-t) : __expf(-t)));
+  return fmaxf(t, 0.f);
+}
+
+// V values per thread and step: pairs, or 16 bytes where rows allow it
+template <typename T, int V>
 __global__ void act_rows_kernel(T* __restrict__ x, long long ldx, int cols, int kind) {
+  struct alignas(V * sizeof(T)) Piece { T v[V]; };
   T* row = x + (size_t)blockIdx.y * ldx;
-  for (int c = (blockIdx.x * blockDim.x + threadIdx.x) * 2; c < cols; c += gridDim.x * blockDim.x * 2) {
-    float2 v = act_load(row + c);
-    float* f = &v.x;
+  for (int c = (blockIdx.x * blockDim.x + threadIdx.x) * V; c < cols; c += gridDim.x * blockDim.x * V) {
+    Piece p = *reinterpret_cast<const Piece*>(row + c);
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const float t = f[i];
-      float r;
-      if (kind == 0) r = 0.5f * t * (1.f + erff(t * 0.70710678118654752f));
-      else if (kind == 1) r = 0.5f * t * (1.f + tanhf(0.7978845608028654f * (t + 0.044715f * t * t * t)));
-      else if (kind == 2) r = t > 0.f ? t * t : 0.f;
-      else if (kind == 3) r = t / (1.f + (sizeof(T) == 4 ? expf(-t) : __expf(-t)));
-      else r = fmaxf(t, 0.f);
-      f[i] = r;
+    for (int i = 0; i < V; i += 2) {
+      float2 f = act_load(p.v + i);
+      f.x = act_value(f.x, kind, sizeof(T) == 4), f.y = act_value(f.y, kind, sizeof(T) == 4);
+      act_store(p.v + i, f);
     }
-    act_store(row + c, v);
+    *reinterpret_cast<Piece*>(row + c) = p;
   }
 }
 
@@ -794,8 +798,11 @@ static void act_rows(T* x, long long ldx, int rows, int cols, int kind, cudaStre
   if (rows <= 0 || cols <= 0) return;
   if ((cols & 1) || (ldx & 1) || (reinterpret_cast<uintptr_t>(x) & (2 * sizeof(T) - 1)) || kind < 0 || kind > 4)
     throw std::runtime_error("act_rows: an even width and leading dimension, pair-aligned rows, kind 0..4");
-  const int bx = std::max(1, std::min((cols / 2 + 255) / 256, 64));
-  act_rows_kernel<T><<<dim3(bx, rows), 256, 0, s>>>(x, ldx, cols, kind);
+  constexpr int V = 16 / sizeof(T);
+  const bool wide = cols % V == 0 && ldx % V == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0;
+  const int step = wide ? V : 2, bx = std::max(1, std::min((cols / step + 255) / 256, 64));
+  if (wide) act_rows_kernel<T, V><<<dim3(bx, rows), 256, 0, s>>>(x, ldx, cols, kind);
+  else act_rows_kernel<T, 2><<<dim3(bx, rows), 256, 0, s>>>(x, ldx, cols, kind);
   cuda_check(cudaGetLastError(), "act_rows_kernel");
 }
 void act_rows_bf16(void* x, long long ldx, int rows, int cols, int kind, cudaStream_t s) {

@@ -175,7 +175,7 @@ void moe_route_fp32(const float* logits, int splits, long long plane, long long 
                     float scale, int* ids, float* weights, cudaStream_t s);
 void moe_route(const void* logits, long long ld, const void* bias, int tokens, int experts, int k, int softmax_all,
                int* ids, float* weights, cudaStream_t s);
-void moe_align(const int* ids, int tokens, int k, int experts, int expert_lo, int expert_hi, int bn, int* row_of,
+void moe_align(const int* ids, int tokens, int k, int expert_lo, int expert_hi, int bn, int* row_of,
                int* token_of, int rows_cap, int* tile_expert, int* tile_row0, int* num_tiles, int max_tiles,
                cudaStream_t s, const float* weights = nullptr, float* row_weight = nullptr);   // row_weight [rows_cap]: weights [tokens * k] by row
 void moe_gather(const void* x, long long ldx, const int* token_of, void* xp, int rows_cap, int hidden, cudaStream_t s,

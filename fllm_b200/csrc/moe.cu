@@ -196,79 +196,91 @@ void moe_route(const void* logits, long long ld, const void* bias, int tokens, i
 // Single CTA. expert_lo/expert_hi select the experts this rank holds; entries routed elsewhere get
 // row -1. Outputs: row_of[tokens*k] (permuted row of each (token, slot) or -1), token_of[rows_cap]
 // (token of each permuted row, -1 = padding), tile_expert / tile_row0 / num_tiles, total_rows.
-__global__ void __launch_bounds__(1024) moe_align_kernel(const int* __restrict__ ids, int entries, int experts,
-                                                         int expert_lo, int expert_hi, int bn, int k,
+// Placement is deterministic: entries of an expert keep their (token, slot) order. Every warp owns a run of
+// consecutive entries: it counts them per expert, a prefix over the warps gives each its first position,
+// and on the second walk the lanes that drew the same expert rank themselves with a match mask. The warps
+// never wait for one another inside a walk.
+__global__ void __launch_bounds__(1024) moe_align_kernel(const int* __restrict__ ids, int entries, int expert_lo, int expert_hi, int bn, int k,
                                                          int* __restrict__ row_of, int* __restrict__ token_of,
                                                          int rows_cap, int* __restrict__ tile_expert,
                                                          int* __restrict__ tile_row0, int* __restrict__ num_tiles,
-                                                         int max_tiles, int staged, const float* __restrict__ weights,
+                                                         int max_tiles, const float* __restrict__ weights,
                                                          float* __restrict__ row_weight) {
-  __shared__ int cnt[512], off[513], fill[512];
-  extern __shared__ int ids_s[];              // the first `staged` ids: the per-expert scans below read them from here
-  for (int e = threadIdx.x; e < 512; e += blockDim.x) { cnt[e] = 0; fill[e] = 0; }
-  __syncthreads();
-  for (int i = threadIdx.x; i < entries; i += blockDim.x) {
-    const int e = ids[i];
-    if (i < staged) ids_s[i] = e;
-    if (e >= expert_lo && e < expert_hi) atomicAdd(&cnt[e - expert_lo], 1);
-  }
-  __syncthreads();
+  __shared__ int off[512], first_tile[512], cnt[512];
+  extern __shared__ int fill[];               // [warp][local expert]: counts, then next positions
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   const int local = expert_hi - expert_lo;
-  if (threadIdx.x == 0) {
-    int o = 0, nt = 0;
-    for (int e = 0; e < local; ++e) {
-      off[e] = o;
-      const int padded = (cnt[e] + bn - 1) / bn * bn;
-      for (int r = 0; r < padded && nt < max_tiles; r += bn) {
-        tile_expert[nt] = e;
-        tile_row0[nt] = o + r;
-        ++nt;
-      }
-      o += padded;
-    }
-    off[local] = o;
-    num_tiles[0] = nt;
-    num_tiles[1] = o;                         // total permuted rows (incl. padding)
-  }
-  __syncthreads();
+  for (int i = threadIdx.x; i < warps * local; i += blockDim.x) fill[i] = 0;
   for (int i = threadIdx.x; i < rows_cap; i += blockDim.x) token_of[i] = -1;
   __syncthreads();
-  // Deterministic placement: entries of an expert keep their (token, slot) order. The entries are taken 1024 at a time,
-  // one per thread; the warps of a round go one after the other, and inside a warp the lanes that drew the same expert
-  // rank themselves with a match mask, so no thread ever scans the list.
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int base = 0; base < entries; base += blockDim.x) {
-    const int i = base + threadIdx.x;
-    const int e = i < entries ? (i < staged ? ids_s[i] : ids[i]) - expert_lo : -1;
-    const bool valid = e >= 0 && e < local;
-    const int warps = min((int)(blockDim.x >> 5), (entries - base + 31) >> 5);
+  int* mine = fill + warp * local;
+  const int run = ((entries + warps - 1) / warps + 31) / 32 * 32, lo = warp * run, hi = min(lo + run, entries);
+  for (int base = lo; base < hi; base += 32) {
+    const int i = base + lane, e = i < hi ? ids[i] - expert_lo : -1;
+    if (e >= 0 && e < local) atomicAdd(&mine[e], 1);
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < local; e += blockDim.x) {
+    int sum = 0;
     for (int w = 0; w < warps; ++w) {
-      if (warp == w) {
-        const unsigned same = __match_any_sync(0xffffffffu, valid ? e : -1 - lane);      // other lanes with this expert
-        if (valid) {
-          const int pos = off[e] + fill[e] + __popc(same & ((1u << lane) - 1u));
-          row_of[i] = pos;
-          if (pos < rows_cap) {
-            token_of[pos] = i / k;
-            if (row_weight) row_weight[pos] = weights[i];
-          }
-        }
-        __syncwarp();
-        if (valid && lane == __ffs(same) - 1) fill[e] += __popc(same);
-      }
-      __syncthreads();
+      const int c = fill[w * local + e];
+      fill[w * local + e] = sum;
+      sum += c;
     }
-    if (i < entries && !valid) row_of[i] = -1;
+    cnt[e] = (sum + bn - 1) / bn;             // tiles of the expert
+  }
+  __syncthreads();
+  if (warp == 0) {                            // prefix of the tiles
+    int done = 0;
+    for (int base = 0; base < local; base += 32) {
+      const int e = base + lane, c = e < local ? cnt[e] : 0;
+      int p = c;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int q = __shfl_up_sync(0xffffffffu, p, o);
+        if (lane >= o) p += q;
+      }
+      if (e < local) first_tile[e] = done + p - c, off[e] = (done + p - c) * bn;
+      done += __shfl_sync(0xffffffffu, p, 31);
+    }
+    if (lane == 0) {
+      num_tiles[0] = min(done, max_tiles);
+      num_tiles[1] = done * bn;               // total permuted rows (incl. padding)
+    }
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < local; e += blockDim.x)
+    for (int t = 0; t < cnt[e] && first_tile[e] + t < max_tiles; ++t) {
+      tile_expert[first_tile[e] + t] = e;
+      tile_row0[first_tile[e] + t] = off[e] + t * bn;
+    }
+  for (int base = lo; base < hi; base += 32) {
+    const int i = base + lane, e = i < hi ? ids[i] - expert_lo : -1;
+    const bool valid = e >= 0 && e < local;
+    const unsigned same = __match_any_sync(0xffffffffu, valid ? e : -1 - lane);      // other lanes with this expert
+    int pos = -1;
+    if (valid) pos = off[e] + mine[e] + __popc(same & ((1u << lane) - 1u));
+    __syncwarp();
+    if (valid && lane == __ffs(same) - 1) mine[e] += __popc(same);
+    __syncwarp();
+    if (i < hi) row_of[i] = pos;
+    if (valid && pos < rows_cap) {
+      token_of[pos] = i / k;
+      if (row_weight) row_weight[pos] = weights[i];
+    }
   }
 }
 
-void moe_align(const int* ids, int tokens, int k, int experts, int expert_lo, int expert_hi, int bn, int* row_of,
+void moe_align(const int* ids, int tokens, int k, int expert_lo, int expert_hi, int bn, int* row_of,
                int* token_of, int rows_cap, int* tile_expert, int* tile_row0, int* num_tiles, int max_tiles,
                cudaStream_t s, const float* weights, float* row_weight) {
   if (expert_hi - expert_lo > 512) throw std::runtime_error("moe_align: at most 512 local experts");
-  const int staged = std::min(tokens * k, 10240);              // 40 KiB of dynamic shared memory at most
-  moe_align_kernel<<<1, 1024, (size_t)staged * sizeof(int), s>>>(ids, tokens * k, experts, expert_lo, expert_hi, bn, k, row_of, token_of,
-                                                                 rows_cap, tile_expert, tile_row0, num_tiles, max_tiles, staged, weights, row_weight);
+  const size_t smem = (size_t)32 * std::max(expert_hi - expert_lo, 1) * sizeof(int);      // 64 KiB at most
+  static bool configured[kMaxDevices] = {};
+  if (first_call_on_device(configured))
+    cuda_check(cudaFuncSetAttribute(moe_align_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024), "moe_align smem");
+  moe_align_kernel<<<1, 1024, smem, s>>>(ids, tokens * k, expert_lo, expert_hi, bn, k, row_of, token_of, rows_cap, tile_expert, tile_row0, num_tiles,
+                                         max_tiles, weights, row_weight);
   cuda_check(cudaGetLastError(), "moe_align_kernel");
 }
 

@@ -667,9 +667,11 @@ __global__ void __launch_bounds__(THREADS) gated_rmsnorm_wide_kernel(const bf16*
   for (int i = 0; i < THREADS / 32; ++i) tot += part[i];
   const float inv = rsqrtf(tot / gs + eps);
   __nv_bfloat162* yr = reinterpret_cast<__nv_bfloat162*>(y + t * ldy + (long long)g * gs);
+  const int w0 = (g * gs) % wlen;
   auto weight = [&](int p) {
-    const int c = (g * gs + 2 * p) % wlen;
-    return make_float2(__bfloat162float(w[c]), __bfloat162float(w[(c + 1) % wlen]));
+    int c = w0 + 2 * p, d = c + 1;
+    if (d >= wlen) c %= wlen, d %= wlen;
+    return make_float2(__bfloat162float(w[c]), __bfloat162float(w[d]));
   };
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
@@ -856,7 +858,9 @@ void gated_rmsnorm(const void* x, long long ldx, const void* z, long long ldz, c
     launch_pdl(kernel, dim3(grid), dim3(threads), 0, stream, static_cast<const bf16*>(x), ldx, static_cast<const bf16*>(z), ldz, static_cast<const bf16*>(w), wlen,
                static_cast<bf16*>(y), ldy, D, group_size, eps, mode);
   };
-  if (group_size > 1024 && pairs_ok) go(gated_rmsnorm_wide_kernel<256, 16>, (unsigned)items, 256);
+  if (group_size > 4096 && pairs_ok) go(gated_rmsnorm_wide_kernel<256, 16>, (unsigned)items, 256);
+  else if (group_size > 2048 && pairs_ok) go(gated_rmsnorm_wide_kernel<256, 8>, (unsigned)items, 256);
+  else if (group_size > 1024 && pairs_ok) go(gated_rmsnorm_wide_kernel<256, 4>, (unsigned)items, 256);
   else if (group_size > 256 && pairs_ok) go(gated_rmsnorm_wide_kernel<128, 4>, (unsigned)items, 128);
   else
     launch_pdl(gated_rmsnorm_kernel<bf16>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, static_cast<const bf16*>(x), ldx, static_cast<const bf16*>(z), ldz,

@@ -253,8 +253,8 @@ int decay_chunk(const SsdScanParams& p, int min_tokens, cudaStream_t s) {
   if (any % 16 || p.ldx % 8 || p.ldb % 8 || p.ldc % 8 || p.ldy % 2 || reinterpret_cast<uintptr_t>(p.y) % 4) return -2;
   const ChunkArgs a{static_cast<const bf16*>(p.Cm), static_cast<const bf16*>(p.Bm), static_cast<const bf16*>(p.x), p.ldc, p.ldb, p.ldx, p.ldy, p.A,
                     p.state, p.q_starts, p.seq_state, p.positions, static_cast<bf16*>(p.y), p.H, p.N, p.P, min_tokens};
-  // few heads: narrower slices, so that more SMs work
-  const bool narrow = (long long)p.H * ((p.P + 31) / 32) * p.B * 2 <= sm_count();
+  // narrower slices (more CTAs, each with the chunk's scores to itself) as long as two CTAs per SM hold them all
+  const bool narrow = (long long)p.H * ((p.P + 15) / 16) * p.B <= 2 * sm_count();
   if (p.N <= 64) narrow ? launch_chunk<64, 16>(a, p.B, s) : launch_chunk<64, 32>(a, p.B, s);
   else narrow ? launch_chunk<128, 16>(a, p.B, s) : launch_chunk<128, 32>(a, p.B, s);
   cuda_check(cudaGetLastError(), "decay_chunk_kernel");
