@@ -47,8 +47,8 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
   const float* part = p.partials ? p.partials + (size_t)t * p.width : nullptr;
   const T* bias = static_cast<const T*>(p.bias);
   auto load1 = [&](int c) {
-    if (!part) return to_f32(xr[c]);
     float v = bias ? to_f32(bias[c]) : 0.f;
+    if (!part) return v + to_f32(xr[c]);
     for (int s = 0; s < p.splits; ++s) v += __ldcg(part + s * p.plane + c);
     return v;
   };
@@ -63,11 +63,13 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
           v.x += q.x, v.y += q.y, v.z += q.z, v.w += q.w;
         }
       }
-      if (!part || bias) {
-        const typename Four<T>::type raw = *reinterpret_cast<const typename Four<T>::type*>((part ? bias : xr) + base + c);
+      auto plus = [&](const T* src) {
+        const typename Four<T>::type raw = *reinterpret_cast<const typename Four<T>::type*>(src + base + c);
         const T* e = reinterpret_cast<const T*>(&raw);
         v.x += to_f32(e[0]), v.y += to_f32(e[1]), v.z += to_f32(e[2]), v.w += to_f32(e[3]);
-      }
+      };
+      if (!part) plus(xr);
+      if (bias) plus(bias);
       return v;
     }
     float* f = &v.x;

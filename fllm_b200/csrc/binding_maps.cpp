@@ -27,7 +27,7 @@ inline void check_pools(const Tensor& k, const Tensor& v, at::ScalarType ty, int
               "pools: [blocks, heads (or twice as many), block_size, width] of one type");
 }
 
-// x [T, >= all segments], or its split-K partial sums [splits][T][width] (bias added here)
+// x [T, >= all segments], or its split-K partial sums [splits][T][width]; bias (optional) [width] is added
 void maps_prepare(const optional<Tensor>& x, const optional<Tensor>& workspace, int64_t splits, int64_t width, const optional<Tensor>& bias,
                   int64_t q_offset, int64_t k_offset, int64_t v_offset, int64_t dim, int64_t v_dim, const Tensor& positions, const Tensor& slots,
                   const Tensor& inv_freq, double rope_factor, const Tensor& q_norm, const Tensor& k_norm, bool full, double eps, Tensor q_out,
@@ -48,13 +48,13 @@ void maps_prepare(const optional<Tensor>& x, const optional<Tensor>& workspace, 
                 "workspace too small for the split-K partials");
     p.partials = reinterpret_cast<const float*>(reinterpret_cast<const uint8_t*>(workspace->data_ptr()) + fllm::kLinearPartialsOffset);
     p.splits = (int)splits, p.width = (int)width, p.plane = T * width;
-    if (given(bias)) {
-      TORCH_CHECK(bias->is_cuda() && bias->scalar_type() == ty && bias->is_contiguous() && bias->numel() >= end, "bias: [width]");
-      p.bias = bias->data_ptr();
-    }
   } else {
     TORCH_CHECK(given(x) && rows_of(*x, ty) && x->size(0) == T && x->size(1) >= end, "x: [T, >= all segments]");
     p.x = x->data_ptr(), p.ldx = x->stride(0);
+  }
+  if (given(bias)) {
+    TORCH_CHECK(bias->is_cuda() && bias->scalar_type() == ty && bias->is_contiguous() && bias->numel() >= end, "bias: [width]");
+    p.bias = bias->data_ptr();
   }
   p.q_offset = (int)q_offset, p.k_offset = (int)k_offset, p.v_offset = (int)v_offset, p.q_heads = (int)HQ, p.k_heads = (int)HK, p.v_heads = (int)G;
   p.dim = (int)dim, p.v_dim = (int)v_dim, p.wk = (int)k_cache.size(3), p.wv = (int)v_cache.size(3), p.block_size = (int)k_cache.size(2), p.tokens = (int)T;

@@ -73,7 +73,7 @@ void mamba2_scan(const Tensor& x, const Tensor& dt, const Tensor& Bm, const Tens
 // chunked: q' = q (activations applied), the sequences with at least min_tokens tokens, over chunks on the tensor cores. Otherwise
 // q' = silu(q), the sequences below skip_from (0: all), token by token.
 void decay_scan(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& decay, Tensor state, const Tensor& q_starts,
-                const Tensor& seq_state, const Tensor& positions, Tensor out, int64_t H, int64_t K, int64_t V, bool chunked, int64_t from) {
+                const Tensor& seq_state, const Tensor& positions, Tensor out, int64_t H, int64_t K, int64_t V, bool chunked, int64_t from, int64_t max_q_len) {
   const auto ty = act_type(v);
   TORCH_CHECK(rows_of(q, ty) && rows_of(k, ty) && rows_of(v, ty) && rows_of(out, ty), "activations: rows of one type");
   TORCH_CHECK(q.size(1) == H * K && k.size(1) == H * K && v.size(1) == H * V && out.size(1) >= H * V && out.size(0) == v.size(0) && decay.numel() == H, "widths");
@@ -89,6 +89,7 @@ void decay_scan(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor&
   p.B = (int)seq_state.numel(), p.tokens = (int)v.size(0), p.H = (int)H, p.P = (int)V, p.G = (int)H, p.N = (int)K;
   p.f32 = ty == at::kFloat ? 1 : 0;
   p.skip_from = chunked ? 0 : (int)from;
+  p.max_q_len = (int)max_q_len;
   const int rc = chunked ? fllm::decay_chunk(p, (int)from, cur_stream()) : fllm::ssd_scan(p, cur_stream());
   TORCH_CHECK(rc == 0, "decay_scan: unsupported arguments (code ", rc, "): key width up to 256; chunked: bf16, widths in multiples of 8, keys up to 128, aligned rows");
 }
@@ -178,7 +179,7 @@ TORCH_LIBRARY_FRAGMENT(fllm_b200, m) {
         "Tensor seq_state, Tensor positions, Tensor(b!) y, int H, int P, int G, int N, float dt_min, float dt_max, int skip_from) -> ()",
         &mamba2_scan);
   m.def("decay_scan(Tensor q, Tensor k, Tensor v, Tensor decay, Tensor(a!) state, Tensor q_starts, Tensor seq_state, Tensor positions, Tensor(b!) out, "
-        "int H, int K, int V, bool chunked, int from_tokens) -> ()", &decay_scan);
+        "int H, int K, int V, bool chunked, int from_tokens, int max_q_len) -> ()", &decay_scan);
   m.def("mamba1_scan(Tensor x, Tensor dt, Tensor Bm, Tensor Cm, Tensor? z, Tensor A, Tensor? D, Tensor? dt_bias, Tensor(a!) state, "
         "Tensor q_starts, Tensor seq_state, Tensor positions, Tensor(b!) y, int seg_len, int segs, Tensor? seg_scratch) -> ()",
         &mamba1_scan);

@@ -530,25 +530,47 @@ __global__ void glu_kernel(const __nv_bfloat16* __restrict__ x, long long ldx,
       if (act_kind == 2) return 2 * f + (up ? 1 : 0);
       return f + (up ? inter : 0);
     };
-    int cg[8], cu[8];
+    if (!ws && layout == 16) {                               // eight neighbours of one block: 16 bytes each
+      const uint4 a = *reinterpret_cast<const uint4*>(xr + col(0, false)), b = *reinterpret_cast<const uint4*>(xr + col(0, true));
+      const uint32_t aw[4] = {a.x, a.y, a.z, a.w}, bw[4] = {b.x, b.y, b.z, b.w};
 #pragma unroll
-    for (int j = 0; j < 8; ++j) { cg[j] = col(j, false); cu[j] = col(j, true); }
-    if (!ws) {
+      for (int j = 0; j < 4; ++j) {
+        const float2 f = unpack_bf16x2(aw[j]), h = unpack_bf16x2(bw[j]);
+        g[2 * j] = f.x, g[2 * j + 1] = f.y, u[2 * j] = h.x, u[2 * j + 1] = h.y;
+      }
+    } else if (!ws) {
 #pragma unroll
-      for (int j = 0; j < 8; ++j) { g[j] = __bfloat162float(xr[cg[j]]); u[j] = __bfloat162float(xr[cu[j]]); }
+      for (int j = 0; j < 8; ++j) { g[j] = __bfloat162float(xr[col(j, false)]); u[j] = __bfloat162float(xr[col(j, true)]); }
     } else {
       const size_t plane = (size_t)rows * 2 * inter;
       const float* src = ws + (size_t)row * 2 * inter;
 #pragma unroll
-      for (int j = 0; j < 8; ++j) { g[j] = __ldcg(src + cg[j]); u[j] = __ldcg(src + cu[j]); }
-#pragma unroll 2
-      for (int sp = 1; sp < splits; ++sp) {
+      for (int j = 0; j < 8; ++j) g[j] = u[j] = 0.f;
+      if (act_kind != 2 || layout == 16) {                    // gate and up values: eight neighbours each
+        const float *sg = src + col(0, false), *su = src + col(0, true);
+#pragma unroll 4
+        for (int sp = 0; sp < splits; ++sp) {
 #pragma unroll
-        for (int j = 0; j < 8; ++j) { g[j] += __ldcg(src + sp * plane + cg[j]); u[j] += __ldcg(src + sp * plane + cu[j]); }
+          for (int j = 0; j < 8; j += 4) {
+            const float4 a = __ldcg(reinterpret_cast<const float4*>(sg + sp * plane + j)), b = __ldcg(reinterpret_cast<const float4*>(su + sp * plane + j));
+            g[j] += a.x, g[j + 1] += a.y, g[j + 2] += a.z, g[j + 3] += a.w;
+            u[j] += b.x, u[j + 1] += b.y, u[j + 2] += b.z, u[j + 3] += b.w;
+          }
+        }
+      } else {                                                // pairs
+        const float* sp0 = src + 2 * i8;
+#pragma unroll 4
+        for (int sp = 0; sp < splits; ++sp) {
+#pragma unroll
+          for (int j = 0; j < 8; j += 2) {
+            const float4 a = __ldcg(reinterpret_cast<const float4*>(sp0 + sp * plane + 2 * j));
+            g[j] += a.x, u[j] += a.y, g[j + 1] += a.z, u[j + 1] += a.w;
+          }
+        }
       }
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
-        if (bias) { g[j] += __bfloat162float(bias[cg[j]]); u[j] += __bfloat162float(bias[cu[j]]); }
+        if (bias) { g[j] += __bfloat162float(bias[col(j, false)]); u[j] += __bfloat162float(bias[col(j, true)]); }
         g[j] = __bfloat162float(__float2bfloat16(g[j]));
         u[j] = __bfloat162float(__float2bfloat16(u[j]));
       }
@@ -580,7 +602,7 @@ __global__ void glu_kernel(const __nv_bfloat16* __restrict__ x, long long ldx,
 #pragma unroll
   for (int j = 0; j < 8; ++j) {
     if (act_kind == 0) {
-      o[j] = g[j] / (1.f + __expf(-g[j])) * u[j];
+      o[j] = __fdividef(g[j], 1.f + __expf(-g[j])) * u[j];
     } else if (act_kind == 1) {
       const float c = 0.7978845608028654f * (g[j] + 0.044715f * g[j] * g[j] * g[j]);
       o[j] = 0.5f * g[j] * (1.f + tanhf(c)) * u[j];

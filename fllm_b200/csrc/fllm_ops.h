@@ -296,6 +296,7 @@ struct SsdScanParams {
   int B, tokens, H, P, G, N;   // tokens: rows of the step (= B: single tokens)
   float dt_min, dt_max;
   int skip_from, f32;
+  int max_q_len;               // decay_chunk: host-side bound on a sequence's tokens in the step
 };
 int ssd_scan(const SsdScanParams& p, cudaStream_t stream);
 // Lightning attention over chunks on the tensor cores (recurrent_chunk.cu), bf16: the sequences with at least min_tokens tokens in
@@ -461,10 +462,10 @@ int attention_tied(const TiedAttnParams& p, int splits, void* workspace, size_t 
 struct MapsPrepareParams {
   const void* x;               // [tokens] rows: query maps from column q_offset, key maps from k_offset, values from v_offset
   long long ldx;
-  const float* partials;       // not null: the rows are the sums of split-K partials [splits][tokens][width] (plus bias), `plane` elements per split
+  const float* partials;       // not null: the rows are the sums of split-K partials [splits][tokens][width], `plane` elements per split
   int splits, width;
   long long plane;
-  const void* bias;            // [width], with partials only
+  const void* bias;            // optional [width], added to the rows
   int q_offset, k_offset, v_offset, q_heads, k_heads, v_heads, dim, v_dim, wk, wv, block_size, tokens;
   const int *positions, *slots;
   const float* inv_freq;       // [rot / 2]: pairs (i, i + rot / 2) of a map's first rot values turn

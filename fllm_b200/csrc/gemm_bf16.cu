@@ -320,14 +320,14 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a,
       __nv_bfloat16* stg = stage_out + (warp - 2) * (32 * 32);
       // gated activation of one (gate, up) pair
       auto gated = [&](float g, float u) -> float {
-        if (p.glu == 1) return g / (1.f + __expf(-g)) * u;
+        if (p.glu == 1) return __fdividef(g, 1.f + __expf(-g)) * u;
         if (p.glu == 2) {
           const float c = 0.7978845608028654f * (g + 0.044715f * g * g * g);
           return 0.5f * g * (1.f + tanhf(c)) * u;
         }
         const float gg = fminf(g, p.glu_limit);
         const float uu = fminf(fmaxf(u, -p.glu_limit), p.glu_limit);
-        return gg / (1.f + __expf(-p.glu_alpha * gg)) * (uu + 1.f);
+        return __fdividef(gg, 1.f + __expf(-p.glu_alpha * gg)) * (uu + 1.f);
       };
       // final values of CH columns of this thread's row -> bias, (activation,) bf16, memory
       auto emit = [&](int c0, const float (&v)[32]) {

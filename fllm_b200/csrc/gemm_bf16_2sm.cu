@@ -192,14 +192,14 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tma_x, const __grid_co
       const uint32_t t_row = tmem_base + buf * P2_TILE + ((uint32_t)(q * 32) << 16);
       __nv_bfloat16* dst = p.out + (size_t)m * p.ldc + n_base;
       auto gated = [&](float g, float u) -> float {
-        if (p.glu == 1) return g / (1.f + __expf(-g)) * u;
+        if (p.glu == 1) return __fdividef(g, 1.f + __expf(-g)) * u;
         if (p.glu == 2) {
           const float c = 0.7978845608028654f * (g + 0.044715f * g * g * g);
           return 0.5f * g * (1.f + tanhf(c)) * u;
         }
         const float gg = fminf(g, p.glu_limit);
         const float uu = fminf(fmaxf(u, -p.glu_limit), p.glu_limit);
-        return gg / (1.f + __expf(-p.glu_alpha * gg)) * (uu + 1.f);
+        return __fdividef(gg, 1.f + __expf(-p.glu_alpha * gg)) * (uu + 1.f);
       };
 #pragma unroll 1
       for (int c0 = 0; c0 < P2_TILE; c0 += 32) {

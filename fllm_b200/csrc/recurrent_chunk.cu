@@ -7,6 +7,8 @@
 // state stays in registers as fp32 accumulators; for the products it travels as the sum of two bf16 values, like the weights
 // d^(i-j) (q_i . k_j); the decayed values of the state's update travel as the sum of three (24 significant bits). q, k and v
 // (bf16, activations applied) are exact operands. States and batch layout as in recurrent_ssd.cu (rows [slot][head][V][K]).
+#include <algorithm>
+
 #include "attention_util.cuh"
 #include "fllm_ops.h"
 #include "ptx.cuh"
@@ -254,7 +256,8 @@ int decay_chunk(const SsdScanParams& p, int min_tokens, cudaStream_t s) {
   const ChunkArgs a{static_cast<const bf16*>(p.Cm), static_cast<const bf16*>(p.Bm), static_cast<const bf16*>(p.x), p.ldc, p.ldb, p.ldx, p.ldy, p.A,
                     p.state, p.q_starts, p.seq_state, p.positions, static_cast<bf16*>(p.y), p.H, p.N, p.P, min_tokens};
   // narrower slices (more CTAs, each with the chunk's scores to itself) as long as two CTAs per SM hold them all
-  const bool narrow = (long long)p.H * ((p.P + 15) / 16) * p.B <= 2 * sm_count();
+  const int longest = std::max(p.max_q_len, 1), walks = std::min(p.B, (p.tokens + longest - 1) / longest);      // about as many as run that long
+  const bool narrow = (long long)p.H * ((p.P + 15) / 16) * walks <= 2 * sm_count();
   if (p.N <= 64) narrow ? launch_chunk<64, 16>(a, p.B, s) : launch_chunk<64, 32>(a, p.B, s);
   else narrow ? launch_chunk<128, 16>(a, p.B, s) : launch_chunk<128, 32>(a, p.B, s);
   cuda_check(cudaGetLastError(), "decay_chunk_kernel");

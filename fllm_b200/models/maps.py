@@ -23,14 +23,14 @@ def _attend(dec, li: int, m, proj, b) -> torch.Tensor:
     inv_freq, factor = dec.layer_rope(c["rope"])
     nq, nk = pad8(H * M * dim), pad8(G * M * dim)
     q = ops.maps_prepare(proj, (0, nq, nq + nk), H * M, dim, v_dim, b.positions, b.slots, inv_freq, factor, m["q_norm"], m["k_norm"],
-                         c["qk_norm"] == "full", eps, keys, values)
+                         c["qk_norm"] == "full", eps, keys, values, m.get("in_bias"))
     combine = Combine(m["lam"], 1.0 - c["diff"], eps) if M == 2 else None
     return ops.attention_maps(q, keys, values, dim, v_dim, b, c["scale"], c["window"], combine, m["wo"].shape[1])
 
 
 def maps_mixer(dec, li: int, lw, h: torch.Tensor, b):
     m, ops = lw.mixer, dec.ops
-    proj = ops.linear(h, m["in_proj"], m.get("in_bias"), defer=dec.defer_to_residual)
+    proj = ops.linear(h, m["in_proj"], defer=dec.defer_to_residual)
     return ops.linear(_attend(dec, li, m, proj, b), m["wo"], defer=dec.defer_to_residual)
 
 
@@ -38,7 +38,7 @@ def maps_lightning_mixer(dec, li: int, lw, h: torch.Tensor, b) -> NormedPair:
     m, ops, s = lw.mixer, dec.ops, dec.cfg.attn_of(li)
     qs, ss, pos = _batch_meta(b)
     H, K, V = s["lin_heads"], s["lin_k_dim"], s["lin_v_dim"]
-    proj = ops.linear(h, m["in_proj"], m.get("in_bias"))
+    proj = ops.linear(h, m["in_proj"])
     ya = ops.linear(_attend(dec, li, m, proj, b), m["wo"])
     at, nk = m["lin_offset"], pad8(H * K)
     q, k, v = proj[:, at:at + H * K], proj[:, at + nk:at + nk + H * K], proj[:, at + 2 * nk:at + 2 * nk + H * V]

@@ -49,15 +49,16 @@ def _rms(x, eps):
 
 
 class MapsRef:
-    def maps_prepare(self, x, offsets, heads, dim, v_dim, positions, slots, inv_freq, rope_factor, q_norm, k_norm, full, eps, k_cache, v_cache):
-        """``x`` [T, ...]: query maps at column offsets[0], key maps at offsets[1], values at offsets[2]. Norms (over a map, or with
+    def maps_prepare(self, x, offsets, heads, dim, v_dim, positions, slots, inv_freq, rope_factor, q_norm, k_norm, full, eps, k_cache, v_cache, bias=None):
+        """``x`` [T, ...] (plus ``bias``): query maps at column offsets[0], key maps at offsets[1], values at offsets[2]. Norms (over a map, or with
         ``full`` over all maps at once), rotates the first 2 len(inv_freq) values of every map, writes the tokens' cache rows
         (slot < 0: none) and returns the queries [T, heads, W], padded like the key rows."""
         T, W, bs = x.shape[0], k_cache.shape[3], k_cache.shape[2]
         rot = 2 * inv_freq.numel()
+        x = x.float() if bias is None else x.float() + bias.float()
 
         def part(off, n, w):
-            t = x[:, off:off + n * dim].float()
+            t = x[:, off:off + n * dim]
             t = _rms(t, eps) * w.float() if full else _rms(t.reshape(T, n, dim), eps) * w.float()
             t = t.reshape(T, n, dim)
             return F.pad(torch.cat([_rotate(t[..., :rot], positions, inv_freq, rope_factor, 0), t[..., rot:]], -1), (0, W - dim)).to(k_cache.dtype)
@@ -111,10 +112,11 @@ class MapsNative:
     """Kernel wrappers; ``self.k`` is the loaded extension and ``self.launches`` the launch counter of the ops object. The
     projection ``maps_prepare`` reads may be deferred: its split-K partial sums are added by the kernel."""
 
-    def maps_prepare(self, x, offsets, heads, dim, v_dim, positions, slots, inv_freq, rope_factor, q_norm, k_norm, full, eps, k_cache, v_cache):
+    def maps_prepare(self, x, offsets, heads, dim, v_dim, positions, slots, inv_freq, rope_factor, q_norm, k_norm, full, eps, k_cache, v_cache, bias=None):
         T, splits = x.shape[0], getattr(x, "splits", 0)
+        bias = bias if bias is not None or not splits else x.bias
         q = torch.empty(T, heads, k_cache.shape[3], dtype=k_cache.dtype, device=k_cache.device)
-        self.k.maps_prepare(None if splits else x, self.workspace if splits else None, int(splits), int(x.shape[1]), x.bias if splits else None,
+        self.k.maps_prepare(None if splits else x, self.workspace if splits else None, int(splits), int(x.shape[1]), bias,
                             int(offsets[0]), int(offsets[1]), int(offsets[2]), int(dim), int(v_dim), positions, slots, inv_freq, float(rope_factor), q_norm,
                             k_norm, bool(full), float(eps), q, k_cache, v_cache)
         self.launches += 1
@@ -151,7 +153,7 @@ class MapsNative:
         aligned = all(t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in (q, k, v)) and out.stride(0) % 2 == 0
         chunks = chunk_from > 0 and max_q_len >= chunk_from and v.dtype == torch.bfloat16 and aligned and K % 8 == 0 and V % 8 == 0 and K <= 128
         if not chunks or min_q_len < chunk_from:
-            self.k.decay_scan(q, k, v, *args, False, int(chunk_from) if chunks else 0)
+            self.k.decay_scan(q, k, v, *args, False, int(chunk_from) if chunks else 0, 0)
             self.launches += 1
         if chunks:
             ld, at = q.stride(0), q.data_ptr()
@@ -160,6 +162,6 @@ class MapsNative:
             else:
                 for t in (q, k, v):
                     self.act_(t, "silu")
-            self.k.decay_scan(q, k, v, *args, True, int(chunk_from))
+            self.k.decay_scan(q, k, v, *args, True, int(chunk_from), int(max_q_len))
             self.launches += 1
         return out
