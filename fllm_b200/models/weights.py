@@ -393,7 +393,8 @@ def init_random_weights(cfg: ModelConfig, device="cpu", dtype=torch.bfloat16, se
             I = cfg.intermediate_size
             g = full((I, H), li, 4)
             u = full((I, H), li, 5)
-            isl = slice(sp.inter_start, sp.inter_start + sp.inter_local)
+            i0, il = (tp_rank * (I // tp), I // tp) if cfg.is_moe else (sp.inter_start, sp.inter_local)      # (the spec's is the experts' width)
+            isl = slice(i0, i0 + il)
             lw.w_gate_up = torch.cat([g[isl], u[isl]], 0).contiguous()
             lw.w_down = full((H, I), li, 6)[:, isl].contiguous()
         pack_layer(lw, weight_format)
