@@ -288,31 +288,40 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const SsdArgs<T> a) {
   }
 }
 
-template <typename T, int NP, bool EXACT, bool LIN>
+// RPT: state rows per thread
+template <typename T, int NP, bool EXACT, bool LIN, int RPT>
 __global__ void __launch_bounds__(128) ssd_decode_kernel(const SsdArgs<T> a) {
   pdl_launch_dependents();
   pdl_wait();
-  constexpr int NPT = 16, TPK = NP / NPT, ROWS = 128 / TPK;
+  constexpr int NPT = 16, TPK = NP / NPT, RG = 128 / TPK, ROWS = RPT * RG;
   const int N = EXACT ? NP : a.N;
   const int ptiles = (a.P + ROWS - 1) / ROWS;
-  const int h = blockIdx.x / ptiles, p = (blockIdx.x % ptiles) * ROWS + threadIdx.x / TPK;
+  const int h = blockIdx.x / ptiles, p0 = (blockIdx.x % ptiles) * ROWS + threadIdx.x / TPK;      // rows p0 + RG r
   const int lk = threadIdx.x % TPK, s = blockIdx.y;
   const int t0 = a.q_starts[s], n = a.q_starts[s + 1] - t0;
   if (n <= 0 || (a.skip_from > 0 && n >= a.skip_from)) return;
-  const int pc = min(p, a.P - 1);
-  float* st = a.state + (((long long)a.seq_state[s] * a.H + h) * a.P + pc) * N;
-  float S[NPT];
+  float* st = a.state + ((long long)a.seq_state[s] * a.H + h) * a.P * N;
+  auto row = [&](int r) { return min(p0 + RG * r, a.P - 1); };
+  float S[RPT][NPT];
 #pragma unroll
-  for (int i = 0; i < NPT; ++i) S[i] = 0.f;
-  if (a.positions[t0] != 0) load_state<TPK, EXACT>(st, lk, N, S);
+  for (int r = 0; r < RPT; ++r)
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) S[r][i] = 0.f;
+  if (a.positions[t0] != 0) {
+#pragma unroll
+    for (int r = 0; r < RPT; ++r) load_state<TPK, EXACT>(st + (long long)row(r) * N, lk, N, S[r]);
+  }
   const float A = a.A[h], D = a.D != nullptr ? a.D[h] : 0.f, dtb = a.dt_bias != nullptr ? a.dt_bias[h] : 0.f;
   const long long go = (long long)(h / (a.H / a.G)) * N;
   for (long long t = t0; t < t0 + n; ++t) {
     const T *bp = a.Bm + t * a.ldb + go, *cp = a.Cm + t * a.ldc + go;
+    float xv[RPT];
+#pragma unroll
+    for (int r = 0; r < RPT; ++r) xv[r] = ld1(a.x + t * a.ldx + (long long)h * a.P + row(r));
     float B[NPT], C[NPT];
     if constexpr (LIN) {                                   // the activations once per CTA
       __shared__ __align__(16) float sb[NP], sc[NP];
-      __syncthreads();
+      if (t > t0) __syncthreads();
       for (int i = threadIdx.x; i < NP; i += 128) sb[i] = i < N ? silu_t<T>(ld1(bp + i)) : 0.f, sc[i] = i < N ? silu_t<T>(ld1(cp + i)) : 0.f;
       __syncthreads();
 #pragma unroll
@@ -323,39 +332,42 @@ __global__ void __launch_bounds__(128) ssd_decode_kernel(const SsdArgs<T> a) {
       }
     } else {
 #pragma unroll
-    for (int j = 0; j < NPT / 4; ++j) {
-      const int c = 4 * (lk + TPK * j);
+      for (int j = 0; j < NPT / 4; ++j) {
+        const int c = 4 * (lk + TPK * j);
 #pragma unroll
-      for (int e = 0; e < 4; e += 2) {
-        float2 b2 = make_float2(0.f, 0.f), c2 = b2;
-        if (EXACT) {
-          b2 = ld2(bp + c + e), c2 = ld2(cp + c + e);
-        } else {
-          if (c + e < N) b2.x = ld1(bp + c + e), c2.x = ld1(cp + c + e);
-          if (c + e + 1 < N) b2.y = ld1(bp + c + e + 1), c2.y = ld1(cp + c + e + 1);
+        for (int e = 0; e < 4; e += 2) {
+          float2 b2 = make_float2(0.f, 0.f), c2 = b2;
+          if (EXACT) {
+            b2 = ld2(bp + c + e), c2 = ld2(cp + c + e);
+          } else {
+            if (c + e < N) b2.x = ld1(bp + c + e), c2.x = ld1(cp + c + e);
+            if (c + e + 1 < N) b2.y = ld1(bp + c + e + 1), c2.y = ld1(cp + c + e + 1);
+          }
+          B[4 * j + e] = b2.x, B[4 * j + e + 1] = b2.y, C[4 * j + e] = c2.x, C[4 * j + e + 1] = c2.y;
         }
-        B[4 * j + e] = b2.x, B[4 * j + e + 1] = b2.y, C[4 * j + e] = c2.x, C[4 * j + e + 1] = c2.y;
       }
     }
+    float d = A, dt = 1.f;
+    if constexpr (!LIN) {
+      dt = fminf(fmaxf(softplus_t<T>(ld1(a.dt + t * a.lddt + h) + dtb), a.dt_min), a.dt_max);
+      d = exp_t<T>(dt * A);
     }
-    float d = A, u = ld1(a.x + t * a.ldx + (long long)h * a.P + pc);
-    const float xv = u;
-    if constexpr (LIN) {
-      u = silu_t<T>(u);
-    } else {
-      const float dt = fminf(fmaxf(softplus_t<T>(ld1(a.dt + t * a.lddt + h) + dtb), a.dt_min), a.dt_max);
-      d = exp_t<T>(dt * A), u = dt * xv;
-    }
-    float o[2] = {0.f, 0.f};
 #pragma unroll
-    for (int i = 0; i < NPT; ++i) {
-      S[i] = fmaf(B[i], u, d * S[i]);
-      o[i & 1] = fmaf(S[i], C[i], o[i & 1]);
+    for (int r = 0; r < RPT; ++r) {
+      const float u = LIN ? silu_t<T>(xv[r]) : dt * xv[r];
+      float o[2] = {0.f, 0.f};
+#pragma unroll
+      for (int i = 0; i < NPT; ++i) {
+        S[r][i] = fmaf(B[i], u, d * S[r][i]);
+        o[i & 1] = fmaf(S[r][i], C[i], o[i & 1]);
+      }
+      const float tot = row_sum<TPK>(o[0] + o[1]);
+      if (lk == 0 && p0 + RG * r < a.P) st1(a.y + t * a.ldy + (long long)h * a.P + p0 + RG * r, fmaf(D, xv[r], tot));
     }
-    const float tot = row_sum<TPK>(o[0] + o[1]);
-    if (lk == 0 && p < a.P) st1(a.y + t * a.ldy + (long long)h * a.P + p, fmaf(D, xv, tot));
   }
-  if (p < a.P) store_state<TPK, EXACT>(st, lk, N, S);
+#pragma unroll
+  for (int r = 0; r < RPT; ++r)
+    if (p0 + RG * r < a.P) store_state<TPK, EXACT>(st + (long long)(p0 + RG * r) * N, lk, N, S[r]);
 }
 }  // namespace
 
@@ -374,10 +386,10 @@ int ssd_scan(const SsdScanParams& p, cudaStream_t stream) {
   // few sequences and heads: two rows per thread instead of four, so that twice as many SMs work
 #define FLLM_SSD(T_, NP_, EXACT_, LIN_)                                                                                     \
   {                                                                                                                   \
-    constexpr int drows = 128 / (NP_ / 16), rows4 = SsdTile<NP_, 4>::ROWS, rows2 = SsdTile<NP_, 2>::ROWS;             \
+    constexpr int drpt = LIN_ ? 2 : 1, drows = drpt * 128 / (NP_ / 16), rows4 = SsdTile<NP_, 4>::ROWS, rows2 = SsdTile<NP_, 2>::ROWS;             \
     const int tiles4 = p.H * ((p.P + rows4 - 1) / rows4), tiles2 = p.H * ((p.P + rows2 - 1) / rows2);                 \
     if (p.tokens == p.B)                                                                                              \
-      launch_pdl(ssd_decode_kernel<T_, NP_, EXACT_, LIN_>, dim3(p.H * ((p.P + drows - 1) / drows), p.B), dim3(128), 0, stream, args(T_{}));  \
+      launch_pdl(ssd_decode_kernel<T_, NP_, EXACT_, LIN_, drpt>, dim3(p.H * ((p.P + drows - 1) / drows), p.B), dim3(128), 0, stream, args(T_{}));  \
     else if (2LL * tiles4 * p.B <= sm_count() && tiles2 > tiles4)                                                     \
       launch_pdl(ssd_scan_kernel<T_, NP_, EXACT_, 2, LIN_>, dim3(tiles2, p.B), dim3(128), 0, stream, args(T_{}));           \
     else                                                                                                              \
