@@ -308,7 +308,7 @@ def test_norm_before_a_sigmoid_gate(ops, D, width, dtype):
 
 # ------------------------------------------------------------------------------------------------ feed-forward, head
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("T,W,E,top,ff,shared", [(1, 64, 6, 2, 32, 48), (37, 200, 12, 1, 48, 0), (300, 256, 7, 7, 16, 32), (64, 128, 40, 5, 32, 64), (5, 24, 1, 1, 16, 16)])
+@pytest.mark.parametrize("T,W,E,top,ff,shared", [(1, 64, 6, 2, 32, 48), (37, 200, 12, 1, 48, 0), (300, 256, 7, 7, 16, 32), (64, 128, 40, 5, 32, 64), (5, 24, 1, 1, 16, 16), (6, 64, 300, 9, 16, 0)])
 def test_routed_experts_weigh_their_input(ops, T, W, E, top, ff, shared, dtype):
     from fllm_b200.models.decoder import Decoder
     from fllm_b200.models.weights import LayerWeights
