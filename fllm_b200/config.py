@@ -47,6 +47,9 @@ class MoeSpec:
     act: str = "swiglu"
     weigh_input: bool = False
     fp32_router: bool = False            # the router's logits stay fp32 (otherwise they take the activation type)
+    masked: float = 0.0                  # what the choice score of an expert outside the kept groups becomes
+    limit: Optional[float] = None        # clamp of the experts' activation (None: the model's)
+    shared_limit: Optional[float] = None # the same of the shared expert's
 
 
 @dataclass
@@ -120,7 +123,7 @@ class ModelConfig:
     layer_kinds: Optional[List[str]] = None      # attention | mla | tied | maps | mamba1 | mamba2 | gated_delta | shortconv | none (FFN-only block)
                                                  # | attention+mamba2 (both read the block's input, their outputs add: Falcon-H1)
                                                  # | maps+lightning (the same, each output normalised, their mean: models.maps)
-    ffn_kinds: Optional[List[str]] = None        # glu | moe | none
+    ffn_kinds: Optional[List[str]] = None        # glu | plain (two matrices in a model of gated networks) | moe | none
     ssm: Dict[str, Any] = field(default_factory=dict)
     # multi-head latent attention (layer kind "mla"): q_lora_rank (0 = one query projection), kv_lora_rank,
     # qk_nope_head_dim, qk_rope_head_dim, v_head_dim; head_dim is then qk_nope + qk_rope and rotary_dim qk_rope
@@ -128,8 +131,10 @@ class ModelConfig:
     # per layer: shapes that differ from layer to layer, laid over `ssm` (recurrent kinds) or `mla` (kind "mla"; there also
     # num_heads, scale, rope_theta, rope_style, head_gate, and kv_from = the layer whose cached rows this one attends to); for
     # kind "tied" all of num_heads, num_kv_heads, head_dim, scale, softcap, temp_coef, temp_every, norm_eps; for kind "maps"
-    # num_heads, num_kv_heads, head_dim, v_dim, maps, window, scale, rope (dims, theta, scaling), qk_norm ("head" | "full"), and
-    # with two maps diff; for "maps+lightning" those and lin_heads, lin_k_dim, lin_v_dim, lin_decay
+    # num_heads, num_kv_heads, head_dim, v_dim, maps, window, scale, rope (dims, theta, scaling; None: no rotation), rope_style
+    # ("neox" | "pair"), qk_norm ("head" | "full" | "unit": without weights | "none"), with two maps diff, with one map conv (taps of a
+    # convolution over the projections), talk (the heads mix their weights) and gate (per head); for "maps+lightning" those and
+    # lin_heads, lin_k_dim, lin_v_dim, lin_decay
     layer_mixers: Optional[List[Dict[str, Any]]] = None
     # per layer: width and activation limit of a feed-forward network that differs from layer to layer (ff, limit), or its
     # routed experts (experts, top, ff, shared_ff, router ...: the fields of MoeSpec)
@@ -138,6 +143,14 @@ class ModelConfig:
     postnorm_alpha: float = 0.0
     # the residual is fp32 and a sublayer reads it as it is; its output is normalised before it is added, x <- x + rms(f(x)) w
     outnorm: bool = False
+    # the residual is fp32 and a sublayer reads its norm, x <- x + f(norm(x)); token_shift: every mixer reads its normed input moved
+    # towards that of the token before, by a learned step per channel
+    prenorm_fp32: bool = False
+    token_shift: bool = False
+    # looped models: the checkpoint layer that every layer of the running order takes its weights from (None: as many layers as the
+    # checkpoint has), and the places in that order where the token embeddings are added to the residual again
+    layer_source: Optional[List[int]] = None
+    embed_again: List[int] = field(default_factory=list)
     # > 0: behind every layer a token's own embedding of that width (one table, a slice per layer) is gated by the residual,
     # projected, normalised and added
     token_side_dim: int = 0
@@ -176,7 +189,12 @@ class ModelConfig:
 
     @property
     def has_recurrent(self) -> bool:
-        return bool(self.layer_kinds) and any(k not in STATELESS_KINDS for k in self.layer_kinds)
+        """Whether a sequence carries a state of fixed size beside its cache rows."""
+        return bool(self.layer_kinds) and (self.token_shift or any(k not in STATELESS_KINDS or self.conv_taps(i) > 1 for i, k in enumerate(self.layer_kinds)))
+
+    def conv_taps(self, layer: int) -> int:
+        """Taps of the convolution over an attention layer's projections (0: none)."""
+        return self.layer_mixers[layer].get("conv", 0) if self.layer_mixers and self.layer_kind(layer) == "maps" else 0
 
     def ssm_of(self, layer: int) -> Dict[str, Any]:
         """Shapes of a recurrent layer."""
@@ -226,14 +244,14 @@ class ModelConfig:
             return "latent"
         if self.postnorm_alpha > 0 and all(k in ("mamba2", "tied") for k in kinds):
             return "tied"
-        if self.outnorm and all(k in ("maps", "maps+lightning") for k in kinds):
+        if (self.outnorm or self.prenorm_fp32) and all(k in ("maps", "maps+lightning") for k in kinds):
             return "maps"
         return ""
 
     @property
     def fp32_residual(self) -> bool:
         """Families whose residual is one or several fp32 streams with an update kernel of their own."""
-        return self.residual_streams > 0 or self.postnorm_alpha > 0 or self.outnorm
+        return self.residual_streams > 0 or self.postnorm_alpha > 0 or self.outnorm or self.prenorm_fp32
 
     @property
     def has_mla(self) -> bool:
@@ -285,6 +303,8 @@ class ModelConfig:
             return divanex_from_config(cls, hf)
         if hf.get("architecture") == "Dorevik":
             return dorevik_from_config(cls, hf)
+        if hf.get("architecture") == "Milenex":
+            return milenex_from_config(cls, hf)
         mt = hf.get("model_type", "llama")
         if mt in ("glm4_moe_lite", "kimi_k2", "youtu"):    # DeepSeek-V3 under another name (Youtu: its dense form): the same tensors, router and latent attention
             hf = dict(hf, model_type="deepseek_v3")
@@ -721,6 +741,76 @@ def dorevik_from_config(cls, c: Dict[str, Any]) -> "ModelConfig":
                logit_softcap=float(c.get("logit_softcap") or 0.0))
 
 
+def _running_order(c: Dict[str, Any]) -> "tuple[List[int], List[int]]":
+    """Layers in running order with the looped ones repeated, and where a repetition begins."""
+    n, loop = len(c["layers"]), c.get("loop") or dict(start=0, stop=0, times=1)
+    start, stop, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+    if not 0 <= start <= stop <= n or times < 1:
+        raise ValueError(f"a loop over layers {start} .. {stop} of {n}, {times} times")
+    order = list(range(stop))
+    again = [] if start == stop else [stop + i * (stop - start) for i in range(times - 1)]
+    for _ in again:
+        order += range(start, stop)
+    return order + list(range(stop, n)), again
+
+
+def _milenex_attention(i: int, kind: str, m: Dict[str, Any]) -> Dict[str, Any]:
+    if m["heads"] % m["kv_heads"]:
+        raise ValueError(f"layer {i}: {m['heads']} query heads over {m['kv_heads']} key heads")
+    if int(m["mask"]["size"]) < 1:
+        raise ValueError(f"layer {i}: a window of {m['mask']['size']} tokens")
+    out = dict(num_heads=m["heads"], num_kv_heads=m["kv_heads"], head_dim=m["dim"], v_dim=m["vdim"], maps=1, window=int(m["mask"]["size"]),
+               scale=float(m["scale"]))
+    if kind == "attention_2":
+        return dict(out, rope=None, qk_norm="none", talk=True, gate=True)
+    rot, taps = m["rot"], int(m["conv"])
+    if not 0 <= rot["dims"] <= m["dim"] or rot["dims"] % 2:
+        raise ValueError(f"layer {i}: a rotation of {rot['dims']} dimensions on heads of {m['dim']}")
+    if not 1 <= taps <= 8:
+        raise ValueError(f"layer {i}: a convolution of {taps} taps (1 to 8)")
+    # (a single tap is a factor per channel; the kernels start at two taps, the earlier one zero)
+    return dict(out, rope=dict(dims=rot["dims"], theta=float(rot["base"])), rope_style="pair", qk_norm="unit", conv=max(taps, 2), taps=taps)
+
+
+def milenex_from_config(cls, c: Dict[str, Any]) -> "ModelConfig":
+    """Milenex: layers of rotary attention behind short convolutions and of talking-heads attention with a distance bias, in any order,
+    each with sizes of its own and a window with a sink; two-matrix GELU networks or routed clamped SwiGLU experts behind them; a token
+    shift in front of every mixer; a run of layers that is repeated with the same weights."""
+    kinds, ffns, mixers, nets = [], [], [], []
+    for i, layer in enumerate(c["layers"]):
+        mlp = layer.get("mlp")
+        if layer["type"] not in ("attention", "attention_2"):
+            raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
+        kinds.append("maps")
+        mixers.append(_milenex_attention(i, layer["type"], layer["mixer"]))
+        if mlp is None:
+            ffns.append("none")
+            nets.append({})
+        elif mlp["kind"] == "dense":
+            ffns.append("plain")
+            nets.append(dict(ff=mlp["ff"], act="gelu"))
+        elif mlp["kind"] == "moe":
+            r, shared = mlp["router"], mlp.get("shared")
+            groups = r.get("groups") or dict(count=1, keep=1)
+            E, count, keep = r["experts"], groups["count"], groups["keep"]
+            if E % count or not 1 <= keep <= count or not 0 < r["top"] <= E // count * keep:
+                raise ValueError(f"layer {i}: the best {r['top']} of {E} experts in the best {keep} of {count} groups")
+            ffns.append("moe")
+            nets.append(dict(experts=E, top=r["top"], ff=mlp["expert"]["ff"], limit=float(mlp["expert"]["limit"]), shared_ff=shared["ff"] if shared else 0,
+                             shared_limit=float(shared["limit"]) if shared else None, router="deepseek_v2", groups=count, topk_groups=keep,
+                             masked=float("-inf"), act="swiglu_oai", fp32_router=True))
+        else:
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+    order, again = _running_order(c)
+    first = mixers[0]
+    ff = max([n["ff"] for k, n in zip(ffns, nets) if k == "plain"] or [16])
+    return cls(arch="milenex", name=c.get("name") or "milenex", vocab_size=c["vocab"], hidden_size=c["width"], num_layers=len(order),
+               num_heads=first["num_heads"], num_kv_heads=first["num_kv_heads"], head_dim=first["head_dim"], intermediate_size=(ff + 15) // 16 * 16,
+               rms_eps=float(c["norm"]["eps"]), norm_weight_offset=1.0, act="swiglu_oai", use_rope=False, layer_kinds=[kinds[i] for i in order],
+               ffn_kinds=[ffns[i] for i in order], layer_mixers=[mixers[i] for i in order], layer_ffns=[nets[i] for i in order],
+               sliding_window=max(m["window"] for m in mixers), prenorm_fp32=True, token_shift=True, layer_source=order, embed_again=again)
+
+
 RECURRENT_MODEL_TYPES = ("falcon_h1", "nemotron_h", "nemotron_h_moe", "mamba", "falcon_mamba", "mamba2", "bamba", "lfm2", "rwkv7", "qwen3_next", "qwen3_5_text", "qwen3_5_moe_text", "jamba", "granitemoehybrid", "granitemoe", "granitemoeshared", "glm4_moe", "ernie4_5_moe", "rwkv6")
 
 
@@ -1152,6 +1242,21 @@ def preset(name: str) -> ModelConfig:
                        mlp=moe if i % 2 else dense) for i in range(8 if tiny else 24)]
         return dorevik_from_config(ModelConfig, dict(
             architecture="Dorevik", name=n, layers=layers, norm=dict(eps=1e-6), logit_softcap=30.0, vocab=512 if tiny else 65536, width=96 if tiny else 2048))
+    if n in ("milenex-tiny", "milenex-3b"):
+        # talking-heads and rotary layers in turn, experts in all but the first; the first half runs twice
+        tiny = n.endswith("tiny")
+        talking = dict(heads=6 if tiny else 16, kv_heads=3 if tiny else 4, dim=20 if tiny else 96, vdim=12 if tiny else 64, mask=dict(size=21 if tiny else 1024))
+        rotary = dict(heads=4 if tiny else 16, kv_heads=2 if tiny else 4, dim=32 if tiny else 128, vdim=24 if tiny else 128, conv=3 if tiny else 4,
+                      mask=dict(size=37 if tiny else 2048), rot=dict(base=1e4, dims=16 if tiny else 64))
+        for m in (talking, rotary):
+            m["scale"] = m["dim"] ** -0.5
+        moe = dict(kind="moe", expert=dict(ff=40 if tiny else 768, limit=7.0), shared=dict(ff=56 if tiny else 1536, limit=7.0),
+                   router=dict(experts=12 if tiny else 32, top=3 if tiny else 4, groups=dict(count=3 if tiny else 8, keep=2 if tiny else 4)))
+        layers = [dict(type="attention" if i % 2 else "attention_2", mixer=rotary if i % 2 else talking,
+                       mlp=moe if i else dict(kind="dense", ff=150 if tiny else 6144)) for i in range(4 if tiny else 16)]
+        return milenex_from_config(ModelConfig, dict(
+            architecture="Milenex", name=n, layers=layers, loop=dict(start=0, stop=len(layers) // 2, times=2), norm=dict(eps=1e-5),
+            vocab=500 if tiny else 65536, width=72 if tiny else 2048))
     raise KeyError(f"unknown model preset {name!r}")
 
 

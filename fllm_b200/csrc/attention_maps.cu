@@ -1,6 +1,10 @@
 // Attention of one or two maps over shared values, with key and value rows of widths of their own and a sliding window:
 //   a_m = softmax_j(scale q_m . k_m,j) v_j over the keys j with 0 <= i - j < window (window 0: all up to i)
 //   one map: out = a_1;  two maps (differential attention): out = rms(a_1 - lam a_2) * out_scale over the head's values
+// With a sink the denominator of one map also holds exp(sink of the head). With a distance bias (one map) r1 ln(1 + r2 (i - j)) of the
+// head is taken off a score. "Spread" attention weighs the values of every key/value head with every head's weights (one value row
+// per token holds them all) and leaves fp32 partial sums; talk_mix adds them up with a matrix over the heads, which is the same as
+// mixing the heads' weights in front of the values, and gates the heads.
 // Rows are padded with zeros to wk and wv (64, 128, or a multiple of 16 above). Pools: keys [block][kv head][map][token][wk],
 // values [block][kv head][token][wv]; queries [token][head][map][wk]. Query rows of a sequence are numbered token * group + head
 // within one kv head.
@@ -12,6 +16,7 @@
 //   maps_decode_kernel   mma.sync, 16 query rows per CTA (two maps: 8 rows of each), each warp streaming its own 16-token pages
 //                        through a private cp.async ring; split over key slices.
 //   maps_simple_kernel   CUDA cores, any width, bf16 and fp32.
+//   talk_mix_kernel      spread attention: partial sums of all heads -> mixed, gated heads.
 //
 // Weights are fp32; for the tensor-core product with the values a weight travels as the sum of two bf16 values (16 significant
 // bits). The maps are combined in fp32 before anything is rounded. Nothing in front of a window's first page is read.
@@ -29,6 +34,7 @@
 
 namespace fllm {
 namespace {
+constexpr float kLn2 = 0.6931471805599453f;
 constexpr int kDecodeRows = 64;           // sequences with at most this many query rows per kv head run in the decode kernel
 
 // ------------------------------------------------------------------------------------------ queries and cache rows
@@ -46,6 +52,22 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
   const T* xr = static_cast<const T*>(p.x) + (long long)t * p.ldx;
   const float* part = p.partials ? p.partials + (size_t)t * p.width : nullptr;
   const T* bias = static_cast<const T*>(p.bias);
+  // short convolution of steps in which every sequence has one token: the taps before it come from the sequence's state row,
+  // which moves on by one token as it is read
+  T* window = p.taps > 0 ? static_cast<T*>(p.conv_state) + (long long)p.seq_state[t] * (p.taps - 1) * p.conv_width : nullptr;
+  const bool fresh = pos == 0;
+  auto conv1 = [&](int c, float u, bool write) {
+    const float* w = p.conv_w + (long long)c * p.taps;
+    float v = w[p.taps - 1] * u, next = u;
+    for (int j = p.taps - 2; j >= 0; --j) {
+      T* at = window + (long long)j * p.conv_width + c;
+      const float old = fresh ? 0.f : to_f32(*at);
+      v = fmaf(w[j], old, v);
+      if (write) *at = from_f32<T>(next);
+      next = old;
+    }
+    return v;
+  };
   auto load1 = [&](int c) {
     float v = bias ? to_f32(bias[c]) : 0.f;
     if (!part) return v + to_f32(xr[c]);
@@ -53,7 +75,7 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
     return v;
   };
   // columns base + c .. c + 3 of a segment of n values, zeros behind it
-  auto load4 = [&](int base, int c, int n) {
+  auto raw4 = [&](int base, int c, int n) {
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (p.vec) {                                                  // n is a multiple of 4
       if (c >= n) return v;
@@ -78,6 +100,17 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
       if (c + e < n) f[e] = load1(base + c + e);
     return v;
   };
+  // behind the convolution, if any: with `write` the state row moves on, so every column is loaded once with it
+  auto load4 = [&](int base, int c, int n, bool write) {
+    float4 v = raw4(base, c, n);
+    if (window) {
+      float* f = &v.x;
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (c + e < n) f[e] = conv1(base + c + e, f[e], write);
+    }
+    return v;
+  };
   auto store4 = [](T* dst, const float (&v)[4]) {
     typename Four<T>::type raw;
     T* e = reinterpret_cast<T*>(&raw);
@@ -95,8 +128,8 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
   float2 all = make_float2(0.f, 0.f);                             // full: 1 / rms of all query maps and of all key maps
   if (p.full) {
     float2 ss = make_float2(0.f, 0.f);
-    for (int c = 4 * threadIdx.x; c < p.q_heads * p.dim; c += 512) ss.x += sq(load4(p.q_offset, c, p.q_heads * p.dim));
-    for (int c = 4 * threadIdx.x; c < p.k_heads * p.dim; c += 512) ss.y += sq(load4(p.k_offset, c, p.k_heads * p.dim));
+    for (int c = 4 * threadIdx.x; c < p.q_heads * p.dim; c += 512) ss.x += sq(load4(p.q_offset, c, p.q_heads * p.dim, false));
+    for (int c = 4 * threadIdx.x; c < p.k_heads * p.dim; c += 512) ss.y += sq(load4(p.k_offset, c, p.k_heads * p.dim, false));
     ss = make_float2(warp_sum(ss.x), warp_sum(ss.y));
     if (lane == 0) red[warp] = ss;
     __syncthreads();
@@ -105,30 +138,42 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
   }
   __syncthreads();
   if (p.lanes > 0) {
-    // maps of 64 or 128 values: 16 or 32 lanes with four values each, so that a warp has one or two maps at a time and a
-    // rotation partner is a shuffle away
+    // maps of up to 64 or 128 values: 16 or 32 lanes with four values each, so that a warp has one or two maps at a time and a
+    // rotation partner is a shuffle away, or in the same lane
     const int maps = p.q_heads + (slot >= 0 ? p.k_heads : 0), per = 32 / p.lanes, sub = lane / p.lanes, li = lane % p.lanes, c = 4 * li;
     const bool low = c < half, turns = c < p.rot;
-    const int mate = turns ? lane + (low ? half / 4 : -half / 4) : lane;
+    const int mate = turns && !p.pairs ? lane + (low ? half / 4 : -half / 4) : lane;
     float2 cs[4];
 #pragma unroll
-    for (int e = 0; e < 4; ++e) cs[e] = turns ? turn[(low ? c : c - half) + e] : make_float2(1.f, 0.f);
+    for (int e = 0; e < 4; ++e) cs[e] = turns ? turn[p.pairs ? (c + e) / 2 : (low ? c : c - half) + e] : make_float2(1.f, 0.f);
     for (int i0 = (blockIdx.y * 4 + warp) * per; i0 < maps; i0 += 4 * per * gridDim.y) {
       const int item = min(i0 + sub, maps - 1);                   // (lanes past the end repeat the last map)
       const bool is_q = item < p.q_heads;
       const int h = is_q ? item : item - p.q_heads;
-      const float4 f = load4((is_q ? p.q_offset : p.k_offset) + h * p.dim, c, p.dim);
+      const float4 f = load4((is_q ? p.q_offset : p.k_offset) + h * p.dim, c, p.dim, i0 + sub < maps);
       float ss = sq(f);
       for (int o = p.lanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-      const float inv = p.full ? (is_q ? all.x : all.y) : 1.f / sqrtf(ss / (float)p.dim + p.eps);
-      const T* w = static_cast<const T*>(is_q ? p.q_norm : p.k_norm) + (p.full ? h * p.dim : 0) + c;
-      const typename Four<T>::type raw = *reinterpret_cast<const typename Four<T>::type*>(w);
-      const T* wv = reinterpret_cast<const T*>(&raw);
-      float v[4] = {f.x * inv * to_f32(wv[0]), f.y * inv * to_f32(wv[1]), f.z * inv * to_f32(wv[2]), f.w * inv * to_f32(wv[3])};
+      const float inv = p.eps < 0.f ? 1.f : (p.full ? (is_q ? all.x : all.y) : 1.f / sqrtf(ss / (float)p.dim + p.eps));
+      float v[4] = {f.x * inv, f.y * inv, f.z * inv, f.w * inv};
+      if (p.q_norm != nullptr && c < p.dim) {
+        const T* w = static_cast<const T*>(is_q ? p.q_norm : p.k_norm) + (p.full ? h * p.dim : 0) + c;
+        const typename Four<T>::type raw = *reinterpret_cast<const typename Four<T>::type*>(w);
+        const T* wv = reinterpret_cast<const T*>(&raw);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float m = __shfl_sync(0xffffffffu, v[e], mate);
-        v[e] = low ? v[e] * cs[e].x - m * cs[e].y : v[e] * cs[e].x + m * cs[e].y;
+        for (int e = 0; e < 4; ++e) v[e] *= to_f32(wv[e]);
+      }
+      if (p.pairs) {
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const float a = v[e], b = v[e + 1];
+          v[e] = a * cs[e].x - b * cs[e].y, v[e + 1] = b * cs[e].x + a * cs[e].y;
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float m = __shfl_sync(0xffffffffu, v[e], mate);
+          v[e] = low ? v[e] * cs[e].x - m * cs[e].y : v[e] * cs[e].x + m * cs[e].y;
+        }
       }
       T* dst = is_q ? static_cast<T*>(p.q_out) + ((long long)t * p.q_heads + h) * p.wk
                     : static_cast<T*>(p.k_cache) + (((long long)(slot / p.block_size) * p.k_heads + h) * p.block_size + slot % p.block_size) * p.wk;
@@ -144,7 +189,7 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
       const int g = item - p.q_heads - p.k_heads;
       T* dst = static_cast<T*>(p.v_cache) + ((block * p.v_heads + g) * p.block_size + at) * p.wv;
       for (int c = 4 * lane; c < p.wv; c += 128) {
-        const float4 f = load4(p.v_offset + g * p.v_dim, c, p.v_dim);
+        const float4 f = load4(p.v_offset + g * p.v_dim, c, p.v_dim, true);
         v[0] = f.x, v[1] = f.y, v[2] = f.z, v[3] = f.w;
         store4(dst + c, v);
       }
@@ -153,19 +198,19 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
     const bool is_q = item < p.q_heads;
     const int h = is_q ? item : item - p.q_heads;
     const int base = (is_q ? p.q_offset : p.k_offset) + h * p.dim;
-    const T* w = static_cast<const T*>(is_q ? p.q_norm : p.k_norm) + (p.full ? h * p.dim : 0);
+    const T* w = p.q_norm ? static_cast<const T*>(is_q ? p.q_norm : p.k_norm) + (p.full ? h * p.dim : 0) : nullptr;
     T* dst = is_q ? static_cast<T*>(p.q_out) + ((long long)t * p.q_heads + h) * p.wk
                   : static_cast<T*>(p.k_cache) + ((block * p.k_heads + h) * p.block_size + at) * p.wk;
     float ss = 0.f;
     for (int c = 4 * lane; c < p.dim; c += 128) {
-      const float4 f = load4(base, c, p.dim);
+      const float4 f = load4(base, c, p.dim, true);
       ss += sq(f);
       buf[c] = f.x;
       if (c + 1 < p.dim) buf[c + 1] = f.y;
       if (c + 2 < p.dim) buf[c + 2] = f.z;
       if (c + 3 < p.dim) buf[c + 3] = f.w;
     }
-    const float own = 1.f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps), inv = p.full ? (is_q ? all.x : all.y) : own;
+    const float own = 1.f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps), inv = p.eps < 0.f ? 1.f : (p.full ? (is_q ? all.x : all.y) : own);
     __syncwarp();
     for (int c = 4 * lane; c < p.wk; c += 128) {
 #pragma unroll
@@ -173,13 +218,13 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
         const int i = c + e;
         v[e] = 0.f;
         if (i >= p.dim) continue;
-        const float n = buf[i] * inv * to_f32(w[i]);
+        const float n = buf[i] * inv * (w ? to_f32(w[i]) : 1.f);
         v[e] = n;
         if (i < p.rot) {
-          const bool low = i < half;
-          const int j = low ? i + half : i - half;
-          const float2 cs = turn[low ? i : j];
-          const float m = buf[j] * inv * to_f32(w[j]);
+          const bool low = p.pairs ? i % 2 == 0 : i < half;
+          const int step = p.pairs ? 1 : half, j = low ? i + step : i - step;
+          const float2 cs = turn[p.pairs ? i / 2 : min(i, j)];
+          const float m = buf[j] * inv * (w ? to_f32(w[j]) : 1.f);
           v[e] = low ? n * cs.x - m * cs.y : n * cs.x + m * cs.y;
         }
       }
@@ -187,19 +232,25 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
     }
     __syncwarp();
   }
+  // further columns of the projection, as fp32
+  if (blockIdx.y == 0)
+    for (int i = threadIdx.x; i < p.extra; i += 128) p.extra_out[(long long)t * p.extra + i] = load1(p.extra_offset + i);
 }
 
 // ------------------------------------------------------------------------------------------ CUDA-core attention
-// One CTA per (head, token); its warps take every NW-th key with an online softmax each and are merged through shared memory.
+// One CTA per (head, token) and, for spread attention, piece of E * 32 value columns; its warps take every NW-th key with an online
+// softmax each and are merged through shared memory.
 template <typename T, int E, int M, int NW>
 __global__ void __launch_bounds__(NW * 32) maps_simple_kernel(const MapsAttnParams p) {
   extern __shared__ float sm[];
+  const int col0 = blockIdx.z * E * 32, v_dim = min(p.v_dim - col0, E * 32);
   float* sq = sm;                              // [M][dim] query rows
   float* sacc = sq + M * p.dim;                // [M][NW][v_dim]
-  float* sml = sacc + M * NW * p.v_dim;        // [M][NW][2] maximum and sum
+  float* sml = sacc + M * NW * v_dim;          // [M][NW][2] maximum and sum
   __shared__ float red[NW];
   const int h = blockIdx.x, t = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = h / (p.H / p.G);
+  const float r1 = p.r1 ? p.r1[h] : 0.f, r2 = p.r1 ? p.r2[h] : 0.f;
   const T* q = static_cast<const T*>(p.q) + ((long long)t * p.H + h) * M * p.wk;
   const T* kc = static_cast<const T*>(p.k_cache);
   const T* vc = static_cast<const T*>(p.v_cache);
@@ -217,20 +268,19 @@ __global__ void __launch_bounds__(NW * 32) maps_simple_kernel(const MapsAttnPara
   for (int j = first + warp; j < kv_len; j += NW) {
     const size_t block = (size_t)table[j / p.block_size] * p.G + g;
     const int at = j % p.block_size;
-    const T* vr = vc + (block * p.block_size + at) * p.wv;
+    const size_t vblock = p.spread ? (size_t)table[j / p.block_size] : block;
+    const T* vr = vc + (vblock * p.block_size + at) * p.wv + col0;
     float v[E];
 #pragma unroll
-    for (int e = 0; e < E; ++e) v[e] = lane + 32 * e < p.v_dim ? to_f32(vr[lane + 32 * e]) : 0.f;
+    for (int e = 0; e < E; ++e) v[e] = lane + 32 * e < v_dim ? to_f32(vr[lane + 32 * e]) : 0.f;
 #pragma unroll
     for (int a = 0; a < M; ++a) {
       const T* kr = kc + ((block * M + a) * p.block_size + at) * p.wk;
       float s = 0.f;
-#pragma unroll
-      for (int e = 0; e < E; ++e) {
-        const int c = lane + 32 * e;
-        if (c < p.dim) s = fmaf(to_f32(kr[c]), sq[a * p.dim + c], s);
-      }
+#pragma unroll 4
+      for (int c = lane; c < p.dim; c += 32) s = fmaf(to_f32(kr[c]), sq[a * p.dim + c], s);
       s = warp_sum(s) * p.scale;
+      if (p.r1) s -= r1 * log1pf(r2 * (float)(kv_len - 1 - j));
       const float mn = fmaxf(m[a], s), corr = expf(m[a] - mn), pr = expf(s - mn);
       l[a] = l[a] * corr + pr;
 #pragma unroll
@@ -242,14 +292,14 @@ __global__ void __launch_bounds__(NW * 32) maps_simple_kernel(const MapsAttnPara
   for (int a = 0; a < M; ++a) {
 #pragma unroll
     for (int e = 0; e < E; ++e)
-      if (lane + 32 * e < p.v_dim) sacc[(a * NW + warp) * p.v_dim + lane + 32 * e] = acc[a][e];
+      if (lane + 32 * e < v_dim) sacc[(a * NW + warp) * v_dim + lane + 32 * e] = acc[a][e];
     if (lane == 0) sml[2 * (a * NW + warp)] = m[a], sml[2 * (a * NW + warp) + 1] = l[a];
   }
   __syncthreads();
-  float c[M][NW], tot[M];
+  float c[M][NW], tot[M], mm;
 #pragma unroll
   for (int a = 0; a < M; ++a) {
-    float mm = -INFINITY;
+    mm = -INFINITY;
 #pragma unroll
     for (int w = 0; w < NW; ++w) mm = fmaxf(mm, sml[2 * (a * NW + w)]);
     tot[a] = 0.f;
@@ -260,13 +310,25 @@ __global__ void __launch_bounds__(NW * 32) maps_simple_kernel(const MapsAttnPara
       tot[a] = fmaf(sml[2 * (a * NW + w) + 1], c[a][w], tot[a]);
     }
   }
+  if (p.spread) {                              // partial sums of one key slice
+    const size_t row = (size_t)t * p.H + h;
+    for (int i = threadIdx.x; i < v_dim; i += NW * 32) {
+      float v = 0.f;
+#pragma unroll
+      for (int w = 0; w < NW; ++w) v = fmaf(sacc[w * v_dim + i], c[0][w], v);
+      p.part_o[row * p.wv + col0 + i] = v;
+    }
+    if (threadIdx.x == 0 && col0 == 0) p.part_ml[2 * row] = mm, p.part_ml[2 * row + 1] = tot[0];
+    return;
+  }
+  if (M == 1 && p.sink) tot[0] += expf(p.sink[h] - mm);
   auto value = [&](int i) {
     float o = 0.f;
 #pragma unroll
     for (int a = 0; a < M; ++a) {
       float v = 0.f;
 #pragma unroll
-      for (int w = 0; w < NW; ++w) v = fmaf(sacc[(a * NW + w) * p.v_dim + i], c[a][w], v);
+      for (int w = 0; w < NW; ++w) v = fmaf(sacc[(a * NW + w) * v_dim + i], c[a][w], v);
       o = a == 0 ? v / tot[0] : o - p.lam * (v / tot[a]);
     }
     return o;
@@ -304,6 +366,9 @@ struct Maps {
   float *ws_o, *ws_ml;                       // partial results of key slices: [T][H][maps][splits][DV], [T][H][maps][splits][2]
   int splits;
   int* status;
+  const float *sink, *r1, *r2;               // [H] each, natural units; r1 null: no distance bias
+  int wv, chunks;                            // spread attention: width of a value row, pieces of DV columns
+  int tab_stride, tab_entries, tab_bufs;     // distance bias of a tile of the prefill kernel: [buffer][head of the group][stride]
 };
 
 // first pool row of the kPage tokens from `token` on, in a pool of `heads` rows per token
@@ -312,11 +377,14 @@ __device__ __forceinline__ int page_row(const Maps& p, const int* table, int tok
 }
 __device__ __forceinline__ int first_key(const Maps& p, int lim) { return p.window > 0 ? max(0, lim - p.window) : 0; }
 
-// one warp, lane holding the values lane + 32 e of every map's weighted sum and the sums of its weights
+// what a head's sink adds to a sum of weights whose reference is m (log2 units)
+__device__ __forceinline__ float sink_weight(const Maps& p, int head, float m) { return p.sink ? ex2(p.sink[head] * kLog2e - m) : 0.f; }
+
+// one warp, lane holding the values lane + 32 e of every map's weighted sum, the sums of its weights and their reference
 template <int M, int E>
-__device__ __forceinline__ void finish_row(const Maps& p, long long tok, int head, const float (&a)[M][E], const float (&l)[M], int lane) {
+__device__ __forceinline__ void finish_row(const Maps& p, long long tok, int head, const float (&a)[M][E], const float (&l)[M], float m, int lane) {
   float y[E], ss = 0.f, f = 1.f;
-  const float i0 = l[0] > 0.f ? 1.f / l[0] : 0.f, i1 = M == 2 && l[M - 1] > 0.f ? p.lam / l[M - 1] : 0.f;
+  const float l0 = M == 1 ? l[0] + sink_weight(p, head, m) : l[0], i0 = l0 > 0.f ? 1.f / l0 : 0.f, i1 = M == 2 && l[M - 1] > 0.f ? p.lam / l[M - 1] : 0.f;
 #pragma unroll
   for (int e = 0; e < E; ++e) {
     y[e] = a[0][e] * i0;
@@ -341,14 +409,15 @@ struct DecodeTile {
   static constexpr int kRowsOf = 16 / M;                   // query rows of a tile: row r of map m is tile row m * kRowsOf + r
 };
 
-template <int DK, int DV, int M>
+template <int DK, int DV, int M, bool SPREAD>
 __global__ void __launch_bounds__(128, 2) maps_decode_kernel(const Maps p, int row_tiles, int max_rows) {
   using L = DecodeTile<DK, DV, M>;
   constexpr int R = L::kRowsOf;
   extern __shared__ __align__(128) uint8_t smem[];
   bf16* qtile = reinterpret_cast<bf16*>(smem);
   uint8_t* ring = smem + L::kQ;
-  const int kvh = blockIdx.x / row_tiles, row0 = (blockIdx.x % row_tiles) * R, seq = blockIdx.y, split = blockIdx.z;
+  const int piece = SPREAD ? blockIdx.x % p.chunks : 0, at = SPREAD ? blockIdx.x / p.chunks : blockIdx.x;
+  const int kvh = at / row_tiles, row0 = (at % row_tiles) * R, seq = blockIdx.y, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_launch_dependents();
   pdl_wait();
@@ -384,6 +453,14 @@ __global__ void __launch_bounds__(128, 2) maps_decode_kernel(const Maps p, int r
     lim[i] = sub < n_rows ? first_pos + (row0 + sub) / p.group + 1 : 0;
     beg[i] = first_key(p, lim[i]);
   }
+  float r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};
+  if (SPREAD && p.r1) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int head = kvh * p.group + (row0 + (g + 8 * i) % R) % p.group;
+      r1[i] = p.r1[head], r2[i] = p.r2[head];
+    }
+  }
   float o[DV / 8][4];
 #pragma unroll
   for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -404,11 +481,12 @@ __global__ void __launch_bounds__(128, 2) maps_decode_kernel(const Maps p, int r
           cp_async16(tile_ptr<DK>(reinterpret_cast<bf16*>(st + a * L::kKey), r, c), src + (size_t)r * DK + c * 8);
         }
       }
-      const bf16* src = p.vc + (long long)page_row(p, table, pg * kPage, p.G, kvh) * DV;
+      const int ldv = SPREAD ? p.wv : DV;
+      const bf16* src = p.vc + (long long)page_row(p, table, pg * kPage, SPREAD ? 1 : p.G, SPREAD ? 0 : kvh) * ldv + piece * DV;
 #pragma unroll
       for (int i = lane; i < kPage * (DV / 8); i += 32) {
         const int r = i / (DV / 8), c = i - r * (DV / 8);
-        cp_async16(tile_ptr<DV>(reinterpret_cast<bf16*>(st + M * L::kKey), r, c), src + (size_t)r * DV + c * 8);
+        cp_async16(tile_ptr<DV>(reinterpret_cast<bf16*>(st + M * L::kKey), r, c), src + (size_t)r * ldv + c * 8);
       }
     }
     cp_async_commit();
@@ -443,7 +521,8 @@ __global__ void __launch_bounds__(128, 2) maps_decode_kernel(const Maps p, int r
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int i = e >> 1, tok = tok_base + nb * 8 + 2 * t4 + (e & 1);
-        const float v = s[M == 2 ? i : 0][nb][e] * p.scale_log2;
+        float v = s[M == 2 ? i : 0][nb][e] * p.scale_log2;
+        if (SPREAD) v -= r1[i] * __log2f(fmaf(r2[i], (float)(lim[i] - 1 - tok), 1.f));
         s[0][nb][e] = tok >= beg[i] && tok < lim[i] ? v : -INFINITY;
         mx[i] = fmaxf(mx[i], s[0][nb][e]);
       }
@@ -525,8 +604,15 @@ __global__ void __launch_bounds__(128, 2) maps_decode_kernel(const Maps p, int r
         for (int e = 0; e < E; ++e) a[k][e] = fmaf(mo[((size_t)w * 16 + r) * DV + lane + 32 * e], c, a[k][e]);
       }
     }
+    if (SPREAD) {
+      const size_t base = (tok * p.H + head) * p.splits + split;
+#pragma unroll
+      for (int e = 0; e < E; ++e) p.ws_o[base * p.wv + piece * DV + lane + 32 * e] = a[0][e];
+      if (lane == 0 && piece == 0) p.ws_ml[base * 2] = ms[0] * kLn2, p.ws_ml[base * 2 + 1] = ls[0];
+      continue;
+    }
     if (p.splits == 1) {
-      finish_row<M, E>(p, tok, head, a, ls, lane);
+      finish_row<M, E>(p, tok, head, a, ls, ms[0], lane);
       continue;
     }
 #pragma unroll
@@ -547,11 +633,11 @@ __global__ void __launch_bounds__(128) maps_merge_kernel(const Maps p, int T) {
   pdl_wait();
   const int item = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (item >= T * p.H) return;
-  float a[M][E], l[M];
+  float a[M][E], l[M], mm;
 #pragma unroll
   for (int k = 0; k < M; ++k) {
     const size_t base = ((size_t)item * M + k) * p.splits;
-    float mm = -INFINITY;
+    mm = -INFINITY;
     l[k] = 0.f;
     for (int s = 0; s < p.splits; ++s) mm = fmaxf(mm, p.ws_ml[(base + s) * 2]);
 #pragma unroll
@@ -565,7 +651,7 @@ __global__ void __launch_bounds__(128) maps_merge_kernel(const Maps p, int T) {
       for (int e = 0; e < E; ++e) a[k][e] = fmaf(p.ws_o[(base + s) * DV + lane + 32 * e], w, a[k][e]);
     }
   }
-  finish_row<M, E>(p, item / p.H, item % p.H, a, l, lane);
+  finish_row<M, E>(p, item / p.H, item % p.H, a, l, mm, lane);
 }
 
 // ------------------------------------------------------------------------------------------ prefill
@@ -575,16 +661,20 @@ __global__ void __launch_bounds__(128) maps_merge_kernel(const Maps p, int T) {
 // Order of the products: S_0, S_1 of the first tile, then per tile O_0, next S_0, O_1, next S_1: while one stream waits for its
 // weights the other's products run. Every wait is bounded.
 constexpr int kThreads = 320;
-template <int DK, int DV, int M>
+constexpr int kTable = 3712;                           // fp32 entries of a stream's distance bias
+template <int DK, int DV, int M, bool SPREAD>
 struct PrefillTile {
-  static constexpr int kQ = 2 * tile_bytes<DK>(), kK = M * tile_bytes<DK>(), kV = tile_bytes<DV>(), kTail = 256 + 2 * 128 * 4 * 2;
+  static constexpr int kQ = 2 * tile_bytes<DK>(), kK = M * tile_bytes<DK>(), kV = tile_bytes<DV>();
+  static constexpr int kTail = 256 + 2 * 128 * 4 * 2 + (SPREAD ? 2 * kTable * 4 : 0);
   static constexpr int kStages = kQ + 2 * (kK + kV) + kTail + 1024 <= 227 * 1024 ? 2 : 1;
   static constexpr int kUsed = kQ + kStages * (kK + kV) + kTail + 1024;
   static constexpr int kTotal = kUsed > 120 * 1024 ? kUsed : 120 * 1024;      // one CTA per SM: it takes all of the tensor memory
 };
 
-template <int DV, bool FULL>
-__device__ __forceinline__ void softmax_tile(uint32_t t_s, uint32_t t_o, float scale_log2, int lo, int hi, bool have_o, float& m_used, float& l) {
+// BIAS: bias[-c] is taken off the score of column c (log2 units)
+template <int DV, bool FULL, bool BIAS>
+__device__ __forceinline__ void softmax_tile(uint32_t t_s, uint32_t t_o, float scale_log2, const float* bias, int lo, int hi, bool have_o, float& m_used,
+                                             float& l) {
   uint32_t sa[32];
   float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll 1
@@ -593,7 +683,7 @@ __device__ __forceinline__ void softmax_tile(uint32_t t_s, uint32_t t_o, float s
     tmem_ld_wait();
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
-      const float v = __uint_as_float(sa[i]) * scale_log2;
+      const float v = BIAS ? fmaf(__uint_as_float(sa[i]), scale_log2, -bias[-(32 * c + i)]) : __uint_as_float(sa[i]) * scale_log2;
       if (FULL || (32 * c + i >= lo && 32 * c + i < hi)) mx[i & 3] = fmaxf(mx[i & 3], v);
     }
   }
@@ -620,7 +710,7 @@ __device__ __forceinline__ void softmax_tile(uint32_t t_s, uint32_t t_o, float s
       float v[2];
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        v[e] = ex2(fmaf(__uint_as_float(sa[i + e]), scale_log2, -m_ref));
+        v[e] = ex2(fmaf(__uint_as_float(sa[i + e]), scale_log2, BIAS ? -m_ref - bias[-(32 * c + i + e)] : -m_ref));
         if (!FULL && (32 * c + i + e < lo || 32 * c + i + e >= hi)) v[e] = 0.f;
         sum[(i + e) & 3] += v[e];
       }
@@ -668,12 +758,13 @@ __device__ __forceinline__ void store_32(const Maps& p, bf16* dst, int c0, const
   }
 }
 
+__device__ __forceinline__ void stream_barrier(int s) { asm volatile("bar.sync %0, 128;" ::"r"(2 + s) : "memory"); }
 __device__ __forceinline__ void softmax_barrier() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
-template <int DK, int DV, int M>
+template <int DK, int DV, int M, bool SPREAD>
 __global__ void __launch_bounds__(kThreads, 1) maps_prefill_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_constant__ CUtensorMap tma_v,
                                                                    const Maps p, int min_rows) {
-  using L = PrefillTile<DK, DV, M>;
+  using L = PrefillTile<DK, DV, M, SPREAD>;
   constexpr int TBK = tile_bytes<DK>(), TBV = tile_bytes<DV>(), NST = L::kStages, CTA_ROWS = M == 2 ? kRows : 2 * kRows;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -690,7 +781,7 @@ __global__ void __launch_bounds__(kThreads, 1) maps_prefill_kernel(const __grid_
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int row0 = (gridDim.x - 1 - blockIdx.x) * CTA_ROWS;          // the tiles with the longest key range start first
-  const int kvh = blockIdx.y, seq = blockIdx.z;
+  const int kvh = SPREAD ? blockIdx.y / p.chunks : blockIdx.y, piece = SPREAD ? blockIdx.y % p.chunks : 0, seq = blockIdx.z;
   const int q0 = p.q_starts[seq], qn = p.q_starts[seq + 1] - q0;
   const int all_rows = qn * p.group;
   if (all_rows < min_rows || row0 >= all_rows) return;
@@ -750,9 +841,9 @@ __global__ void __launch_bounds__(kThreads, 1) maps_prefill_kernel(const __grid_
         mbar_expect_tx(&v_full[b], TBV);
 #pragma unroll
         for (int pg = 0; pg < kTile / kPage; ++pg) {
-          const int row = page_row(p, table, tok[pg], p.G, kvh);
+          const int row = page_row(p, table, tok[pg], SPREAD ? 1 : p.G, SPREAD ? 0 : kvh);
 #pragma unroll
-          for (int h = 0; h < DV / 64; ++h) tma_load_2d(sv + b * L::kV + h * kHalf + pg * (kPage * 128), &tma_v, &v_full[b], 64 * h, row);
+          for (int h = 0; h < DV / 64; ++h) tma_load_2d(sv + b * L::kV + h * kHalf + pg * (kPage * 128), &tma_v, &v_full[b], piece * DV + 64 * h, row);
         }
       }
     }
@@ -815,14 +906,29 @@ __global__ void __launch_bounds__(kThreads, 1) maps_prefill_kernel(const __grid_
     const int lim_first = first_pos + srow0 / p.group + 1, beg_last = first_key(p, first_pos + (srow0 + kRows - 1) / p.group + 1);
     float m_used = -INFINITY, l = 0.f;
     bool ok = true;
+    const int off = (srow0 + r) / p.group - srow0 / p.group, hh = (srow0 + r) % p.group;      // of the row: token behind the stream's first, head of the group
+    float* table = swap_ss + 2 * kRows + s * kTable;
     for (int it = 0; it < n_tiles; ++it) {
       const int tok0 = begin + it * kTile;
+      const float* bias = nullptr;
+      if (SPREAD && n_rows > 0) {
+        // the bias of every distance between the stream's tokens and the tile's, per head; entry e is off + 127 - column
+        float* buf = table + (p.tab_bufs == 2 && (it & 1) ? p.tab_entries : 0);
+        if (p.tab_bufs == 1 && it > 0) stream_barrier(s);
+        const int base = first_pos + srow0 / p.group - tok0 - (kTile - 1);
+        for (int i = (warp & 3) * 32 + lane; i < p.tab_entries; i += 128) {
+          const int head = kvh * p.group + i / p.tab_stride, d = base + i % p.tab_stride;
+          buf[i] = p.r1 && d > 0 ? p.r1[head] * __log2f(fmaf(p.r2[head], (float)d, 1.f)) : 0.f;
+        }
+        stream_barrier(s);
+        bias = buf + hh * p.tab_stride + off + (kTile - 1);
+      }
       if (!mbar_wait(&s_full[s], it & 1, abort_flag)) { ok = false; break; }
       tc_fence_after_sync();
       if (n_rows == kRows && tok0 + kTile <= lim_first && tok0 >= beg_last)      // every row of the stream sees the whole tile
-        softmax_tile<DV, true>(t_s, t_o, p.scale_log2, 0, 0, it > 0, m_used, l);
-      else
-        softmax_tile<DV, false>(t_s, t_o, p.scale_log2, beg - tok0, lim - tok0, it > 0, m_used, l);
+        softmax_tile<DV, true, SPREAD>(t_s, t_o, p.scale_log2, bias, 0, 0, it > 0, m_used, l);
+      else if (!SPREAD || n_rows > 0)
+        softmax_tile<DV, false, SPREAD>(t_s, t_o, p.scale_log2, bias, beg - tok0, lim - tok0, it > 0, m_used, l);
       tc_fence_before_sync();
       __syncwarp();
       if (lane == 0) mbar_arrive(&p_ready[s]);
@@ -863,7 +969,22 @@ __global__ void __launch_bounds__(kThreads, 1) maps_prefill_kernel(const __grid_
           store_32(p, dst, (s * N + n) * 32, y[n]);
         }
       }
+    } else if (ok && SPREAD) {
+      const long long at = (long long)(q0 + row / p.group) * p.H + kvh * p.group + row % p.group;
+#pragma unroll 1
+      for (int c = 0; c < DV / 32; ++c) {
+        uint32_t a[32];
+        tmem_ld_32x32(t_o + 32 * c, a);
+        tmem_ld_wait();
+        if (!valid) continue;
+        float4* to = reinterpret_cast<float4*>(p.ws_o + at * p.wv + piece * DV + 32 * c);
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+          to[i] = make_float4(__uint_as_float(a[4 * i]), __uint_as_float(a[4 * i + 1]), __uint_as_float(a[4 * i + 2]), __uint_as_float(a[4 * i + 3]));
+      }
+      if (valid && piece == 0) p.ws_ml[2 * at] = m_used * kLn2, p.ws_ml[2 * at + 1] = l;
     } else if (ok) {
+      if (valid) l += sink_weight(p, kvh * p.group + row % p.group, m_used);
       const float inv = l > 0.f ? 1.f / l : 0.f;
 #pragma unroll 1
       for (int c = 0; c < DV / 32; ++c) {
@@ -905,23 +1026,24 @@ const CUtensorMap& pool_map(const void* pool, uint64_t rows, int D) {
   return it->second;
 }
 
-template <int DK, int DV, int M>
+template <int DK, int DV, int M, bool SPREAD = false>
 int launch_tc(Maps a, const MapsAttnParams& p, int splits, cudaStream_t s) {
   using D = DecodeTile<DK, DV, M>;
-  using P = PrefillTile<DK, DV, M>;
+  using P = PrefillTile<DK, DV, M, SPREAD>;
   static bool configured[kMaxDevices] = {};
   if (first_call_on_device(configured)) {
-    cuda_check(cudaFuncSetAttribute(maps_decode_kernel<DK, DV, M>, cudaFuncAttributeMaxDynamicSharedMemorySize, D::kTotal), "maps_decode smem");
-    cuda_check(cudaFuncSetAttribute(maps_prefill_kernel<DK, DV, M>, cudaFuncAttributeMaxDynamicSharedMemorySize, P::kTotal), "maps_prefill smem");
+    cuda_check(cudaFuncSetAttribute(maps_decode_kernel<DK, DV, M, SPREAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, D::kTotal), "maps_decode smem");
+    cuda_check(cudaFuncSetAttribute(maps_prefill_kernel<DK, DV, M, SPREAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, P::kTotal), "maps_prefill smem");
   }
   int launches = 0;
   const int max_rows = p.max_q_len * a.group;
   if (p.min_q_len * a.group <= kDecodeRows) {
     a.splits = max_rows <= kDecodeRows ? splits : 1;      // partial results of longer sequences do not exist
     const int row_tiles = (std::min(max_rows, kDecodeRows) + D::kRowsOf - 1) / D::kRowsOf;
-    launch_pdl(maps_decode_kernel<DK, DV, M>, dim3(a.G * row_tiles, p.num_seqs, a.splits), dim3(128), D::kTotal, s, a, row_tiles, (int)kDecodeRows);
+    launch_pdl(maps_decode_kernel<DK, DV, M, SPREAD>, dim3(a.G * row_tiles * a.chunks, p.num_seqs, a.splits), dim3(128), D::kTotal, s, a, row_tiles,
+               (int)kDecodeRows);
     ++launches;
-    if (a.splits > 1) {
+    if (!SPREAD && a.splits > 1) {
       launch_pdl(maps_merge_kernel<DV, M>, dim3((p.tokens * a.H + 3) / 4), dim3(128), 0, s, a, p.tokens);
       ++launches;
     }
@@ -930,8 +1052,8 @@ int launch_tc(Maps a, const MapsAttnParams& p, int splits, cudaStream_t s) {
     constexpr int rows = M == 2 ? kRows : 2 * kRows;
     const uint64_t n = (uint64_t)p.num_blocks * a.G * a.block_size;
     // (copies: a second lookup may move the first entry)
-    const CUtensorMap km = pool_map(p.k_cache, n * M, DK), vm = pool_map(p.v_cache, n, DV);
-    maps_prefill_kernel<DK, DV, M><<<dim3((max_rows + rows - 1) / rows, a.G, p.num_seqs), kThreads, P::kTotal, s>>>(km, vm, a, kDecodeRows + 1);
+    const CUtensorMap km = pool_map(p.k_cache, n * M, DK), vm = SPREAD ? pool_map(p.v_cache, n / a.G, a.wv) : pool_map(p.v_cache, n, DV);
+    maps_prefill_kernel<DK, DV, M, SPREAD><<<dim3((max_rows + rows - 1) / rows, a.G * a.chunks, p.num_seqs), kThreads, P::kTotal, s>>>(km, vm, a, kDecodeRows + 1);
     ++launches;
   }
   cuda_check(cudaGetLastError(), "attention_maps launch");
@@ -941,9 +1063,9 @@ int launch_tc(Maps a, const MapsAttnParams& p, int splits, cudaStream_t s) {
 template <typename T, int M>
 void launch_simple(const MapsAttnParams& p, cudaStream_t s) {
   constexpr int NW = 4;
-  const size_t smem = (size_t)(M * p.dim + M * NW * p.v_dim + M * 2 * NW) * sizeof(float);
-  const dim3 grid(p.H, p.tokens);
-  const int widest = std::max(p.dim, p.v_dim);
+  const int piece = std::min(p.v_dim, 512), widest = p.spread ? piece : std::max(p.dim, p.v_dim);
+  const size_t smem = (size_t)(M * p.dim + M * NW * piece + M * 2 * NW) * sizeof(float);
+  const dim3 grid(p.H, p.tokens, p.spread ? (p.v_dim + 511) / 512 : 1);
   if (widest <= 64) maps_simple_kernel<T, 2, M, NW><<<grid, NW * 32, smem, s>>>(p);
   else if (widest <= 128) maps_simple_kernel<T, 4, M, NW><<<grid, NW * 32, smem, s>>>(p);
   else if (widest <= 256) maps_simple_kernel<T, 8, M, NW><<<grid, NW * 32, smem, s>>>(p);
@@ -951,10 +1073,84 @@ void launch_simple(const MapsAttnParams& p, cudaStream_t s) {
   else throw std::runtime_error("attention_maps: heads of at most 512 values");
   cuda_check(cudaGetLastError(), "maps_simple_kernel");
 }
+
+// ------------------------------------------------------------------------------------------ spread attention: the heads mixed
+// One CTA per token, a thread per value column (g, i) at a time: with a[f] the column of head f's output, head h of group g is
+// sigmoid(gate_h) sum_f talk[h, f] a[f]. The key slices of a head are merged on the way, and the sink joins its denominator.
+constexpr int kMixHeads = 8;
+template <typename T>
+__global__ void __launch_bounds__(256) talk_mix_kernel(const TalkMixParams p) {
+  extern __shared__ float sm[];
+  float* mat = sm;                             // [H][H]
+  float* coef = mat + p.H * p.H;               // [H][splits]
+  const int t = blockIdx.x, H = p.H, group = H / p.G, S = p.splits;
+  pdl_launch_dependents();
+  for (int i = threadIdx.x; i < H * H; i += blockDim.x) mat[i] = p.talk[i];
+  pdl_wait();
+  for (int h = threadIdx.x; h < H; h += blockDim.x) {
+    const float2* ml = reinterpret_cast<const float2*>(p.part_ml) + ((size_t)t * H + h) * S;
+    float m = p.sink ? p.sink[h] : -INFINITY, l = 0.f;
+    for (int s = 0; s < S; ++s) m = fmaxf(m, ml[s].x);
+    if (p.sink) l = expf(p.sink[h] - m);
+    for (int s = 0; s < S; ++s) {
+      const float2 v = ml[s];
+      const float c = v.x == -INFINITY ? 0.f : expf(v.x - m);
+      coef[h * S + s] = c;
+      l = fmaf(v.y, c, l);
+    }
+    for (int s = 0; s < S; ++s) coef[h * S + s] /= l;
+  }
+  __syncthreads();
+  T* out = static_cast<T*>(p.out) + (long long)t * p.ldo;
+  const float* src = p.part_o + (size_t)t * H * S * p.wv;
+  const float* gate = p.gate ? p.gate + (long long)t * p.ld_gate : nullptr;
+  for (int c = threadIdx.x; c < p.G * p.v_dim; c += blockDim.x) {
+    const int g = c / p.v_dim, i = c - g * p.v_dim;
+    for (int h0 = 0; h0 < group; h0 += kMixHeads) {
+      float acc[kMixHeads];
+#pragma unroll
+      for (int e = 0; e < kMixHeads; ++e) acc[e] = 0.f;
+      const int n = min(kMixHeads, group - h0);
+      const float* row = mat + (size_t)(g * group + h0) * H;
+#pragma unroll 4
+      for (int f = 0; f < H; ++f) {
+        float a = 0.f;
+        for (int s = 0; s < S; ++s) {
+          const float w = coef[f * S + s];
+          if (w != 0.f) a = fmaf(__ldcg(src + ((size_t)f * S + s) * p.wv + c), w, a);
+        }
+#pragma unroll
+        for (int e = 0; e < kMixHeads; ++e)
+          if (e < n) acc[e] = fmaf(row[e * H + f], a, acc[e]);
+      }
+#pragma unroll
+      for (int e = 0; e < kMixHeads; ++e) {
+        if (e >= n) continue;
+        const int h = g * group + h0 + e;
+        out[(long long)h * p.v_dim + i] = from_f32<T>(gate ? acc[e] / (1.f + expf(-gate[h])) : acc[e]);
+      }
+    }
+  }
+  for (int c = H * p.v_dim + threadIdx.x; c < p.cols; c += blockDim.x) out[c] = from_f32<T>(0.f);
+}
+
+// the table of a stream's distance bias: heads of a group x distances, rows spaced so that the lanes of a warp hit distinct banks
+void plan_table(Maps& a) {
+  const int n = 127 / a.group + 1 + kTile, shift = (32 + a.group - 1) / a.group % 32;
+  a.tab_stride = n + ((shift - n) % 32 + 32) % 32;
+  a.tab_entries = a.group * a.tab_stride;
+  a.tab_bufs = 2 * a.tab_entries <= kTable ? 2 : 1;
+}
 }  // namespace
 
 bool attention_maps_tc_supported(int wk, int wv, int block_size, int f32) {
   return !f32 && (wk == 64 || wk == 128) && (wv == 64 || wv == 128) && block_size % kPage == 0;
+}
+bool attention_spread_tc_supported(int group, int wk, int wv, int block_size, int f32) {
+  Maps a{};
+  a.group = group;
+  plan_table(a);
+  return !f32 && (wk == 64 || wk == 128) && (wv == 64 || wv % 128 == 0) && block_size % kPage == 0 && a.tab_entries <= kTable;
 }
 
 // key slices the tensor-core path uses for a step (1: no workspace needed)
@@ -974,13 +1170,18 @@ int attention_maps(const MapsAttnParams& p, int splits, void* workspace, size_t 
   if (p.tokens <= 0) return 0;
   if (p.tokens > 65535 || p.num_seqs > 65535) throw std::runtime_error("attention_maps: at most 65535 rows and sequences in a step");
   if (p.maps != 1 && p.maps != 2) throw std::runtime_error("attention_maps: one or two maps");
-  if (!tensor_cores || !attention_maps_tc_supported(p.wk, p.wv, p.block_size, p.f32)) {
+  if (p.maps == 2 && (p.sink || p.r1 || p.spread)) throw std::runtime_error("attention_maps: sinks, distance biases and spread values go with one map");
+  if (p.spread && (!p.part_o || !p.part_ml)) throw std::runtime_error("attention_maps: spread values need room for partial sums");
+  const bool fast = p.spread ? attention_spread_tc_supported(p.H / p.G, p.wk, p.wv, p.block_size, p.f32)
+                             : !p.r1 && attention_maps_tc_supported(p.wk, p.wv, p.block_size, p.f32);
+  if (!tensor_cores || !fast) {
+    if (p.spread && splits > 1) throw std::runtime_error("attention_maps: key slices are the tensor-core path's");
     if (p.f32) p.maps == 2 ? launch_simple<float, 2>(p, s) : launch_simple<float, 1>(p, s);
     else p.maps == 2 ? launch_simple<bf16, 2>(p, s) : launch_simple<bf16, 1>(p, s);
     return 1;
   }
   splits = std::max(splits, 1);
-  if (workspace_bytes < attention_maps_workspace_bytes(p.tokens, p.H * p.maps, p.wv, splits))
+  if (!p.spread && workspace_bytes < attention_maps_workspace_bytes(p.tokens, p.H * p.maps, p.wv, splits))
     throw std::runtime_error("attention_maps: workspace too small for the requested key slices");
   Maps a{};
   a.q = static_cast<const bf16*>(p.q), a.kc = static_cast<const bf16*>(p.k_cache), a.vc = static_cast<const bf16*>(p.v_cache);
@@ -992,6 +1193,13 @@ int attention_maps(const MapsAttnParams& p, int splits, void* workspace, size_t 
   a.ws_o = static_cast<float*>(workspace);
   a.ws_ml = a.ws_o != nullptr ? a.ws_o + (size_t)p.tokens * p.H * p.maps * splits * p.wv : nullptr;
   a.status = status;
+  a.sink = p.sink, a.r1 = p.r1, a.r2 = p.r2, a.chunks = 1;
+  if (p.spread) {
+    a.ws_o = p.part_o, a.ws_ml = p.part_ml, a.wv = p.wv, a.chunks = p.wv == 64 ? 1 : p.wv / 128;
+    plan_table(a);
+    if (p.wk == 64) return p.wv == 64 ? launch_tc<64, 64, 1, true>(a, p, splits, s) : launch_tc<64, 128, 1, true>(a, p, splits, s);
+    return p.wv == 64 ? launch_tc<128, 64, 1, true>(a, p, splits, s) : launch_tc<128, 128, 1, true>(a, p, splits, s);
+  }
 #define FLLM_MAPS(K_, V_) return p.maps == 2 ? launch_tc<K_, V_, 2>(a, p, splits, s) : launch_tc<K_, V_, 1>(a, p, splits, s);
   if (p.wk == 64 && p.wv == 64) { FLLM_MAPS(64, 64) }
   if (p.wk == 64) { FLLM_MAPS(64, 128) }
@@ -1000,14 +1208,30 @@ int attention_maps(const MapsAttnParams& p, int splits, void* workspace, size_t 
 #undef FLLM_MAPS
 }
 
+void talk_mix(const TalkMixParams& p, cudaStream_t s) {
+  if (p.tokens <= 0) return;
+  const size_t smem = ((size_t)p.H * p.H + (size_t)p.H * p.splits) * sizeof(float);
+  static bool configured[kMaxDevices] = {};
+  if (smem > 200 * 1024) throw std::runtime_error("talk_mix: too many heads");
+  if (first_call_on_device(configured)) {
+    cuda_check(cudaFuncSetAttribute(talk_mix_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024), "talk_mix smem");
+    cuda_check(cudaFuncSetAttribute(talk_mix_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024), "talk_mix smem");
+  }
+  const dim3 threads(std::min(256, (p.G * p.v_dim + 31) / 32 * 32));
+  if (p.f32) launch_pdl(talk_mix_kernel<float>, dim3(p.tokens), threads, smem, s, p);
+  else launch_pdl(talk_mix_kernel<bf16>, dim3(p.tokens), threads, smem, s, p);
+  cuda_check(cudaGetLastError(), "talk_mix_kernel");
+}
+
 void maps_prepare(const MapsPrepareParams& params, cudaStream_t s) {
   if (params.tokens <= 0) return;
   MapsPrepareParams p = params;
+  if (p.taps > 0 && p.full) throw std::runtime_error("maps_prepare: a norm over all maps does not go with a convolution");
   const uintptr_t any = reinterpret_cast<uintptr_t>(p.x) | reinterpret_cast<uintptr_t>(p.bias) | reinterpret_cast<uintptr_t>(p.partials);
   p.vec = p.dim % 4 == 0 && p.v_dim % 4 == 0 && p.q_offset % 4 == 0 && p.k_offset % 4 == 0 && p.v_offset % 4 == 0 && any % 16 == 0 &&
           (p.partials ? p.width % 4 == 0 && p.plane % 4 == 0 : p.ldx % 4 == 0);
   const uintptr_t norms = reinterpret_cast<uintptr_t>(p.q_norm) | reinterpret_cast<uintptr_t>(p.k_norm);
-  p.lanes = p.vec && (p.dim == 64 || p.dim == 128) && p.wk == p.dim && p.rot % 8 == 0 && norms % 16 == 0 ? p.dim / 4 : 0;
+  p.lanes = p.vec && (p.wk == 64 || p.wk == 128) && (p.pairs ? p.rot % 4 == 0 : p.rot % 8 == 0) && norms % 16 == 0 ? p.wk / 4 : 0;
   const int heads = p.q_heads + p.k_heads + p.v_heads;
   const int shares = std::max(1, std::min((heads + 3) / 4, 4 * sm_count() / std::max(p.tokens, 1)));
   const size_t smem = (size_t)(p.rot + 4 * p.dim) * sizeof(float);

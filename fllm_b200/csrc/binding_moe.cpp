@@ -36,9 +36,10 @@ void moe_route_scored(const Tensor& logits, const optional<Tensor>& select_bias,
                          renorm ? 1 : 0, (float)scale, ids.data_ptr<int>(), weights.data_ptr<float>(), cur_stream());
 }
 
-// logits fp32 [T, ld], or their split-K partial sums [splits][T][ld] in `workspace`
+// logits fp32 [T, ld], or their split-K partial sums [splits][T][ld] in `workspace`; gate_out (optional) [T]: the sigmoid of column `experts`
 void moe_route_fp32(const optional<Tensor>& logits, const optional<Tensor>& workspace, int64_t splits, int64_t ld, int64_t experts, int64_t k,
-                    int64_t score_kind, bool renorm, double scale, Tensor ids, Tensor weights) {
+                    int64_t score_kind, bool renorm, double scale, Tensor ids, Tensor weights, const optional<Tensor>& select_bias, int64_t groups,
+                    int64_t keep, double masked, const optional<Tensor>& gate_out) {
   TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == at::kInt && ids.dim() == 2 && ids.size(1) == k && weights.scalar_type() == at::kFloat &&
                   ids.is_contiguous() && weights.is_contiguous() && weights.numel() == ids.numel() && experts <= ld, "ids int32, weights fp32 [T, k]");
   const int64_t T = ids.size(0);
@@ -52,9 +53,19 @@ void moe_route_fp32(const optional<Tensor>& logits, const optional<Tensor>& work
                     logits->size(0) == T && logits->size(1) == ld, "logits: contiguous fp32 [T, ld]");
     z = logits->data_ptr<float>();
   }
+  const float* sb = nullptr;
+  if (select_bias.has_value() && select_bias->defined()) {
+    TORCH_CHECK(select_bias->is_cuda() && select_bias->scalar_type() == at::kFloat && select_bias->is_contiguous() && select_bias->numel() == experts, "select_bias: fp32 [experts]");
+    sb = select_bias->data_ptr<float>();
+  }
+  float* gate = nullptr;
+  if (gate_out.has_value() && gate_out->defined()) {
+    TORCH_CHECK(gate_out->is_cuda() && gate_out->scalar_type() == at::kFloat && gate_out->is_contiguous() && gate_out->numel() == T && experts < ld, "gate_out: fp32 [T]");
+    gate = gate_out->data_ptr<float>();
+  }
   c10::cuda::CUDAGuard guard(ids.device());
   fllm::moe_route_fp32(z, (int)std::max<int64_t>(splits, 1), T * ld, ld, (int)T, (int)experts, (int)k, (int)score_kind, renorm ? 1 : 0, (float)scale,
-                       ids.data_ptr<int>(), weights.data_ptr<float>(), cur_stream());
+                       ids.data_ptr<int>(), weights.data_ptr<float>(), cur_stream(), sb, fllm::RouteGroups{(int)groups, (int)keep, (float)masked}, gate);
 }
 
 void moe_align(const Tensor& ids, int64_t experts, int64_t expert_lo, int64_t expert_hi, int64_t bn, Tensor row_of,
@@ -121,15 +132,19 @@ int64_t moe_grouped_linear(const Tensor& xp, const Tensor& w_stack, const option
                                        num_tiles.data_ptr<int>(), (int)tile_expert.numel(), (int)bn, st, cur_stream());
 }
 
-void moe_combine(const Tensor& y, const Tensor& row_of, const optional<Tensor>& weights, Tensor out, const optional<Tensor>& add) {
+void moe_combine(const Tensor& y, const Tensor& row_of, const optional<Tensor>& weights, Tensor out, const optional<Tensor>& add,
+                 const optional<Tensor>& add_gate) {
   const bool f32 = f32_rows(y), plus = add.has_value() && add->defined();
   TORCH_CHECK(out.scalar_type() == y.scalar_type() && out.stride(1) == 1 && y.size(1) == out.size(1) && y.size(1) % 4 == 0 && y.stride(0) % 4 == 0 &&
                   out.stride(0) % 4 == 0, "moe_combine: shapes");
   TORCH_CHECK(!plus || (f32_rows(*add) == f32 && add->sizes() == out.sizes() && add->stride(0) % 4 == 0), "add: rows like out");
+  const bool gated = add_gate.has_value() && add_gate->defined();
+  TORCH_CHECK(!gated || (plus && add_gate->is_cuda() && add_gate->scalar_type() == at::kFloat && add_gate->is_contiguous() && add_gate->numel() == out.size(0)),
+              "add_gate: fp32, one per row");
   c10::cuda::CUDAGuard guard(y.device());
   fllm::moe_combine(y.data_ptr(), y.stride(0), row_of.data_ptr<int>(), weights.has_value() && weights->defined() ? weights->data_ptr<float>() : nullptr,
                     (int)out.size(0), (int)row_of.size(1), out.data_ptr(), out.stride(0), (int)out.size(1), cur_stream(), plus ? add->data_ptr() : nullptr,
-                    plus ? add->stride(0) : 0, f32 ? 1 : 0);
+                    plus ? add->stride(0) : 0, f32 ? 1 : 0, gated ? add_gate->data_ptr<float>() : nullptr);
 }
 }  // namespace
 
@@ -138,11 +153,12 @@ TORCH_LIBRARY_FRAGMENT(fllm_b200, m) {
         &moe_route_scored);
   m.def("moe_route(Tensor logits, Tensor? bias, int k, bool softmax_all, Tensor(a!) ids, Tensor(b!) weights) -> ()", &moe_route);
   m.def("moe_route_fp32(Tensor? logits, Tensor? workspace, int splits, int ld, int experts, int k, int score_kind, bool renorm, float scale, "
-        "Tensor(a!) ids, Tensor(b!) weights) -> ()", &moe_route_fp32);
+        "Tensor(a!) ids, Tensor(b!) weights, Tensor? select_bias=None, int groups=1, int keep=1, float masked=0.0, Tensor(c!)? gate_out=None) -> ()",
+        &moe_route_fp32);
   m.def("moe_grouped_linear_f32(Tensor xp, Tensor w_stack, Tensor(a!) y, Tensor tile_expert, Tensor tile_row0, Tensor num_tiles, int bn) -> ()",
         &moe_grouped_linear_f32);
   m.def("moe_align(Tensor ids, int experts, int expert_lo, int expert_hi, int bn, Tensor(a!) row_of, Tensor(b!) token_of, Tensor(c!) tile_expert, Tensor(d!) tile_row0, Tensor(e!) num_tiles, Tensor? weights=None, Tensor(f!)? row_weight=None) -> ()", &moe_align);
   m.def("moe_gather(Tensor x, Tensor token_of, Tensor(a!) xp, Tensor? row_weight=None) -> ()", &moe_gather);
   m.def("moe_grouped_linear(Tensor xp, Tensor w_stack, Tensor? bias_stack, Tensor(a!) y, Tensor tile_expert, Tensor tile_row0, Tensor num_tiles, int bn, Tensor? status) -> int", &moe_grouped_linear);
-  m.def("moe_combine(Tensor y, Tensor row_of, Tensor? weights, Tensor(a!) out, Tensor? add=None) -> ()", &moe_combine);
+  m.def("moe_combine(Tensor y, Tensor row_of, Tensor? weights, Tensor(a!) out, Tensor? add=None, Tensor? add_gate=None) -> ()", &moe_combine);
 }

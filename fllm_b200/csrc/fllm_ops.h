@@ -171,8 +171,15 @@ int moe_grouped_linear_bf16(const void* xp, long long ldx, const void* w_stack, 
 void moe_route_scored(const void* logits, long long ld, const float* select_bias, int tokens, int experts, int k, int score_kind,
                       int renorm, float scale, int* ids, float* weights, cudaStream_t s);
 // the same rule (without a selection bias) on fp32 logits: the sum of `splits` planes of [tokens][ld], `plane` elements each
+// groups of neighbouring experts: only experts of the `keep` groups with the best choice can be taken, the others' choice counts as
+// `masked`; gate_out (optional): column `experts` of the logits, through a sigmoid
+struct RouteGroups {
+  int groups = 1, keep = 1;
+  float masked = 0.f;
+};
 void moe_route_fp32(const float* logits, int splits, long long plane, long long ld, int tokens, int experts, int k, int score_kind, int renorm,
-                    float scale, int* ids, float* weights, cudaStream_t s);
+                    float scale, int* ids, float* weights, cudaStream_t s, const float* select_bias = nullptr, const RouteGroups& groups = RouteGroups{},
+                    float* gate_out = nullptr);
 void moe_route(const void* logits, long long ld, const void* bias, int tokens, int experts, int k, int softmax_all,
                int* ids, float* weights, cudaStream_t s);
 void moe_align(const int* ids, int tokens, int k, int expert_lo, int expert_hi, int bn, int* row_of,
@@ -182,7 +189,8 @@ void moe_gather(const void* x, long long ldx, const int* token_of, void* xp, int
                 const float* row_weight = nullptr, int f32 = 0);
 // weights null: the rows are summed as they are; add (optional): [tokens] rows added to the result
 void moe_combine(const void* y, long long ldy, const int* row_of, const float* weights, int tokens, int k, void* out,
-                 long long ldo, int hidden, cudaStream_t s, const void* add = nullptr, long long ld_add = 0, int f32 = 0);
+                 long long ldo, int hidden, cudaStream_t s, const void* add = nullptr, long long ld_add = 0, int f32 = 0,
+                 const float* add_gate = nullptr);
 
 // ---- elementwise --------------------------------------------------------------------
 void embed_bf16(const int* ids, const void* table, void* out, int tokens, int hidden, int vocab,
@@ -471,9 +479,18 @@ struct MapsPrepareParams {
   const float* inv_freq;       // [rot / 2]: pairs (i, i + rot / 2) of a map's first rot values turn
   int rot;
   float rope_factor;           // on cosine and sine
-  const void *q_norm, *k_norm; // [dim], or with full [heads * dim]
+  int pairs;                   // 1: pairs (2 i, 2 i + 1) turn instead
+  const void *q_norm, *k_norm; // [dim], or with full [heads * dim]; null: norms without weights
   int full;                    // 1: one root mean square over all maps, 0: one per map
-  float eps;
+  float eps;                   // < 0: no norms
+  // taps > 0: a causal convolution over the rows comes first; every sequence of the step has one token, whose row is its index.
+  // State rows [taps - 1][conv_width] hold the columns of the tokens before it and move on by one token.
+  const float* conv_w;         // [conv_width][taps]
+  void* conv_state;
+  const int* seq_state;
+  int taps, conv_width;
+  float* extra_out;            // [tokens][extra]: further columns of the rows, from extra_offset on, as fp32
+  int extra_offset, extra;
   void* q_out;                 // [tokens][q_heads][wk]
   void *k_cache, *v_cache;     // [blocks][k_heads][block_size][wk], [blocks][v_heads][block_size][wv]
   int f32;
@@ -494,7 +511,25 @@ struct MapsAttnParams {
   int window;                  // keys a query sees, itself included (0: all)
   float lam, out_scale, eps;   // two maps: out = rms(a1 - lam a2) * out_scale
   int f32;
+  const float *sink;           // one map, optional [H]: exp(sink) joins a head's denominator
+  const float *r1, *r2;        // one map, optional [H]: r1 ln(1 + r2 distance) is taken off a head's scores (tensor cores: with spread values)
+  // 1: value rows [blocks][block_size][wv] hold all heads' values (v_dim of them) and every head weighs all of them: part_o
+  // [tokens][H][splits][wv] and part_ml [tokens][H][splits][2] (reference, sum of weights; the sink is left to talk_mix)
+  int spread;
+  float *part_o, *part_ml;
 };
+// out head h of group g = sigmoid(gate_h) sum_f talk[h, f] (head f's weights over the values of group g)
+struct TalkMixParams {
+  const float *part_o, *part_ml;
+  const float *sink, *talk;    // [H] (optional), [H][H]
+  const float* gate;           // optional: fp32 rows of H logits
+  long long ld_gate;
+  void* out;                   // [tokens] rows of `cols` columns, zero beyond H * v_dim
+  long long ldo;
+  int tokens, H, G, splits, v_dim, wv, cols, f32;
+};
+void talk_mix(const TalkMixParams& p, cudaStream_t s);
+bool attention_spread_tc_supported(int group, int wk, int wv, int block_size, int f32);
 bool attention_maps_tc_supported(int wk, int wv, int block_size, int f32);
 int attention_maps_splits(int num_seqs, int max_q_len, int H, int G, int maps, int max_kv_len, int window);
 size_t attention_maps_workspace_bytes(int tokens, int q_heads, int wv, int splits);
@@ -529,6 +564,34 @@ struct PostNormParams {
   int write, f32;
 };
 void postnorm(const PostNormParams& p, cudaStream_t s);
+// ---- residual with the norm in front of a sublayer, token shift (prenorm.cu) ---------------------------------------------------
+struct PreNormParams {
+  const float* x;              // [rows][ld] fp32, zero beyond `width`; null: the sum starts at zero
+  float* x_out;                // the new residual (null: not written); may be x without a token shift
+  const int* ids;              // not null: table[ids[row]] is added
+  const void* table;
+  int vocab;
+  long long ld_table;
+  const void* y;               // output of the sublayer (optional), or the split-K partial sums [splits][rows][ld] of its projection
+  long long ld_y;
+  const float* partials;
+  int splits;
+  long long plane;
+  const void* norm_w;
+  float w_offset;              // h = x / rms(x) * (w_offset + w)
+  const int* rows;             // optional row selection of the outputs
+  void* h;
+  long long ld_h;
+  const void* shift;           // not null: h_t + (h_(t-1) - h_t) shift within each sequence
+  float* state;                // [slots][ld]: h of every sequence's last token
+  const int *q_starts, *seq_state, *row_seq, *positions;
+  int single;                  // every sequence has one row, its index
+  int rows_per;                // set by prenorm
+  int n_out, width, ld;
+  float eps;
+  int f32;
+};
+void prenorm(const PreNormParams& p, cudaStream_t s);
 struct SideGateParams {
   const void* gate;            // [tokens] rows, or split-K partial sums [splits][tokens][cols]
   long long ld_gate;

@@ -80,7 +80,8 @@ __global__ void moe_route_kernel(const __nv_bfloat16* __restrict__ logits, long 
 
 // Routers that weigh experts by their score: score = softmax over all experts (score_kind 1) or sigmoid (2) of the logit; the
 // k experts with the largest score + select_bias are taken (the bias only steers the choice: DeepSeek-V3, GLM-4.5, ERNIE 4.5);
-// weights = the scores of the chosen experts, renormalised on request, times `scale`. One warp per token, up to 256 experts.
+// weights = the scores of the chosen experts, renormalised on request, times `scale`. With groups of neighbouring experts only the
+// experts of the best groups (by their best choice score) can be taken. One warp per token, up to 256 experts.
 // Logits: bf16, or (Sum) fp32 as the sum of planes, then with the accurate exponential.
 struct Bf16Logits {
   const __nv_bfloat16* p;
@@ -101,7 +102,9 @@ struct SumLogits {
 };
 template <typename Logits>
 __global__ void moe_route_scored_kernel(const Logits logits, const float* __restrict__ select_bias, int tokens, int experts, int k,
-                                        int score_kind, int renorm, float scale, int* __restrict__ ids, float* __restrict__ weights) {
+                                        int score_kind, int renorm, float scale, const RouteGroups gr, int* __restrict__ ids,
+                                        float* __restrict__ weights, float* __restrict__ gate_out) {
+  __shared__ float choice[4][256], best_of[4][256];
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (t >= tokens) return;
@@ -135,6 +138,31 @@ __global__ void moe_route_scored_kernel(const Logits logits, const float* __rest
     const int e = lane + 32 * i;
     ch[i] = e < experts ? sc[i] + (select_bias ? select_bias[e] : 0.f) : -INFINITY;
   }
+  if (gr.groups > 1) {
+    float* mine = choice[threadIdx.x >> 5];
+    float* group = best_of[threadIdx.x >> 5];
+    const int per = experts / gr.groups;
+#pragma unroll
+    for (int i = 0; i < MAXPL; ++i) mine[lane + 32 * i] = ch[i];
+    __syncwarp();
+    for (int g = lane; g < gr.groups; g += 32) {
+      float m = -INFINITY;
+      for (int e = g * per; e < (g + 1) * per; ++e) m = fmaxf(m, mine[e]);
+      group[g] = m;
+    }
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < MAXPL; ++i) {
+      const int e = lane + 32 * i;
+      if (e >= experts) continue;
+      const int g = e / per;
+      const float own = group[g];
+      int ahead = 0;
+      for (int o = 0; o < gr.groups; ++o) ahead += group[o] > own || (group[o] == own && o < g);
+      if (ahead >= gr.keep) ch[i] = gr.masked;
+    }
+  }
+  if (gate_out != nullptr && lane == 0) gate_out[t] = 1.f / (1.f + ex(-logits(t, experts)));
   float sel_s[8];
   int sel_e[8];
   for (int j = 0; j < k; ++j) {
@@ -171,16 +199,17 @@ void moe_route_scored(const void* logits, long long ld, const float* select_bias
   if (tokens <= 0) return;
   if (experts > 256 || k > 8 || (score_kind != 1 && score_kind != 2)) throw std::runtime_error("moe_route_scored: at most 256 experts, top-8, score kind 1 or 2");
   moe_route_scored_kernel<<<(tokens + 3) / 4, 128, 0, s>>>(Bf16Logits{(const __nv_bfloat16*)logits, ld}, select_bias, tokens, experts, k,
-                                                           score_kind, renorm, scale, ids, weights);
+                                                           score_kind, renorm, scale, RouteGroups{}, ids, weights, (float*)nullptr);
   cuda_check(cudaGetLastError(), "moe_route_scored_kernel");
 }
 
 void moe_route_fp32(const float* logits, int splits, long long plane, long long ld, int tokens, int experts, int k, int score_kind, int renorm,
-                    float scale, int* ids, float* weights, cudaStream_t s) {
+                    float scale, int* ids, float* weights, cudaStream_t s, const float* select_bias, const RouteGroups& groups, float* gate_out) {
   if (tokens <= 0) return;
   if (experts > 256 || k > 8 || (score_kind != 1 && score_kind != 2)) throw std::runtime_error("moe_route_fp32: at most 256 experts, top-8, score kind 1 or 2");
-  moe_route_scored_kernel<<<(tokens + 3) / 4, 128, 0, s>>>(SumLogits{logits, ld, plane, splits}, (const float*)nullptr, tokens, experts, k, score_kind,
-                                                           renorm, scale, ids, weights);
+  if (groups.groups < 1 || experts % groups.groups || groups.keep < 1) throw std::runtime_error("moe_route_fp32: equal groups of experts");
+  moe_route_scored_kernel<<<(tokens + 3) / 4, 128, 0, s>>>(SumLogits{logits, ld, plane, splits}, select_bias, tokens, experts, k, score_kind,
+                                                           renorm, scale, groups, ids, weights, gate_out);
   cuda_check(cudaGetLastError(), "moe_route_fp32");
 }
 
@@ -327,11 +356,13 @@ void moe_gather(const void* x, long long ldx, const int* token_of, void* xp, int
   cuda_check(cudaGetLastError(), "moe_gather_kernel");
 }
 
-// weights (optional; none: the rows are summed as they are), add (optional): rows added to the result
+// weights (optional; none: the rows are summed as they are), add (optional): rows added to the result, each times add_gate (optional)
 template <typename T>
 __global__ void moe_combine_kernel(const T* __restrict__ y, long long ldy, const int* __restrict__ row_of, const float* __restrict__ weights, int k,
-                                   const T* __restrict__ add, long long ld_add, T* __restrict__ out, long long ldo, int hidden) {
+                                   const T* __restrict__ add, long long ld_add, const float* __restrict__ add_gate, T* __restrict__ out, long long ldo,
+                                   int hidden) {
   const int t = blockIdx.x;
+  const float ga = add_gate != nullptr ? add_gate[t] : 1.f;
   for (int i = threadIdx.x; i < hidden / 4; i += blockDim.x) {
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int j = 0; j < k; ++j) {
@@ -343,20 +374,21 @@ __global__ void moe_combine_kernel(const T* __restrict__ y, long long ldy, const
     }
     if (add != nullptr) {
       const float4 v = row4(add + (size_t)t * ld_add + 4 * i);
-      acc.x += v.x, acc.y += v.y, acc.z += v.z, acc.w += v.w;
+      acc.x = fmaf(ga, v.x, acc.x), acc.y = fmaf(ga, v.y, acc.y), acc.z = fmaf(ga, v.z, acc.z), acc.w = fmaf(ga, v.w, acc.w);
     }
     put4(out + (size_t)t * ldo + 4 * i, acc);
   }
 }
 
 void moe_combine(const void* y, long long ldy, const int* row_of, const float* weights, int tokens, int k, void* out,
-                 long long ldo, int hidden, cudaStream_t s, const void* add, long long ld_add, int f32) {
+                 long long ldo, int hidden, cudaStream_t s, const void* add, long long ld_add, int f32, const float* add_gate) {
   if (tokens <= 0) return;
   if (f32)
-    moe_combine_kernel<float><<<tokens, 128, 0, s>>>((const float*)y, ldy, row_of, weights, k, (const float*)add, ld_add, (float*)out, ldo, hidden);
+    moe_combine_kernel<float><<<tokens, 128, 0, s>>>((const float*)y, ldy, row_of, weights, k, (const float*)add, ld_add, add_gate, (float*)out, ldo,
+                                                      hidden);
   else
     moe_combine_kernel<__nv_bfloat16><<<tokens, 128, 0, s>>>((const __nv_bfloat16*)y, ldy, row_of, weights, k, (const __nv_bfloat16*)add, ld_add,
-                                                              (__nv_bfloat16*)out, ldo, hidden);
+                                                              add_gate, (__nv_bfloat16*)out, ldo, hidden);
   cuda_check(cudaGetLastError(), "moe_combine_kernel");
 }
 

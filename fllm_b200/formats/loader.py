@@ -58,6 +58,9 @@ def load_hf_checkpoint(directory: str, device="cuda", tp: int = 1, tp_rank: int 
         if cfg.arch == "dorevik":
             from .dorevik_loader import dorevik_weights
             return cfg, dorevik_weights(cfg, get, device, dtype), tok
+        if cfg.arch == "milenex":
+            from .milenex_loader import milenex_weights
+            return cfg, milenex_weights(cfg, get, device, dtype), tok
         from .sovanex_loader import sovanex_weights
         return cfg, sovanex_weights(cfg, get, device, dtype), tok
     if cfg.arch in CLASSIC_MODEL_TYPES:

@@ -18,6 +18,8 @@ from typing import List, Optional
 import torch
 
 from ..config import ModelConfig, RopeScaling, rope_inv_freq, scaled_inv_freq
+from ..ops.prenorm import TokenShift
+from .maps import MAPS_MIXERS
 from .moe import ACT_KIND
 from .weights import DecoderWeights, ShardSpec, make_shard_spec
 
@@ -164,7 +166,7 @@ class Decoder:
         scaling = rope.get("scaling") or {}
         key = (rope["dims"], rope["theta"], tuple(sorted(scaling.items())))
         if key not in self._rope_tables:
-            inv, factor = scaled_inv_freq(rope["dims"], rope["theta"], RopeScaling(**scaling))
+            inv, factor = ([], 1.0) if rope["dims"] == 0 else scaled_inv_freq(rope["dims"], rope["theta"], RopeScaling(**scaling))
             self._rope_tables[key] = (torch.tensor(inv, dtype=torch.float32, device=self.w.final_norm.device), factor)
         return self._rope_tables[key]
 
@@ -233,17 +235,18 @@ class Decoder:
                 if cfg.mlp_kind == "plain":
                     act = ops.act_(ops.linear(h, lw.shared_gate_up), cfg.act)
                 else:
-                    act = ops.linear_glu(h, lw.shared_gate_up, None, ACT_KIND.get(spec_of(cfg, lw).act, 0), cfg.swiglu_alpha, cfg.swiglu_limit,
-                                         lw.shared_layout)
+                    s = spec_of(cfg, lw)
+                    act = ops.linear_glu(h, lw.shared_gate_up, None, ACT_KIND.get(s.act, 0), cfg.swiglu_alpha,
+                                         cfg.swiglu_limit if s.shared_limit is None else s.shared_limit, lw.shared_layout)
                 ys = ops.linear(act, lw.shared_down)
-                if lw.shared_gate_w is not None:
+                if lw.shared_gate_w is not None and not spec_of(cfg, lw).fp32_router:     # (with an fp32 router the gate is one of its columns)
                     ys = (ys.float() * torch.sigmoid(ops.linear(h, lw.shared_gate_w)[:, :1].float())).to(ys.dtype)
             if lw.moe_latent_in is not None:         # the router reads the hidden state, the experts a projection of it
                 y = ops.linear(moe_ffn(self, lw, h, ops.linear(h, lw.moe_latent_in)), lw.moe_latent_out)
                 return y if ys is None else y + ys
             return moe_ffn(self, lw, h, add=ys)
-        if cfg.mlp_kind == "plain":               # two matrices and an activation between them
-            u = ops.act_(ops.linear(h, lw.w_gate_up, lw.b_up), cfg.act)
+        if cfg.mlp_kind == "plain" or lw.plain_act:    # two matrices and an activation between them
+            u = ops.act_(ops.linear(h, lw.w_gate_up, lw.b_up), lw.plain_act or cfg.act)
             return ops.linear(u, lw.w_down, lw.b_down, defer=self.defer_to_residual)
         act = ops.linear_glu(h, lw.w_gate_up, None, self.act_kind, cfg.swiglu_alpha, cfg.swiglu_limit if lw.act_limit is None else lw.act_limit,
                              getattr(lw, "glu_layout", 0))
@@ -265,6 +268,8 @@ class Decoder:
             return self._forward_streams(b)
         if cfg.postnorm_alpha > 0 or cfg.outnorm:
             return self._forward_postnorm(b)
+        if cfg.prenorm_fp32:
+            return self._forward_prenorm(b)
         if self.first_stage:
             x = ops.embed(b.token_ids, self.w.embed, cfg.embed_scale)
             if cfg.learned_positions:              # the same row gather on the position table
@@ -336,8 +341,7 @@ class Decoder:
             if cfg.layer_kind(li) == "tied":
                 from .tied import tied_attention_mixer
                 y = tied_attention_mixer(self, li, lw, h, b)
-            elif cfg.layer_kind(li) in ("maps", "maps+lightning"):
-                from .maps import MAPS_MIXERS
+            elif cfg.layer_kind(li) in MAPS_MIXERS:
                 y = MAPS_MIXERS[cfg.layer_kind(li)](self, li, lw, h, b)
             else:
                 from .recurrent import MIXERS
@@ -354,6 +358,27 @@ class Decoder:
             if self._nvtx:
                 torch.cuda.nvtx.range_pop()
         return x, pending
+
+    def _forward_prenorm(self, b: StepBatch):
+        """The layers of a model with norms in front of its sublayers and an fp32 residual. A sublayer's output is added together with
+        the next one's norm, and with the token shift where the model has one; in front of a repeated run of layers the tokens'
+        embeddings are added again. Returns (residual, output of the last sublayer)."""
+        cfg, ops = self.cfg, self.ops
+        how = (cfg.hidden_size, cfg.rms_eps, cfg.norm_weight_offset)
+        x = y = None
+        for li, lw in zip(self.layer_range, self.w.layers):
+            if self._nvtx:
+                torch.cuda.nvtx.range_push(f"layer{li}")
+            ids = b.token_ids if x is None or li in cfg.embed_again else None
+            shift = TokenShift(lw.shift, self.rstate.shift[li], b) if cfg.token_shift else None
+            x, h = ops.prenorm_step(x, y, lw.attn_norm, *how, ids=ids, table=None if ids is None else self.w.embed, shift=shift)
+            y = MAPS_MIXERS[cfg.layer_kind(li)](self, li, lw, h, b)
+            if cfg.ffn_kind(li) != "none":
+                x, h = ops.prenorm_step(x, y, lw.ffn_norm, *how)
+                y = self._ffn_block(lw, h)
+            if self._nvtx:
+                torch.cuda.nvtx.range_pop()
+        return x, y
 
     def _sublayers(self):
         """(stream coefficients, norm weight, norm bias, layer index, layer weights, is the mixer) in running order."""
@@ -480,6 +505,12 @@ class Decoder:
                 self.last_hidden = hs / cfg.logit_scale
             lg = ops.linear(hs, self.w.lm_head)
             return ops.softcap_(lg, cfg.logit_softcap) if cfg.logit_softcap > 0 else lg
+        if cfg.prenorm_fp32:                    # last update, final norm, wanted rows: one kernel
+            rows = None if b.all_decode and b.logit_rows.numel() == x.shape[0] else b.logit_rows
+            _, hs = ops.prenorm_step(x, delta, self.w.final_norm, cfg.hidden_size, cfg.rms_eps, cfg.norm_weight_offset, rows=rows)
+            if self.capture_hidden:
+                self.last_hidden = hs
+            return ops.linear(hs, self.w.lm_head)
         if cfg.arch in ("rwkv7", "rwkv6"):
             from .rwkv import rwkv7_final_norm
             h = rwkv7_final_norm(self, x)

@@ -3,14 +3,17 @@ kinds of the decoder runner. One projection makes [queries | keys | values], fol
 [queries | keys | values | gate] of the recurrent half; every segment starts on a multiple of 8 rows.
 
 Two maps are differential attention: the difference of two softmax attentions, normalised per head. Lightning attention is a
-linear attention whose state decays by a constant per head; its output is normalised over all heads and gated."""
+linear attention whose state decays by a constant per head; its output is normalised over all heads and gated. One map may have a
+short convolution over time on its projections, norms without weights, a sink, a distance bias, heads that mix their weights
+(talking heads: the values of all key/value heads then share a cache row) and a gate per head (its logits are further columns of
+the projection)."""
 from __future__ import annotations
 
 from typing import Dict, Optional
 
 import torch
 
-from ..ops.maps import Combine, NormedPair
+from ..ops.maps import Combine, ConvWindow, NormedPair
 from .recurrent import _batch_meta, pad8, pad_cols, pad_rows
 
 
@@ -20,17 +23,31 @@ def _attend(dec, li: int, m, proj, b) -> torch.Tensor:
     H, G, M, dim, v_dim = c["num_heads"], c["num_kv_heads"], c["maps"], c["head_dim"], c["v_dim"]
     at, eps = dec.kv_index[li], dec.cfg.rms_eps
     keys, values = dec.kv.layer(at), dec.kv.values(at)
-    inv_freq, factor = dec.layer_rope(c["rope"])
+    inv_freq, factor = dec.layer_rope(c["rope"] or dict(dims=0, theta=1.0))
     nq, nk = pad8(H * M * dim), pad8(G * M * dim)
-    q = ops.maps_prepare(proj, (0, nq, nq + nk), H * M, dim, v_dim, b.positions, b.slots, inv_freq, factor, m["q_norm"], m["k_norm"],
-                         c["qk_norm"] == "full", eps, keys, values, m.get("in_bias"))
+    talk, conv, gate = m.get("talk"), None, None
+    if "conv" in m:
+        qs, ss, pos = _batch_meta(b)
+        if b.max_q_len == 1:                               # one token per sequence: inside the next kernel
+            conv = ConvWindow(m["conv"], dec.rstate.conv[li], ss)
+        else:
+            proj = ops.causal_conv1d(proj[:, :m["conv"].shape[0]], m["conv"], None, dec.rstate.conv[li], qs, ss, pos, act=False, max_q_len=b.max_q_len)
+    if c.get("gate"):
+        gate = torch.empty(proj.shape[0], H, dtype=torch.float32, device=keys.device)
+    q = ops.maps_prepare(proj, (0, nq, nq + nk), H * M, dim, v_dim if talk is None else G * v_dim, b.positions, b.slots, inv_freq, factor, m.get("q_norm"),
+                         m.get("k_norm"), c["qk_norm"] == "full", -1.0 if c["qk_norm"] == "none" else eps, keys, values, m.get("in_bias"),
+                         pairs=c.get("rope_style") == "pair", conv=conv, extra_out=gate, extra_offset=nq + nk + pad8(G * v_dim))
+    terms = dict(sink=m.get("sink"), r1=m.get("r1"), r2=m.get("r2"), out_cols=m["wo"].shape[1])
+    if talk is not None:
+        return ops.attention_talk(q, keys, values, dim, v_dim, b, c["scale"], talk, c["window"], gate=gate, **terms)
     combine = Combine(m["lam"], 1.0 - c["diff"], eps) if M == 2 else None
-    return ops.attention_maps(q, keys, values, dim, v_dim, b, c["scale"], c["window"], combine, m["wo"].shape[1])
+    return ops.attention_maps(q, keys, values, dim, v_dim, b, c["scale"], c["window"], combine, **terms)
 
 
 def maps_mixer(dec, li: int, lw, h: torch.Tensor, b):
     m, ops = lw.mixer, dec.ops
-    proj = ops.linear(h, m["in_proj"], defer=dec.defer_to_residual)
+    # (the convolution of longer portions reads finished rows)
+    proj = ops.linear(h, m["in_proj"], defer=dec.defer_to_residual and not ("conv" in m and b.max_q_len > 1))
     return ops.linear(_attend(dec, li, m, proj, b), m["wo"], defer=dec.defer_to_residual)
 
 
@@ -51,13 +68,21 @@ def maps_lightning_mixer(dec, li: int, lw, h: torch.Tensor, b) -> NormedPair:
 MAPS_MIXERS = {"maps": maps_mixer, "maps+lightning": maps_lightning_mixer}
 
 
-def pack_maps(q, k, v, q_norm, k_norm, o_proj, dtype, device, biases=None, lambdas=None, diff: float = 0.0) -> Dict[str, object]:
+def pack_maps(q, k, v, q_norm, k_norm, o_proj, dtype, device, biases=None, lambdas=None, diff: float = 0.0, gate=None, convs=None,
+              terms: Optional[Dict[str, torch.Tensor]] = None) -> Dict[str, object]:
     """q [H * maps * dim, in], k [G * maps * dim, in], v [G * v_dim, in], o_proj [out, H * v_dim]; ``biases``: those of q, k and v;
-    ``lambdas``: the vectors lq1, lk1, lq2, lk2 of two maps."""
+    ``lambdas``: the vectors lq1, lk1, lq2, lk2 of two maps; norm weights may be None; ``gate`` [H, in]; ``convs``: the taps [rows, taps]
+    of q, k and v; ``terms``: fp32 numbers per head (sink, r1, r2) and the matrix over the heads (talk)."""
     put = lambda t: t.to(device=device, dtype=dtype).contiguous()
     p8 = lambda t: pad_rows(t, pad8(t.shape[0]))
-    m: Dict[str, object] = dict(in_proj=put(torch.cat([p8(t) for t in (q, k, v)], 0)), wo=put(pad_cols(o_proj, pad8(o_proj.shape[1]))),
-                                q_norm=put(q_norm), k_norm=put(k_norm))
+    f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
+    m: Dict[str, object] = dict(in_proj=put(torch.cat([p8(t) for t in ((q, k, v) if gate is None else (q, k, v, gate))], 0)),
+                                wo=put(pad_cols(o_proj, pad8(o_proj.shape[1]))))
+    if q_norm is not None:
+        m.update(q_norm=put(q_norm), k_norm=put(k_norm))
+    if convs is not None:
+        m["conv"] = f32(torch.cat([p8(t) for t in convs], 0))
+    m.update({n: f32(t) for n, t in (terms or {}).items()})
     if biases is not None:
         m["in_bias"] = put(torch.cat([p8(t) for t in biases], 0))
     if lambdas is not None:

@@ -24,14 +24,15 @@ def spec_of(cfg, lw=None) -> MoeSpec:
     return cfg if isinstance(cfg, MoeSpec) else (getattr(lw, "moe", None) or cfg.moe)
 
 
-def _act(cfg, gu: torch.Tensor, act: str) -> torch.Tensor:
+def _act(cfg, gu: torch.Tensor, act: str, limit: Optional[float] = None) -> torch.Tensor:
     if cfg.mlp_kind == "plain":                  # experts of two matrices: the activation alone
         return {"gelu": F.gelu, "gelu_tanh": lambda t: F.gelu(t, approximate="tanh"), "relu2": lambda t: F.relu(t).square(),
                 "silu": F.silu, "relu": F.relu}[act](gu)
     if act == "swiglu_oai":
         g, u = gu[..., 0::2], gu[..., 1::2]
-        g = g.clamp(max=cfg.swiglu_limit)
-        u = u.clamp(min=-cfg.swiglu_limit, max=cfg.swiglu_limit)
+        limit = cfg.swiglu_limit if limit is None else limit
+        g = g.clamp(max=limit)
+        u = u.clamp(min=-limit, max=limit)
         return g * torch.sigmoid(cfg.swiglu_alpha * g) * (u + 1)
     I = gu.shape[-1] // 2
     g, u = gu[..., :I], gu[..., I:]
@@ -40,7 +41,7 @@ def _act(cfg, gu: torch.Tensor, act: str) -> torch.Tensor:
 
 def route_deepseek(cfg, logits: torch.Tensor, bias: Optional[torch.Tensor]):
     """The DeepSeek routers in plain tensor ops (the selection is [T, E]-sized work). V2: softmax scores, experts
-    outside the best groups (by their best expert) masked, top-k, weights = scores. V3: sigmoid scores, selection on
+    outside the best groups (by their best expert) masked (their choice score becomes ``masked``), top-k, weights = scores. V3: sigmoid scores, selection on
     scores + bias with groups ranked by the sum of their two best, weights = unbiased scores, renormalised. Both scale
     the weights by ``scale``. ``cfg``: a model's configuration or a layer's MoeSpec."""
     spec = spec_of(cfg)
@@ -56,7 +57,7 @@ def route_deepseek(cfg, logits: torch.Tensor, bias: Optional[torch.Tensor]):
         group_rank = choice.view(-1, G, E // G).max(-1).values
     if G > 1:
         keep = torch.zeros_like(group_rank).scatter_(1, group_rank.topk(spec.topk_groups, dim=-1)[1], 1.0)
-        choice = choice.masked_fill(keep[:, :, None].expand(-1, G, E // G).reshape(-1, E) == 0, 0.0)
+        choice = choice.masked_fill(keep[:, :, None].expand(-1, G, E // G).reshape(-1, E) == 0, spec.masked)
     ids = choice.topk(k, dim=-1)[1]
     w = scores.gather(1, ids)
     if spec.norm_topk:
@@ -106,7 +107,7 @@ def moe_reference(cfg, lw, h: torch.Tensor, expert_lo: int = 0, round_bf16: bool
         gu = x @ lw.exp_gate_up[e].float().t()
         if lw.exp_gate_up_b is not None:
             gu = gu + lw.exp_gate_up_b[e].float()
-        a = r(_act(cfg, r(gu), spec.act))
+        a = r(_act(cfg, r(gu), spec.act, spec.limit))
         y = a @ lw.exp_down[e].float().t()
         if lw.exp_down_b is not None:
             y = y + lw.exp_down_b[e].float()
@@ -144,16 +145,19 @@ def _grouped(k_ops, ops, x, w, bias, y, tile_e, tile_r, ntiles, bn):
         k_ops.moe_grouped_linear(x, w, bias, y, tile_e, tile_r, ntiles, bn, ops.status)
 
 
-def _padded_router(lw):
-    """Router weight and bias with the expert count padded to a multiple of 8 (e.g. 60 experts)."""
+def _padded_router(lw, gate=None):
+    """Router weight and bias with the expert count padded to a multiple of 8 (e.g. 60 experts); ``gate`` [.., H]: its first row follows
+    the experts'."""
     E = lw.router_w.shape[0]
-    if E % 8 == 0:
+    if E % 8 == 0 and gate is None:
         return lw.router_w, lw.router_b
     pad = getattr(lw, "_router_pad", None)
     if pad is None:
-        Ep = (E + 7) // 8 * 8
+        Ep = (E + (gate is not None) + 7) // 8 * 8
         wp = torch.zeros(Ep, lw.router_w.shape[1], dtype=lw.router_w.dtype, device=lw.router_w.device)
         wp[:E] = lw.router_w
+        if gate is not None:
+            wp[E] = gate[0]
         bp = None
         if lw.router_b is not None:
             bp = torch.zeros(Ep, dtype=lw.router_b.dtype, device=lw.router_b.device)
@@ -168,15 +172,17 @@ def _router_logits(ops, lw, h: torch.Tensor) -> torch.Tensor:
     return ops.linear(h, w, b)[:, :lw.router_w.shape[0]]
 
 
-def _route_fp32(ops, spec: MoeSpec, lw, h: torch.Tensor, ids, wts):
-    """Selection by scores of fp32 logits: the GEMM's split-K partial sums, which the routing kernel adds, or an fp32 product."""
-    w, _ = _padded_router(lw)
+def _route_fp32(ops, spec: MoeSpec, lw, h: torch.Tensor, ids, wts, gate=None):
+    """Selection by scores of fp32 logits: the GEMM's split-K partial sums, which the routing kernel adds, or an fp32 product.
+    ``gate`` [T]: receives the sigmoid of the shared experts' gate, one more row of the router."""
+    w, _ = _padded_router(lw, lw.shared_gate_w)
     z = ops.linear(h, w, force_splits=2, defer=True) if h.dtype != torch.float32 and h.shape[1] > 64 else None
     splits = getattr(z, "splits", 0)
     if not splits:                               # narrow models, products the GEMM does not split, fp32 serving
         z = ops.linear(h.float(), w.float())
     ops.k.moe_route_fp32(None if splits else z, ops.workspace if splits else None, int(splits), int(w.shape[0]), spec.experts, spec.top,
-                         2 if spec.router == "deepseek_v3" else 1, bool(spec.norm_topk), float(spec.scale), ids, wts)
+                         2 if spec.router == "deepseek_v3" else 1, bool(spec.norm_topk), float(spec.scale), ids, wts, getattr(lw, "router_select_b", None),
+                         max(spec.groups, 1), max(spec.topk_groups, 1), float(spec.masked), gate)
 
 
 def moe_ffn(dec, lw, h: torch.Tensor, xe: Optional[torch.Tensor] = None, add: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -184,8 +190,11 @@ def moe_ffn(dec, lw, h: torch.Tensor, xe: Optional[torch.Tensor] = None, add: Op
     added to the result (always-on experts)."""
     cfg, ops, sp, spec = dec.cfg, dec.ops, dec.spec, spec_of(dec.cfg, lw)
     lo = sp.expert_start if sp.expert_parallel else 0
+    gated = add is not None and spec.fp32_router and lw.shared_gate_w is not None      # the gate of `add` is a column of the router
     if not hasattr(ops, "k") or not h.is_cuda:
         y = moe_reference(cfg, _dense_experts(lw), h, lo, h.dtype != torch.float32, xe)
+        if gated:
+            add = add.float() * torch.sigmoid(h.float() @ lw.shared_gate_w[0].float())[:, None]
         return (y if add is None else y + add.float()).to(h.dtype)
     k_ops = ops.k
     T, H = (h if xe is None else xe).shape
@@ -195,12 +204,19 @@ def moe_ffn(dec, lw, h: torch.Tensor, xe: Optional[torch.Tensor] = None, add: Op
     wts = torch.empty(T, k, dtype=torch.float32, device=h.device)
     small = spec.experts <= 256 and k <= 8       # the routing kernels' register budget; beyond it the same rule in tensor ops
     scored = spec.router in ("deepseek_v2", "deepseek_v3")
-    if spec.fp32_router and scored and spec.groups <= 1 and small:
-        _route_fp32(ops, spec, lw, h, ids, wts)
+    gate = torch.empty(T, dtype=torch.float32, device=h.device) if gated else None
+    if spec.fp32_router and scored and small:
+        _route_fp32(ops, spec, lw, h, ids, wts, gate)
     else:
-        logits = ops.linear(h.float(), _padded_router(lw)[0].float())[:, :spec.experts] if spec.fp32_router else _router_logits(ops, lw, h)
+        if spec.fp32_router:
+            logits = ops.linear(h.float(), _padded_router(lw, lw.shared_gate_w)[0].float())
+            if gated:
+                gate = torch.sigmoid(logits[:, spec.experts]).contiguous()
+            logits = logits[:, :spec.experts]
+        else:
+            logits = _router_logits(ops, lw, h)
         if scored:
-            if spec.groups <= 1 and small:       # one kernel; grouped selection stays in tensor ops
+            if spec.groups <= 1 and small:       # one kernel; grouped selection by bf16 logits stays in tensor ops
                 k_ops.moe_route_scored(logits, getattr(lw, "router_select_b", None), k, 2 if spec.router == "deepseek_v3" else 1,
                                        bool(spec.norm_topk), float(spec.scale), ids, wts)
             else:
@@ -225,11 +241,12 @@ def moe_ffn(dec, lw, h: torch.Tensor, xe: Optional[torch.Tensor] = None, add: Op
     k_ops.moe_gather(h if xe is None else xe, token_of, xp, row_w)
     gu = torch.empty(rows_cap, lw.exp_gate_up.shape[1], dtype=h.dtype, device=h.device)
     _grouped(k_ops, ops, xp, lw.exp_gate_up, lw.exp_gate_up_b, gu, tile_e, tile_r, ntiles, bn)
-    act = ops.act_(gu, spec.act) if cfg.mlp_kind == "plain" else ops.glu(gu, ACT_KIND.get(spec.act, 0), cfg.swiglu_alpha, cfg.swiglu_limit)
+    act = ops.act_(gu, spec.act) if cfg.mlp_kind == "plain" else \
+        ops.glu(gu, ACT_KIND.get(spec.act, 0), cfg.swiglu_alpha, cfg.swiglu_limit if spec.limit is None else spec.limit)
     y = torch.empty(rows_cap, H, dtype=h.dtype, device=h.device)
     _grouped(k_ops, ops, act, lw.exp_down, lw.exp_down_b, y, tile_e, tile_r, ntiles, bn)
     out = torch.empty(T, H, dtype=h.dtype, device=h.device)
-    k_ops.moe_combine(y, row_of, None if spec.weigh_input else wts, out, add)
+    k_ops.moe_combine(y, row_of, None if spec.weigh_input else wts, out, add, gate)
     ops.launches += 6
     return out
 

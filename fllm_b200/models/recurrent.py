@@ -39,6 +39,8 @@ def conv_channels(cfg: ModelConfig, kind: str, layer: int = 0) -> int:
         return 2 * pad8(s["num_k_heads"] * s["head_k_dim"]) + pad8(s["num_v_heads"] * s["head_v_dim"])
     if kind in ("shortconv", "rwkv7", "rwkv6"):
         return cfg.hidden_size
+    if kind == "maps":
+        return pad8(s["num_heads"] * s["maps"] * s["head_dim"]) + pad8(s["num_kv_heads"] * s["maps"] * s["head_dim"]) + pad8(s["num_kv_heads"] * s["v_dim"])
     raise ValueError(kind)
 
 
@@ -59,15 +61,23 @@ def scan_state_shape(cfg: ModelConfig, kind: str, layer: int = 0):
 
 class RecurrentState:
     """State pools of this stage's recurrent layers: per layer a convolution window [slots, W - 1, C] in the activation type (bf16 on a GPU; none for
-    lightning attention) and (except for the short convolution) an fp32 scan state [slots, ...]. The last row is the scratch row of padding sequences."""
+    lightning attention) and (except for the short convolution) an fp32 scan state [slots, ...]. Attention of kind "maps" has a convolution window where
+    its projections pass through one, and with a token shift in front of the mixers every layer has an fp32 row [slots, padded width]. The last row is
+    the scratch row of padding sequences."""
 
     def __init__(self, cfg: ModelConfig, layer_range: range, slots: int, device, act_dtype=torch.bfloat16):
         self.slots = slots
         self.conv: Dict[int, torch.Tensor] = {}
         self.scan: Dict[int, torch.Tensor] = {}
         self.shift2: Dict[int, torch.Tensor] = {}          # RWKV: the channel mix has a token shift of its own
+        self.shift: Dict[int, torch.Tensor] = {}           # the normalised input of every sequence's last token
         for li in layer_range:
             kind = _state_kind(cfg.layer_kind(li))
+            if cfg.token_shift:
+                self.shift[li] = torch.zeros(slots, pad8(cfg.hidden_size), dtype=torch.float32, device=device)
+            taps = cfg.conv_taps(li)
+            if taps > 1:
+                self.conv[li] = torch.zeros(slots, taps - 1, conv_channels(cfg, kind, li), dtype=act_dtype, device=device)
             if kind in STATELESS_KINDS:
                 continue
             W = cfg.ssm_of(li).get("d_conv", 4)
@@ -84,6 +94,10 @@ class RecurrentState:
         n = 0
         for li in layer_range:
             kind = _state_kind(cfg.layer_kind(li))
+            if cfg.token_shift:
+                n += pad8(cfg.hidden_size) * 4
+            if cfg.conv_taps(li) > 1:
+                n += (cfg.conv_taps(li) - 1) * conv_channels(cfg, kind, li) * elem
             if kind in STATELESS_KINDS:
                 continue
             W = cfg.ssm_of(li).get("d_conv", 4)
@@ -98,7 +112,7 @@ class RecurrentState:
         return n
 
     def nbytes(self) -> int:
-        return sum(t.numel() * t.element_size() for d in (self.conv, self.scan, self.shift2) for t in d.values())
+        return sum(t.numel() * t.element_size() for d in (self.conv, self.scan, self.shift2, self.shift) for t in d.values())
 
 
 def _batch_meta(b):

@@ -10,7 +10,7 @@ import torch
 
 from ..config import ModelConfig
 from ..ops.latent import latent_width
-from ..ops.maps import maps_width
+from ..ops.maps import maps_width, spread_width
 from ..ops.tied import tied_width
 
 
@@ -70,7 +70,9 @@ class RowCache:
                 out.append(RowSpec(tied_width(c["head_dim"]), c["num_kv_heads"]))
             elif cfg.layer_kind(li) in ("maps", "maps+lightning"):
                 c = cfg.attn_of(li)
-                out.append(RowSpec(maps_width(c["head_dim"]), c["num_kv_heads"] * c["maps"], maps_width(c["v_dim"]), c["num_kv_heads"]))
+                one = c.get("talk")                # heads that mix their weights read the values of all heads as one row
+                out.append(RowSpec(maps_width(c["head_dim"]), c["num_kv_heads"] * c["maps"], spread_width(c["num_kv_heads"] * c["v_dim"]) if one else
+                                   maps_width(c["v_dim"]), 1 if one else c["num_kv_heads"]))
         return out
 
     @staticmethod

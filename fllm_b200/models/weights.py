@@ -79,6 +79,8 @@ class LayerWeights:
     streams1: Optional["StreamMix"] = None
     streams2: Optional["StreamMix"] = None
     side: Optional["SideInput"] = None              # per-layer token input behind the layer
+    shift: Optional[torch.Tensor] = None            # token shift: step towards the token before, per channel
+    plain_act: str = ""                             # a dense network of two matrices in a model of gated ones: its activation
     act_limit: Optional[float] = None               # clamp of this layer's gated activation (None: the model's)
     moe: Optional[MoeSpec] = None                   # routed experts that differ from layer to layer (None: the model's)
     # packed formats keep their payload here (format name -> tensors)
@@ -291,6 +293,11 @@ def init_random_weights(cfg: ModelConfig, device="cpu", dtype=torch.bfloat16, se
         if tp > 1 or (layers is not None and len(layers) != cfg.num_layers):
             raise NotImplementedError("models with a residual in fp32 run on one rank and one pipeline stage")
         return dorevik_weights(cfg, random_tensors(cfg, seed, device), device, dtype)
+    if cfg.arch == "milenex":
+        from ..formats.milenex_loader import milenex_weights, random_tensors
+        if tp > 1 or (layers is not None and len(layers) != cfg.num_layers):
+            raise NotImplementedError("models with a residual in fp32 run on one rank and one pipeline stage")
+        return milenex_weights(cfg, random_tensors(cfg, seed, device), device, dtype)
     sp = make_shard_spec(cfg, tp, tp_rank, expert_parallel)
     D, H = cfg.head_dim, cfg.hidden_size
     layers = range(cfg.num_layers) if layers is None else layers

@@ -14,6 +14,7 @@ import torch
 from ._lib import load_cuda
 from .latent import LatentNative
 from .maps import MapsNative
+from .prenorm import PreNormNative
 from .recurrent import RecurrentNative
 from .tied import TiedNative
 
@@ -33,7 +34,7 @@ class Deferred:
         return (self.rows, self.cols)
 
 
-class NativeOps(RecurrentNative, LatentNative, TiedNative, MapsNative):
+class NativeOps(RecurrentNative, LatentNative, TiedNative, MapsNative, PreNormNative):
     name = "sm100a"
 
     def __init__(self, device: torch.device, workspace_bytes: int = 96 << 20, part: str = ""):

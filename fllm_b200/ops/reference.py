@@ -13,11 +13,12 @@ import torch.nn.functional as F
 
 from .latent import LatentRef
 from .maps import MapsRef
+from .prenorm import PreNormRef
 from .tied import TiedRef
 from .recurrent import RecurrentRef
 
 
-class RefOps(RecurrentRef, LatentRef, TiedRef, MapsRef):
+class RefOps(RecurrentRef, LatentRef, TiedRef, MapsRef, PreNormRef):
     name = "reference"
 
     # ---------------------------------------------------------------- dense

@@ -25,7 +25,7 @@ class StateCheckpoints:
 
     def _pools(self) -> List[torch.Tensor]:
         r = self.rstate
-        return [d[li] for d in (r.conv, r.scan, r.shift2) for li in sorted(d)]
+        return [d[li] for d in (r.conv, r.scan, r.shift2, r.shift) for li in sorted(d)]
 
     def has(self, h: bytes) -> bool:
         return h in self.items
