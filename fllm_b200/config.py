@@ -1245,7 +1245,7 @@ def preset(name: str) -> ModelConfig:
     if n in ("milenex-tiny", "milenex-3b"):
         # talking-heads and rotary layers in turn, experts in all but the first; the first half runs twice
         tiny = n.endswith("tiny")
-        talking = dict(heads=6 if tiny else 16, kv_heads=3 if tiny else 4, dim=20 if tiny else 96, vdim=12 if tiny else 64, mask=dict(size=21 if tiny else 1024))
+        talking = dict(heads=8 if tiny else 16, kv_heads=2 if tiny else 4, dim=20 if tiny else 96, vdim=12 if tiny else 64, mask=dict(size=21 if tiny else 1024))
         rotary = dict(heads=4 if tiny else 16, kv_heads=2 if tiny else 4, dim=32 if tiny else 128, vdim=24 if tiny else 128, conv=3 if tiny else 4,
                       mask=dict(size=37 if tiny else 2048), rot=dict(base=1e4, dims=16 if tiny else 64))
         for m in (talking, rotary):
