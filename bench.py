@@ -157,7 +157,7 @@ def main() -> None:
     ap.add_argument("--profile-step", action="store_true",
                     help="bracket ONE replay of the decode step with cudaProfilerStart/Stop (for a profiler's "
                          "launch list, run with --profile-from-start off) and exit")
-    ap.add_argument("--compare", default=None, choices=["sovanex", "divanex", "dorevik"],
+    ap.add_argument("--compare", default=None, choices=["sovanex", "divanex", "dorevik", "milenex"],
                     help="instead of the workload above: prefill and decode throughput of this design beside the closest other "
                          "model at equal sizes (random weights), one JSON line")
     ap.add_argument("--sizes", default="1b,3b,7b", help="with --compare: model sizes")

@@ -35,7 +35,7 @@ _COMMON = ("binding", "binding_recurrent", "binding_f32", "elementwise", "sampli
 PARTS = {
     "latent": _COMMON + ("binding_latent", "attention_latent", "streams"),
     "tied": _COMMON + ("binding_tied", "binding_postnorm", "attention_tied", "postnorm"),
-    "maps": _COMMON + ("binding_maps", "binding_postnorm", "binding_prenorm", "binding_moe", "attention_maps", "postnorm", "prenorm", "moe"),
+    "maps": _COMMON + ("binding_maps", "binding_postnorm", "binding_prenorm", "binding_moe", "attention_maps", "attention_talk", "postnorm", "prenorm", "moe"),
 }
 
 

@@ -1,4 +1,5 @@
-"""Throughput of a design beside the framework's closest other model at equal size (``bench.py --compare sovanex|divanex|dorevik``).
+"""Throughput of a design beside the framework's closest other model at equal size (``bench.py --compare
+sovanex|divanex|dorevik|milenex``).
 
 The closest other model of Sovanex is a hybrid of the layer kinds it shares with other families: the gated delta rule
 (Qwen3-Next) and 512 + 64 wide latent attention (DeepSeek), with the same layer order, heads, widths and squared-ReLU
@@ -8,7 +9,9 @@ layer order, sizes and clamped SwiGLU networks (gpt-oss), but separate values, n
 residual, and no token input. That of Dorevik is a hybrid of windowed grouped-query attention with normalised queries and keys,
 of that attention beside Mamba-2 (Falcon-H1) and of routed experts beside a shared one (DeepSeek-V3's router), with the same
 layer order and as many weights and products, but one softmax per head, weights on the experts' outputs, and norms in front of
-the blocks around one bf16 residual. Both models run random weights through the engine: prompts of 1024 tokens in 2048-token
+the blocks around one bf16 residual. That of Milenex is a stack of windowed grouped-query attention with sinks and of clamped SwiGLU
+networks and experts (gpt-oss) with a shared expert, as many layers as Milenex runs and as many weights in each, but no
+convolution, no mixing of heads, no token shift, and one bf16 residual. Both models run random weights through the engine: prompts of 1024 tokens in 2048-token
 steps, then captured decode steps. ``--kernels`` times the kernels that differ, each beside its like kernel on the same sizes.
 """
 from __future__ import annotations
@@ -19,7 +22,7 @@ from typing import Dict, List
 
 import torch
 
-from .config import EngineConfig, ModelConfig, divanex_from_config, dorevik_from_config, sovanex_from_config
+from .config import EngineConfig, ModelConfig, divanex_from_config, dorevik_from_config, milenex_from_config, sovanex_from_config
 
 # name -> width, layers, feed-forward width, value heads / key heads of the delta rule, attention heads
 SIZES = {"1b": (2048, 12, 8192, 32, 16, 16), "3b": (3072, 24, 12288, 48, 24, 24), "7b": (4096, 32, 16384, 64, 32, 32)}
@@ -101,6 +104,33 @@ def dorevik_twin_config(size: str) -> ModelConfig:
                        router_kind="deepseek_v3", layer_kinds=["attention+mamba2" if i % 4 == 3 else "attention" for i in range(L)],
                        ffn_kinds=["moe" if i % 2 else "glu" for i in range(L)],
                        ssm=dict(d_inner=H * 128, d_state=128, d_conv=4, n_groups=H, head_dim=64, n_heads=2 * H, norm_groups=1, conv_bias=True, dt_min=0.0, dt_max=1e30))
+
+
+# name -> width, layers (the first quarter runs twice), feed-forward width of two matrices, query / key heads (of 128, values of 64 in the
+# talking-heads layers), experts (in 8 groups, the best 4 kept), their width, shared width, tokens of every window
+MILENEX_SIZES = {"1b": (2048, 12, 9216, 16, 4, 32, 768, 1536, 1024), "3b": (3072, 16, 13824, 24, 6, 32, 1024, 2048, 1024),
+                 "7b": (4096, 20, 18432, 32, 8, 32, 1536, 3072, 1024)}
+MILENEX_TOP = 4
+
+
+def milenex_config(size: str) -> ModelConfig:
+    W, L, ff, H, G, E, fe, fs, window = MILENEX_SIZES[size]
+    heads = dict(heads=H, kv_heads=G, dim=128, scale=128 ** -0.5, mask=dict(size=window))
+    rotary, talking = dict(heads, vdim=128, conv=4, rot=dict(base=1e6, dims=128)), dict(heads, vdim=64)
+    moe = dict(kind="moe", expert=dict(ff=fe, limit=7.0), router=dict(experts=E, top=MILENEX_TOP, groups=dict(count=8, keep=4)), shared=dict(ff=fs, limit=7.0))
+    layers = [dict(type="attention" if i % 4 in (1, 2) else "attention_2", mixer=rotary if i % 4 in (1, 2) else talking, mlp=moe if i % 2 else dict(kind="dense", ff=ff))
+              for i in range(L)]
+    return milenex_from_config(ModelConfig, dict(architecture="Milenex", name=f"milenex-{size}", layers=layers, loop=dict(start=0, stop=L // 4, times=2),
+                                                 norm=dict(eps=1e-6), vocab=VOCAB, width=W))
+
+
+def milenex_twin_config(size: str) -> ModelConfig:
+    W, L, ff, H, G, E, fe, fs, window = MILENEX_SIZES[size]
+    order = milenex_config(size).layer_source
+    return ModelConfig(arch="hybrid", name=f"gqa-sink-moe-{size}", vocab_size=VOCAB, hidden_size=W, num_layers=len(order), num_heads=H, num_kv_heads=G, head_dim=128,
+                       rope_theta=1e6, attn_sinks=True, sliding_window=window, intermediate_size=ff * 2 // 3, act="swiglu_oai", tie_embeddings=False, num_experts=E,
+                       experts_per_token=MILENEX_TOP, moe_intermediate_size=fe, shared_intermediate_size=fs, router_kind="deepseek_v2",
+                       layer_kinds=["attention"] * len(order), ffn_kinds=["moe" if i % 2 else "glu" for i in order])
 
 
 def throughput(cfg: ModelConfig, batch: int, prompt_len: int, steps: int, warmup: int, device, graphs: bool = True) -> Dict[str, float]:
@@ -377,7 +407,87 @@ def dorevik_kernels(device, size: str = "1b") -> List[dict]:
     return tab.rows
 
 
-DESIGNS = {"dorevik": (dorevik_config, dorevik_twin_config, dorevik_kernels), "sovanex": (sovanex_config, twin_config, sovanex_kernels), "divanex": (divanex_config, divanex_twin_config, divanex_kernels)}
+def milenex_kernels(device, size: str = "1b") -> List[dict]:
+    from .ops.maps import ConvWindow
+    from .ops.prenorm import TokenShift
+    tab = _Table(device)
+    ops, rnd, floor, bf = tab.ops, tab.rnd, tab.floor, torch.bfloat16
+    W, _, ff, H, G, E, fe, fs, _ = MILENEX_SIZES[size]
+    D, V = 128, 64
+    per_head = lambda: torch.rand(H, device=device)
+    for shape, lens, ctxs, windows in (("decode 64 x 1152", [1] * 64, [1152] * 64, (0, 512)), ("decode 8 x 4096", [1] * 8, [4096] * 8, (0, 512)),
+                                       ("prompt 2048", [2048], [2048], (0, 512)), ("prompt 8192", [8192], [8192], (0, 1024)),
+                                       ("prompt 4 x 512 at 2048", [512] * 4, [2048] * 4, (0, 512))):
+        b = _batch(lens, ctxs, device)
+        T = b.tokens
+        b.min_q_len, b.seq_lens = min(lens), torch.tensor(ctxs, dtype=torch.int32, device=device)
+        kc, vc, joint = rnd(b.blocks, G, 16, D), rnd(b.blocks, G, 16, D), rnd(b.blocks, 1, 16, G * V)
+        q, sink, r1, r2, gate = rnd(T, H, D), per_head(), per_head(), per_head(), rnd(T, H, dtype=torch.float32)
+        mix, sinks = torch.eye(H, device=device) + 0.1, sink.float()
+        for window in windows:
+            see = lambda i: min(i + 1, window or i + 1)
+            keys = sum(see(i) for n, c in zip(lens, ctxs) for i in range(c - n, c))
+            rows = sum(min(c, n + (window or c) - 1) for n, c in zip(lens, ctxs))
+            fl = floor(rows * G * 4 * D + 4 * T * H * D, 4.0 * keys * H * D)
+            talk_bytes = rows * G * 2 * (D + V) + 2 * T * H * (D + V)
+            like = tab.time(lambda: ops.attention(q.view(T, -1), kc, vc, b.block_tables, b.row_seq, b.positions, H, G, D, D ** -0.5, window, sinks, 0.0, meta=b))
+            at = f"{shape}, window {window}" if window else shape
+            tab.add(at, "attention_maps, sink", tab.time(lambda: ops.attention_maps(q, kc, vc, D, D, b, D ** -0.5, window, sink=sink)), fl, "attention, sink", like, fl)
+            us = tab.time(lambda: ops.attention_talk(q, kc, joint, D, V, b, D ** -0.5, mix, window, sink, r1, r2, gate, reach=9.0))
+            # products: scores, mixed weights, values once per head; or the values of all key/value heads per head, as one pass over the keys needs
+            tab.add(at, "attention_talk", us, floor(talk_bytes, 2.0 * keys * H * (D + V + H)), "attention, sink", like, fl)
+            tab.add(at, "attention_talk, products of one pass", us, floor(talk_bytes, 2.0 * keys * H * (D + G * V)), "attention, sink", like, fl)
+        if len(lens) == 4:
+            continue
+        N = (H + 2 * G) * D
+        x, w, inv, qs, none = rnd(T, N), torch.ones(D, device=device, dtype=bf), torch.rand(D // 2, device=device), b.q_starts, torch.zeros(0, device=device)
+        fl = floor(2 * T * (2 * H + 4 * G) * D)
+        like = tab.time(lambda: ops.rope_kv_write(x, b.positions, b.slots, inv, w, w, kc, vc, H, G, D, D, 0, 1e-5))
+        prepare = lambda conv=None: ops.maps_prepare(x, (0, H * D, (H + G) * D), H, D, D, b.positions, b.slots, inv, 1.0, None, None, False, 1e-5, kc, vc, pairs=True,
+                                                     conv=conv)
+        tab.add(shape, "maps_prepare, norms without weights", tab.time(prepare), fl, "rope_kv_write", like, fl)
+        cw, state = torch.rand(N, 4, device=device), torch.zeros(b.num_seqs, 3, N, device=device, dtype=bf)
+        if lens[0] == 1:
+            tab.add(shape, "maps_prepare behind a convolution", tab.time(lambda: prepare(ConvWindow(cw, state, b.seq_state))),
+                    floor(2 * T * (2 * H + 4 * G) * D + 12 * T * N + 16 * N), "rope_kv_write", like, fl)
+        else:
+            us = tab.time(lambda: ops.causal_conv1d(x, cw, None, state, qs, b.seq_state, b.positions, False, b.max_q_len))
+            us2 = tab.time(lambda: ops.causal_conv1d(x, cw, None, state, qs, b.seq_state, b.positions, True, b.max_q_len))
+            tab.add(shape, "convolution", us, floor(4 * T * N), "the same with an activation", us2, floor(4 * T * N))
+        gates, xt = torch.empty(T, H, device=device), rnd(T, H * D + G * (D + V) + H)
+        tab.add(shape, "maps_prepare, joint values and gates", tab.time(lambda: ops.maps_prepare(
+            xt, (0, H * D, (H + G) * D), H, D, G * V, b.positions, b.slots, none, 1.0, None, None, False, -1.0, kc, joint, extra_out=gates, extra_offset=(H + G) * D + G * V)),
+            floor(2 * T * (2 * H * D + 2 * G * (D + V) + 3 * H)), "rope_kv_write", like, fl)
+    for T in (64, 2048):
+        shape = f"{T} rows"
+        b = _batch([1] * T if T == 64 else [T], [1024] * T if T == 64 else [T], device)
+        x, y, y2, res, w = rnd(T, W, dtype=torch.float32), rnd(T, W), rnd(T, W), rnd(T, W), torch.ones(W, device=device, dtype=bf)
+        state = torch.zeros(b.num_seqs, W, device=device)
+        norm, norm_fl = tab.time(lambda: ops.rmsnorm(res, y, w, 1e-5)), floor(T * W * 8)
+        tab.add(shape, "prenorm", tab.time(lambda: ops.prenorm_step(x, y, w, W, 1e-5)), floor(T * W * 12), "residual add + rmsnorm", norm, norm_fl)
+        tab.add(shape, "prenorm with a token shift", tab.time(lambda: ops.prenorm_step(x, y, w, W, 1e-5, shift=TokenShift(w, state, b))),
+                floor(T * W * 12 + state.numel() * 8), "residual add + rmsnorm", norm, norm_fl)
+        rw, rw8, bias = rnd(E, W), rnd(E + 8, W), torch.zeros(E, device=device)
+        ids, wts, gate = torch.empty(T, MILENEX_TOP, dtype=torch.int32, device=device), torch.empty(T, MILENEX_TOP, device=device), torch.empty(T, device=device)
+
+        def routed(grouped):
+            if grouped:
+                z = ops.linear(y, rw8, force_splits=2, defer=True)
+                ops.k.moe_route_fp32(None, ops.workspace, z.splits, E + 8, E, MILENEX_TOP, 1, False, 1.0, ids, wts, bias, 8, 4, float("-inf"), gate)
+            else:
+                ops.k.moe_route_scored(ops.linear(y, rw), bias, MILENEX_TOP, 1, False, 1.0, ids, wts)
+        fl = floor(2 * (T * W + E * W))
+        tab.add(shape, "router, fp32 logits, groups, shared gate", tab.time(lambda: routed(True)), fl, "router, bf16 logits", tab.time(lambda: routed(False)), fl)
+        n = T * MILENEX_TOP
+        xp, row_of = rnd(n, W), torch.arange(n, device=device).int().view(T, -1)
+        tab.add(shape, "combine with the gated shared expert", tab.time(lambda: ops.k.moe_combine(xp, row_of, wts, y2, res, gate)), floor(2 * (2 * T + n) * W), "combine",
+                tab.time(lambda: ops.k.moe_combine(xp, row_of, wts, y2)), floor(2 * (T + n) * W))
+        u, gu = rnd(T, ff), rnd(T, 2 * ff)
+        tab.add(shape, "gelu", tab.time(lambda: ops.act_(u, "gelu")), floor(4 * T * ff), "clamped SwiGLU", tab.time(lambda: ops.glu(gu, 2)), floor(6 * T * ff))
+    return tab.rows
+
+
+DESIGNS = {"milenex": (milenex_config, milenex_twin_config, milenex_kernels), "dorevik": (dorevik_config, dorevik_twin_config, dorevik_kernels), "sovanex": (sovanex_config, twin_config, sovanex_kernels), "divanex": (divanex_config, divanex_twin_config, divanex_kernels)}
 
 
 def main(args) -> dict:

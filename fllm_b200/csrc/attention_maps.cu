@@ -16,7 +16,7 @@
 //   maps_decode_kernel   mma.sync, 16 query rows per CTA (two maps: 8 rows of each), each warp streaming its own 16-token pages
 //                        through a private cp.async ring; split over key slices.
 //   maps_simple_kernel   CUDA cores, any width, bf16 and fp32.
-//   talk_mix_kernel      spread attention: partial sums of all heads -> mixed, gated heads.
+// (Spread attention on the tensor cores and the mixing of its heads: attention_talk.cu.)
 //
 // Weights are fp32; for the tensor-core product with the values a weight travels as the sum of two bf16 values (16 significant
 // bits). The maps are combined in fp32 before anything is rounded. Nothing in front of a window's first page is read.
@@ -34,12 +34,12 @@
 
 namespace fllm {
 namespace {
-constexpr float kLn2 = 0.6931471805599453f;
 constexpr int kDecodeRows = 64;           // sequences with at most this many query rows per kv head run in the decode kernel
 
 // ------------------------------------------------------------------------------------------ queries and cache rows
 // One CTA per (token, share of its maps and value heads), a warp per map at a time.
-template <typename T>
+constexpr int kMaxTaps = 8;
+template <typename T, bool CONV>
 __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPrepareParams p) {
   extern __shared__ float sm[];
   float2* turn = reinterpret_cast<float2*>(sm);                   // [rot / 2] cosine, sine
@@ -53,8 +53,8 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
   const float* part = p.partials ? p.partials + (size_t)t * p.width : nullptr;
   const T* bias = static_cast<const T*>(p.bias);
   // short convolution of steps in which every sequence has one token: the taps before it come from the sequence's state row,
-  // which moves on by one token as it is read
-  T* window = p.taps > 0 ? static_cast<T*>(p.conv_state) + (long long)p.seq_state[t] * (p.taps - 1) * p.conv_width : nullptr;
+  // which moves on by one token where `write` is set
+  T* window = CONV ? static_cast<T*>(p.conv_state) + (long long)p.seq_state[t] * (p.taps - 1) * p.conv_width : nullptr;
   const bool fresh = pos == 0;
   auto conv1 = [&](int c, float u, bool write) {
     const float* w = p.conv_w + (long long)c * p.taps;
@@ -65,6 +65,46 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
       v = fmaf(w[j], old, v);
       if (write) *at = from_f32<T>(next);
       next = old;
+    }
+    return v;
+  };
+  auto conv4 = [&](int c, const float4& u, bool write) {          // four columns from a multiple of 4 on: all loads in flight at once
+    using Raw = typename Four<T>::type;
+    Raw old[kMaxTaps - 1];
+    float4 w[kMaxTaps];
+#pragma unroll
+    for (int j = 0; j < kMaxTaps - 1; ++j)
+      if (j < p.taps - 1) old[j] = fresh ? Raw{} : *reinterpret_cast<const Raw*>(window + (long long)j * p.conv_width + c);
+    const float* wc = p.conv_w + (long long)c * p.taps;
+    if (p.taps == 4) {                                            // 4 x 4, a row per column
+      const float4 r0 = *reinterpret_cast<const float4*>(wc), r1 = *reinterpret_cast<const float4*>(wc + 4), r2 = *reinterpret_cast<const float4*>(wc + 8),
+                   r3 = *reinterpret_cast<const float4*>(wc + 12);
+      w[0] = make_float4(r0.x, r1.x, r2.x, r3.x), w[1] = make_float4(r0.y, r1.y, r2.y, r3.y);
+      w[2] = make_float4(r0.z, r1.z, r2.z, r3.z), w[3] = make_float4(r0.w, r1.w, r2.w, r3.w);
+    } else {
+#pragma unroll
+      for (int j = 0; j < kMaxTaps; ++j)
+        if (j < p.taps) w[j] = make_float4(wc[j], wc[p.taps + j], wc[2 * p.taps + j], wc[3 * p.taps + j]);
+    }
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j < kMaxTaps; ++j) {
+      if (j < p.taps - 1) {
+        const T* e = reinterpret_cast<const T*>(&old[min(j, kMaxTaps - 2)]);
+        v.x = fmaf(w[j].x, to_f32(e[0]), v.x), v.y = fmaf(w[j].y, to_f32(e[1]), v.y);
+        v.z = fmaf(w[j].z, to_f32(e[2]), v.z), v.w = fmaf(w[j].w, to_f32(e[3]), v.w);
+        if (write && j > 0) *reinterpret_cast<Raw*>(window + (long long)(j - 1) * p.conv_width + c) = old[min(j, kMaxTaps - 2)];
+      } else if (j == p.taps - 1) {
+        v.x = fmaf(w[j].x, u.x, v.x), v.y = fmaf(w[j].y, u.y, v.y), v.z = fmaf(w[j].z, u.z, v.z), v.w = fmaf(w[j].w, u.w, v.w);
+      }
+    }
+    if (write) {
+      const float f[4] = {u.x, u.y, u.z, u.w};
+      Raw raw;
+      T* e = reinterpret_cast<T*>(&raw);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) e[i] = from_f32<T>(f[i]);
+      *reinterpret_cast<Raw*>(window + (long long)(p.taps - 2) * p.conv_width + c) = raw;
     }
     return v;
   };
@@ -103,7 +143,9 @@ __global__ void __launch_bounds__(128) maps_prepare_kernel(const MapsPreparePara
   // behind the convolution, if any: with `write` the state row moves on, so every column is loaded once with it
   auto load4 = [&](int base, int c, int n, bool write) {
     float4 v = raw4(base, c, n);
-    if (window) {
+    if (CONV && p.vec) {
+      if (c < n) v = conv4(base + c, v, write);
+    } else if (CONV) {
       float* f = &v.x;
 #pragma unroll
       for (int e = 0; e < 4; ++e)
@@ -366,9 +408,7 @@ struct Maps {
   float *ws_o, *ws_ml;                       // partial results of key slices: [T][H][maps][splits][DV], [T][H][maps][splits][2]
   int splits;
   int* status;
-  const float *sink, *r1, *r2;               // [H] each, natural units; r1 null: no distance bias
-  int wv, chunks;                            // spread attention: width of a value row, pieces of DV columns
-  int tab_stride, tab_entries, tab_bufs;     // distance bias of a tile of the prefill kernel: [buffer][head of the group][stride]
+  const float* sink;                         // optional [H], natural units
 };
 
 // first pool row of the kPage tokens from `token` on, in a pool of `heads` rows per token
@@ -409,15 +449,14 @@ struct DecodeTile {
   static constexpr int kRowsOf = 16 / M;                   // query rows of a tile: row r of map m is tile row m * kRowsOf + r
 };
 
-template <int DK, int DV, int M, bool SPREAD>
+template <int DK, int DV, int M>
 __global__ void __launch_bounds__(128, 2) maps_decode_kernel(const Maps p, int row_tiles, int max_rows) {
   using L = DecodeTile<DK, DV, M>;
   constexpr int R = L::kRowsOf;
   extern __shared__ __align__(128) uint8_t smem[];
   bf16* qtile = reinterpret_cast<bf16*>(smem);
   uint8_t* ring = smem + L::kQ;
-  const int piece = SPREAD ? blockIdx.x % p.chunks : 0, at = SPREAD ? blockIdx.x / p.chunks : blockIdx.x;
-  const int kvh = at / row_tiles, row0 = (at % row_tiles) * R, seq = blockIdx.y, split = blockIdx.z;
+  const int kvh = blockIdx.x / row_tiles, row0 = (blockIdx.x % row_tiles) * R, seq = blockIdx.y, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_launch_dependents();
   pdl_wait();
@@ -453,14 +492,6 @@ __global__ void __launch_bounds__(128, 2) maps_decode_kernel(const Maps p, int r
     lim[i] = sub < n_rows ? first_pos + (row0 + sub) / p.group + 1 : 0;
     beg[i] = first_key(p, lim[i]);
   }
-  float r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};
-  if (SPREAD && p.r1) {
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int head = kvh * p.group + (row0 + (g + 8 * i) % R) % p.group;
-      r1[i] = p.r1[head], r2[i] = p.r2[head];
-    }
-  }
   float o[DV / 8][4];
 #pragma unroll
   for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -481,12 +512,11 @@ __global__ void __launch_bounds__(128, 2) maps_decode_kernel(const Maps p, int r
           cp_async16(tile_ptr<DK>(reinterpret_cast<bf16*>(st + a * L::kKey), r, c), src + (size_t)r * DK + c * 8);
         }
       }
-      const int ldv = SPREAD ? p.wv : DV;
-      const bf16* src = p.vc + (long long)page_row(p, table, pg * kPage, SPREAD ? 1 : p.G, SPREAD ? 0 : kvh) * ldv + piece * DV;
+      const bf16* src = p.vc + (long long)page_row(p, table, pg * kPage, p.G, kvh) * DV;
 #pragma unroll
       for (int i = lane; i < kPage * (DV / 8); i += 32) {
         const int r = i / (DV / 8), c = i - r * (DV / 8);
-        cp_async16(tile_ptr<DV>(reinterpret_cast<bf16*>(st + M * L::kKey), r, c), src + (size_t)r * ldv + c * 8);
+        cp_async16(tile_ptr<DV>(reinterpret_cast<bf16*>(st + M * L::kKey), r, c), src + (size_t)r * DV + c * 8);
       }
     }
     cp_async_commit();
@@ -521,8 +551,7 @@ __global__ void __launch_bounds__(128, 2) maps_decode_kernel(const Maps p, int r
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int i = e >> 1, tok = tok_base + nb * 8 + 2 * t4 + (e & 1);
-        float v = s[M == 2 ? i : 0][nb][e] * p.scale_log2;
-        if (SPREAD) v -= r1[i] * __log2f(fmaf(r2[i], (float)(lim[i] - 1 - tok), 1.f));
+        const float v = s[M == 2 ? i : 0][nb][e] * p.scale_log2;
         s[0][nb][e] = tok >= beg[i] && tok < lim[i] ? v : -INFINITY;
         mx[i] = fmaxf(mx[i], s[0][nb][e]);
       }
@@ -604,13 +633,6 @@ __global__ void __launch_bounds__(128, 2) maps_decode_kernel(const Maps p, int r
         for (int e = 0; e < E; ++e) a[k][e] = fmaf(mo[((size_t)w * 16 + r) * DV + lane + 32 * e], c, a[k][e]);
       }
     }
-    if (SPREAD) {
-      const size_t base = (tok * p.H + head) * p.splits + split;
-#pragma unroll
-      for (int e = 0; e < E; ++e) p.ws_o[base * p.wv + piece * DV + lane + 32 * e] = a[0][e];
-      if (lane == 0 && piece == 0) p.ws_ml[base * 2] = ms[0] * kLn2, p.ws_ml[base * 2 + 1] = ls[0];
-      continue;
-    }
     if (p.splits == 1) {
       finish_row<M, E>(p, tok, head, a, ls, ms[0], lane);
       continue;
@@ -661,20 +683,16 @@ __global__ void __launch_bounds__(128) maps_merge_kernel(const Maps p, int T) {
 // Order of the products: S_0, S_1 of the first tile, then per tile O_0, next S_0, O_1, next S_1: while one stream waits for its
 // weights the other's products run. Every wait is bounded.
 constexpr int kThreads = 320;
-constexpr int kTable = 3712;                           // fp32 entries of a stream's distance bias
-template <int DK, int DV, int M, bool SPREAD>
+template <int DK, int DV, int M>
 struct PrefillTile {
-  static constexpr int kQ = 2 * tile_bytes<DK>(), kK = M * tile_bytes<DK>(), kV = tile_bytes<DV>();
-  static constexpr int kTail = 256 + 2 * 128 * 4 * 2 + (SPREAD ? 2 * kTable * 4 : 0);
+  static constexpr int kQ = 2 * tile_bytes<DK>(), kK = M * tile_bytes<DK>(), kV = tile_bytes<DV>(), kTail = 256 + 2 * 128 * 4 * 2;
   static constexpr int kStages = kQ + 2 * (kK + kV) + kTail + 1024 <= 227 * 1024 ? 2 : 1;
   static constexpr int kUsed = kQ + kStages * (kK + kV) + kTail + 1024;
   static constexpr int kTotal = kUsed > 120 * 1024 ? kUsed : 120 * 1024;      // one CTA per SM: it takes all of the tensor memory
 };
 
-// BIAS: bias[-c] is taken off the score of column c (log2 units)
-template <int DV, bool FULL, bool BIAS>
-__device__ __forceinline__ void softmax_tile(uint32_t t_s, uint32_t t_o, float scale_log2, const float* bias, int lo, int hi, bool have_o, float& m_used,
-                                             float& l) {
+template <int DV, bool FULL>
+__device__ __forceinline__ void softmax_tile(uint32_t t_s, uint32_t t_o, float scale_log2, int lo, int hi, bool have_o, float& m_used, float& l) {
   uint32_t sa[32];
   float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll 1
@@ -683,7 +701,7 @@ __device__ __forceinline__ void softmax_tile(uint32_t t_s, uint32_t t_o, float s
     tmem_ld_wait();
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
-      const float v = BIAS ? fmaf(__uint_as_float(sa[i]), scale_log2, -bias[-(32 * c + i)]) : __uint_as_float(sa[i]) * scale_log2;
+      const float v = __uint_as_float(sa[i]) * scale_log2;
       if (FULL || (32 * c + i >= lo && 32 * c + i < hi)) mx[i & 3] = fmaxf(mx[i & 3], v);
     }
   }
@@ -710,7 +728,7 @@ __device__ __forceinline__ void softmax_tile(uint32_t t_s, uint32_t t_o, float s
       float v[2];
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        v[e] = ex2(fmaf(__uint_as_float(sa[i + e]), scale_log2, BIAS ? -m_ref - bias[-(32 * c + i + e)] : -m_ref));
+        v[e] = ex2(fmaf(__uint_as_float(sa[i + e]), scale_log2, -m_ref));
         if (!FULL && (32 * c + i + e < lo || 32 * c + i + e >= hi)) v[e] = 0.f;
         sum[(i + e) & 3] += v[e];
       }
@@ -758,13 +776,12 @@ __device__ __forceinline__ void store_32(const Maps& p, bf16* dst, int c0, const
   }
 }
 
-__device__ __forceinline__ void stream_barrier(int s) { asm volatile("bar.sync %0, 128;" ::"r"(2 + s) : "memory"); }
 __device__ __forceinline__ void softmax_barrier() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
-template <int DK, int DV, int M, bool SPREAD>
+template <int DK, int DV, int M>
 __global__ void __launch_bounds__(kThreads, 1) maps_prefill_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_constant__ CUtensorMap tma_v,
                                                                    const Maps p, int min_rows) {
-  using L = PrefillTile<DK, DV, M, SPREAD>;
+  using L = PrefillTile<DK, DV, M>;
   constexpr int TBK = tile_bytes<DK>(), TBV = tile_bytes<DV>(), NST = L::kStages, CTA_ROWS = M == 2 ? kRows : 2 * kRows;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -781,7 +798,7 @@ __global__ void __launch_bounds__(kThreads, 1) maps_prefill_kernel(const __grid_
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int row0 = (gridDim.x - 1 - blockIdx.x) * CTA_ROWS;          // the tiles with the longest key range start first
-  const int kvh = SPREAD ? blockIdx.y / p.chunks : blockIdx.y, piece = SPREAD ? blockIdx.y % p.chunks : 0, seq = blockIdx.z;
+  const int kvh = blockIdx.y, seq = blockIdx.z;
   const int q0 = p.q_starts[seq], qn = p.q_starts[seq + 1] - q0;
   const int all_rows = qn * p.group;
   if (all_rows < min_rows || row0 >= all_rows) return;
@@ -841,9 +858,9 @@ __global__ void __launch_bounds__(kThreads, 1) maps_prefill_kernel(const __grid_
         mbar_expect_tx(&v_full[b], TBV);
 #pragma unroll
         for (int pg = 0; pg < kTile / kPage; ++pg) {
-          const int row = page_row(p, table, tok[pg], SPREAD ? 1 : p.G, SPREAD ? 0 : kvh);
+          const int row = page_row(p, table, tok[pg], p.G, kvh);
 #pragma unroll
-          for (int h = 0; h < DV / 64; ++h) tma_load_2d(sv + b * L::kV + h * kHalf + pg * (kPage * 128), &tma_v, &v_full[b], piece * DV + 64 * h, row);
+          for (int h = 0; h < DV / 64; ++h) tma_load_2d(sv + b * L::kV + h * kHalf + pg * (kPage * 128), &tma_v, &v_full[b], 64 * h, row);
         }
       }
     }
@@ -906,29 +923,14 @@ __global__ void __launch_bounds__(kThreads, 1) maps_prefill_kernel(const __grid_
     const int lim_first = first_pos + srow0 / p.group + 1, beg_last = first_key(p, first_pos + (srow0 + kRows - 1) / p.group + 1);
     float m_used = -INFINITY, l = 0.f;
     bool ok = true;
-    const int off = (srow0 + r) / p.group - srow0 / p.group, hh = (srow0 + r) % p.group;      // of the row: token behind the stream's first, head of the group
-    float* table = swap_ss + 2 * kRows + s * kTable;
     for (int it = 0; it < n_tiles; ++it) {
       const int tok0 = begin + it * kTile;
-      const float* bias = nullptr;
-      if (SPREAD && n_rows > 0) {
-        // the bias of every distance between the stream's tokens and the tile's, per head; entry e is off + 127 - column
-        float* buf = table + (p.tab_bufs == 2 && (it & 1) ? p.tab_entries : 0);
-        if (p.tab_bufs == 1 && it > 0) stream_barrier(s);
-        const int base = first_pos + srow0 / p.group - tok0 - (kTile - 1);
-        for (int i = (warp & 3) * 32 + lane; i < p.tab_entries; i += 128) {
-          const int head = kvh * p.group + i / p.tab_stride, d = base + i % p.tab_stride;
-          buf[i] = p.r1 && d > 0 ? p.r1[head] * __log2f(fmaf(p.r2[head], (float)d, 1.f)) : 0.f;
-        }
-        stream_barrier(s);
-        bias = buf + hh * p.tab_stride + off + (kTile - 1);
-      }
       if (!mbar_wait(&s_full[s], it & 1, abort_flag)) { ok = false; break; }
       tc_fence_after_sync();
       if (n_rows == kRows && tok0 + kTile <= lim_first && tok0 >= beg_last)      // every row of the stream sees the whole tile
-        softmax_tile<DV, true, SPREAD>(t_s, t_o, p.scale_log2, bias, 0, 0, it > 0, m_used, l);
-      else if (!SPREAD || n_rows > 0)
-        softmax_tile<DV, false, SPREAD>(t_s, t_o, p.scale_log2, bias, beg - tok0, lim - tok0, it > 0, m_used, l);
+        softmax_tile<DV, true>(t_s, t_o, p.scale_log2, 0, 0, it > 0, m_used, l);
+      else
+        softmax_tile<DV, false>(t_s, t_o, p.scale_log2, beg - tok0, lim - tok0, it > 0, m_used, l);
       tc_fence_before_sync();
       __syncwarp();
       if (lane == 0) mbar_arrive(&p_ready[s]);
@@ -969,20 +971,6 @@ __global__ void __launch_bounds__(kThreads, 1) maps_prefill_kernel(const __grid_
           store_32(p, dst, (s * N + n) * 32, y[n]);
         }
       }
-    } else if (ok && SPREAD) {
-      const long long at = (long long)(q0 + row / p.group) * p.H + kvh * p.group + row % p.group;
-#pragma unroll 1
-      for (int c = 0; c < DV / 32; ++c) {
-        uint32_t a[32];
-        tmem_ld_32x32(t_o + 32 * c, a);
-        tmem_ld_wait();
-        if (!valid) continue;
-        float4* to = reinterpret_cast<float4*>(p.ws_o + at * p.wv + piece * DV + 32 * c);
-#pragma unroll
-        for (int i = 0; i < 8; ++i)
-          to[i] = make_float4(__uint_as_float(a[4 * i]), __uint_as_float(a[4 * i + 1]), __uint_as_float(a[4 * i + 2]), __uint_as_float(a[4 * i + 3]));
-      }
-      if (valid && piece == 0) p.ws_ml[2 * at] = m_used * kLn2, p.ws_ml[2 * at + 1] = l;
     } else if (ok) {
       if (valid) l += sink_weight(p, kvh * p.group + row % p.group, m_used);
       const float inv = l > 0.f ? 1.f / l : 0.f;
@@ -1006,44 +994,23 @@ __global__ void __launch_bounds__(kThreads, 1) maps_prefill_kernel(const __grid_
 }
 
 // ------------------------------------------------------------------------------------------ host
-const CUtensorMap& pool_map(const void* pool, uint64_t rows, int D) {
-  struct Key {
-    const void* base;
-    uint64_t rows;
-    int d;
-    bool operator==(const Key& o) const { return base == o.base && rows == o.rows && d == o.d; }
-  };
-  struct Hash {
-    size_t operator()(const Key& k) const { return std::hash<const void*>()(k.base) ^ std::hash<uint64_t>()(k.rows * 2 + k.d / 128); }
-  };
-  static std::unordered_map<Key, CUtensorMap, Hash> maps;
-  const Key key{pool, rows, D};
-  auto it = maps.find(key);
-  if (it == maps.end()) {
-    if (maps.size() > 4096) maps.clear();
-    it = maps.emplace(key, make_tmap_2d(pool, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows, D, D * 2, kPage, 64, true)).first;
-  }
-  return it->second;
-}
-
-template <int DK, int DV, int M, bool SPREAD = false>
+template <int DK, int DV, int M>
 int launch_tc(Maps a, const MapsAttnParams& p, int splits, cudaStream_t s) {
   using D = DecodeTile<DK, DV, M>;
-  using P = PrefillTile<DK, DV, M, SPREAD>;
+  using P = PrefillTile<DK, DV, M>;
   static bool configured[kMaxDevices] = {};
   if (first_call_on_device(configured)) {
-    cuda_check(cudaFuncSetAttribute(maps_decode_kernel<DK, DV, M, SPREAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, D::kTotal), "maps_decode smem");
-    cuda_check(cudaFuncSetAttribute(maps_prefill_kernel<DK, DV, M, SPREAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, P::kTotal), "maps_prefill smem");
+    cuda_check(cudaFuncSetAttribute(maps_decode_kernel<DK, DV, M>, cudaFuncAttributeMaxDynamicSharedMemorySize, D::kTotal), "maps_decode smem");
+    cuda_check(cudaFuncSetAttribute(maps_prefill_kernel<DK, DV, M>, cudaFuncAttributeMaxDynamicSharedMemorySize, P::kTotal), "maps_prefill smem");
   }
   int launches = 0;
   const int max_rows = p.max_q_len * a.group;
   if (p.min_q_len * a.group <= kDecodeRows) {
     a.splits = max_rows <= kDecodeRows ? splits : 1;      // partial results of longer sequences do not exist
     const int row_tiles = (std::min(max_rows, kDecodeRows) + D::kRowsOf - 1) / D::kRowsOf;
-    launch_pdl(maps_decode_kernel<DK, DV, M, SPREAD>, dim3(a.G * row_tiles * a.chunks, p.num_seqs, a.splits), dim3(128), D::kTotal, s, a, row_tiles,
-               (int)kDecodeRows);
+    launch_pdl(maps_decode_kernel<DK, DV, M>, dim3(a.G * row_tiles, p.num_seqs, a.splits), dim3(128), D::kTotal, s, a, row_tiles, (int)kDecodeRows);
     ++launches;
-    if (!SPREAD && a.splits > 1) {
+    if (a.splits > 1) {
       launch_pdl(maps_merge_kernel<DV, M>, dim3((p.tokens * a.H + 3) / 4), dim3(128), 0, s, a, p.tokens);
       ++launches;
     }
@@ -1052,8 +1019,8 @@ int launch_tc(Maps a, const MapsAttnParams& p, int splits, cudaStream_t s) {
     constexpr int rows = M == 2 ? kRows : 2 * kRows;
     const uint64_t n = (uint64_t)p.num_blocks * a.G * a.block_size;
     // (copies: a second lookup may move the first entry)
-    const CUtensorMap km = pool_map(p.k_cache, n * M, DK), vm = SPREAD ? pool_map(p.v_cache, n / a.G, a.wv) : pool_map(p.v_cache, n, DV);
-    maps_prefill_kernel<DK, DV, M, SPREAD><<<dim3((max_rows + rows - 1) / rows, a.G * a.chunks, p.num_seqs), kThreads, P::kTotal, s>>>(km, vm, a, kDecodeRows + 1);
+    const CUtensorMap km = pool_map(p.k_cache, n * M, DK), vm = pool_map(p.v_cache, n, DV);
+    maps_prefill_kernel<DK, DV, M><<<dim3((max_rows + rows - 1) / rows, a.G, p.num_seqs), kThreads, P::kTotal, s>>>(km, vm, a, kDecodeRows + 1);
     ++launches;
   }
   cuda_check(cudaGetLastError(), "attention_maps launch");
@@ -1074,85 +1041,11 @@ void launch_simple(const MapsAttnParams& p, cudaStream_t s) {
   cuda_check(cudaGetLastError(), "maps_simple_kernel");
 }
 
-// ------------------------------------------------------------------------------------------ spread attention: the heads mixed
-// One CTA per token, a thread per value column (g, i) at a time: with a[f] the column of head f's output, head h of group g is
-// sigmoid(gate_h) sum_f talk[h, f] a[f]. The key slices of a head are merged on the way, and the sink joins its denominator.
-constexpr int kMixHeads = 8;
-template <typename T>
-__global__ void __launch_bounds__(256) talk_mix_kernel(const TalkMixParams p) {
-  extern __shared__ float sm[];
-  float* mat = sm;                             // [H][H]
-  float* coef = mat + p.H * p.H;               // [H][splits]
-  const int t = blockIdx.x, H = p.H, group = H / p.G, S = p.splits;
-  pdl_launch_dependents();
-  for (int i = threadIdx.x; i < H * H; i += blockDim.x) mat[i] = p.talk[i];
-  pdl_wait();
-  for (int h = threadIdx.x; h < H; h += blockDim.x) {
-    const float2* ml = reinterpret_cast<const float2*>(p.part_ml) + ((size_t)t * H + h) * S;
-    float m = p.sink ? p.sink[h] : -INFINITY, l = 0.f;
-    for (int s = 0; s < S; ++s) m = fmaxf(m, ml[s].x);
-    if (p.sink) l = expf(p.sink[h] - m);
-    for (int s = 0; s < S; ++s) {
-      const float2 v = ml[s];
-      const float c = v.x == -INFINITY ? 0.f : expf(v.x - m);
-      coef[h * S + s] = c;
-      l = fmaf(v.y, c, l);
-    }
-    for (int s = 0; s < S; ++s) coef[h * S + s] /= l;
-  }
-  __syncthreads();
-  T* out = static_cast<T*>(p.out) + (long long)t * p.ldo;
-  const float* src = p.part_o + (size_t)t * H * S * p.wv;
-  const float* gate = p.gate ? p.gate + (long long)t * p.ld_gate : nullptr;
-  for (int c = threadIdx.x; c < p.G * p.v_dim; c += blockDim.x) {
-    const int g = c / p.v_dim, i = c - g * p.v_dim;
-    for (int h0 = 0; h0 < group; h0 += kMixHeads) {
-      float acc[kMixHeads];
-#pragma unroll
-      for (int e = 0; e < kMixHeads; ++e) acc[e] = 0.f;
-      const int n = min(kMixHeads, group - h0);
-      const float* row = mat + (size_t)(g * group + h0) * H;
-#pragma unroll 4
-      for (int f = 0; f < H; ++f) {
-        float a = 0.f;
-        for (int s = 0; s < S; ++s) {
-          const float w = coef[f * S + s];
-          if (w != 0.f) a = fmaf(__ldcg(src + ((size_t)f * S + s) * p.wv + c), w, a);
-        }
-#pragma unroll
-        for (int e = 0; e < kMixHeads; ++e)
-          if (e < n) acc[e] = fmaf(row[e * H + f], a, acc[e]);
-      }
-#pragma unroll
-      for (int e = 0; e < kMixHeads; ++e) {
-        if (e >= n) continue;
-        const int h = g * group + h0 + e;
-        out[(long long)h * p.v_dim + i] = from_f32<T>(gate ? acc[e] / (1.f + expf(-gate[h])) : acc[e]);
-      }
-    }
-  }
-  for (int c = H * p.v_dim + threadIdx.x; c < p.cols; c += blockDim.x) out[c] = from_f32<T>(0.f);
-}
-
-// the table of a stream's distance bias: heads of a group x distances, rows spaced so that the lanes of a warp hit distinct banks
-void plan_table(Maps& a) {
-  const int n = 127 / a.group + 1 + kTile, shift = (32 + a.group - 1) / a.group % 32;
-  a.tab_stride = n + ((shift - n) % 32 + 32) % 32;
-  a.tab_entries = a.group * a.tab_stride;
-  a.tab_bufs = 2 * a.tab_entries <= kTable ? 2 : 1;
-}
 }  // namespace
 
 bool attention_maps_tc_supported(int wk, int wv, int block_size, int f32) {
   return !f32 && (wk == 64 || wk == 128) && (wv == 64 || wv == 128) && block_size % kPage == 0;
 }
-bool attention_spread_tc_supported(int group, int wk, int wv, int block_size, int f32) {
-  Maps a{};
-  a.group = group;
-  plan_table(a);
-  return !f32 && (wk == 64 || wk == 128) && (wv == 64 || wv % 128 == 0) && block_size % kPage == 0 && a.tab_entries <= kTable;
-}
-
 // key slices the tensor-core path uses for a step (1: no workspace needed)
 int attention_maps_splits(int num_seqs, int max_q_len, int H, int G, int maps, int max_kv_len, int window) {
   const int rows = max_q_len * (H / G), per_tile = 16 / maps;
@@ -1172,7 +1065,7 @@ int attention_maps(const MapsAttnParams& p, int splits, void* workspace, size_t 
   if (p.maps != 1 && p.maps != 2) throw std::runtime_error("attention_maps: one or two maps");
   if (p.maps == 2 && (p.sink || p.r1 || p.spread)) throw std::runtime_error("attention_maps: sinks, distance biases and spread values go with one map");
   if (p.spread && (!p.part_o || !p.part_ml)) throw std::runtime_error("attention_maps: spread values need room for partial sums");
-  const bool fast = p.spread ? attention_spread_tc_supported(p.H / p.G, p.wk, p.wv, p.block_size, p.f32)
+  const bool fast = p.spread ? attention_spread_tc_supported(p.H / p.G, p.wk, p.wv, p.block_size, p.f32) && p.scale > 0.f && p.bias_range <= kTalkBiasRange
                              : !p.r1 && attention_maps_tc_supported(p.wk, p.wv, p.block_size, p.f32);
   if (!tensor_cores || !fast) {
     if (p.spread && splits > 1) throw std::runtime_error("attention_maps: key slices are the tensor-core path's");
@@ -1180,8 +1073,9 @@ int attention_maps(const MapsAttnParams& p, int splits, void* workspace, size_t 
     else p.maps == 2 ? launch_simple<bf16, 2>(p, s) : launch_simple<bf16, 1>(p, s);
     return 1;
   }
+  if (p.spread) return attention_spread_tc(p, splits, status, s);
   splits = std::max(splits, 1);
-  if (!p.spread && workspace_bytes < attention_maps_workspace_bytes(p.tokens, p.H * p.maps, p.wv, splits))
+  if (workspace_bytes < attention_maps_workspace_bytes(p.tokens, p.H * p.maps, p.wv, splits))
     throw std::runtime_error("attention_maps: workspace too small for the requested key slices");
   Maps a{};
   a.q = static_cast<const bf16*>(p.q), a.kc = static_cast<const bf16*>(p.k_cache), a.vc = static_cast<const bf16*>(p.v_cache);
@@ -1193,13 +1087,7 @@ int attention_maps(const MapsAttnParams& p, int splits, void* workspace, size_t 
   a.ws_o = static_cast<float*>(workspace);
   a.ws_ml = a.ws_o != nullptr ? a.ws_o + (size_t)p.tokens * p.H * p.maps * splits * p.wv : nullptr;
   a.status = status;
-  a.sink = p.sink, a.r1 = p.r1, a.r2 = p.r2, a.chunks = 1;
-  if (p.spread) {
-    a.ws_o = p.part_o, a.ws_ml = p.part_ml, a.wv = p.wv, a.chunks = p.wv == 64 ? 1 : p.wv / 128;
-    plan_table(a);
-    if (p.wk == 64) return p.wv == 64 ? launch_tc<64, 64, 1, true>(a, p, splits, s) : launch_tc<64, 128, 1, true>(a, p, splits, s);
-    return p.wv == 64 ? launch_tc<128, 64, 1, true>(a, p, splits, s) : launch_tc<128, 128, 1, true>(a, p, splits, s);
-  }
+  a.sink = p.sink;
 #define FLLM_MAPS(K_, V_) return p.maps == 2 ? launch_tc<K_, V_, 2>(a, p, splits, s) : launch_tc<K_, V_, 1>(a, p, splits, s);
   if (p.wk == 64 && p.wv == 64) { FLLM_MAPS(64, 64) }
   if (p.wk == 64) { FLLM_MAPS(64, 128) }
@@ -1208,24 +1096,11 @@ int attention_maps(const MapsAttnParams& p, int splits, void* workspace, size_t 
 #undef FLLM_MAPS
 }
 
-void talk_mix(const TalkMixParams& p, cudaStream_t s) {
-  if (p.tokens <= 0) return;
-  const size_t smem = ((size_t)p.H * p.H + (size_t)p.H * p.splits) * sizeof(float);
-  static bool configured[kMaxDevices] = {};
-  if (smem > 200 * 1024) throw std::runtime_error("talk_mix: too many heads");
-  if (first_call_on_device(configured)) {
-    cuda_check(cudaFuncSetAttribute(talk_mix_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024), "talk_mix smem");
-    cuda_check(cudaFuncSetAttribute(talk_mix_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024), "talk_mix smem");
-  }
-  const dim3 threads(std::min(256, (p.G * p.v_dim + 31) / 32 * 32));
-  if (p.f32) launch_pdl(talk_mix_kernel<float>, dim3(p.tokens), threads, smem, s, p);
-  else launch_pdl(talk_mix_kernel<bf16>, dim3(p.tokens), threads, smem, s, p);
-  cuda_check(cudaGetLastError(), "talk_mix_kernel");
-}
-
 void maps_prepare(const MapsPrepareParams& params, cudaStream_t s) {
   if (params.tokens <= 0) return;
   MapsPrepareParams p = params;
+  if (p.taps > kMaxTaps || (p.taps > 0 && (p.conv_width % 4 || reinterpret_cast<uintptr_t>(p.conv_w) % 16 || reinterpret_cast<uintptr_t>(p.conv_state) % 16)))
+    throw std::runtime_error("maps_prepare: a convolution of at most 8 taps, columns in multiples of 4");
   if (p.taps > 0 && p.full) throw std::runtime_error("maps_prepare: a norm over all maps does not go with a convolution");
   const uintptr_t any = reinterpret_cast<uintptr_t>(p.x) | reinterpret_cast<uintptr_t>(p.bias) | reinterpret_cast<uintptr_t>(p.partials);
   p.vec = p.dim % 4 == 0 && p.v_dim % 4 == 0 && p.q_offset % 4 == 0 && p.k_offset % 4 == 0 && p.v_offset % 4 == 0 && any % 16 == 0 &&
@@ -1236,8 +1111,14 @@ void maps_prepare(const MapsPrepareParams& params, cudaStream_t s) {
   const int shares = std::max(1, std::min((heads + 3) / 4, 4 * sm_count() / std::max(p.tokens, 1)));
   const size_t smem = (size_t)(p.rot + 4 * p.dim) * sizeof(float);
   if (smem > 48 * 1024) throw std::runtime_error("maps_prepare: heads too wide");
-  if (p.f32) launch_pdl(maps_prepare_kernel<float>, dim3(p.tokens, shares), dim3(128), smem, s, p);
-  else launch_pdl(maps_prepare_kernel<bf16>, dim3(p.tokens, shares), dim3(128), smem, s, p);
+  const dim3 grid(p.tokens, shares);
+  if (p.taps > 0) {
+    if (p.f32) launch_pdl(maps_prepare_kernel<float, true>, grid, dim3(128), smem, s, p);
+    else launch_pdl(maps_prepare_kernel<bf16, true>, grid, dim3(128), smem, s, p);
+  } else {
+    if (p.f32) launch_pdl(maps_prepare_kernel<float, false>, grid, dim3(128), smem, s, p);
+    else launch_pdl(maps_prepare_kernel<bf16, false>, grid, dim3(128), smem, s, p);
+  }
   cuda_check(cudaGetLastError(), "maps_prepare_kernel");
 }
 

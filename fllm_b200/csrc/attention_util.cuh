@@ -5,7 +5,10 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include <unordered_map>
+
 #include "ptx.cuh"
+#include "tma_host.h"
 
 namespace fllm {
 namespace {
@@ -74,6 +77,27 @@ constexpr int tile_bytes() { return (D / 64) * kHalf; }
 template <int D>
 __device__ __forceinline__ uint64_t desc_mn_major(uint32_t saddr) {
   return (uint64_t)((saddr & 0x3FFFFu) >> 4) | (uint64_t)((D > 64 ? kHalf : 1024) >> 4) << 16 | (uint64_t)(1024 >> 4) << 32 | (uint64_t)1 << 46 | (uint64_t)2 << 61;
+}
+
+// tensor map of a pool of `rows` rows of D values, in boxes of a page's rows and 64 columns
+inline const CUtensorMap& pool_map(const void* pool, uint64_t rows, int D) {
+  struct Key {
+    const void* base;
+    uint64_t rows;
+    int d;
+    bool operator==(const Key& o) const { return base == o.base && rows == o.rows && d == o.d; }
+  };
+  struct Hash {
+    size_t operator()(const Key& k) const { return std::hash<const void*>()(k.base) ^ std::hash<uint64_t>()(k.rows * 2 + k.d / 128); }
+  };
+  static std::unordered_map<Key, CUtensorMap, Hash> maps;
+  const Key key{pool, rows, D};
+  auto it = maps.find(key);
+  if (it == maps.end()) {
+    if (maps.size() > 4096) maps.clear();
+    it = maps.emplace(key, make_tmap_2d(pool, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows, D, D * 2, kPage, 64, true)).first;
+  }
+  return it->second;
 }
 }  // namespace
 }  // namespace fllm

@@ -144,7 +144,7 @@ int64_t attention_talk(const Tensor& q, const Tensor& k_cache, const Tensor& v_c
                        const Tensor& row_seq, const Tensor& positions, const Tensor& q_starts, Tensor out, int64_t num_seqs, int64_t max_q_len,
                        int64_t min_q_len, double scale, int64_t window, const optional<Tensor>& sink, const optional<Tensor>& r1,
                        const optional<Tensor>& r2, const Tensor& talk, const optional<Tensor>& gate, Tensor part_o, Tensor part_ml, bool tensor_cores,
-                       const optional<Tensor>& status) {
+                       double bias_range, const optional<Tensor>& status) {
   const auto ty = act_type(q);
   TORCH_CHECK(k_cache.dim() == 4 && v_cache.dim() == 4, "pools: [blocks, heads, block_size, width]");
   const int64_t T = q.size(0), G = k_cache.size(1), H = q.size(1), wv = v_cache.size(3);
@@ -167,6 +167,7 @@ int64_t attention_talk(const Tensor& q, const Tensor& k_cache, const Tensor& v_c
   p.H = (int)H, p.G = (int)G, p.maps = 1, p.dim = (int)dim, p.v_dim = (int)(G * v_dim), p.wk = (int)k_cache.size(3), p.wv = (int)wv;
   p.block_size = (int)k_cache.size(2), p.num_blocks = k_cache.size(0), p.scale = (float)scale, p.window = (int)window, p.f32 = ty == at::kFloat ? 1 : 0;
   p.r1 = per_head(r1, H), p.r2 = per_head(r2, H), p.spread = 1, p.part_o = part_o.data_ptr<float>(), p.part_ml = part_ml.data_ptr<float>();
+  p.bias_range = (float)bias_range;
   TORCH_CHECK((p.r1 != nullptr) == (p.r2 != nullptr), "a distance bias has two numbers per head");
   fllm::TalkMixParams m{};
   m.part_o = p.part_o, m.part_ml = p.part_ml, m.sink = per_head(sink, H), m.talk = talk.data_ptr<float>();
@@ -177,6 +178,9 @@ int64_t attention_talk(const Tensor& q, const Tensor& k_cache, const Tensor& v_c
   const int n = fllm::attention_maps(p, m.splits, nullptr, 0, tensor_cores, given(status) ? status->data_ptr<int>() : nullptr, cur_stream());
   fllm::talk_mix(m, cur_stream());
   return n + 1;
+}
+int64_t attention_spread_splits(int64_t num_seqs, int64_t max_q_len, int64_t H, int64_t G, int64_t wv, int64_t max_kv_len, int64_t window) {
+  return fllm::attention_spread_splits((int)num_seqs, (int)max_q_len, (int)H, (int)G, (int)wv, (int)max_kv_len, (int)window);
 }
 bool attention_spread_tc_supported(int64_t group, int64_t wk, int64_t wv, int64_t block_size) {
   return fllm::attention_spread_tc_supported((int)group, (int)wk, (int)wv, (int)block_size, 0);
@@ -193,8 +197,9 @@ TORCH_LIBRARY_FRAGMENT(fllm_b200, m) {
   m.def("attention_maps(Tensor q, Tensor k_cache, Tensor v_cache, int dim, int v_dim, Tensor block_tables, Tensor row_seq, Tensor positions, Tensor q_starts, "
         "Tensor(a!) out, int num_seqs, int max_q_len, int min_q_len, float scale, int window, float lam, float out_scale, float eps, int splits, "
         "Tensor? workspace, bool tensor_cores, Tensor? status, Tensor? sink=None, Tensor? r1=None, Tensor? r2=None) -> int", &attention_maps);
+  m.def("attention_spread_splits(int num_seqs, int max_q_len, int H, int G, int wv, int max_kv_len, int window) -> int", &attention_spread_splits);
   m.def("attention_spread_tc_supported(int group, int wk, int wv, int block_size) -> bool", &attention_spread_tc_supported);
   m.def("attention_talk(Tensor q, Tensor k_cache, Tensor v_cache, int dim, int v_dim, Tensor block_tables, Tensor row_seq, Tensor positions, Tensor q_starts, "
         "Tensor(a!) out, int num_seqs, int max_q_len, int min_q_len, float scale, int window, Tensor? sink, Tensor? r1, Tensor? r2, Tensor talk, Tensor? gate, "
-        "Tensor(b!) part_o, Tensor(c!) part_ml, bool tensor_cores, Tensor? status) -> int", &attention_talk);
+        "Tensor(b!) part_o, Tensor(c!) part_ml, bool tensor_cores, float bias_range, Tensor? status) -> int", &attention_talk);
 }

@@ -517,7 +517,12 @@ struct MapsAttnParams {
   // [tokens][H][splits][wv] and part_ml [tokens][H][splits][2] (reference, sum of weights; the sink is left to talk_mix)
   int spread;
   float *part_o, *part_ml;
+  float bias_range;            // spread, tensor cores: the most a bias changes inside a tile of keys, log2 units (see kTalkBiasRange)
 };
+// spread attention on the tensor cores (attention_talk.cu); returns the number of kernels launched
+int attention_spread_tc(const MapsAttnParams& p, int splits, int* status, cudaStream_t s);
+int attention_spread_splits(int num_seqs, int max_q_len, int H, int G, int wv, int max_kv_len, int window);      // key slices for a step
+constexpr float kTalkBiasRange = 100.f;
 // out head h of group g = sigmoid(gate_h) sum_f talk[h, f] (head f's weights over the values of group g)
 struct TalkMixParams {
   const float *part_o, *part_ml;
@@ -527,6 +532,7 @@ struct TalkMixParams {
   void* out;                   // [tokens] rows of `cols` columns, zero beyond H * v_dim
   long long ldo;
   int tokens, H, G, splits, v_dim, wv, cols, f32;
+  int vec;                     // set by talk_mix: output rows can be stored four values at a time
 };
 void talk_mix(const TalkMixParams& p, cudaStream_t s);
 bool attention_spread_tc_supported(int group, int wk, int wv, int block_size, int f32);

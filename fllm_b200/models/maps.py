@@ -13,7 +13,7 @@ from typing import Dict, Optional
 
 import torch
 
-from ..ops.maps import Combine, ConvWindow, NormedPair
+from ..ops.maps import Combine, ConvWindow, NormedPair, bias_range
 from .recurrent import _batch_meta, pad8, pad_cols, pad_rows
 
 
@@ -39,7 +39,7 @@ def _attend(dec, li: int, m, proj, b) -> torch.Tensor:
                          pairs=c.get("rope_style") == "pair", conv=conv, extra_out=gate, extra_offset=nq + nk + pad8(G * v_dim))
     terms = dict(sink=m.get("sink"), r1=m.get("r1"), r2=m.get("r2"), out_cols=m["wo"].shape[1])
     if talk is not None:
-        return ops.attention_talk(q, keys, values, dim, v_dim, b, c["scale"], talk, c["window"], gate=gate, **terms)
+        return ops.attention_talk(q, keys, values, dim, v_dim, b, c["scale"], talk, c["window"], gate=gate, reach=m["bias_range"], **terms)
     combine = Combine(m["lam"], 1.0 - c["diff"], eps) if M == 2 else None
     return ops.attention_maps(q, keys, values, dim, v_dim, b, c["scale"], c["window"], combine, **terms)
 
@@ -83,6 +83,8 @@ def pack_maps(q, k, v, q_norm, k_norm, o_proj, dtype, device, biases=None, lambd
     if convs is not None:
         m["conv"] = f32(torch.cat([p8(t) for t in convs], 0))
     m.update({n: f32(t) for n, t in (terms or {}).items()})
+    if "talk" in m:
+        m["bias_range"] = bias_range(m.get("r1"), m.get("r2"))
     if biases is not None:
         m["in_bias"] = put(torch.cat([p8(t) for t in biases], 0))
     if lambdas is not None:

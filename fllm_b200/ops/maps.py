@@ -35,6 +35,14 @@ def spread_width(dim: int) -> int:
     return 64 if dim <= 64 else (dim + 127) // 128 * 128
 
 
+MAX_BIAS_RANGE = 100.0           # (log2 units) a distance bias that changes more inside a tile of keys runs on the CUDA cores
+
+
+def bias_range(r1, r2) -> float:
+    """The most a distance bias can change between the tokens and the keys of one tile (within 320 of each other), in log2 units."""
+    return 0.0 if r1 is None else float((r1.double().abs() * torch.log2(1 + r2.double() * 320)).nan_to_num(1e9).max())
+
+
 @dataclass
 class ConvWindow:
     """A causal convolution in front of the preparation of a step whose sequences have one token each: weights fp32 [columns, taps],
@@ -142,9 +150,10 @@ class MapsRef:
         return out
 
     def attention_talk(self, q, k_cache, v_cache, dim, v_dim, b, scale, talk, window=0, sink=None, r1=None, r2=None, gate=None, out_cols=0, tensor_cores=True,
-                       splits=None):
+                       splits=None, reach=None):
         """Talking heads: head h weighs the values of its key/value head with sum_f talk[h, f] (weights of head f); its output is
-        scaled by sigmoid(gate[:, h]). Value rows [.., 1, .., width] hold all heads' values (``v_dim`` each)."""
+        scaled by sigmoid(gate[:, h]). Value rows [.., 1, .., width] hold all heads' values (``v_dim`` each). ``reach``: the
+        ``bias_range`` of r1 and r2 (None: it is computed, which waits for the device)."""
         T, H = q.shape[:2]
         G, bs = k_cache.shape[1], k_cache.shape[2]
         out = torch.zeros(T, max(out_cols, H * v_dim), dtype=q.dtype, device=q.device)
@@ -219,18 +228,21 @@ class MapsNative:
         return out
 
     def attention_talk(self, q, k_cache, v_cache, dim, v_dim, b, scale, talk, window=0, sink=None, r1=None, r2=None, gate=None, out_cols=0, tensor_cores=True,
-                       splits=None):
+                       splits=None, reach=None):
         T, H = q.shape[:2]
         G, wv = k_cache.shape[1], v_cache.shape[3]
-        fast = tensor_cores and q.dtype == torch.bfloat16 and self.k.attention_spread_tc_supported(H // G, k_cache.shape[3], wv, k_cache.shape[2])
-        most = int(self.k.attention_maps_splits(b.num_seqs, b.max_q_len, H, G, 1, b.max_kv_len, int(window)))
-        splits = 1 if not fast else most if splits is None else splits
+        reach = bias_range(r1, r2) if reach is None else reach
+        fast = tensor_cores and q.dtype == torch.bfloat16 and reach <= MAX_BIAS_RANGE and scale > 0 and self.k.attention_spread_tc_supported(H // G, k_cache.shape[3], wv, k_cache.shape[2])
+        if not fast:
+            splits = 1
+        elif splits is None:
+            splits = int(self.k.attention_spread_splits(b.num_seqs, b.max_q_len, H, G, wv, b.max_kv_len, int(window)))
         out = torch.empty(T, max(out_cols, H * v_dim), dtype=q.dtype, device=q.device)
         part_o = torch.empty(T, H, splits, wv, dtype=torch.float32, device=q.device)
         part_ml = torch.empty(T, H, splits, 2, dtype=torch.float32, device=q.device)
         self.launches += self.k.attention_talk(q, k_cache, v_cache, int(dim), int(v_dim), b.block_tables, b.row_seq, b.positions, b.q_starts, out, b.num_seqs,
                                                b.max_q_len, b.min_q_len, float(scale), int(window), sink, r1, r2, talk, gate, part_o, part_ml,
-                                               bool(fast), self.status)
+                                               bool(fast), float(reach), self.status)
         return out
 
     def decay_scan(self, q, k, v, decay, state, q_starts, seq_state, positions, H, K, V, width=0, max_q_len=0, min_q_len=0, chunk_from=DECAY_CHUNK_TOKENS):
