@@ -6,12 +6,12 @@
 //   out_h = sigmoid(gate_h) sum_f talk[h, f] A_f(values of h's group) / (l_f + exp(sink_f - m_f))
 // which equals mixing the heads' weights in front of the values.
 //
-// talk_prefill_kernel: one stream of 128 query rows (token * group + head) of one key head per CTA and up to 256 value columns. Warps 0 and 1
-// bring tiles of 128 keys by TMA, K whole and V in pieces of 128 columns: a lane per page of 16 tokens finds its place in the pool, one
-// lane issues the boxes (one thread that also walks the pages is slower than the products). Warp 3 issues the MMAs. Sixteen warps are the softmax: a row belongs to
-// four threads with 32 columns each, which stay in registers between the maximum and the weights. Tensor memory: two score / weight
-// buffers of 128 columns and 256 columns of output, so that the softmax of a tile runs under the products of the one before and the
-// scores of the one after it. The weights travel as two bf16 terms, as in attention_maps.cu.
+// talk_prefill_kernel: one stream of 128 query rows (token * group + head) of one key head per CTA and up to 256 value columns. Warps 0 and 2
+// bring tiles of 128 keys by TMA, warp 1 their values, all columns of a 16-token page in one box (issuing a box takes its thread as long as
+// an MMA takes the tensor cores, whatever its size): a lane per page finds its place in the pool, one lane issues. Warp 3 issues the
+// MMAs. Sixteen warps are the softmax: a row belongs to four threads with 32 columns each, which stay in registers between the maximum
+// and the weights. Tensor memory: two score / weight buffers of 128 columns and 256 columns of output, so that the softmax of a tile runs
+// under the products of the one before and the scores of the one after it. The weights travel as two bf16 terms, as in attention_maps.cu.
 //
 // talk_decode_kernel: mma.sync, 16 query rows (token * heads + head, so usually all heads of a token) and up to 256 value columns per CTA.
 // The scores of all key heads fall into one accumulator: a row's queries are zero against every key head but its own. Each warp streams
@@ -35,9 +35,10 @@ namespace fllm {
 namespace {
 constexpr float kLn2 = 0.6931471805599453f;
 constexpr int kMmaWarp = 3, kFirstSoftmax = 128, kSoftmax = 512, kThreads = kFirstSoftmax + kSoftmax;
-constexpr int kPiece = 128;                              // value columns of one product
+constexpr int kCols = 256;                               // most value columns of a CTA
+constexpr int kPiece = 128;                              // value columns of an item of the decode kernel's ring
 constexpr int kTable = 2592;                             // fp32 entries of a tile's factors (16 heads of a group)
-constexpr int kVStages = 3;
+constexpr int kVStages = 3, kVPages = 4;                 // V comes in stages of four pages
 
 struct Talk {
   const bf16 *q, *kc, *vc;
@@ -54,7 +55,7 @@ struct Talk {
 
 template <int DK>
 struct TalkTile {
-  static constexpr int kQ = tile_bytes<DK>(), kK = tile_bytes<DK>(), kV = tile_bytes<kPiece>();
+  static constexpr int kQ = tile_bytes<DK>(), kK = tile_bytes<DK>(), kV = kVPages * kPage * kCols * 2;
   static constexpr int kTail = 256 + 2 * 4 * kRows * 4 + 4 * kRows * 4 + 2 * 16 * 4 + kTable * 4;
   static constexpr int kTotal = kQ + 2 * kK + kVStages * kV + kTail + 1024;
   static_assert(kTotal <= 227 * 1024, "shared memory");
@@ -127,6 +128,11 @@ __device__ __forceinline__ float largest(const uint32_t (&sa)[32], int lo, int h
   return fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
 }
 
+// MN-major operand of 16 tokens: 1024 bytes between groups of eight tokens, 2048 between 64-column parts
+__device__ __forceinline__ uint64_t desc_page(uint32_t saddr) {
+  return (uint64_t)((saddr & 0x3FFFFu) >> 4) | (uint64_t)(kPage * 128 >> 4) << 16 | (uint64_t)(1024 >> 4) << 32 | (uint64_t)1 << 46 | (uint64_t)2 << 61;
+}
+
 template <int DK>
 __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_constant__ CUtensorMap tma_v,
                                                                    const Talk p, int min_rows, int col_ctas) {
@@ -135,7 +141,7 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sq = smem;
   uint8_t* sk = smem + L::kQ;                                        // [2]
-  uint8_t* sv = sk + 2 * L::kK;                                      // [kVStages] pieces of 128 columns
+  uint8_t* sv = sk + 2 * L::kK;                                      // [kVStages][page][64-column part][token], 128-byte swizzled rows
   uint64_t* bars = reinterpret_cast<uint64_t*>(sv + kVStages * L::kV);
   uint64_t *k_full = bars, *k_empty = bars + 2, *s_full = bars + 4, *p_ready = bars + 6, *o_done = bars + 7;
   uint64_t *v_full = bars + 8, *v_empty = bars + 8 + kVStages;
@@ -148,8 +154,8 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int row0 = (gridDim.x - 1 - blockIdx.x) * kRows;             // the tiles with the longest key range start first
-  const int kvh = blockIdx.y / col_ctas, col0 = blockIdx.y % col_ctas * 2 * kPiece, seq = blockIdx.z;
-  const int cols = min(2 * kPiece, p.wv - col0), step = min(cols, kPiece), pieces = (cols + kPiece - 1) / kPiece;
+  const int kvh = blockIdx.y / col_ctas, col0 = blockIdx.y % col_ctas * kCols, seq = blockIdx.z;
+  const int cols = min(kCols, p.wv - col0), v_page = kPage * 2 * min(kCols, p.wv);      // bytes of a page as it is fetched (zeros beyond the row)
   const int q0 = p.q_starts[seq], qn = p.q_starts[seq + 1] - q0;
   const int all_rows = qn * p.group;
   if (all_rows < min_rows || row0 >= all_rows) return;
@@ -159,7 +165,7 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
   const int n_tiles = (first_pos + (row0 + n_rows - 1) / p.group + 1 - begin + kTile - 1) / kTile;
 
   if (threadIdx.x == 0) {
-    for (int i = 0; i < 2; ++i) mbar_init(&k_full[i], 1), mbar_init(&k_empty[i], 1), mbar_init(&s_full[i], 1);
+    for (int i = 0; i < 2; ++i) mbar_init(&k_full[i], 2), mbar_init(&k_empty[i], 1), mbar_init(&s_full[i], 1);
     for (int i = 0; i < kVStages; ++i) mbar_init(&v_full[i], 1), mbar_init(&v_empty[i], 1);
     mbar_init(p_ready, kSoftmax / 32), mbar_init(o_done, 1);
     *abort_flag = 0;
@@ -182,7 +188,7 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
   tc_fence_after_sync();
   const uint32_t tmem_base = *tmem_slot;
 
-  if (warp < 2) {
+  if (warp < kMmaWarp) {
     constexpr int PAGES = kTile / kPage;
     const int* blocks = p.block_tables + (size_t)seq * p.max_blocks;
     const int last = (kv_len - 1) / kPage * kPage;                     // pages past the sequence repeat its last one (finite values)
@@ -191,19 +197,20 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
       const int tok = min(begin + it * kTile + lane % PAGES * kPage, last);
       return (blocks[tok / p.block_size] * heads + head) * p.block_size + tok % p.block_size;
     };
-    if (warp == 0) {
+    if (warp != 1) {                                                   // half of the pages' keys
+      const int pg0 = warp == 0 ? 0 : PAGES / 2;
       int row = first_row(0, p.G, kvh);
       for (int it = 0; it < n_tiles; ++it) {
         const int now = row, b = it & 1, use = it >> 1;
         if (it + 1 < n_tiles) row = first_row(it + 1, p.G, kvh);
         if (!__all_sync(0xffffffffu, use == 0 || mbar_wait(&k_empty[b], (use - 1) & 1, abort_flag))) break;
-        if (lane == 0) mbar_expect_tx(&k_full[b], tile_bytes<DK>());
+        if (lane == 0) mbar_expect_tx(&k_full[b], tile_bytes<DK>() / 2);
 #pragma unroll
-        for (int pg = 0; pg < PAGES; ++pg) {
-          const int y = __shfl_sync(0xffffffffu, now, pg);
+        for (int pg = 0; pg < PAGES / 2; ++pg) {
+          const int y = __shfl_sync(0xffffffffu, now, pg0 + pg);
           if (lane == 0) {
 #pragma unroll
-            for (int h = 0; h < DK / 64; ++h) tma_load_2d(sk + b * L::kK + h * kHalf + pg * (kPage * 128), &tma_k, &k_full[b], 64 * h, y);
+            for (int h = 0; h < DK / 64; ++h) tma_load_2d(sk + b * L::kK + h * kHalf + (pg0 + pg) * (kPage * 128), &tma_k, &k_full[b], 64 * h, y);
           }
         }
       }
@@ -213,16 +220,14 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
       for (int it = 0; ok && it < n_tiles; ++it) {
         const int now = row;
         if (it + 1 < n_tiles) row = first_row(it + 1, 1, 0);
-        for (int c = 0; c < pieces; ++c) {
+#pragma unroll 1
+        for (int c = 0; c < PAGES; c += kVPages) {
           if (!(ok = __all_sync(0xffffffffu, v_use == 0 || mbar_wait(&v_empty[vs], (v_use - 1) & 1, abort_flag)))) break;
-          if (lane == 0) mbar_expect_tx(&v_full[vs], step / 64 * kHalf);
+          if (lane == 0) mbar_expect_tx(&v_full[vs], kVPages * v_page);
 #pragma unroll
-          for (int pg = 0; pg < PAGES; ++pg) {
-            const int y = __shfl_sync(0xffffffffu, now, pg);
-            if (lane == 0) {
-              tma_load_2d(sv + vs * L::kV + pg * (kPage * 128), &tma_v, &v_full[vs], col0 + c * kPiece, y);
-              if (step > 64) tma_load_2d(sv + vs * L::kV + kHalf + pg * (kPage * 128), &tma_v, &v_full[vs], col0 + c * kPiece + 64, y);
-            }
+          for (int pg = 0; pg < kVPages; ++pg) {
+            const int y = __shfl_sync(0xffffffffu, now, c + pg);
+            if (lane == 0) tma_load_3d(sv + vs * L::kV + pg * v_page, &tma_v, &v_full[vs], 0, y, col0 / 64);
           }
           if (++vs == kVStages) vs = 0, ++v_use;
         }
@@ -231,7 +236,7 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
   } else if (warp == kMmaWarp) {
     if (lane == 0) {
       constexpr uint32_t idesc_s = make_idesc(128, 128, 1, 1);
-      const uint32_t idesc_pv = make_idesc(128, step, 1, 1) | (1u << 16);      // B is MN-major
+      const uint32_t idesc_pv = make_idesc(128, cols, 1, 1) | (1u << 16);      // B is MN-major
       const uint32_t q_addr = smem_u32(sq), k_addr = smem_u32(sk), v_addr = smem_u32(sv);
       bool ok = true;
       auto scores = [&](int it) {
@@ -252,16 +257,16 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
       for (int it = 0; ok && it < n_tiles; ++it) {
         const uint32_t t_p = tmem_base + 128 * (it & 1);
         if (!(ok = mbar_wait(p_ready, it & 1, abort_flag))) break;
-        for (int c = 0; c < pieces; ++c) {
+        for (int c = 0; c < kTile / kPage; c += kVPages) {
           if (!(ok = mbar_wait(&v_full[vs], v_use & 1, abort_flag))) break;
           tc_fence_after_sync();
-          const uint32_t t_o = tmem_base + 256 + kPiece * c;
 #pragma unroll
-          for (int k = 0; k < kTile / 16; ++k) {
+          for (int pg = 0; pg < kVPages; ++pg) {
+            const int k = c + pg;
             const uint32_t a = t_p + 32 * (k >> 1) + 8 * (k & 1);
-            const uint64_t v = desc_mn_major<kPiece>(v_addr + vs * L::kV + k * 2048);
-            tc_mma_bf16_ts(t_o, a, v, idesc_pv, it > 0 || k > 0);
-            tc_mma_bf16_ts(t_o, a + 16, v, idesc_pv, 1);
+            const uint64_t v = desc_page(v_addr + vs * L::kV + pg * v_page);
+            tc_mma_bf16_ts(tmem_base + 256, a, v, idesc_pv, it > 0 || k > 0);
+            tc_mma_bf16_ts(tmem_base + 256, a + 16, v, idesc_pv, 1);
           }
           tc_commit(&v_empty[vs]);
           if (++vs == kVStages) vs = 0, ++v_use;
@@ -765,15 +770,24 @@ void launch_decode(const Talk& a, const MapsAttnParams& p, int splits, cudaStrea
   cuda_check(cudaGetLastError(), "talk_decode_kernel");
 }
 
+// tensor map of a pool of rows of wv values as [64-column part][row][64 values], in boxes of a page's rows and up to kCols columns
+CUtensorMap value_map(const void* pool, uint64_t rows, int wv) {
+  static std::unordered_map<std::string, CUtensorMap> maps;
+  const std::string key = std::to_string(reinterpret_cast<uintptr_t>(pool)) + "/" + std::to_string(rows) + "/" + std::to_string(wv);
+  auto it = maps.find(key);
+  if (it != maps.end()) return it->second;
+  if (maps.size() > 4096) maps.clear();
+  return maps.emplace(key, make_tmap_parts(pool, rows, wv, kPage, std::min(kCols, wv) / 64)).first->second;
+}
+
 template <int DK>
 void launch_prefill(const Talk& a, const MapsAttnParams& p, int min_rows, cudaStream_t s) {
   static bool configured[kMaxDevices] = {};
   if (first_call_on_device(configured))
     cuda_check(cudaFuncSetAttribute(talk_prefill_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, TalkTile<DK>::kTotal), "talk_prefill smem");
   const uint64_t n = (uint64_t)p.num_blocks * a.block_size;
-  // (copies: a second lookup may move the first entry)
-  const CUtensorMap km = pool_map(p.k_cache, n * a.G, DK), vm = pool_map(p.v_cache, n, a.wv);
-  const int col_ctas = (a.wv + 2 * kPiece - 1) / (2 * kPiece);
+  const CUtensorMap km = pool_map(p.k_cache, n * a.G, DK), vm = value_map(p.v_cache, n, a.wv);
+  const int col_ctas = (a.wv + kCols - 1) / kCols;
   const dim3 grid((p.max_q_len * a.group + kRows - 1) / kRows, a.G * col_ctas, p.num_seqs);
   talk_prefill_kernel<DK><<<grid, kThreads, TalkTile<DK>::kTotal, s>>>(km, vm, a, min_rows, col_ctas);
   cuda_check(cudaGetLastError(), "talk_prefill_kernel");

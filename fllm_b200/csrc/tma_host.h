@@ -61,6 +61,21 @@ inline CUtensorMap make_tmap_2d(const void* base, CUtensorMapDataType dt, int el
   return m;
 }
 
+// bf16 rows of `cols` values (a multiple of 64) as a 3-D tensor [cols / 64][rows][64]: a box of `box_parts` 64-column parts of
+// `box_rows` rows lands as [part][row][64], 128-byte swizzled. Parts beyond the row read as zero.
+inline CUtensorMap make_tmap_parts(const void* base, uint64_t rows, uint64_t cols, uint32_t box_rows, uint32_t box_parts) {
+  CUtensorMap m;
+  cuuint64_t dims[3] = {64, rows, cols / 64};
+  cuuint64_t strides[2] = {cols * 2, 128};
+  cuuint32_t box[3] = {64, box_rows, box_parts};
+  cuuint32_t estr[3] = {1, 1, 1};
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || cols % 64) throw std::runtime_error("fllm_b200: TMA operand must be 16-byte aligned, rows of whole 64-column parts");
+  CUresult r = get_encode_tiled()(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                                  CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) throw std::runtime_error("fllm_b200: cuTensorMapEncodeTiled failed with code " + std::to_string((int)r));
+  return m;
+}
+
 // Programmatic dependent launch: the kernel may start while its predecessor in the stream is
 // still running; it must execute griddepcontrol.wait before it touches anything the predecessor
 // produces. FLLM_PDL=0 turns the attribute off (plain stream order).
