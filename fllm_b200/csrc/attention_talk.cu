@@ -9,7 +9,7 @@
 // talk_prefill_kernel: one stream of 128 query rows (token * group + head) of one key head per CTA and up to 256 value columns. Warps 0 and 2
 // bring tiles of 128 keys by TMA, warp 1 their values, all columns of a 16-token page in one box (issuing a box takes its thread as long as
 // an MMA takes the tensor cores, whatever its size): a lane per page finds its place in the pool, one lane issues. Warp 3 issues the
-// MMAs. Sixteen warps are the softmax: a row belongs to four threads with 32 columns each, which stay in registers between the maximum
+// MMAs. Eight warps are the softmax: a row belongs to two threads with 64 columns each, which stay in registers between the maximum
 // and the weights. Tensor memory: two score / weight buffers of 128 columns and 256 columns of output, so that the softmax of a tile runs
 // under the products of the one before and the scores of the one after it. The weights travel as two bf16 terms, as in attention_maps.cu.
 //
@@ -34,7 +34,8 @@
 namespace fllm {
 namespace {
 constexpr float kLn2 = 0.6931471805599453f;
-constexpr int kMmaWarp = 3, kFirstSoftmax = 128, kSoftmax = 512, kThreads = kFirstSoftmax + kSoftmax;
+constexpr int kParts = 2, kSpan = kTile / kParts;        // threads of a row, columns of each
+constexpr int kMmaWarp = 3, kFirstSoftmax = 128, kSoftmax = kRows * kParts, kThreads = kFirstSoftmax + kSoftmax;
 constexpr int kCols = 256;                               // most value columns of a CTA
 constexpr int kPiece = 128;                              // value columns of an item of the decode kernel's ring
 constexpr int kTable = 2592;                             // fp32 entries of a tile's factors (16 heads of a group)
@@ -56,12 +57,12 @@ struct Talk {
 template <int DK>
 struct TalkTile {
   static constexpr int kQ = tile_bytes<DK>(), kK = tile_bytes<DK>(), kV = kVPages * kPage * kCols * 2;
-  static constexpr int kTail = 256 + 2 * 4 * kRows * 4 + 4 * kRows * 4 + 2 * 16 * 4 + kTable * 4;
+  static constexpr int kTail = 256 + 2 * kParts * kRows * 4 + kParts * kRows * 4 + 4 * 16 * 4 + kTable * 4;
   static constexpr int kTotal = kQ + 2 * kK + kVStages * kV + kTail + 1024;
   static_assert(kTotal <= 227 * 1024, "shared memory");
 };
 
-__device__ __forceinline__ void softmax_barrier() { asm volatile("bar.sync 1, 512;" ::: "memory"); }
+__device__ __forceinline__ void softmax_barrier() { asm volatile("bar.sync 1, %0;" ::"n"(kSoftmax) : "memory"); }
 // two fp32 operations at once
 __device__ __forceinline__ uint64_t pair(float a, float b) {
   uint64_t r;
@@ -89,43 +90,58 @@ __device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
   return r;
 }
 
-// weights of 32 columns of a row: sa holds the raw scores; columns [lo, hi) are visible (FULL: all); fac[-c] is the factor of column c.
+__device__ __forceinline__ float lg2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float max3(float a, float b, float c) {
+  float y;
+  asm("max.f32 %0, %1, %2, %3;" : "=f"(y) : "f"(a), "f"(b), "f"(c));
+  return y;
+}
+
+// weights of kSpan columns of a row: sa holds the raw scores; columns [lo, hi) are visible (FULL: all); fac[-c] is the factor of column c.
 // A weight is cut after its leading bf16 term, the second term is the rounded rest.
 template <bool FULL>
-__device__ __forceinline__ float weigh(uint32_t t_s, const uint32_t (&sa)[32], float scale_log2, float ref, const float* fac, int lo, int hi) {
+__device__ __forceinline__ float weigh(uint32_t t_s, const uint32_t (&sa)[kSpan / 32][32], float scale_log2, float ref, const float* fac, int lo, int hi) {
   const uint64_t sc = pair(scale_log2, scale_log2), off = pair(-ref, -ref), minus = pair(-1.f, -1.f);
   uint64_t sum[2] = {0, 0};
-  uint32_t ph[16], pl[16];
 #pragma unroll
-  for (int c = 0; c < 32; c += 2) {
-    const float2 t = unpair(fma2(pair(__uint_as_float(sa[c]), __uint_as_float(sa[c + 1])), sc, off));
-    uint64_t v = mul2(pair(ex2(t.x), ex2(t.y)), pair(fac[-c], fac[-c - 1]));
-    if (!FULL) {
-      float2 w = unpair(v);
-      if (c < lo || c >= hi) w.x = 0.f;
-      if (c + 1 < lo || c + 1 >= hi) w.y = 0.f;
-      v = pair(w.x, w.y);
+  for (int b = 0; b < kSpan / 32; ++b) {
+    uint32_t ph[16], pl[16];
+#pragma unroll
+    for (int i = 0; i < 32; i += 2) {
+      const int c = 32 * b + i;
+      const float2 t = unpair(fma2(pair(__uint_as_float(sa[b][i]), __uint_as_float(sa[b][i + 1])), sc, off));
+      uint64_t v = mul2(pair(ex2(t.x), ex2(t.y)), pair(fac[-c], fac[-c - 1]));
+      if (!FULL) {
+        float2 w = unpair(v);
+        if (c < lo || c >= hi) w.x = 0.f;
+        if (c + 1 < lo || c + 1 >= hi) w.y = 0.f;
+        v = pair(w.x, w.y);
+      }
+      sum[(i >> 1) & 1] = add2(sum[(i >> 1) & 1], v);
+      const float2 w = unpair(v);
+      const uint32_t x = __float_as_uint(w.x), y = __float_as_uint(w.y);
+      ph[i / 2] = __byte_perm(x, y, 0x7632);
+      const float2 rest = unpair(fma2(pair(__uint_as_float(x & 0xffff0000u), __uint_as_float(y & 0xffff0000u)), minus, v));
+      pl[i / 2] = pack_bf16x2(rest.x, rest.y);
     }
-    sum[(c >> 1) & 1] = add2(sum[(c >> 1) & 1], v);
-    const float2 w = unpair(v);
-    const uint32_t x = __float_as_uint(w.x), y = __float_as_uint(w.y);
-    ph[c / 2] = __byte_perm(x, y, 0x7632);
-    const float2 rest = unpair(fma2(pair(__uint_as_float(x & 0xffff0000u), __uint_as_float(y & 0xffff0000u)), minus, v));
-    pl[c / 2] = pack_bf16x2(rest.x, rest.y);
+    tmem_st_32x16(t_s + 32 * b, ph);
+    tmem_st_32x16(t_s + 32 * b + 16, pl);
   }
-  tmem_st_32x16(t_s, ph);
-  tmem_st_32x16(t_s + 16, pl);
   const float2 all = unpair(add2(sum[0], sum[1]));
   return all.x + all.y;
 }
-// the largest of 32 scores, or of the visible ones
+// the largest of kSpan scores, or of the visible ones
 template <bool FULL>
-__device__ __forceinline__ float largest(const uint32_t (&sa)[32], int lo, int hi) {
+__device__ __forceinline__ float largest(const uint32_t (&sa)[kSpan / 32][32], int lo, int hi) {
+  auto at = [&](int c) { return FULL || (c >= lo && c < hi) ? __uint_as_float(sa[c >> 5][c & 31]) : -INFINITY; };
   float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-  for (int c = 0; c < 32; ++c)
-    if (FULL || (c >= lo && c < hi)) mx[c & 3] = fmaxf(mx[c & 3], __uint_as_float(sa[c]));
-  return fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+  for (int c = 0; c < kSpan; c += 2) mx[(c >> 1) & 3] = max3(mx[(c >> 1) & 3], at(c), at(c + 1));
+  return fmaxf(max3(mx[0], mx[1], mx[2]), mx[3]);
 }
 
 // MN-major operand of 16 tokens: 1024 bytes between groups of eight tokens, 2048 between 64-column parts
@@ -148,10 +164,13 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 8 + 2 * kVStages);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   float* swap_m = reinterpret_cast<float*>(bars + 32);               // [buffer][part][row]
-  float* swap_l = swap_m + 8 * kRows;                                // [part][row]
-  float* rates = swap_l + 4 * kRows;                                 // [head of the group] r1, then r2
-  float* table = rates + 2 * 16;
+  float* swap_l = swap_m + 2 * kParts * kRows;                       // [part][row]
+  float* rates = swap_l + kParts * kRows;                                 // [head of the group] r1, then r2
+  float* near_bias = rates + 2 * 16;                                 // [buffer][head of the group]: bias of a tile's smallest distance
+  float* table = near_bias + 2 * 16;
 
+  pdl_launch_dependents();
+  pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int row0 = (gridDim.x - 1 - blockIdx.x) * kRows;             // the tiles with the longest key range start first
   const int kvh = blockIdx.y / col_ctas, col0 = blockIdx.y % col_ctas * kCols, seq = blockIdx.z;
@@ -174,7 +193,13 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
   if (threadIdx.x == 0) tma_prefetch_desc(&tma_k);
   if (threadIdx.x == 32) tma_prefetch_desc(&tma_v);
   if (warp == kMmaWarp) tmem_alloc(tmem_slot, 512), tmem_relinquish();
-  for (int i = threadIdx.x; i < p.group; i += kThreads) rates[i] = p.r1 ? p.r1[kvh * p.group + i] : 0.f, rates[16 + i] = p.r1 ? p.r2[kvh * p.group + i] : 0.f;
+  auto bias = [](float a, float b, int d) { return a * lg2(fmaf(b, (float)d, 1.f)); };
+  auto nearest = [&](int it) { return max(i0 - (begin + it * kTile) - (kTile - 1), 0); };
+  if (threadIdx.x < p.group) {
+    const int head = kvh * p.group + threadIdx.x;
+    const float a = p.r1 ? p.r1[head] : 0.f, b = p.r1 ? p.r2[head] : 0.f;
+    rates[threadIdx.x] = a, rates[16 + threadIdx.x] = b, near_bias[threadIdx.x] = bias(a, b, nearest(0));
+  }
   // query rows -> shared memory in the layout TMA's 128-byte swizzle would have produced
   for (int i = threadIdx.x; i < kRows * (DK / 8); i += kThreads) {
     const int r = i / (DK / 8), c = i % (DK / 8), row = row0 + r;
@@ -277,16 +302,15 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
       }
     }
   } else if (warp >= kFirstSoftmax / 32) {                             // (warp 2 has no work)
-    // thread of a row's columns 32 part .. 32 part + 31; the row is in the lane quarter this warp may touch
+    // thread of a row's columns kSpan part .. + kSpan - 1; the row is in the lane quarter this warp may touch
     const int part = (warp - kFirstSoftmax / 32) >> 2, r = (warp & 3) * 32 + lane, id = threadIdx.x - kFirstSoftmax;
     const uint32_t lane_off = (uint32_t)((warp & 3) * 32) << 16;
     const bool valid = r < n_rows;
     const int lim = valid ? first_pos + (row0 + r) / p.group + 1 : 0, beg = p.window > 0 ? max(0, lim - p.window) : 0;
-    const int lim_first = i0 + 1, last_lim = first_pos + (row0 + n_rows - 1) / p.group + 1, beg_last = p.window > 0 ? max(0, last_lim - p.window) : 0;
+    const int last_lim = first_pos + (row0 + n_rows - 1) / p.group + 1, beg_last = p.window > 0 ? max(0, last_lim - p.window) : 0;
     const int off = (row0 + r) / p.group - row0 / p.group, hh = (row0 + r) % p.group;      // token behind the CTA's first, head of the group
-    const float my_r1 = rates[hh], my_r2 = rates[16 + hh];
-    auto bias = [](float a, float b, int d) { return a * __log2f(fmaf(b, (float)d, 1.f)); };
     const int e_head = id / p.tab_stride, e_at = id % p.tab_stride, jump_head = kSoftmax / p.tab_stride, jump_at = kSoftmax % p.tab_stride;
+    float* my_max = swap_m + r;
     float m_used = -INFINITY, l = 0.f;
     bool ok = true;
     for (int it = 0; it < n_tiles; ++it) {
@@ -295,12 +319,13 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
       float* buf = table + (p.tab_bufs == 2 && (it & 1) ? p.tab_entries : 0);
       if (p.tab_bufs == 1 && it > 0) softmax_barrier();
       for (int head = e_head, at = e_at, i = id; i < p.tab_entries; i += kSoftmax) {
-        const float a = rates[head], b = rates[16 + head];
-        buf[i] = ex2(bias(a, b, d0) - bias(a, b, max(base + at, d0)));
+        buf[i] = ex2(near_bias[(it & 1) * 16 + head] - bias(rates[head], rates[16 + head], max(base + at, d0)));
         head += jump_head, at += jump_at;
         if (at >= p.tab_stride) at -= p.tab_stride, ++head;
       }
-      const uint32_t t_s = tmem_base + 128 * (it & 1) + 32 * part + lane_off;
+      const float b0 = near_bias[(it & 1) * 16 + hh];
+      if (id < p.group) near_bias[(~it & 1) * 16 + id] = bias(rates[id], rates[16 + id], nearest(it + 1));
+      const uint32_t t_s = tmem_base + 128 * (it & 1) + kSpan * part + lane_off;
       // every thread waits for every tile's output products, in order: before it touches the output, or at its end
       bool waited = it == 0;
       auto wait_output = [&]() {
@@ -311,18 +336,21 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
       };
       if (!mbar_wait(&s_full[it & 1], (it >> 1) & 1, abort_flag)) ok = false;
       tc_fence_after_sync();
-      uint32_t sa[32];
-      tmem_ld_32x32(t_s, sa);
+      uint32_t sa[kSpan / 32][32];
+#pragma unroll
+      for (int b = 0; b < kSpan / 32; ++b) tmem_ld_32x32(t_s + 32 * b, sa[b]);
       tmem_ld_wait();
-      const int lo = beg - tok0 - 32 * part, hi = lim - tok0 - 32 * part;
-      const bool full = n_rows == kRows && tok0 + kTile <= lim_first && tok0 >= beg_last;
-      float* mine = swap_m + (it & 1) * 4 * kRows + r;
-      mine[part * kRows] = full ? largest<true>(sa, 0, 0) : largest<false>(sa, lo, hi);
+      const int lo = beg - tok0 - kSpan * part, hi = lim - tok0 - kSpan * part;
+      const bool full = n_rows == kRows && tok0 + kTile <= i0 + 1 && tok0 >= beg_last;
+      float* row_max = my_max + (it & 1) * kParts * kRows;
+      row_max[part * kRows] = full ? largest<true>(sa, 0, 0) : largest<false>(sa, lo, hi);
       softmax_barrier();
-      const float raw = fmaxf(fmaxf(mine[0], mine[kRows]), fmaxf(mine[2 * kRows], mine[3 * kRows])), b0 = bias(my_r1, my_r2, d0);
+      float raw = row_max[0];
+#pragma unroll
+      for (int k = 1; k < kParts; ++k) raw = fmaxf(raw, row_max[k * kRows]);
       const float top = raw == -INFINITY ? -INFINITY : fmaf(raw, p.scale_log2, -b0);
       // a row keeps its old reference unless the new maximum is far above it; the decision is per warp because the tensor
-      // memory accesses of the rescale are warp-wide, and the four warps of the rows take the same one
+      // memory accesses of the rescale are warp-wide, and all warps of the rows take the same one
       if (__any_sync(0xffffffffu, top > m_used + kLazyRescale || (m_used == -INFINITY && top > -INFINITY))) {
         const float m_new = fmaxf(m_used, top), corr = m_new == -INFINITY ? 1.f : ex2(m_used - m_new);
         m_used = m_new;
@@ -330,7 +358,7 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
         if (it > 0) {
           wait_output();
 #pragma unroll 1
-          for (int c = part * 32; c < cols; c += 128) {
+          for (int c = part * 32; c < cols; c += 32 * kParts) {
             uint32_t o[32];
             const uint32_t t_o = tmem_base + 256 + c + lane_off;
             tmem_ld_32x32(t_o, o);
@@ -347,7 +375,7 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
         }
       }
       const float ref = (m_used == -INFINITY ? 0.f : m_used) + b0;
-      const float* fac = buf + hh * p.tab_stride + off + (kTile - 1) - 32 * part;
+      const float* fac = buf + hh * p.tab_stride + off + (kTile - 1) - kSpan * part;
       l += full ? weigh<true>(t_s, sa, p.scale_log2, ref, fac, 0, 0) : weigh<false>(t_s, sa, p.scale_log2, ref, fac, lo, hi);
       tmem_st_wait();
       wait_output();
@@ -359,10 +387,13 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
     tc_fence_after_sync();
     swap_l[part * kRows + r] = l;
     softmax_barrier();
+    l = 0.f;
+#pragma unroll
+    for (int k = 0; k < kParts; ++k) l += swap_l[k * kRows + r];
     const int row = row0 + r;
     const long long at = (long long)(q0 + row / p.group) * p.H + kvh * p.group + row % p.group;
 #pragma unroll 1
-    for (int c = part * 32; c < cols; c += 128) {
+    for (int c = part * 32; c < cols; c += 32 * kParts) {
       uint32_t o[32];
       tmem_ld_32x32(tmem_base + 256 + c + lane_off, o);
       tmem_ld_wait();
@@ -372,8 +403,7 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
       for (int i = 0; i < 8; ++i)
         to[i] = make_float4(__uint_as_float(o[4 * i]), __uint_as_float(o[4 * i + 1]), __uint_as_float(o[4 * i + 2]), __uint_as_float(o[4 * i + 3]));
     }
-    if (ok && valid && part == 0 && col0 == 0)
-      p.part_ml[2 * at] = m_used * kLn2, p.part_ml[2 * at + 1] = (l + swap_l[kRows + r]) + (swap_l[2 * kRows + r] + swap_l[3 * kRows + r]);
+    if (ok && valid && part == 0 && col0 == 0) p.part_ml[2 * at] = m_used * kLn2, p.part_ml[2 * at + 1] = l;
   }
   tc_fence_before_sync();
   __syncthreads();
@@ -654,7 +684,71 @@ __global__ void __launch_bounds__(256) talk_mix_rows_kernel(const TalkMixParams 
   for (int c = H * p.v_dim + threadIdx.x; c < p.cols; c += blockDim.x) out[c] = from_f32<T>(0.f);
 }
 
-// One CTA per token and NC of its value columns (g, i), 256 / NC threads per column: the normalised column of every head's output is
+// Several key slices, or few tokens: a CTA per token, blockDim.x threads with four columns each times blockDim.y shares of the heads, whose
+// parts of four mixed heads are added up through shared memory.
+template <typename T>
+__global__ void __launch_bounds__(512) talk_mix_slices_kernel(const TalkMixParams p) {
+  extern __shared__ __align__(16) float sm[];
+  const int H = p.H, S = p.splits, group = H / p.G, t = blockIdx.x, X = blockDim.x, Y = blockDim.y, x = threadIdx.x, y = threadIdx.y;
+  const int id = y * X + x, n = X * Y, warp = id >> 5, lane = id & 31;
+  float4* part = reinterpret_cast<float4*>(sm);          // [4][Y][X]
+  float* mat = sm + 16 * n;                              // [f][h]
+  float* coef = mat + H * H;                             // [f][slice]
+  pdl_launch_dependents();
+  for (int i = id; i < H * H; i += n) mat[i % H * H + i / H] = p.talk[i];
+  pdl_wait();
+  for (int h = warp; h < H; h += n / 32) {               // a lane per key slice
+    const float2 v = lane < S ? __ldcg(reinterpret_cast<const float2*>(p.part_ml) + ((size_t)t * H + h) * S + lane) : make_float2(-INFINITY, 0.f);
+    const float m = warp_max(v.x), c = v.x == -INFINITY ? 0.f : expf(v.x - m), l = warp_sum(v.y * c) + (p.sink ? expf(p.sink[h] - m) : 0.f);
+    if (lane < S) coef[h * S + lane] = c / l;
+  }
+  __syncthreads();
+  T* out = static_cast<T*>(p.out) + (long long)t * p.ldo;
+  const int cols = p.G * p.v_dim;
+  for (int c0 = 0; c0 < cols; c0 += 4 * X) {
+    const int c = c0 + 4 * x, g = min(c, cols - 4) / p.v_dim, i = c - g * p.v_dim;
+    const float* src = p.part_o + (size_t)t * H * S * p.wv + c;
+    for (int e0 = 0; e0 < group; e0 += 4) {
+      const int h0 = g * group + e0, k = min(4, group - e0);
+      float4 acc[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[e] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < cols) {
+        for (int f = y; f < H; f += Y) {
+          float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+          for (int s = 0; s < S; ++s) {
+            const float4 v = __ldcg(reinterpret_cast<const float4*>(src + ((size_t)f * S + s) * p.wv));
+            const float z = coef[f * S + s];
+            a.x = fmaf(z, v.x, a.x), a.y = fmaf(z, v.y, a.y), a.z = fmaf(z, v.z, a.z), a.w = fmaf(z, v.w, a.w);
+          }
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float w = mat[f * H + h0 + min(e, k - 1)];
+            acc[e].x = fmaf(w, a.x, acc[e].x), acc[e].y = fmaf(w, a.y, acc[e].y), acc[e].z = fmaf(w, a.z, acc[e].z), acc[e].w = fmaf(w, a.w, acc[e].w);
+          }
+        }
+      }
+      __syncthreads();
+#pragma unroll
+      for (int e = 0; e < 4; ++e) part[e * n + id] = acc[e];
+      __syncthreads();
+      for (int e = y; e < k && c < cols; e += Y) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int j = 0; j < Y; ++j) {
+          const float4 q = part[e * n + j * X + x];
+          v.x += q.x, v.y += q.y, v.z += q.z, v.w += q.w;
+        }
+        const float z = p.gate ? 1.f / (1.f + expf(-p.gate[(long long)t * p.ld_gate + h0 + e])) : 1.f;
+        T* to = out + (long long)(h0 + e) * p.v_dim + i;
+        to[0] = from_f32<T>(v.x * z), to[1] = from_f32<T>(v.y * z), to[2] = from_f32<T>(v.z * z), to[3] = from_f32<T>(v.w * z);
+      }
+    }
+  }
+  for (int c = H * p.v_dim + id; c < p.cols; c += n) out[c] = from_f32<T>(0.f);
+}
+
+// Any value width: one CTA per token and NC of its value columns (g, i), 256 / NC threads per column: the normalised column of every head's output is
 // put together from its key slices, then each thread mixes some of the heads of group g.
 constexpr int kMixHeads = 8;
 template <typename T, int NC>
@@ -728,6 +822,16 @@ __global__ void __launch_bounds__(256) talk_mix_kernel(const TalkMixParams p) {
 }
 
 template <typename T>
+void launch_mix_slices(const TalkMixParams& p, cudaStream_t s) {
+  const int x = std::min(128, (p.G * p.v_dim / 4 + 31) / 32 * 32), y = std::max(1, std::min(512 / x, p.H));
+  const size_t smem = ((size_t)16 * x * y + (size_t)p.H * p.H + (size_t)p.H * p.splits) * sizeof(float);
+  static bool configured[kMaxDevices] = {};
+  if (first_call_on_device(configured))
+    cuda_check(cudaFuncSetAttribute(talk_mix_slices_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024), "talk_mix smem");
+  launch_pdl(talk_mix_slices_kernel<T>, dim3(p.tokens), dim3(x, y), smem, s, p);
+  cuda_check(cudaGetLastError(), "talk_mix_slices_kernel");
+}
+template <typename T>
 void launch_mix_rows(const TalkMixParams& p, cudaStream_t s) {
   const int x = std::min(256, (p.G * p.v_dim / 4 + 31) / 32 * 32), y = p.tokens >= 8 * sm_count() ? std::max(1, 256 / x) : 1;
   const size_t smem = ((size_t)p.H * p.H + (size_t)y * p.H) * sizeof(float);
@@ -789,7 +893,7 @@ void launch_prefill(const Talk& a, const MapsAttnParams& p, int min_rows, cudaSt
   const CUtensorMap km = pool_map(p.k_cache, n * a.G, DK), vm = value_map(p.v_cache, n, a.wv);
   const int col_ctas = (a.wv + kCols - 1) / kCols;
   const dim3 grid((p.max_q_len * a.group + kRows - 1) / kRows, a.G * col_ctas, p.num_seqs);
-  talk_prefill_kernel<DK><<<grid, kThreads, TalkTile<DK>::kTotal, s>>>(km, vm, a, min_rows, col_ctas);
+  launch_pdl(talk_prefill_kernel<DK>, grid, dim3(kThreads), TalkTile<DK>::kTotal, s, km, vm, a, min_rows, col_ctas);
   cuda_check(cudaGetLastError(), "talk_prefill_kernel");
 }
 }  // namespace
@@ -835,7 +939,12 @@ int attention_spread_tc(const MapsAttnParams& p, int splits, int* status, cudaSt
 void talk_mix(const TalkMixParams& p, cudaStream_t s) {
   if (p.tokens <= 0) return;
   if (p.splits > 32) throw std::runtime_error("talk_mix: at most 32 key slices");
-  if (p.splits == 1 && p.v_dim % 4 == 0 && p.H <= 96) {
+  if (p.v_dim % 4 == 0 && p.H <= 96 && (p.splits > 1 || p.tokens < 2 * sm_count())) {
+    if (p.f32) launch_mix_slices<float>(p, s);
+    else launch_mix_slices<bf16>(p, s);
+    return;
+  }
+  if (p.v_dim % 4 == 0 && p.H <= 96) {
     TalkMixParams q = p;
     q.vec = p.ldo % 4 == 0 && reinterpret_cast<uintptr_t>(p.out) % (p.f32 ? 16 : 8) == 0;
     if (p.f32) launch_mix_rows<float>(q, s);
