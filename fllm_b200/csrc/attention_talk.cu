@@ -159,7 +159,7 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
   uint8_t* sk = smem + L::kQ;                                        // [2]
   uint8_t* sv = sk + 2 * L::kK;                                      // [kVStages][page][64-column part][token], 128-byte swizzled rows
   uint64_t* bars = reinterpret_cast<uint64_t*>(sv + kVStages * L::kV);
-  uint64_t *k_full = bars, *k_empty = bars + 2, *s_full = bars + 4, *p_ready = bars + 6, *o_done = bars + 7;
+  uint64_t *k_full = bars, *k_empty = bars + 2, *s_full = bars + 4, *p_ready = bars + 6, *o_done = bars + 7, *q_full = bars + 31;
   uint64_t *v_full = bars + 8, *v_empty = bars + 8 + kVStages;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 8 + 2 * kVStages);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
@@ -186,7 +186,7 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
   if (threadIdx.x == 0) {
     for (int i = 0; i < 2; ++i) mbar_init(&k_full[i], 2), mbar_init(&k_empty[i], 1), mbar_init(&s_full[i], 1);
     for (int i = 0; i < kVStages; ++i) mbar_init(&v_full[i], 1), mbar_init(&v_empty[i], 1);
-    mbar_init(p_ready, kSoftmax / 32), mbar_init(o_done, 1);
+    mbar_init(p_ready, kSoftmax / 32), mbar_init(o_done, 1), mbar_init(q_full, kSoftmax);
     *abort_flag = 0;
     fence_barrier_init();
   }
@@ -200,14 +200,6 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
     const float a = p.r1 ? p.r1[head] : 0.f, b = p.r1 ? p.r2[head] : 0.f;
     rates[threadIdx.x] = a, rates[16 + threadIdx.x] = b, near_bias[threadIdx.x] = bias(a, b, nearest(0));
   }
-  // query rows -> shared memory in the layout TMA's 128-byte swizzle would have produced
-  for (int i = threadIdx.x; i < kRows * (DK / 8); i += kThreads) {
-    const int r = i / (DK / 8), c = i % (DK / 8), row = row0 + r;
-    uint4 v = make_uint4(0, 0, 0, 0);
-    if (row < all_rows) v = *reinterpret_cast<const uint4*>(p.q + ((long long)(q0 + row / p.group) * p.H + kvh * p.group + row % p.group) * DK + c * 8);
-    *reinterpret_cast<uint4*>(sq + (c >> 3) * kHalf + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
-  }
-  fence_proxy_async_smem();
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
@@ -276,7 +268,8 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
         tc_commit(&s_full[b]);
         tc_commit(&k_empty[b]);
       };
-      scores(0);
+      ok = mbar_wait(q_full, 0, abort_flag);
+      if (ok) scores(0);
       if (ok && n_tiles > 1) scores(1);
       int vs = 0, v_use = 0;
       for (int it = 0; ok && it < n_tiles; ++it) {
@@ -304,6 +297,25 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
   } else if (warp >= kFirstSoftmax / 32) {                             // (warp 2 has no work)
     // thread of a row's columns kSpan part .. + kSpan - 1; the row is in the lane quarter this warp may touch
     const int part = (warp - kFirstSoftmax / 32) >> 2, r = (warp & 3) * 32 + lane, id = threadIdx.x - kFirstSoftmax;
+    // the query rows go to shared memory in the layout TMA's 128-byte swizzle would have produced, all loads of a thread in flight at once
+    {
+      constexpr int CHUNKS = DK / 8, STEP = kSoftmax / CHUNKS, N = kRows / STEP;
+      const int c = id % CHUNKS;
+      uint4 v[N];
+#pragma unroll
+      for (int k = 0; k < N; ++k) {
+        const int row = row0 + id / CHUNKS + k * STEP, tok = row / p.group;
+        v[k] = make_uint4(0, 0, 0, 0);
+        if (row < all_rows) v[k] = *reinterpret_cast<const uint4*>(p.q + ((long long)(q0 + tok) * p.H + kvh * p.group + row - tok * p.group) * DK + c * 8);
+      }
+#pragma unroll
+      for (int k = 0; k < N; ++k) {
+        const int rr = id / CHUNKS + k * STEP;
+        *reinterpret_cast<uint4*>(sq + (c >> 3) * kHalf + rr * 128 + (((c & 7) ^ (rr & 7)) << 4)) = v[k];
+      }
+      fence_proxy_async_smem();
+      mbar_arrive(q_full);
+    }
     const uint32_t lane_off = (uint32_t)((warp & 3) * 32) << 16;
     const bool valid = r < n_rows;
     const int lim = valid ? first_pos + (row0 + r) / p.group + 1 : 0, beg = p.window > 0 ? max(0, lim - p.window) : 0;
@@ -390,19 +402,33 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
     l = 0.f;
 #pragma unroll
     for (int k = 0; k < kParts; ++k) l += swap_l[k * kRows + r];
-    const int row = row0 + r;
-    const long long at = (long long)(q0 + row / p.group) * p.H + kvh * p.group + row % p.group;
+    // blocks of 32 rows x 32 columns go out through shared memory (the keys' place), so that eight lanes write 128 bytes of a row
+    constexpr int LD = 36;
+    static_assert(2 * L::kK + kVStages * L::kV >= kSoftmax / 32 * 32 * LD * 4, "room for the output blocks");
+    float* turn = reinterpret_cast<float*>(sk) + (warp - kFirstSoftmax / 32) * (32 * LD);
+    long long to[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const int row = row0 + (warp & 3) * 32 + 4 * k + lane / 8, tok = row / p.group;
+      to[k] = ok && row < all_rows ? ((long long)(q0 + tok) * p.H + kvh * p.group + row - tok * p.group) * p.wv + col0 + 4 * (lane % 8) : -1;
+    }
 #pragma unroll 1
     for (int c = part * 32; c < cols; c += 32 * kParts) {
       uint32_t o[32];
       tmem_ld_32x32(tmem_base + 256 + c + lane_off, o);
       tmem_ld_wait();
-      if (!ok || !valid) continue;
-      float4* to = reinterpret_cast<float4*>(p.part_o + at * p.wv + col0 + c);
 #pragma unroll
-      for (int i = 0; i < 8; ++i)
-        to[i] = make_float4(__uint_as_float(o[4 * i]), __uint_as_float(o[4 * i + 1]), __uint_as_float(o[4 * i + 2]), __uint_as_float(o[4 * i + 3]));
+      for (int i = 0; i < 32; i += 4) *reinterpret_cast<uint4*>(turn + lane * LD + i) = make_uint4(o[i], o[i + 1], o[i + 2], o[i + 3]);
+      __syncwarp();
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        const float4 v = *reinterpret_cast<const float4*>(turn + (4 * k + lane / 8) * LD + 4 * (lane % 8));
+        if (to[k] >= 0) *reinterpret_cast<float4*>(p.part_o + to[k] + c) = v;
+      }
+      __syncwarp();
     }
+    const int row = row0 + r;
+    const long long at = (long long)(q0 + row / p.group) * p.H + kvh * p.group + row % p.group;
     if (ok && valid && part == 0 && col0 == 0) p.part_ml[2 * at] = m_used * kLn2, p.part_ml[2 * at + 1] = l;
   }
   tc_fence_before_sync();
