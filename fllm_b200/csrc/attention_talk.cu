@@ -169,8 +169,6 @@ __global__ void __launch_bounds__(kThreads, 1) talk_prefill_kernel(const __grid_
   float* near_bias = rates + 2 * 16;                                 // [buffer][head of the group]: bias of a tile's smallest distance
   float* table = near_bias + 2 * 16;
 
-  pdl_launch_dependents();
-  pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int row0 = (gridDim.x - 1 - blockIdx.x) * kRows;             // the tiles with the longest key range start first
   const int kvh = blockIdx.y / col_ctas, col0 = blockIdx.y % col_ctas * kCols, seq = blockIdx.z;
@@ -919,7 +917,8 @@ void launch_prefill(const Talk& a, const MapsAttnParams& p, int min_rows, cudaSt
   const CUtensorMap km = pool_map(p.k_cache, n * a.G, DK), vm = value_map(p.v_cache, n, a.wv);
   const int col_ctas = (a.wv + kCols - 1) / kCols;
   const dim3 grid((p.max_q_len * a.group + kRows - 1) / kRows, a.G * col_ctas, p.num_seqs);
-  launch_pdl(talk_prefill_kernel<DK>, grid, dim3(kThreads), TalkTile<DK>::kTotal, s, km, vm, a, min_rows, col_ctas);
+  // in plain stream order: a kernel that takes all tensor memory of its SMs neither starts early nor lets others start
+  talk_prefill_kernel<DK><<<grid, kThreads, TalkTile<DK>::kTotal, s>>>(km, vm, a, min_rows, col_ctas);
   cuda_check(cudaGetLastError(), "talk_prefill_kernel");
 }
 }  // namespace

@@ -760,7 +760,7 @@ static void launch_gemm(const CUtensorMap& ta, const CUtensorMap& tb, const Gemm
   using S = GemmSmem<BN>;
   configure_gemm<BN>();
   if (a.cluster_red)
-    launch_pdl_cluster(gemm_bf16_kernel<BN>, dim3(grid), dim3(kGemmThreads), S::kTotal, stream, (unsigned)a.k_splits, ta,
+    launch_cluster(true, gemm_bf16_kernel<BN>, dim3(grid), dim3(kGemmThreads), S::kTotal, stream, (unsigned)a.k_splits, ta,
                        tb, a);
   else
     launch_pdl(gemm_bf16_kernel<BN>, dim3(grid), dim3(kGemmThreads), S::kTotal, stream, ta, tb, a);

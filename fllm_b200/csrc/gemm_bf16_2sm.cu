@@ -129,14 +129,14 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tma_x, const __grid_co
   const uint32_t tmem_base = *tmem_slot;
   // No early trigger for the dependents: with one, steps stalled at random where a one-CTA GEMM followed closely. Its
   // CTAs could allocate tensor memory on an SM that one CTA of a pair had left while the other still freed the pair's
-  // columns. The next kernel starts when the whole grid is done.
+  // columns. The next kernel starts when the whole grid is done, and for the same reason this one does not start before
+  // the kernels ahead of it are done: pairs and single CTAs never hold tensor memory at the same time.
 
   const int tiles = p.m_tiles * p.n_tiles;
   const int n_clusters = gridDim.x >> 1, cluster_id = blockIdx.x >> 1;
 
   if (warp == 0) {
     if (lane == 0) {
-      pdl_wait();
       int stage = 0;
       uint32_t phase = 0;
       bool ok = true;
@@ -282,7 +282,7 @@ int linear_bf16_pair(const void* x, long long ldx, const void* w, long long ldw,
     cuda_check(cudaFuncSetAttribute(gemm_bf16_pair_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kP2Smem),
                "cudaFuncSetAttribute(gemm_bf16_pair_kernel)");
   const int clusters = std::min(a.m_tiles * a.n_tiles, sm_count() / 2);
-  launch_pdl_cluster(gemm_bf16_pair_kernel, dim3(2 * clusters), dim3(kP2Threads), (size_t)kP2Smem, stream, 2u, tx, tw, a);
+  launch_cluster(false, gemm_bf16_pair_kernel, dim3(2 * clusters), dim3(kP2Threads), (size_t)kP2Smem, stream, 2u, tx, tw, a);
   return 1;
 }
 

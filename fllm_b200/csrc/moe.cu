@@ -47,13 +47,20 @@ __global__ void moe_route_kernel(const __nv_bfloat16* __restrict__ logits, long 
   }
   float sel_v[8];
   int sel_e[8];
+  // a logit that is not a number counts as -inf, and a winner is marked as taken: the k experts are valid and distinct whatever comes in
+  unsigned open = 0;
+#pragma unroll
+  for (int i = 0; i < MAXPL; ++i) {
+    if (v[i] != v[i]) v[i] = -INFINITY;
+    open |= lane + 32 * i < experts ? 1u << i : 0u;
+  }
   for (int j = 0; j < k; ++j) {
     float best = -INFINITY;
     int best_e = 0x7fffffff;
 #pragma unroll
     for (int i = 0; i < MAXPL; ++i) {
       const int e = lane + 32 * i;
-      if (v[i] > best || (v[i] == best && e < best_e)) { best = v[i]; best_e = e; }
+      if ((open >> i & 1) && (v[i] > best || (v[i] == best && e < best_e))) { best = v[i]; best_e = e; }
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
@@ -63,7 +70,7 @@ __global__ void moe_route_kernel(const __nv_bfloat16* __restrict__ logits, long 
     }
     sel_v[j] = best;
     sel_e[j] = best_e;
-    if ((best_e & 31) == lane) v[best_e >> 5] = -INFINITY;    // remove the winner
+    if ((best_e & 31) == lane) open &= ~(1u << (best_e >> 5));    // remove the winner
   }
   if (lane == 0) {
     float w[8], sum = 0.f;
@@ -165,13 +172,19 @@ __global__ void moe_route_scored_kernel(const Logits logits, const float* __rest
   if (gate_out != nullptr && lane == 0) gate_out[t] = 1.f / (1.f + ex(-logits(t, experts)));
   float sel_s[8];
   int sel_e[8];
+  unsigned open = 0;      // as in moe_route_kernel: valid and distinct experts whatever the scores are
+#pragma unroll
+  for (int i = 0; i < MAXPL; ++i) {
+    if (ch[i] != ch[i]) ch[i] = -INFINITY;
+    open |= lane + 32 * i < experts ? 1u << i : 0u;
+  }
   for (int j = 0; j < k; ++j) {
     float best = -INFINITY, best_s = 0.f;
     int best_e = 0x7fffffff;
 #pragma unroll
     for (int i = 0; i < MAXPL; ++i) {
       const int e = lane + 32 * i;
-      if (ch[i] > best || (ch[i] == best && e < best_e)) { best = ch[i]; best_e = e; best_s = sc[i]; }
+      if ((open >> i & 1) && (ch[i] > best || (ch[i] == best && e < best_e))) { best = ch[i]; best_e = e; best_s = sc[i]; }
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
@@ -181,7 +194,7 @@ __global__ void moe_route_scored_kernel(const Logits logits, const float* __rest
     }
     sel_s[j] = best_s;
     sel_e[j] = best_e;
-    if ((best_e & 31) == lane) ch[best_e >> 5] = -INFINITY;    // remove the winner
+    if ((best_e & 31) == lane) open &= ~(1u << (best_e >> 5));    // remove the winner
   }
   if (lane == 0) {
     float sum = 0.f;
@@ -197,7 +210,7 @@ __global__ void moe_route_scored_kernel(const Logits logits, const float* __rest
 void moe_route_scored(const void* logits, long long ld, const float* select_bias, int tokens, int experts, int k, int score_kind,
                       int renorm, float scale, int* ids, float* weights, cudaStream_t s) {
   if (tokens <= 0) return;
-  if (experts > 256 || k > 8 || (score_kind != 1 && score_kind != 2)) throw std::runtime_error("moe_route_scored: at most 256 experts, top-8, score kind 1 or 2");
+  if (experts > 256 || k > 8 || k > experts || (score_kind != 1 && score_kind != 2)) throw std::runtime_error("moe_route_scored: at most 256 experts, top-8, score kind 1 or 2");
   moe_route_scored_kernel<<<(tokens + 3) / 4, 128, 0, s>>>(Bf16Logits{(const __nv_bfloat16*)logits, ld}, select_bias, tokens, experts, k,
                                                            score_kind, renorm, scale, RouteGroups{}, ids, weights, (float*)nullptr);
   cuda_check(cudaGetLastError(), "moe_route_scored_kernel");
@@ -206,7 +219,7 @@ void moe_route_scored(const void* logits, long long ld, const float* select_bias
 void moe_route_fp32(const float* logits, int splits, long long plane, long long ld, int tokens, int experts, int k, int score_kind, int renorm,
                     float scale, int* ids, float* weights, cudaStream_t s, const float* select_bias, const RouteGroups& groups, float* gate_out) {
   if (tokens <= 0) return;
-  if (experts > 256 || k > 8 || (score_kind != 1 && score_kind != 2)) throw std::runtime_error("moe_route_fp32: at most 256 experts, top-8, score kind 1 or 2");
+  if (experts > 256 || k > 8 || k > experts || (score_kind != 1 && score_kind != 2)) throw std::runtime_error("moe_route_fp32: at most 256 experts, top-8, score kind 1 or 2");
   if (groups.groups < 1 || experts % groups.groups || groups.keep < 1) throw std::runtime_error("moe_route_fp32: equal groups of experts");
   moe_route_scored_kernel<<<(tokens + 3) / 4, 128, 0, s>>>(SumLogits{logits, ld, plane, splits}, select_bias, tokens, experts, k, score_kind,
                                                            renorm, scale, groups, ids, weights, gate_out);

@@ -104,10 +104,10 @@ inline void launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t s
   cuda_check(cudaLaunchKernelEx(&cfg, kernel, KArgs(std::forward<Args>(args))...), "cudaLaunchKernelEx");
 }
 
-// Same, with the grid cut into thread-block clusters of `cluster_x` consecutive CTAs.
+// Same, with the grid cut into thread-block clusters of `cluster_x` consecutive CTAs; `early` = false: plain stream order.
 template <typename... KArgs, typename... Args>
-inline void launch_pdl_cluster(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
-                               unsigned cluster_x, Args&&... args) {
+inline void launch_cluster(bool early, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
+                           unsigned cluster_x, Args&&... args) {
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = grid;
   cfg.blockDim = block;
@@ -115,7 +115,7 @@ inline void launch_pdl_cluster(void (*kernel)(KArgs...), dim3 grid, dim3 block, 
   cfg.stream = stream;
   cudaLaunchAttribute attr[2];
   attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attr[0].val.programmaticStreamSerializationAllowed = pdl_enabled() ? 1 : 0;
+  attr[0].val.programmaticStreamSerializationAllowed = early && pdl_enabled() ? 1 : 0;
   attr[1].id = cudaLaunchAttributeClusterDimension;
   attr[1].val.clusterDim.x = cluster_x;
   attr[1].val.clusterDim.y = 1;

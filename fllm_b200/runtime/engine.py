@@ -388,11 +388,12 @@ class LLMEngine:
                     rows.append(t + n - 1)
             max_kv = max(max_kv, s.start + n)
             t += n
-        if Tp > T:           # padding rows of a graph bucket: no KV write, row 0's table
+        if Tp > T:           # padding rows of a graph bucket: no KV write, the first token of block 0 as their only key
             ids[T:Tp] = 0
             pos[T:Tp] = 0
             slots[T:Tp] = -1
-            rseq[T:Tp] = 0
+            rseq[T:Tp] = np.arange(B, Bp, dtype=np.int32)
+            tab[B:Bp, 0] = 0                              # (a sequence's own first block may have fallen behind the window)
             rows.extend(range(T, Tp))
             qst[B:Bp] = np.arange(T, Tp, dtype=np.int32)      # one padding row per padding sequence
             kvl[B:Bp] = 1

@@ -141,6 +141,31 @@ def test_generation_through_the_scheduler_gives_back_pages_behind_the_windows():
     _best(cfg, w, prompts, eng.generate(prompts, SamplingParams(max_tokens=30, ignore_eos=True)), 30)
 
 
+def test_padding_rows_of_a_captured_step_point_at_a_real_block():
+    """Rows that fill a decode step up to its captured size have one key, the first of block 0, whatever the staging buffer held:
+    entries of sequences whose first pages fell behind the window (-1) stay out of them."""
+    cfg = S.CONFIGS["odd"]
+    eng = S.engine(cfg, S.tensors(cfg), chunk=16, seqs=4, spare=4, blocks=48)
+    build, seen = eng._build_batch, []
+
+    def checked(step, pad_to=0, slot=0):
+        if step.all_decode:
+            n, b = len(step.seqs), build(step, pad_to=4, slot=slot)
+            t = b.block_tables
+            seen.append((n, int((t[:n, 0] < 0).sum())))
+            assert t.shape[0] == 4 and t[n:, 0].tolist() == [0] * (4 - n)
+            assert b.row_seq.tolist() == list(range(4)) and b.seq_lens[n:].tolist() == [1] * (4 - n) and b.slots[n:].tolist() == [-1] * (4 - n)
+            assert b.seq_state[n:].tolist() == [eng.rstate.slots - 1] * (4 - n)
+        return build(step, pad_to=pad_to, slot=slot)
+
+    eng._build_batch = checked
+    for k, n in enumerate((60, 64, 55, 58)):
+        eng.add_request(S.prompt(cfg, n, n), SamplingParams(max_tokens=24 + 4 * k, ignore_eos=True))
+    while eng.scheduler.has_work():
+        eng.step()
+    assert any(pruned for _, pruned in seen) and {n for n, _ in seen} == {1, 2, 3, 4}      # pruned first pages, then fewer and fewer sequences
+
+
 def test_a_cached_prefix_restores_the_states():
     """Prompts that share a prefix: the later ones continue from kept copies of the shift and convolution rows."""
     cfg = S.CONFIGS["odd"]

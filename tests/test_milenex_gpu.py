@@ -444,6 +444,60 @@ def test_generation_through_the_scheduler(f32):
     assert not f32 or alone[0] == outs[0]
 
 
+@pytest.mark.parametrize("f32", [True, False])
+def test_captured_steps_with_padding_rows(f32):
+    """Requests that end one after another behind their windows: the captured steps of four rows hold more and more padding, whose
+    results stay finite and leave the other rows alone."""
+    cfg = S.CONFIGS["odd"]
+    w = S.tensors(cfg, 0, not f32)
+    eng = S.engine(cfg, w, DEV, f32, chunk=64, seqs=4, spare=8, blocks=40, max_len=256, graph_buckets=[4])
+    build, widths = eng._build_batch, []
+
+    def watched(step, pad_to=0, slot=0):
+        b = build(step, pad_to=pad_to, slot=slot)
+        if pad_to:
+            widths.append(len(step.seqs))
+            assert b.block_tables[len(step.seqs):, 0].tolist() == [0] * (pad_to - len(step.seqs))
+        return b
+
+    eng._build_batch = watched
+    prompts = [S.prompt(cfg, n, n) for n in (40, 90, 50, 70)]
+    reqs = [eng.requests[eng.add_request(p, SamplingParams(max_tokens=12 + 9 * k, ignore_eos=True))] for k, p in enumerate(prompts)]
+    while not all(r.finish_reason for r in reqs):
+        eng.step()
+        for g in eng._graphs.values():
+            assert torch.isfinite(g.logits).all()
+    assert set(widths) >= {1, 2, 3, 4} and eng.ops.check_status() == 0
+    for p, r in zip(prompts, reqs):
+        lg = O.forward(cfg, w, p + list(r.output))[len(p) - 1:-1]
+        gap = (lg.max(-1).values - lg.gather(1, torch.tensor(list(r.output))[:, None])[:, 0]) / (lg.max(-1).values - lg.min(-1).values)
+        assert float(gap.max()) < (1e-4 if f32 else 0.05)
+
+
+@pytest.mark.parametrize("E,k", [(5, 3), (8, 8), (60, 6), (256, 8)])
+def test_routes_of_rows_that_are_not_numbers(ops, E, k):
+    """Scores that are NaN or infinite still give k different experts of the layer, and the other rows do not notice."""
+    z = torch.randn(9, E, device=DEV, generator=gen(E))
+    clean = z.clone()
+    z[1], z[3], z[5, : E // 2], z[7] = float("nan"), float("-inf"), float("nan"), float("inf")
+    bad = [1, 3, 5, 7]
+    good = [i for i in range(9) if i not in bad]
+
+    def run(call, x):
+        ids, wts = torch.empty(9, k, dtype=torch.int32, device=DEV), torch.empty(9, k, device=DEV)
+        call(x, ids, wts)
+        return ids, wts
+
+    calls = [lambda x, i, w: ops.k.moe_route(x.bfloat16(), None, k, False, i, w), lambda x, i, w: ops.k.moe_route(x.bfloat16(), None, k, True, i, w),
+             lambda x, i, w: ops.k.moe_route_scored(x.bfloat16(), None, k, 1, True, 1.0, i, w),
+             lambda x, i, w: ops.k.moe_route_scored(x.bfloat16(), None, k, 2, True, 1.0, i, w),
+             lambda x, i, w: ops.k.moe_route_fp32(x, None, 0, E, E, k, 1, False, 1.0, i, w, None, 1, 1, float("-inf"), None)]
+    for call in calls:
+        (ids, wts), (ids0, wts0) = run(call, z), run(call, clean)
+        assert int(ids.min()) >= 0 and int(ids.max()) < E and all(len(set(r)) == k for r in ids.tolist())
+        assert torch.equal(ids[good], ids0[good]) and torch.equal(wts[good], wts0[good])
+
+
 def test_replay_program(tmp_path):
     """bin/trace_run as a process: steps on standard input, one logits file and one 'done' line per step."""
     cfg, w, toks, want = S.expected("odd", 140, 2)
